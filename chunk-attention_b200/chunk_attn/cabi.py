@@ -14,7 +14,7 @@ _LIB_PATH = os.path.join(os.path.dirname(os.path.abspath(__file__)), "lib", "lib
 
 CA_OK = 0
 CA_ERR_INVALID, CA_ERR_CUDA, CA_ERR_STATE, CA_ERR_DEVICE_STATUS = -1, -2, -3, -4
-CA_DTYPE_F16, CA_DTYPE_F32 = 0, 1
+CA_DTYPE_F16, CA_DTYPE_F32, CA_DTYPE_BF16 = 0, 1, 2
 CA_OPT_SPLIT_PHASES, CA_OPT_NUM_CTAS, CA_OPT_SEQ_FIRST_TENSOR, CA_OPT_TRACE, CA_OPT_DEPENDENT_LAUNCH = 1, 2, 3, 4, 5
 CA_OPT_WIDE_RUNS, CA_OPT_WAIT_LIMIT_CYCLES, CA_OPT_TEST_WITHHOLD_ITEM, CA_OPT_OVERLAP_KERNELS, CA_OPT_FINISH_IN_TAILS = 6, 7, 8, 9, 10
 STATUS_FULL_WAIT_TIMEOUT, STATUS_EMPTY_WAIT_TIMEOUT, STATUS_DRAIN_TIMEOUT, STATUS_BAD_WORK_LIST, STATUS_BAD_POSITION = 1, 2, 3, 4, 5
@@ -31,6 +31,8 @@ EXPORTED = [
     "ca_context_read_trace",
     "ca_plan_build", "ca_plan_build_for_context", "ca_refresh_from_plan", "ca_plan_array", "ca_plan_stats_get", "ca_plan_destroy", "ca_attention_static", "ca_attention_static_status",
     "ca_rms_norm", "ca_fused_add_rms_norm", "ca_rotary_embedding",
+    "ca_chunk_bytes_shaped", "ca_context_create_shaped", "ca_store_qkv", "ca_attention_rows", "ca_rows_block", "ca_token_shift", "ca_gated_norm_add",
+    "ca_norm_rows", "ca_gelu_tanh", "ca_conv_silu", "ca_scan_scratch_floats", "ca_selective_scan", "ca_decay_attention",
 ]
 CA_STATIC_MAX_SLOTS = 16384
 

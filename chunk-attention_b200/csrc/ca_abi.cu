@@ -48,6 +48,18 @@ struct DeviceGuard {
 };
 
 int esize_of(int dtype) { return dtype == CA_DTYPE_F16 ? 2 : (dtype == CA_DTYPE_F32 ? 4 : 0); }
+int shaped_esize_of(int dtype) { return dtype == CA_DTYPE_BF16 ? 2 : esize_of(dtype); }
+
+// pool geometry of a head shape: heads padded to whole 16-byte granules
+ca::Geometry shaped_geometry(const ca_head_shape& sh, int chunk_size, int esize) {
+    const int per16 = 16 / esize;
+    auto pad = [&](int d) { return (d + per16 - 1) / per16 * per16; };
+    return ca::make_geometry(sh.n_kv_heads, pad(sh.d_key), chunk_size, esize, pad(sh.d_value));
+}
+bool shape_ok(const ca_head_shape* sh) {
+    return sh && sh->n_heads > 0 && sh->n_kv_heads > 0 && sh->n_heads % sh->n_kv_heads == 0 && sh->d_key > 0 && sh->d_value > 0 &&
+           sh->d_key <= 256 && sh->d_value <= 256;
+}
 
 size_t align_up(size_t x, size_t a) { return (x + a - 1) / a * a; }
 
@@ -80,6 +92,9 @@ struct ca_context {
     int64_t max_chunks = 0;
     int tpp_threshold = 1;
     bool fast = false;
+    bool shaped = false;          // made by ca_context_create_shaped: `shape` describes the heads
+    ca_head_shape shape{};
+    int group = 1;                // query heads per key/value head
     int num_sms = 1;
     bool opt_split = false;
     int opt_ctas = 0;
@@ -167,14 +182,8 @@ int64_t ca_tile_elem_offset(int d_head, int chunk_size, int dtype, int token, in
     return ca::tile_elem_offset(g, token, elem);
 }
 
-int ca_context_create(ca_context** out, int device, int n_heads, int d_head, int chunk_size, int dtype,
-                      void* pool, int64_t max_chunks, int tpp_threshold) {
-    if (!out) return fail(CA_ERR_INVALID, "out is null");
-    *out = nullptr;
-    const int es = esize_of(dtype);
-    if (es == 0) return fail(CA_ERR_INVALID, "unsupported dtype (fp16 and fp32 only)");
-    if (n_heads <= 0 || d_head <= 0 || chunk_size <= 0) return fail(CA_ERR_INVALID, "n_heads, d_head, chunk_size must be positive");
-    if (d_head > 256) return fail(CA_ERR_INVALID, "d_head above 256 is not supported");
+static int make_context(ca_context** out, int device, const ca_head_shape* shape, const ca::Geometry& geo, int dtype, void* pool,
+                        int64_t max_chunks, int tpp_threshold) {
     if (max_chunks < 0 || (max_chunks > 0 && !pool)) return fail(CA_ERR_INVALID, "pool is null");
     if (reinterpret_cast<uintptr_t>(pool) % 256 != 0) return fail(CA_ERR_INVALID, "pool must be 256-byte aligned");
     int n_dev = 0;
@@ -190,11 +199,16 @@ int ca_context_create(ca_context** out, int device, int n_heads, int d_head, int
     if (!c) return fail(CA_ERR_INVALID, "out of host memory");
     c->device = device;
     c->dtype = dtype;
-    c->geo = ca::make_geometry(n_heads, d_head, chunk_size, es);
+    c->geo = geo;
+    if (shape) {
+        c->shaped = true;
+        c->shape = *shape;
+        c->group = shape->n_heads / shape->n_kv_heads;
+    }
     c->pool = pool;
     c->max_chunks = max_chunks;
     c->tpp_threshold = tpp_threshold < 1 ? 1 : tpp_threshold;
-    c->fast = (dtype == CA_DTYPE_F16 && d_head == ca::FAST_D && chunk_size == ca::FAST_C);
+    c->fast = (!shape && dtype == CA_DTYPE_F16 && geo.d_head == ca::FAST_D && geo.chunk_size == ca::FAST_C);
     c->num_sms = prop.multiProcessorCount;
     cudaError_t e = cudaEventCreateWithFlags(&c->upload_done, cudaEventDisableTiming);
     if (e == cudaSuccess) e = cudaEventCreateWithFlags(&c->paths_done, cudaEventDisableTiming);
@@ -213,6 +227,34 @@ int ca_context_create(ca_context** out, int device, int n_heads, int d_head, int
     }
     *out = c;
     return CA_OK;
+}
+
+int ca_context_create(ca_context** out, int device, int n_heads, int d_head, int chunk_size, int dtype,
+                      void* pool, int64_t max_chunks, int tpp_threshold) {
+    if (!out) return fail(CA_ERR_INVALID, "out is null");
+    *out = nullptr;
+    const int es = esize_of(dtype);
+    if (es == 0) return fail(CA_ERR_INVALID, "unsupported dtype (fp16 and fp32 only)");
+    if (n_heads <= 0 || d_head <= 0 || chunk_size <= 0) return fail(CA_ERR_INVALID, "n_heads, d_head, chunk_size must be positive");
+    if (d_head > 256) return fail(CA_ERR_INVALID, "d_head above 256 is not supported");
+    return make_context(out, device, nullptr, ca::make_geometry(n_heads, d_head, chunk_size, es), dtype, pool, max_chunks, tpp_threshold);
+}
+
+int64_t ca_chunk_bytes_shaped(const ca_head_shape* shape, int chunk_size, int dtype) {
+    const int es = shaped_esize_of(dtype);
+    if (es == 0 || !shape_ok(shape) || chunk_size <= 0) return -1;
+    return shaped_geometry(*shape, chunk_size, es).chunk_elems * es;
+}
+
+int ca_context_create_shaped(ca_context** out, int device, const ca_head_shape* shape, int chunk_size, int dtype, void* pool,
+                             int64_t max_chunks, int tpp_threshold) {
+    if (!out) return fail(CA_ERR_INVALID, "out is null");
+    *out = nullptr;
+    const int es = shaped_esize_of(dtype);
+    if (es == 0) return fail(CA_ERR_INVALID, "unsupported dtype (fp16, bf16 and fp32 only)");
+    if (!shape_ok(shape)) return fail(CA_ERR_INVALID, "bad head shape: n_kv_heads must divide n_heads, head sizes must lie in 1 .. 256");
+    if (chunk_size <= 0) return fail(CA_ERR_INVALID, "chunk_size must be positive");
+    return make_context(out, device, shape, shaped_geometry(*shape, chunk_size, es), dtype, pool, max_chunks, tpp_threshold);
 }
 
 void ca_context_destroy(ca_context* c) {
@@ -484,6 +526,7 @@ static int check_attention_args(ca_context* c, const void* q, int n_seqs) {
     if (!c->valid) return fail(CA_ERR_STATE, "work list is stale: call ca_refresh_kernel_context first");
     if (n_seqs != c->meta.n_seqs) return fail(CA_ERR_INVALID, "n_seqs differs from the refreshed work list");
     if (n_seqs > 0 && !q) return fail(CA_ERR_INVALID, "q is null");
+    if (c->shaped) return fail(CA_ERR_INVALID, "a context with a head shape is served by ca_attention_rows");
     if (reinterpret_cast<uintptr_t>(q) % 16 != 0 && c->fast) return fail(CA_ERR_INVALID, "q must be 16-byte aligned");
     return CA_OK;
 }
@@ -822,10 +865,103 @@ int ca_attention(ca_context* c, const void* q, void* out, int n_seqs, int partit
     g.path_off = c->d_path_off;
     g.path_chunks = c->d_path_chunks;
     g.path_tokens = c->d_path_tokens;
-    g.n_seqs = n_seqs;
+    g.n_rows = n_seqs;
+    g.out_width = c->geo.d_value;
     g.delta_tokens = c->delta_tokens;
     g.scale = 1.0f / std::sqrt((float)c->geo.d_head);
     CA_CUDA(ca::launch_attn_seq_generic(g, c->dtype, static_cast<cudaStream_t>(stream_)));
+    return CA_OK;
+}
+
+int ca_store_qkv(ca_context* c, const ca_qkv_args* a, ca_stream stream_) {
+    if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
+    if (!c->shaped) return fail(CA_ERR_INVALID, "store_qkv needs a context with a head shape");
+    if (a->n_tokens < 0) return fail(CA_ERR_INVALID, "negative token count");
+    if (a->n_tokens == 0) return CA_OK;
+    if (!a->qkv || !a->q_out || !a->positions) return fail(CA_ERR_INVALID, "qkv, q_out or positions is null");
+    if (reinterpret_cast<uintptr_t>(a->q_out) % 16) return fail(CA_ERR_INVALID, "q_out must be 16-byte aligned");
+    if (a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > c->shape.d_key) return fail(CA_ERR_INVALID, "rot_dims must be even and at most d_key");
+    const bool append = a->tok_slot == nullptr;
+    if (append) {
+        if (!c->valid) return fail(CA_ERR_STATE, "work list is stale: call ca_refresh_kernel_context first");
+        if (a->n_tokens != c->meta.n_seqs) return fail(CA_ERR_INVALID, "one token per row of the refreshed work list is required");
+        if (c->max_tail_tokens + c->delta_tokens >= c->geo.chunk_size)
+            return fail(CA_ERR_STATE, "a tail chunk is full: reserve a new tail and refresh before appending");
+    }
+    DeviceGuard guard(c->device);
+    if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
+    ca::QkvParams p;
+    p.pool = c->pool;
+    p.geo = c->geo;
+    p.group = c->group;
+    p.d_key = c->shape.d_key;
+    p.d_value = c->shape.d_value;
+    p.qkv = a->qkv;
+    p.row_stride = a->row_stride;
+    p.q_out = a->q_out;
+    p.q_norm = a->q_norm;
+    p.k_norm = a->k_norm;
+    p.eps = a->eps;
+    p.rot_dims = a->rot_dims;
+    p.key_freq = a->key_freq;
+    p.value_freq = a->value_freq;
+    p.positions = a->positions;
+    p.tok_slot = a->tok_slot;
+    p.tail_chunk = c->d_tail_chunk;
+    p.tail_tokens = c->d_tail_tokens;
+    p.delta_tokens = c->delta_tokens;
+    p.n_tokens = a->n_tokens;
+    CA_CUDA(ca::launch_store_qkv(p, c->dtype, static_cast<cudaStream_t>(stream_)));
+    if (append) c->delta_tokens += 1;
+    return CA_OK;
+}
+
+int ca_rows_block(const ca_head_shape* shape) {
+    if (!shape_ok(shape)) return 1;
+    const int group = shape->n_heads / shape->n_kv_heads;  // a block holds the query heads of a group: 128 query rows
+    return group >= 128 ? 1 : 128 / group;
+}
+
+int ca_attention_rows(ca_context* c, const ca_rows_args* a, ca_stream stream_) {
+    if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
+    if (!c->shaped) return fail(CA_ERR_INVALID, "attention_rows needs a context with a head shape");
+    if (a->n_rows < 0) return fail(CA_ERR_INVALID, "negative row count");
+    if (a->n_rows == 0) return CA_OK;
+    if (!a->q || !a->out) return fail(CA_ERR_INVALID, "q or out is null");
+    if (reinterpret_cast<uintptr_t>(a->q) % 16) return fail(CA_ERR_INVALID, "q must be 16-byte aligned");
+    const bool decode = a->path_off == nullptr;
+    if (decode) {
+        if (!c->valid) return fail(CA_ERR_STATE, "work list is stale: call ca_refresh_kernel_context first");
+        if (a->n_rows != c->meta.n_seqs) return fail(CA_ERR_INVALID, "n_rows differs from the refreshed work list");
+    } else if (!a->row_entry || !a->path_chunks || !a->positions || !a->blocks) {
+        return fail(CA_ERR_INVALID, "portions need row_entry, positions, path_chunks and blocks");
+    }
+    if (a->value_freq && !a->positions) return fail(CA_ERR_INVALID, "rotated values need positions");
+    DeviceGuard guard(c->device);
+    if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
+    cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+    if (decode) {
+        const int rc = ensure_paths(c, stream);
+        if (rc != CA_OK) return rc;
+    }
+    ca::GenericParams g;
+    g.pool = c->pool;
+    g.geo = c->geo;
+    g.q = a->q;
+    g.out = a->out;
+    g.path_off = decode ? c->d_path_off : a->path_off;
+    g.path_chunks = decode ? c->d_path_chunks : a->path_chunks;
+    g.path_tokens = decode ? c->d_path_tokens : nullptr;
+    g.n_rows = a->n_rows;
+    g.delta_tokens = c->delta_tokens;
+    g.scale = c->shape.scale;
+    g.group = c->group;
+    g.out_width = c->shape.d_value;
+    g.sink = c->shape.sink;
+    g.row_entry = decode ? nullptr : a->row_entry;
+    g.positions = a->positions;
+    g.value_freq = a->value_freq;
+    CA_CUDA(ca::launch_attn_seq_generic(g, c->dtype, stream));
     return CA_OK;
 }
 
@@ -843,7 +979,10 @@ int ca_scatter_prefill(ca_context* c, const void* k, const void* v, int64_t stri
     if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
     const int es = c->geo.esize;
     const char* kb = static_cast<const char*>(k) + (int64_t)first_token * stride_token * es;
-    const char* vb = static_cast<const char*>(v) + (int64_t)first_token * stride_token * es;
+    // values of another width than the keys are dense rows
+    const bool same = c->geo.d_value == c->geo.d_head;
+    const int64_t v_st = same ? stride_token : (int64_t)c->geo.n_heads * c->geo.d_value, v_sh = same ? stride_head : c->geo.d_value;
+    const char* vb = static_cast<const char*>(v) + (int64_t)first_token * v_st * es;
     // 16-byte moves need every source row to start on a 16-byte boundary
     const bool vec16 = c->geo.epg > 1 && reinterpret_cast<uintptr_t>(kb) % 16 == 0 &&
                        reinterpret_cast<uintptr_t>(vb) % 16 == 0 && (stride_token * es) % 16 == 0 &&
@@ -854,9 +993,11 @@ int ca_scatter_prefill(ca_context* c, const void* k, const void* v, int64_t stri
         p.pool = c->pool;
         p.geo = c->geo;
         p.k = kb + (int64_t)c0 * C * stride_token * es;
-        p.v = vb + (int64_t)c0 * C * stride_token * es;
+        p.v = vb + (int64_t)c0 * C * v_st * es;
         p.stride_token = stride_token;
         p.stride_head = stride_head;
+        p.v_stride_token = v_st;
+        p.v_stride_head = v_sh;
         const int tok_end = (c0 + nc) * C < n_tokens ? (c0 + nc) * C : n_tokens;
         p.n_tokens = tok_end - c0 * C;
         std::memcpy(p.chunk_ids, chunk_ids + c0, nc * sizeof(int32_t));
@@ -881,6 +1022,8 @@ int ca_scatter_rows(ca_context* c, const void* k, const void* v, int64_t stride_
     const bool vec16 = c->geo.epg > 1 && reinterpret_cast<uintptr_t>(k) % 16 == 0 &&
                        reinterpret_cast<uintptr_t>(v) % 16 == 0 && (stride_token * es) % 16 == 0 &&
                        (stride_head * es) % 16 == 0;
+    const bool same = c->geo.d_value == c->geo.d_head;
+    const int64_t v_st = same ? stride_token : (int64_t)c->geo.n_heads * c->geo.d_value, v_sh = same ? stride_head : c->geo.d_value;
     // the plan's tail fill counts no longer describe the pool: the next step needs a fresh work list
     c->valid = false;
     for (int t0 = 0; t0 < n_tokens; t0 += ca::SCATTER_MAX_ROWS) {
@@ -889,9 +1032,11 @@ int ca_scatter_rows(ca_context* c, const void* k, const void* v, int64_t stride_
         p.pool = c->pool;
         p.geo = c->geo;
         p.k = static_cast<const char*>(k) + (int64_t)t0 * stride_token * es;
-        p.v = static_cast<const char*>(v) + (int64_t)t0 * stride_token * es;
+        p.v = static_cast<const char*>(v) + (int64_t)t0 * v_st * es;
         p.stride_token = stride_token;
         p.stride_head = stride_head;
+        p.v_stride_token = v_st;
+        p.v_stride_head = v_sh;
         p.n_tokens = nt;
         std::memcpy(p.chunk_ids, chunk_ids + t0, nt * sizeof(int32_t));
         std::memcpy(p.rows, rows + t0, nt * sizeof(int32_t));

@@ -129,20 +129,50 @@ struct PeerBarrierParams {
 };
 cudaError_t launch_peer_barrier(const PeerBarrierParams& p, cudaStream_t stream);
 
-// ---- generic path: any d_head <= 256, any chunk size, fp16 or fp32 ----------------------------------
+// ---- generic path: any d_head <= 256, any chunk size, fp16, bf16 or fp32 -----------------------------
 struct GenericParams {
     const void* pool;
     Geometry geo;
-    const void* q;
-    void* out;
-    const int32_t* path_off;     // [n_seqs + 1]
+    const void* q;               // [n_rows, n_heads * group, d_head]
+    void* out;                   // [n_rows, n_heads * group, out_width]
+    const int32_t* path_off;     // [paths + 1]
     const int32_t* path_chunks;
-    const int32_t* path_tokens;
-    int n_seqs;
+    const int32_t* path_tokens;  // tokens stored in each chunk; null: only `positions` bounds what a row sees
+    int n_rows;
     int delta_tokens;
-    float scale;                 // 1 / sqrt(d_head)
+    float scale;
+    int group = 1;               // query heads per key/value head
+    int out_width = 0;           // elements of an output row (d_value without the padding)
+    int sink = 0;                // 1: one is added to the softmax denominator
+    const int32_t* row_entry = nullptr;  // path of each row; null: row r walks path r, all of it
+    const int32_t* positions = nullptr;  // position of each row's token (needed with row_entry or value_freq)
+    const float* value_freq = nullptr;   // radians per position of value pair i; null: values are not rotated
 };
 cudaError_t launch_attn_seq_generic(const GenericParams& p, int dtype, cudaStream_t stream);
+
+// ---- projections to attention operands (ca_qkv.cu) ------------------------------------------------------
+struct QkvParams {
+    void* pool;
+    Geometry geo;                // padded head sizes
+    int group;                   // query heads per key/value head
+    int d_key, d_value;          // head sizes without padding
+    const void* qkv;             // [n_tokens, row_stride]: q heads | k heads | v heads
+    int64_t row_stride;
+    void* q_out;                 // [n_tokens, n_heads * group, geo.d_head]
+    const float* q_norm;         // [d_key] or null: no norm
+    const float* k_norm;
+    float eps;
+    int rot_dims;                // leading elements of q and k that are rotated (pairs 2i, 2i + 1)
+    const float* key_freq;       // [rot_dims / 2] radians per position, or null
+    const float* value_freq;     // [d_value / 2] or null
+    const int32_t* positions;    // [n_tokens]
+    const int32_t* tok_slot;     // pool row (chunk * chunk_size + row) of each token, -1: not written; or null:
+    const int32_t* tail_chunk;   // token s goes to row tail_tokens[s] + delta_tokens of tail_chunk[s]
+    const int32_t* tail_tokens;
+    int delta_tokens;
+    int n_tokens;
+};
+cudaError_t launch_store_qkv(const QkvParams& p, int dtype, cudaStream_t stream);
 
 // ---- pool maintenance ------------------------------------------------------------------------------------
 struct AppendParams {
@@ -164,7 +194,8 @@ struct ScatterParams {
     Geometry geo;
     const void* k;
     const void* v;
-    int64_t stride_token, stride_head;  // in elements
+    int64_t stride_token, stride_head;  // of k, in elements
+    int64_t v_stride_token, v_stride_head;
     int n_tokens;
     int32_t chunk_ids[SCATTER_MAX_CHUNKS];
 };
@@ -177,7 +208,8 @@ struct ScatterRowsParams {
     Geometry geo;
     const void* k;
     const void* v;
-    int64_t stride_token, stride_head;  // in elements
+    int64_t stride_token, stride_head;  // of k, in elements
+    int64_t v_stride_token, v_stride_head;
     int n_tokens;
     int32_t chunk_ids[SCATTER_MAX_ROWS];
     int32_t rows[SCATTER_MAX_ROWS];

@@ -14,6 +14,10 @@
 // no TMA swizzle mode.  The same XOR makes the ldmatrix patterns of the mma.sync path (8 consecutive tokens x
 // one granule, plain for K, .trans for V) and row-wise 128-bit readers bank-conflict free.
 // Other geometries (rows that are not a multiple of 128 bytes) are stored row-major, unswizzled.
+//
+// Keys and values may differ in width (d_head, d_value); each tile then follows the rules above for its own row
+// width.  A layer with fewer key/value heads than query heads (grouped heads) has one tile pair per KEY/VALUE head:
+// n_heads below counts those.
 #pragma once
 #include <stdint.h>
 
@@ -26,30 +30,50 @@
 namespace ca {
 
 struct Geometry {
-    int n_heads;
+    int n_heads;  // key/value heads
     int d_head;
     int chunk_size;
     int esize;  // bytes per element
     int epg;    // elements per 16-byte granule, or 1 when rows are not a whole number of granules
     int gpr;    // granules per token row (d_head / epg)
     int swz;    // 7 when the tile is stored as swizzled 128-byte panels, else 0 (row-major)
-    int64_t tile_elems;   // chunk_size * d_head
-    int64_t chunk_elems;  // n_heads * 2 * tile_elems
+    int64_t tile_elems;   // chunk_size * d_head: one K tile
+    int64_t chunk_elems;  // n_heads * (K tile + V tile)
+    int d_value;          // the same for the V tiles
+    int v_gpr;
+    int v_swz;
+    int64_t v_tile_elems;
 };
 
-CA_HD Geometry make_geometry(int n_heads, int d_head, int chunk_size, int esize) {
+CA_HD Geometry make_geometry(int n_heads, int d_head, int chunk_size, int esize, int d_value = 0) {
     Geometry g;
+    if (d_value <= 0) d_value = d_head;
     g.n_heads = n_heads;
     g.d_head = d_head;
+    g.d_value = d_value;
     g.chunk_size = chunk_size;
     g.esize = esize;
     int per16 = 16 / esize;
-    g.epg = (d_head % per16 == 0) ? per16 : 1;
+    g.epg = (d_head % per16 == 0 && d_value % per16 == 0) ? per16 : 1;
     g.gpr = d_head / g.epg;
+    g.v_gpr = d_value / g.epg;
     g.swz = (g.epg > 1 && g.gpr % 8 == 0) ? 7 : 0;
+    g.v_swz = (g.epg > 1 && g.v_gpr % 8 == 0) ? 7 : 0;
     g.tile_elems = (int64_t)chunk_size * d_head;
-    g.chunk_elems = (int64_t)n_heads * 2 * g.tile_elems;
+    g.v_tile_elems = (int64_t)chunk_size * d_value;
+    g.chunk_elems = (int64_t)n_heads * (g.tile_elems + g.v_tile_elems);
     return g;
+}
+
+// the geometry as seen by code that handles "a tile": the K side (kv = 0) or the V side (kv = 1)
+CA_HD Geometry tile_side(const Geometry& g, int kv) {
+    Geometry s = g;
+    if (kv) {
+        s.d_head = g.d_value;
+        s.gpr = g.v_gpr;
+        s.swz = g.v_swz;
+    }
+    return s;
 }
 
 // index, in 16-byte units from the start of the tile, of granule `gran` of token row t (geometries with
@@ -69,7 +93,7 @@ CA_HD int64_t tile_elem_offset(const Geometry& g, int t, int e) {
 
 // element offset of the K tile (kv = 0) or V tile (kv = 1) of (chunk, head) inside the pool
 CA_HD int64_t tile_base_elems(const Geometry& g, int64_t chunk, int head, int kv) {
-    return chunk * g.chunk_elems + ((int64_t)head * 2 + kv) * g.tile_elems;
+    return chunk * g.chunk_elems + (int64_t)head * (g.tile_elems + g.v_tile_elems) + (kv ? g.tile_elems : 0);
 }
 
 }  // namespace ca

@@ -20,6 +20,11 @@ template <typename U>
 __device__ __forceinline__ int units_per_row(const Geometry& g) {
     return sizeof(U) == 16 ? g.gpr : g.d_head;
 }
+// units of the wider of the two sides: what the grids are sized by
+template <typename U>
+__device__ __forceinline__ int max_units_per_row(const Geometry& g) {
+    return sizeof(U) == 16 ? max(g.gpr, g.v_gpr) : max(g.d_head, g.d_value);
+}
 template <typename U>
 __device__ __forceinline__ void move_unit(void* dst_tile, const void* src_row, const Geometry& g, int t, int unit) {
     if (sizeof(U) == 16) {
@@ -32,7 +37,7 @@ __device__ __forceinline__ void move_unit(void* dst_tile, const void* src_row, c
 template <typename U>
 __global__ void append_kv_kernel(const AppendParams p) {
     const Geometry& g = p.geo;
-    const int upr = units_per_row<U>(g);
+    const int upr = max_units_per_row<U>(g);
     const int64_t total = (int64_t)p.n_seqs * g.n_heads * 2 * upr;
     const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -44,16 +49,18 @@ __global__ void append_kv_kernel(const AppendParams p) {
     const int s = (int)(r / g.n_heads);
     const int t = p.tail_tokens[s] + p.delta_tokens;  // slot inside the tail chunk
     if (t >= g.chunk_size) return;                    // rejected on the host; never write past the tile
+    const Geometry side = tile_side(g, kv);
+    if (unit >= units_per_row<U>(side)) return;
     const char* src = reinterpret_cast<const char*>(kv ? p.v : p.k) +
-                      ((int64_t)s * g.n_heads + h) * g.d_head * g.esize;
+                      ((int64_t)s * g.n_heads + h) * side.d_head * g.esize;
     char* dst = reinterpret_cast<char*>(p.pool) + tile_base_elems(g, p.tail_chunk[s], h, kv) * g.esize;
-    move_unit<U>(dst, src, g, t, unit);
+    move_unit<U>(dst, src, side, t, unit);
 }
 
 template <typename U>
 __global__ void scatter_prefill_kernel(const ScatterParams p) {
     const Geometry& g = p.geo;
-    const int upr = units_per_row<U>(g);
+    const int upr = max_units_per_row<U>(g);
     const int64_t total = (int64_t)p.n_tokens * g.n_heads * 2 * upr;
     const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -65,16 +72,18 @@ __global__ void scatter_prefill_kernel(const ScatterParams p) {
     const int tok = (int)(r / g.n_heads);
     const int chunk = p.chunk_ids[tok / g.chunk_size];
     const int t = tok % g.chunk_size;
-    const char* src = reinterpret_cast<const char*>(kv ? p.v : p.k) +
-                      ((int64_t)tok * p.stride_token + (int64_t)h * p.stride_head) * g.esize;
+    const Geometry side = tile_side(g, kv);
+    if (unit >= units_per_row<U>(side)) return;
+    const int64_t st = kv ? p.v_stride_token : p.stride_token, sh = kv ? p.v_stride_head : p.stride_head;
+    const char* src = reinterpret_cast<const char*>(kv ? p.v : p.k) + ((int64_t)tok * st + (int64_t)h * sh) * g.esize;
     char* dst = reinterpret_cast<char*>(p.pool) + tile_base_elems(g, chunk, h, kv) * g.esize;
-    move_unit<U>(dst, src, g, t, unit);
+    move_unit<U>(dst, src, side, t, unit);
 }
 
 template <typename U>
 __global__ void scatter_rows_kernel(const ScatterRowsParams p) {
     const Geometry& g = p.geo;
-    const int upr = units_per_row<U>(g);
+    const int upr = max_units_per_row<U>(g);
     const int64_t total = (int64_t)p.n_tokens * g.n_heads * 2 * upr;
     const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -84,10 +93,12 @@ __global__ void scatter_rows_kernel(const ScatterRowsParams p) {
     r >>= 1;
     const int h = (int)(r % g.n_heads);
     const int tok = (int)(r / g.n_heads);
-    const char* src = reinterpret_cast<const char*>(kv ? p.v : p.k) +
-                      ((int64_t)tok * p.stride_token + (int64_t)h * p.stride_head) * g.esize;
+    const Geometry side = tile_side(g, kv);
+    if (unit >= units_per_row<U>(side)) return;
+    const int64_t st = kv ? p.v_stride_token : p.stride_token, sh = kv ? p.v_stride_head : p.stride_head;
+    const char* src = reinterpret_cast<const char*>(kv ? p.v : p.k) + ((int64_t)tok * st + (int64_t)h * sh) * g.esize;
     char* dst = reinterpret_cast<char*>(p.pool) + tile_base_elems(g, p.chunk_ids[tok], h, kv) * g.esize;
-    move_unit<U>(dst, src, g, p.rows[tok], unit);
+    move_unit<U>(dst, src, side, p.rows[tok], unit);
 }
 
 template <typename U>
@@ -103,16 +114,16 @@ __global__ void copy_chunks_kernel(const CopyParams p) {
 template <typename E>
 __global__ void read_chunk_kernel(const ReadChunkParams p) {
     const Geometry& g = p.geo;
-    const int64_t total = (int64_t)g.n_heads * p.n_tokens * g.d_head;
+    const int kv = blockIdx.y;
+    const Geometry side = tile_side(g, kv);
+    const int64_t total = (int64_t)g.n_heads * p.n_tokens * side.d_head;
     const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
-    const int e = (int)(idx % g.d_head);
-    const int t = (int)((idx / g.d_head) % p.n_tokens);
-    const int h = (int)(idx / ((int64_t)g.d_head * p.n_tokens));
+    const int e = (int)(idx % side.d_head);
+    const int t = (int)((idx / side.d_head) % p.n_tokens);
+    const int h = (int)(idx / ((int64_t)side.d_head * p.n_tokens));
     const E* pool = reinterpret_cast<const E*>(p.pool);
-    const int64_t off = tile_elem_offset(g, t, e);
-    reinterpret_cast<E*>(p.k_out)[idx] = pool[tile_base_elems(g, p.chunk_id, h, 0) + off];
-    reinterpret_cast<E*>(p.v_out)[idx] = pool[tile_base_elems(g, p.chunk_id, h, 1) + off];
+    reinterpret_cast<E*>(kv ? p.v_out : p.k_out)[idx] = pool[tile_base_elems(g, p.chunk_id, h, kv) + tile_elem_offset(side, t, e)];
 }
 
 inline int blocks_for(int64_t total, int threads) { return (int)((total + threads - 1) / threads); }
@@ -120,7 +131,7 @@ inline int blocks_for(int64_t total, int threads) { return (int)((total + thread
 }  // namespace
 
 cudaError_t launch_append_kv(const AppendParams& p, bool vec16, cudaStream_t stream) {
-    const int upr = vec16 ? p.geo.gpr : p.geo.d_head;
+    const int upr = vec16 ? std::max(p.geo.gpr, p.geo.v_gpr) : std::max(p.geo.d_head, p.geo.d_value);
     const int64_t total = (int64_t)p.n_seqs * p.geo.n_heads * 2 * upr;
     if (total <= 0) return cudaSuccess;
     if (vec16) {
@@ -134,7 +145,7 @@ cudaError_t launch_append_kv(const AppendParams& p, bool vec16, cudaStream_t str
 }
 
 cudaError_t launch_scatter_prefill(const ScatterParams& p, bool vec16, cudaStream_t stream) {
-    const int upr = vec16 ? p.geo.gpr : p.geo.d_head;
+    const int upr = vec16 ? std::max(p.geo.gpr, p.geo.v_gpr) : std::max(p.geo.d_head, p.geo.d_value);
     const int64_t total = (int64_t)p.n_tokens * p.geo.n_heads * 2 * upr;
     if (total <= 0) return cudaSuccess;
     if (vec16) {
@@ -148,7 +159,7 @@ cudaError_t launch_scatter_prefill(const ScatterParams& p, bool vec16, cudaStrea
 }
 
 cudaError_t launch_scatter_rows(const ScatterRowsParams& p, bool vec16, cudaStream_t stream) {
-    const int upr = vec16 ? p.geo.gpr : p.geo.d_head;
+    const int upr = vec16 ? std::max(p.geo.gpr, p.geo.v_gpr) : std::max(p.geo.d_head, p.geo.d_value);
     const int64_t total = (int64_t)p.n_tokens * p.geo.n_heads * 2 * upr;
     if (total <= 0) return cudaSuccess;
     if (vec16) {
@@ -178,12 +189,13 @@ cudaError_t launch_copy_chunks(const CopyParams& p, cudaStream_t stream) {
 }
 
 cudaError_t launch_read_chunk(const ReadChunkParams& p, cudaStream_t stream) {
-    const int64_t total = (int64_t)p.geo.n_heads * p.n_tokens * p.geo.d_head;
+    const int64_t total = (int64_t)p.geo.n_heads * p.n_tokens * std::max(p.geo.d_head, p.geo.d_value);
     if (total <= 0) return cudaSuccess;
+    const dim3 grid(blocks_for(total, 256), 2);  // y: K, V
     if (p.geo.esize == 2) {
-        read_chunk_kernel<uint16_t><<<blocks_for(total, 256), 256, 0, stream>>>(p);
+        read_chunk_kernel<uint16_t><<<grid, 256, 0, stream>>>(p);
     } else {
-        read_chunk_kernel<uint32_t><<<blocks_for(total, 256), 256, 0, stream>>>(p);
+        read_chunk_kernel<uint32_t><<<grid, 256, 0, stream>>>(p);
     }
     return cudaGetLastError();
 }

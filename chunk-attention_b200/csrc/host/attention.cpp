@@ -1,5 +1,6 @@
 #include "attention.h"
 
+#include <algorithm>
 #include <chrono>
 
 #include <c10/cuda/CUDAGuard.h>
@@ -28,9 +29,19 @@ Attention::Attention(int n_heads, int d_head, int chunk_size, int memory_mb, boo
 
 Attention::Attention(Attention& other)
   : n_heads_(other.n_heads_), d_head_(other.d_head_), chunk_size_(other.chunk_size_), memory_mb_(other.memory_mb_),
-    tpp_threshold_(other.tpp_threshold_), share_prefix_(other.share_prefix_), options_(other.options_) {
+    tpp_threshold_(other.tpp_threshold_), shaped_(other.shaped_), shape_(other.shape_), share_prefix_(other.share_prefix_),
+    options_(other.options_) {
     init();
     shared_plan_ = other.shared_plan_;  // same configuration, same sequence of tree operations: same work lists
+    shared_tables_ = other.shared_tables_;
+}
+
+Attention::Attention(const ca_head_shape& shape, int chunk_size, int memory_mb, bool share_prefix, int tpp_threshold,
+                     torch::Dtype dtype, torch::Device device)
+  : n_heads_(shape.n_heads), d_head_(shape.d_key), chunk_size_(chunk_size), memory_mb_(memory_mb),
+    tpp_threshold_(tpp_threshold), shaped_(true), shape_(shape), share_prefix_(share_prefix),
+    options_(torch::TensorOptions().dtype(dtype).layout(torch::kStrided).device(device).requires_grad(false)) {
+    init();
 }
 
 void Attention::init() {
@@ -45,22 +56,36 @@ void Attention::init() {
         ca_dtype_ = CA_DTYPE_F16;
     } else if (st == torch::kFloat32) {
         ca_dtype_ = CA_DTYPE_F32;
+    } else if (st == torch::kBFloat16 && shaped_) {
+        ca_dtype_ = CA_DTYPE_BF16;
     } else {
         throw std::runtime_error(std::string("unsupported dtype ") + c10::toString(st));
     }
     if (!options_.device().has_index())
         options_ = options_.device(torch::Device(torch::kCUDA, c10::cuda::current_device()));
-    chunk_bytes_ = ca_chunk_bytes(n_heads_, d_head_, chunk_size_, ca_dtype_);
+    if (shaped_) {
+        chunk_bytes_ = ca_chunk_bytes_shaped(&shape_, chunk_size_, ca_dtype_);
+        if (chunk_bytes_ <= 0) throw std::runtime_error("n_kv_heads must divide n_heads, head sizes must lie in 1 .. 256");
+        const int per16 = 16 / (ca_dtype_ == CA_DTYPE_F32 ? 4 : 2);
+        k_padded_ = (shape_.d_key + per16 - 1) / per16 * per16;
+        v_padded_ = (shape_.d_value + per16 - 1) / per16 * per16;
+    } else {
+        chunk_bytes_ = ca_chunk_bytes(n_heads_, d_head_, chunk_size_, ca_dtype_);
+        k_padded_ = v_padded_ = d_head_;
+    }
     // same sizing rule as the reference's allocator: as many whole chunks as memory_mb holds
     max_chunks_ = (int64_t)((double)memory_mb_ * 1024.0 * 1024.0 / (double)chunk_bytes_);
     c10::cuda::CUDAGuard guard(options_.device());
     pool_ = torch::empty({std::max<int64_t>(max_chunks_, 1) * chunk_bytes_}, options_.dtype(torch::kUInt8));
     tree_.reset(new PrefixTree(chunk_size_, max_chunks_, chunk_bytes_, share_prefix_));
-    check_rc(ca_context_create(&ctx_, options_.device().index(), n_heads_, d_head_, chunk_size_, ca_dtype_,
-                               pool_.data_ptr(), max_chunks_, tpp_threshold_),
+    check_rc(shaped_ ? ca_context_create_shaped(&ctx_, options_.device().index(), &shape_, chunk_size_, ca_dtype_,
+                                                pool_.data_ptr(), max_chunks_, tpp_threshold_)
+                     : ca_context_create(&ctx_, options_.device().index(), n_heads_, d_head_, chunk_size_, ca_dtype_,
+                                         pool_.data_ptr(), max_chunks_, tpp_threshold_),
              "chunk_attn: context");
     valid_ = false;
     shared_plan_ = std::make_shared<SharedPlan>();
+    shared_tables_ = std::make_shared<SharedTables>();
 }
 
 Attention::SharedPlan::~SharedPlan() {
@@ -104,10 +129,19 @@ torch::Tensor Attention::to_cache(torch::Tensor t) const {
     return t;
 }
 
+void Attention::check_kv(const torch::Tensor& k, const torch::Tensor& v, int64_t n, const char* what) const {
+    const int dv = shaped_ ? shape_.d_value : d_head_;
+    if (k.dim() != 3 || v.dim() != 3 || k.size(0) != n || v.size(0) != n || k.size(1) != kv_heads() || v.size(1) != kv_heads() ||
+        k.size(2) != d_head_ || v.size(2) != dv)
+        throw std::runtime_error(what);
+}
+
+torch::Tensor Attention::pad_heads(torch::Tensor t, int padded) const {
+    return t.size(2) == padded ? t : torch::constant_pad_nd(t, {0, padded - t.size(2)});
+}
+
 int Attention::add_seq(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v) {
-    if (k.dim() != 3 || v.dim() != 3 || k.size(0) != v.size(0) || k.size(1) != n_heads_ || v.size(1) != n_heads_ ||
-        k.size(2) != d_head_ || v.size(2) != d_head_)
-        throw std::runtime_error("add_seq: k and v must be [n_tokens, n_heads, d_head]");
+    check_kv(k, v, k.dim() > 0 ? k.size(0) : 0, "add_seq: k and v must be [n_tokens, n_heads, d_head]");
     // rows past the last token (a right-padded prompt) are ignored, as the reference's slices do
     if (k.size(0) < (int64_t)tokens.size()) throw std::runtime_error("add_seq: one K/V row per token is required");
     std::vector<NewChunk> created;
@@ -116,9 +150,9 @@ int Attention::add_seq(const std::vector<int>& tokens, torch::Tensor k, torch::T
     if (!created.empty()) {
         // the new chunks hold one contiguous token range: a single scatter fills them all.  K/V of
         // the matched prefix are not read (the first sequence that brought a chunk wrote it).
-        k = to_cache(k);
-        v = to_cache(v);
-        if (k.strides() != v.strides()) {
+        k = pad_heads(to_cache(k), k_padded_);
+        v = pad_heads(to_cache(v), v_padded_);
+        if (k.strides() != v.strides() || k_padded_ != v_padded_) {
             k = k.contiguous();
             v = v.contiguous();
         }
@@ -164,16 +198,14 @@ std::shared_ptr<std::future<int>> Attention::add_seq_async(const std::vector<int
 
 int Attention::append_completion(int seq_idx, const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v) {
     const int64_t n = (int64_t)tokens.size();
-    if (k.dim() != 3 || v.dim() != 3 || k.size(0) != n || v.size(0) != n || k.size(1) != n_heads_ || v.size(1) != n_heads_ ||
-        k.size(2) != d_head_ || v.size(2) != d_head_)
-        throw std::runtime_error("append_completion: k and v must be [n_tokens, n_heads, d_head]");
+    check_kv(k, v, n, "append_completion: k and v must be [n_tokens, n_heads, d_head]");
     std::vector<std::pair<Chunk*, Chunk*>> pairs;
     std::vector<std::pair<Chunk*, int>> slots;
     tree_->append_completion(seq_idx, tokens, pairs, slots);
     valid_ = false;
-    k = to_cache(k);
-    v = to_cache(v);
-    if (k.strides() != v.strides()) {
+    k = pad_heads(to_cache(k), k_padded_);
+    v = pad_heads(to_cache(v), v_padded_);
+    if (k.strides() != v.strides() || k_padded_ != v_padded_) {
         k = k.contiguous();
         v = v.contiguous();
     }
@@ -246,13 +278,11 @@ void Attention::refresh_kernel_context(bool force) {
 std::vector<Chunk*> Attention::append_token(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v, bool) {
     if (tree_->tails().size() != tokens.size()) throw std::runtime_error("num of seqs is not equal to num of tokens");
     const int64_t n = (int64_t)tokens.size();
-    if (k.dim() != 3 || v.dim() != 3 || k.size(0) != n || v.size(0) != n || k.size(1) != n_heads_ ||
-        v.size(1) != n_heads_ || k.size(2) != d_head_ || v.size(2) != d_head_)
-        throw std::runtime_error("append_token: k and v must be [n_seqs, n_heads, d_head]");
+    check_kv(k, v, n, "append_token: k and v must be [n_seqs, n_heads, d_head]");
     std::vector<Chunk*> fresh = reserve();
     refresh_kernel_context(false);
-    k = to_cache(k).contiguous();
-    v = to_cache(v).contiguous();
+    k = pad_heads(to_cache(k), k_padded_).contiguous();
+    v = pad_heads(to_cache(v), v_padded_).contiguous();
     c10::cuda::CUDAGuard guard(options_.device());
     check_rc(ca_append_kv(ctx_, k.data_ptr(), v.data_ptr(), (int)n, stream()), "append_token");
     tree_->append_token_ids(tokens);
@@ -328,6 +358,168 @@ void Attention::forward_to_peers(torch::Tensor q, const std::vector<int64_t>& pe
     check_rc(ca_attention_to_peers(ctx_, q.data_ptr(), ptrs.data(), (int)ptrs.size(), reinterpret_cast<void*>(multicast_ptr),
                                    total_heads, head_offset, (int)q.size(0), stream()),
              "forward_to_peers");
+}
+
+std::vector<int> Attention::extend(const std::vector<int>& rows, const std::vector<std::vector<int>>& tokens) {
+    const size_t n = rows.size();
+    if (tokens.size() != n) throw std::runtime_error("extend: one token list per row is required");
+    // everything that can be refused is refused before anything changes
+    std::vector<char> seen(tree_->n_seqs(), 0);
+    int64_t need = 0;
+    for (size_t i = 0; i < n; i++) {
+        if (tokens[i].empty()) throw std::runtime_error("extend: an entry has no tokens");
+        if (rows[i] >= 0) {
+            need += tree_->extend_need(rows[i], (int)tokens[i].size());
+            if (seen[rows[i]]++) throw std::runtime_error("extend: a row is named twice");
+        } else {
+            need += (int64_t)tokens[i].size() / chunk_size_ + 1;
+        }
+    }
+    if (tree_->pool().max_chunks() - tree_->pool().in_use() < need) throw std::runtime_error("ChunkAllocator: capacity reached");
+    valid_ = false;
+    tables_.n_tokens = -1;
+
+    std::vector<int> out(rows);
+    std::vector<std::vector<int32_t>> slot_of(n);
+    std::vector<Chunk*> tail(n);
+    for (size_t i = 0; i < n; i++) {
+        if (rows[i] < 0) continue;
+        std::vector<std::pair<Chunk*, int>> slots;
+        tree_->extend_seq(rows[i], tokens[i], slots);
+        for (const auto& s : slots) slot_of[i].push_back(s.first->id * chunk_size_ + s.second);
+        tail[i] = tree_->tails()[rows[i]];
+    }
+    for (size_t i = 0; i < n; i++) {
+        if (rows[i] >= 0) continue;
+        std::vector<NewChunk> created;
+        out[i] = tree_->add_seq(tokens[i], created);
+        slot_of[i].assign(tokens[i].size(), -1);  // tokens of a matched prefix are in the pool already
+        for (const NewChunk& nc : created)
+            for (int j = 0; j < nc.n_tokens; j++) slot_of[i][nc.token_start + j] = nc.chunk->id * chunk_size_ + j;
+        tail[i] = tree_->tails()[out[i]];
+    }
+
+    // tables: tok_slot | path_off | path_chunks | blocks (16-byte aligned)
+    std::vector<int32_t> data;
+    for (const auto& s : slot_of) data.insert(data.end(), s.begin(), s.end());
+    tables_.path_off = (int64_t)data.size();
+    std::vector<int32_t> off{0}, chunks;
+    for (size_t i = 0; i < n; i++) {
+        const size_t b = chunks.size();
+        for (Chunk* c = tail[i]; c->parent != nullptr; c = c->parent) chunks.push_back(c->id);
+        std::reverse(chunks.begin() + b, chunks.end());
+        off.push_back((int32_t)chunks.size());
+    }
+    data.insert(data.end(), off.begin(), off.end());
+    tables_.path_chunks = (int64_t)data.size();
+    data.insert(data.end(), chunks.begin(), chunks.end());
+    while (data.size() % 4) data.push_back(0);
+    tables_.blocks = (int64_t)data.size();
+    tables_.block_rows = ca_rows_block(&shape_);
+    tables_.n_blocks = 0;
+    int32_t base = 0;
+    for (size_t i = 0; i < n; i++) {
+        const int len = (int)tokens[i].size();
+        // the last blocks of a portion see the most context: they go first
+        for (int b = (len - 1) / tables_.block_rows; b >= 0; b--) {
+            const int lo = b * tables_.block_rows, hi = std::min(len, lo + tables_.block_rows);
+            data.insert(data.end(), {(int32_t)i, base + lo, base + hi, 0});
+            tables_.n_blocks++;
+        }
+        base += len;
+    }
+    c10::cuda::CUDAGuard guard(options_.device());
+    SharedTables& st = *shared_tables_;
+    if (!st.device.defined() || st.data != data) {
+        torch::Tensor host = torch::empty({(int64_t)data.size()}, torch::TensorOptions().dtype(torch::kInt32).pinned_memory(true));
+        std::memcpy(host.data_ptr(), data.data(), data.size() * sizeof(int32_t));
+        st.device = host.to(options_.device(), torch::kInt32, /*non_blocking=*/true);
+        st.data.swap(data);
+    }
+    tables_.device = st.device;
+    tables_.n_tokens = base;
+    return out;
+}
+
+namespace {
+const float* f32_ptr(const c10::optional<torch::Tensor>& t, int64_t n, const char* msg) {
+    if (!t.has_value()) return nullptr;
+    if (!t->is_cuda() || t->scalar_type() != torch::kFloat32 || !t->is_contiguous() || t->numel() != n) throw std::runtime_error(msg);
+    return t->data_ptr<float>();
+}
+const int32_t* i32_ptr(const torch::Tensor& t, int64_t n, const char* msg) {
+    if (!t.is_cuda() || t.scalar_type() != torch::kInt32 || !t.is_contiguous() || t.numel() != n) throw std::runtime_error(msg);
+    return t.data_ptr<int32_t>();
+}
+}  // namespace
+
+torch::Tensor Attention::store_qkv(torch::Tensor qkv, torch::Tensor positions, c10::optional<torch::Tensor> q_norm,
+                                   c10::optional<torch::Tensor> k_norm, double eps, int rot_dims,
+                                   c10::optional<torch::Tensor> key_freq, c10::optional<torch::Tensor> value_freq,
+                                   c10::optional<std::vector<int>> append_tokens) {
+    if (!shaped_) throw std::runtime_error("store_qkv needs a cache with a head shape");
+    const int64_t n = qkv.dim() == 2 ? qkv.size(0) : -1;
+    if (n < 0 || qkv.size(1) < (int64_t)(n_heads_ + kv_heads()) * d_head_ + (int64_t)kv_heads() * shape_.d_value || qkv.stride(1) != 1 ||
+        qkv.device() != options_.device() || qkv.scalar_type() != c10::typeMetaToScalarType(options_.dtype()))
+        throw std::runtime_error("store_qkv: qkv must be [n_tokens, q | k | v heads] with the dtype and device of the cache");
+    ca_qkv_args a{};
+    a.qkv = qkv.data_ptr();
+    a.row_stride = qkv.stride(0);
+    a.q_norm = f32_ptr(q_norm, d_head_, "store_qkv: q_norm must be fp32 [d_key]");
+    a.k_norm = f32_ptr(k_norm, d_head_, "store_qkv: k_norm must be fp32 [d_key]");
+    a.eps = (float)eps;
+    a.rot_dims = rot_dims;
+    a.key_freq = f32_ptr(key_freq, rot_dims / 2, "store_qkv: key_freq must be fp32 [rot_dims / 2]");
+    a.value_freq = f32_ptr(value_freq, shape_.d_value / 2, "store_qkv: value_freq must be fp32 [d_value / 2]");
+    a.positions = i32_ptr(positions, n, "store_qkv: positions must be int32 [n_tokens]");
+    a.n_tokens = (int32_t)n;
+    c10::cuda::CUDAGuard guard(options_.device());
+    torch::Tensor q = torch::empty({n, n_heads_, k_padded_}, options_);
+    a.q_out = q.data_ptr();
+    if (append_tokens.has_value()) {
+        if (tree_->tails().size() != append_tokens->size() || (int64_t)append_tokens->size() != n)
+            throw std::runtime_error("num of seqs is not equal to num of tokens");
+        reserve();
+        refresh_kernel_context(false);
+        check_rc(ca_store_qkv(ctx_, &a, stream()), "store_qkv");
+        tree_->append_token_ids(*append_tokens);
+    } else {
+        if (tables_.n_tokens != n) throw std::runtime_error("store_qkv: extend must have described these tokens");
+        a.tok_slot = tables_.device.data_ptr<int32_t>();
+        check_rc(ca_store_qkv(ctx_, &a, stream()), "store_qkv");
+    }
+    return q;
+}
+
+torch::Tensor Attention::forward_rows(torch::Tensor q, torch::Tensor positions, c10::optional<torch::Tensor> value_freq,
+                                      c10::optional<torch::Tensor> row_entry) {
+    if (!shaped_) throw std::runtime_error("forward_rows needs a cache with a head shape");
+    if (q.dim() != 3 || q.size(1) != n_heads_ || q.size(2) != k_padded_ || !q.is_contiguous() || q.device() != options_.device() ||
+        q.scalar_type() != c10::typeMetaToScalarType(options_.dtype()))
+        throw std::runtime_error("forward_rows: q must be what store_qkv returned");
+    const int64_t n = q.size(0);
+    c10::cuda::CUDAGuard guard(options_.device());
+    torch::Tensor out = torch::empty({n, n_heads_, shape_.d_value}, options_);
+    ca_rows_args a{};
+    a.q = q.data_ptr();
+    a.out = out.data_ptr();
+    a.n_rows = (int32_t)n;
+    a.positions = i32_ptr(positions, n, "forward_rows: positions must be int32 [n_rows]");
+    a.value_freq = f32_ptr(value_freq, shape_.d_value / 2, "forward_rows: value_freq must be fp32 [d_value / 2]");
+    if (row_entry.has_value()) {
+        if (tables_.n_tokens != n) throw std::runtime_error("forward_rows: extend must have described these tokens");
+        const int32_t* t = tables_.device.data_ptr<int32_t>();
+        a.row_entry = i32_ptr(*row_entry, n, "forward_rows: row_entry must be int32 [n_rows]");
+        a.path_off = t + tables_.path_off;
+        a.path_chunks = t + tables_.path_chunks;
+        a.blocks = t + tables_.blocks;
+        a.n_blocks = tables_.n_blocks;
+        a.block_rows = tables_.block_rows;
+    } else {
+        refresh_kernel_context(false);
+    }
+    check_rc(ca_attention_rows(ctx_, &a, stream()), "forward_rows");
+    return out;
 }
 
 void Attention::print(Chunk* root, int level) {

@@ -29,6 +29,10 @@ class Attention {
     Attention(int n_heads, int d_head, int chunk_size, int memory_mb = 2048, bool share_prefix = true,
               int tpp_threshold = 1, torch::Dtype dtype = torch::kFloat16,
               torch::Device device = torch::Device(torch::kCUDA));
+    // heads described by a ca_head_shape (grouped key/value heads, values of another width, a unit term in the
+    // softmax denominator, any scale): the cache of layers driven through extend / store_qkv / forward_rows
+    Attention(const ca_head_shape& shape, int chunk_size, int memory_mb, bool share_prefix, int tpp_threshold,
+              torch::Dtype dtype, torch::Device device);
     // same configuration, fresh empty cache (one per transformer layer in the reference's model)
     Attention(Attention& other);
     ~Attention();
@@ -40,6 +44,20 @@ class Attention {
     // no other method of this object may be called (the tree is not locked).
     std::shared_ptr<std::future<int>> add_seq_async(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v);
     void remove_seq(int seq_idx);
+    // One step of portions, tree side: entry i brings the next tokens of row rows[i] as the rows are now, or of a new
+    // sequence (rows[i] < 0).  Returns the row of each entry (a new one's at the moment it was inserted, existing ones
+    // are handled first).  store_qkv and forward_rows then work on these entries' tokens, laid end to end, until the
+    // next change of the tree.
+    std::vector<int> extend(const std::vector<int>& rows, const std::vector<std::vector<int>>& tokens);
+    // Projections [n_tokens, q heads | k heads | v heads] to attention operands: k and v go into the pool, q is returned
+    // ([n_tokens, n_heads, padded d_key]).  With append_tokens: one token per row, appended to every row as
+    // append_token does.
+    torch::Tensor store_qkv(torch::Tensor qkv, torch::Tensor positions, c10::optional<torch::Tensor> q_norm,
+                            c10::optional<torch::Tensor> k_norm, double eps, int rot_dims, c10::optional<torch::Tensor> key_freq,
+                            c10::optional<torch::Tensor> value_freq, c10::optional<std::vector<int>> append_tokens);
+    // [n_rows, n_heads, d_value]: decode over every row (row_entry not given), or the tokens of the last extend
+    torch::Tensor forward_rows(torch::Tensor q, torch::Tensor positions, c10::optional<torch::Tensor> value_freq,
+                               c10::optional<torch::Tensor> row_entry);
     std::vector<Chunk*> append_token(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v, bool fused = true);
     void refresh_kernel_context(bool force = false);
     std::vector<Chunk*> reserve();
@@ -86,7 +104,14 @@ class Attention {
     void* stream() const;
     torch::Tensor to_cache(torch::Tensor t) const;  // dtype/device of the cache, last dim contiguous
 
+    int kv_heads() const { return shaped_ ? shape_.n_kv_heads : n_heads_; }
+    torch::Tensor pad_heads(torch::Tensor t, int padded) const;  // zeros up to the pool's head size
+    void check_kv(const torch::Tensor& k, const torch::Tensor& v, int64_t n, const char* what) const;
+
     int n_heads_, d_head_, chunk_size_, memory_mb_, tpp_threshold_;
+    bool shaped_ = false;
+    ca_head_shape shape_{};
+    int k_padded_ = 0, v_padded_ = 0;  // head sizes in the pool
     bool share_prefix_;
     torch::TensorOptions options_;
     int ca_dtype_ = 0;
@@ -109,6 +134,18 @@ class Attention {
         ~SharedPlan();
     };
     std::shared_ptr<SharedPlan> shared_plan_;
+
+    // The device tables of the current portions (extend), shared the same way: equal tables are uploaded once.
+    struct SharedTables {
+        std::vector<int32_t> data;
+        torch::Tensor device;
+    };
+    std::shared_ptr<SharedTables> shared_tables_;
+    struct {
+        torch::Tensor device;      // tok_slot | path_off | path_chunks | blocks
+        int64_t n_tokens = -1, path_off = 0, path_chunks = 0, blocks = 0;
+        int n_blocks = 0, block_rows = 1;
+    } tables_;
 
     // add_seq_async: one worker thread, started on first use, runs the queued insertions in order
     void worker_loop();

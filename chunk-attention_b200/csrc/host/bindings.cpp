@@ -15,6 +15,7 @@ using ca_host::PrefixTree;
 
 namespace ca_host {
 void init_ops(py::module& m);
+void init_block_ops(py::module& m, py::module& ops);
 }
 
 namespace {
@@ -73,6 +74,32 @@ PYBIND11_MODULE(chunk_attn_c, m) {
            py::arg("share_prefix") = true, py::arg("tpp_threshold") = 1, py::arg("dtype") = py::none(),
            py::arg("device") = py::none())
       .def(py::init<Attention&>())
+      // a cache whose heads are described by a head shape: grouped key/value heads, values of another width than the
+      // keys, any scale, a unit term in the softmax denominator; fp32, fp16, bf16
+      .def_static("shaped",
+           [](int n_heads, int n_kv_heads, int d_key, int d_value, double scale, bool sink, int chunk_size, int memory_mb,
+              bool share_prefix, int tpp_threshold, py::object dtype, py::object device) {
+               ca_head_shape sh{};
+               sh.n_heads = n_heads;
+               sh.n_kv_heads = n_kv_heads;
+               sh.d_key = d_key;
+               sh.d_value = d_value;
+               sh.sink = sink ? 1 : 0;
+               sh.scale = (float)scale;
+               if (py::isinstance<py::str>(device)) device = py::module_::import("torch").attr("device")(device);
+               return std::make_shared<Attention>(sh, chunk_size, memory_mb, share_prefix, tpp_threshold,
+                                                  torch::python::detail::py_object_to_dtype(dtype),
+                                                  torch::python::detail::py_object_to_device(device));
+           },
+           py::arg("n_heads"), py::arg("n_kv_heads"), py::arg("d_key"), py::arg("d_value"), py::arg("scale"),
+           py::arg("sink") = false, py::arg("chunk_size") = 64, py::arg("memory_mb") = 1024, py::arg("share_prefix") = true,
+           py::arg("tpp_threshold") = 1, py::arg("dtype"), py::arg("device"))
+      .def("extend", &Attention::extend, py::arg("rows"), py::arg("tokens"))
+      .def("store_qkv", &Attention::store_qkv, py::arg("qkv"), py::arg("positions"), py::arg("q_norm") = py::none(),
+           py::arg("k_norm") = py::none(), py::arg("eps") = 0.0, py::arg("rot_dims") = 0, py::arg("key_freq") = py::none(),
+           py::arg("value_freq") = py::none(), py::arg("append_tokens") = py::none())
+      .def("forward_rows", &Attention::forward_rows, py::arg("q"), py::arg("positions"), py::arg("value_freq") = py::none(),
+           py::arg("row_entry") = py::none())
       .def("forward", &Attention::forward, py::arg("q"), py::arg("partition") = 0)
       .def("add_seq", &Attention::add_seq, py::arg("tokens"), py::arg("k"), py::arg("v"))
       .def("add_seq_async", &Attention::add_seq_async, py::arg("tokens"), py::arg("k"), py::arg("v"))
@@ -114,6 +141,7 @@ PYBIND11_MODULE(chunk_attn_c, m) {
     // the reference carries this submodule whenever it is built for CUDA (python_exports.cpp:83-86)
     py::module ops = m.def_submodule("ops");
     ca_host::init_ops(ops);
+    ca_host::init_block_ops(m, ops);
 
     py::class_<PrefixTree>(m, "PrefixTree", py::module_local())
       .def(py::init([](int chunk_size, int64_t max_chunks, bool share_prefix) {
@@ -137,6 +165,15 @@ PYBIND11_MODULE(chunk_attn_c, m) {
            },
            py::arg("tokens"))
       .def("remove_seq", &PrefixTree::remove_seq, py::arg("seq_idx"))
+      .def("extend_seq",
+           [](PrefixTree& t, int seq_idx, const std::vector<int>& tokens) {
+               std::vector<std::pair<Chunk*, int>> slots;
+               t.extend_seq(seq_idx, tokens, slots);
+               std::vector<std::pair<int, int>> out;  // (chunk id, row) of every token
+               for (auto& x : slots) out.emplace_back(x.first->id, x.second);
+               return out;
+           },
+           py::arg("seq_idx"), py::arg("tokens"))
       .def("reserve", &PrefixTree::reserve, py::return_value_policy::reference)
       .def("append_token",
            [](PrefixTree& t, const std::vector<int>& tokens) {

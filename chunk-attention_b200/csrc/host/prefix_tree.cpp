@@ -82,6 +82,33 @@ void PrefixTree::remove_seq(int seq_idx) {
     tails_.erase(tails_.begin() + seq_idx);
 }
 
+int PrefixTree::extend_need(int seq_idx, int n_tokens) const {
+    if (seq_idx < 0 || seq_idx >= (int)tails_.size()) throw std::runtime_error("seq_idx out of range");
+    if (n_tokens <= 0) return 0;
+    const int room = chunk_size_ - tails_[seq_idx]->n_tokens();
+    // the last chunk is never left full: (n - room) / chunk_size full ones and one more below them
+    return n_tokens < room ? 0 : (n_tokens - room) / chunk_size_ + 1;
+}
+
+void PrefixTree::extend_seq(int seq_idx, const std::vector<int>& tokens, std::vector<std::pair<Chunk*, int>>& slots) {
+    slots.clear();
+    const int total = (int)tokens.size();
+    const int need = extend_need(seq_idx, total);
+    if (total == 0) return;
+    if (pool_.max_chunks() - pool_.in_use() < need) throw std::runtime_error("ChunkAllocator: capacity reached");
+    slots.reserve(total);
+    Chunk* tail = tails_[seq_idx];
+    for (int i = 0; i < total;) {
+        if (tail->full()) tail = tail->add_child(pool_.allocate());
+        const int n = std::min(total - i, chunk_size_ - tail->n_tokens());
+        for (int j = 0; j < n; j++) slots.emplace_back(tail, tail->n_tokens() + j);
+        tail->append_tokens(tokens, i, i + n);
+        i += n;
+    }
+    if (tail->full()) tail = tail->add_child(pool_.allocate());
+    tails_[seq_idx] = tail;
+}
+
 std::vector<Chunk*> PrefixTree::reserve() {
     std::vector<Chunk*> fresh;
     int need = 0;

@@ -28,6 +28,12 @@ class PrefixTree {
     // listed).
     int add_seq(const std::vector<int>& tokens, std::vector<NewChunk>& created);
     void remove_seq(int seq_idx);
+    // Continue row `seq_idx` with more tokens (the next portion of its prompt): they fill its tail and new chunks
+    // below it, and a chunk that ends up full gets an empty successor, as after add_seq.  `slots` receives, per
+    // token, the (chunk, row in chunk) its K/V must be written to.  Nothing is changed when the pool cannot hold it.
+    void extend_seq(int seq_idx, const std::vector<int>& tokens, std::vector<std::pair<Chunk*, int>>& slots);
+    // chunks a call of extend_seq would allocate
+    int extend_need(int seq_idx, int n_tokens) const;
     // Give every full tail an empty child; returns the new chunks.
     std::vector<Chunk*> reserve();
     // Record one new token id per sequence in its tail (the K/V rows are written on the device).

@@ -38,6 +38,7 @@ extern "C" {
 /* element types of q/k/v/out and of the chunk pool */
 #define CA_DTYPE_F16 0
 #define CA_DTYPE_F32 1
+#define CA_DTYPE_BF16 2 /* contexts with a head shape (ca_context_create_shaped) and the block kernels */
 
 /* `partition` of ca_attention, the reference's meaning (cpp/chunk_attn/attention.h:46):
  * 0 auto, 1 chunk-first then sequence-first, 2 sequence-first only. */
@@ -86,6 +87,24 @@ CA_API int64_t ca_tile_elem_offset(int d_head, int chunk_size, int dtype, int to
 CA_API int ca_context_create(ca_context** out, int device, int n_heads, int d_head, int chunk_size,
                              int dtype, void* pool, int64_t max_chunks, int tpp_threshold);
 CA_API void ca_context_destroy(ca_context* ctx);
+
+/* A context whose heads are not one K/V head per query head of one width.  Query head h reads key/value head
+ * h / (n_heads / n_kv_heads); the pool has one tile pair per KEY/VALUE head.  d_key and d_value are padded with zeros to
+ * whole 16-byte granules in the pool and in q ([rows, n_heads, padded d_key]); outputs are not padded.
+ * score = (q . k) * scale; with `sink` the softmax denominator has one added (a score of 0 without a value).
+ * fp32, fp16 and bf16.  Served by ca_store_qkv, ca_attention_rows and the pool functions; the counterpart of the
+ * fixed-geometry calls for models with grouped heads. */
+typedef struct ca_head_shape {
+    int32_t n_heads;     /* query heads                                   */
+    int32_t n_kv_heads;  /* divides n_heads                               */
+    int32_t d_key;       /* <= 256                                        */
+    int32_t d_value;     /* <= 256                                        */
+    int32_t sink;        /* 1: unit term in the softmax denominator       */
+    float scale;
+} ca_head_shape;
+CA_API int64_t ca_chunk_bytes_shaped(const ca_head_shape* shape, int chunk_size, int dtype);
+CA_API int ca_context_create_shaped(ca_context** out, int device, const ca_head_shape* shape, int chunk_size, int dtype,
+                                    void* pool, int64_t max_chunks, int tpp_threshold);
 
 /* 0: one launch walks shared runs and private tails together (default);
  * 1: the chunk-first items and the sequence-first items are launched as two kernels. */
@@ -288,6 +307,101 @@ CA_API int ca_rotary_embedding(const int64_t* positions, void* query, void* key,
                                int rot_dim, int64_t query_stride, int64_t key_stride, int num_heads,
                                int num_kv_heads, int head_size, int64_t num_tokens, int is_neox, int dtype,
                                int64_t max_position, int32_t* status, ca_stream stream);
+
+/* ---- batches of spans: portions of sequences, and the block kernels that work on them ---------------------
+ * A step runs the next tokens of several sequences ("spans"), laid end to end: span e holds tokens
+ * [cu[e], cu[e + 1]) of the batch, the first of which is at position start[e] of its sequence, and keeps its recurrent
+ * states in row slot[e] of the state arrays.  A state is taken as zero when start[e] is 0.  Device pointers, except the
+ * counts.  The pieces cut every span into runs of at most work_len tokens, in order. */
+typedef struct ca_spans {
+    int32_t n_entries;
+    int32_t n_tokens;
+    int32_t max_tokens;       /* longest span                                                        */
+    int32_t n_work;           /* pieces                                                              */
+    int32_t work_len;         /* tokens of a full piece                                              */
+    const int32_t* cu;        /* [n_entries + 1]                                                     */
+    const int32_t* start;     /* [n_entries]                                                         */
+    const int32_t* slot;      /* [n_entries]                                                         */
+    const int32_t* entry_of;  /* [n_tokens]                                                          */
+    const int32_t* work;      /* [n_work][4]: span, first token, end token, number within the span   */
+    const int32_t* work_off;  /* [n_entries + 1]: first piece of each span                           */
+} ca_spans;
+
+/* Operands of attention from a batch's projections, for a context with a head shape: per-head RMS norm of q and k
+ * (q_norm, k_norm: fp32 [d_key], may be NULL), rotation of the first rot_dims elements of q and k in interleaved pairs
+ * by position * key_freq[i] (NULL: none), rotation of v over all pairs by position * value_freq[i] (NULL: none), q to
+ * q_out, k and v into the pool.  qkv: [n_tokens, row_stride] of the context's type, q heads | k heads | v heads.
+ * tok_slot (device, [n_tokens]): pool row chunk * chunk_size + row of each token, -1 for a token that is not written;
+ * NULL: one token per row of the current work list goes to that row's tail, as ca_append_kv does, and is counted. */
+typedef struct ca_qkv_args {
+    const void* qkv;
+    int64_t row_stride;
+    void* q_out;
+    const float* q_norm;
+    const float* k_norm;
+    float eps;
+    int32_t rot_dims;
+    const float* key_freq;
+    const float* value_freq;
+    const int32_t* positions;
+    const int32_t* tok_slot;
+    int32_t n_tokens;
+} ca_qkv_args;
+CA_API int ca_store_qkv(ca_context* ctx, const ca_qkv_args* args, ca_stream stream);
+
+/* Attention of a context with a head shape.
+ * Decode (path_off NULL): one row per row of the current work list, each over all of its context.
+ * Portions: row r belongs to span row_entry[r], walks the pool chunks path_chunks[path_off[e] ..] of that span and sees
+ * the tokens up to its own position.  blocks (n_blocks of {span, first row, end row, 0}) cut the rows of every span into
+ * runs of at most block_rows.
+ * value_freq != NULL: values were stored rotated by their positions; output rows are turned back by theirs. */
+typedef struct ca_rows_args {
+    const void* q;              /* [n_rows, n_heads, padded d_key]  */
+    void* out;                  /* [n_rows, n_heads, d_value]       */
+    int32_t n_rows;
+    const int32_t* positions;   /* [n_rows]                         */
+    const float* value_freq;
+    const int32_t* row_entry;   /* [n_rows]                         */
+    const int32_t* path_off;    /* [n_entries + 1]                  */
+    const int32_t* path_chunks;
+    const int32_t* blocks;
+    int32_t n_blocks;
+    int32_t block_rows;
+} ca_rows_args;
+/* rows of a block the kernels want (ca_rows_args.block_rows) */
+CA_API int ca_rows_block(const ca_head_shape* shape);
+CA_API int ca_attention_rows(ca_context* ctx, const ca_rows_args* args, ca_stream stream);
+
+/* Block kernels (fp32 residual stream x, activations of `dtype`).  Vectors of weights are fp32.
+ * ca_token_shift: plain = x, shifted = x + (previous token's x - x) * mu; state [slots, width].
+ * ca_gated_norm_add: g = r * sigmoid(gate + bias); x += g / sqrt(mean(g^2) + eps) * weight; plain (optional) = x.  With
+ *   next_mu (one token per span only) also the token shift of the result.
+ * ca_norm_rows: out[i] = row rows[i] (NULL: i) of x, RMS-normed, times weight, times sigmoid(gate[i]) if given.
+ * ca_gelu_tanh: the tanh form.
+ * ca_conv_silu: depthwise causal convolution with bias (taps [channels, n_taps], last tap = current token), then
+ *   SiLU; state [slots, n_taps - 1, channels], oldest first.
+ * ca_selective_scan: dt = softplus(dt + dt_bias); S[c, n] = exp(dt A) S + dt x B_n; y = (S . C + D x) * silu(z);
+ *   bc row: B then C; state [slots, channels, n_states]; scratch of ca_scan_scratch_floats() floats.
+ * ca_decay_attention: q, k, v = silu of the heads of qkv; S = decay_h S + k v^T, out = S^T q; state
+ *   [slots, heads, d_key, d_value]. */
+CA_API int ca_token_shift(const float* x, const float* mu, float* state, void* plain, void* shifted, const ca_spans* spans,
+                          int width, int dtype, ca_stream stream);
+CA_API int ca_gated_norm_add(float* x, const void* r, int64_t r_stride, const void* gate, int64_t gate_stride,
+                             const float* bias, const float* weight, float eps, void* plain, const float* next_mu,
+                             float* next_state, void* next_shifted, const ca_spans* spans, int64_t n_tokens, int width,
+                             int dtype, ca_stream stream);
+CA_API int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const int32_t* rows, const float* weight,
+                        const void* gate, int64_t gate_stride, float eps, int64_t n_rows, int width, int dtype,
+                        ca_stream stream);
+CA_API int ca_gelu_tanh(void* out, const void* in, int64_t in_stride, int64_t n_rows, int width, int dtype, ca_stream stream);
+CA_API int ca_conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, const float* bias, float* state,
+                        const ca_spans* spans, int channels, int n_taps, int dtype, ca_stream stream);
+CA_API int64_t ca_scan_scratch_floats(const ca_spans* spans, int channels, int n_states);
+CA_API int ca_selective_scan(void* y, const void* x, const void* z, int64_t z_stride, const float* dt, const float* dt_bias,
+                             const float* A, const float* bc, int64_t bc_stride, const float* D, float* state, float* scratch,
+                             const ca_spans* spans, int channels, int n_states, int dtype, ca_stream stream);
+CA_API int ca_decay_attention(void* out, const void* qkv, int64_t row_stride, const float* decay, float* state,
+                              const ca_spans* spans, int n_heads, int d_key, int d_value, int dtype, ca_stream stream);
 
 /* ---- allocation-free decode step ---------------------------------------------------------------
  * No counterpart in the reference: this entry point exists for callers that cannot allocate device
