@@ -92,6 +92,7 @@ struct ca_context {
     int64_t max_chunks = 0;
     int tpp_threshold = 1;
     bool fast = false;
+    bool items = false;           // work lists hold items (fast contexts and 16-bit head shapes), else per-row paths
     bool shaped = false;          // made by ca_context_create_shaped: `shape` describes the heads
     ca_head_shape shape{};
     int group = 1;                // query heads per key/value head
@@ -101,6 +102,7 @@ struct ca_context {
     bool opt_sf_tensor = true;
     int opt_pdl = 3;
     int opt_wide = 1;
+    int opt_span_tensor = 1;      // CA_OPT_SPAN_TENSOR
     bool opt_overlap = false;
     cudaStream_t side_stream = nullptr;   // the short-tails kernel runs here beside the wide-runs kernel
     cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
@@ -204,11 +206,13 @@ static int make_context(ca_context** out, int device, const ca_head_shape* shape
         c->shaped = true;
         c->shape = *shape;
         c->group = shape->n_heads / shape->n_kv_heads;
+        c->items = dtype == CA_DTYPE_BF16;
     }
     c->pool = pool;
     c->max_chunks = max_chunks;
     c->tpp_threshold = tpp_threshold < 1 ? 1 : tpp_threshold;
     c->fast = (!shape && dtype == CA_DTYPE_F16 && geo.d_head == ca::FAST_D && geo.chunk_size == ca::FAST_C);
+    c->items = c->items || c->fast;
     c->num_sms = prop.multiProcessorCount;
     cudaError_t e = cudaEventCreateWithFlags(&c->upload_done, cudaEventDisableTiming);
     if (e == cudaSuccess) e = cudaEventCreateWithFlags(&c->paths_done, cudaEventDisableTiming);
@@ -319,6 +323,10 @@ int ca_context_set_option(ca_context* c, int option, int64_t value) {
         if (value != 0 && value != 1) return fail(CA_ERR_INVALID, "CA_OPT_FINISH_IN_TAILS takes 0 or 1");
         c->opt_finish_in_tails = (int)value;
         return CA_OK;
+    } else if (option == CA_OPT_SPAN_TENSOR) {
+        if (value < 0 || value > 2) return fail(CA_ERR_INVALID, "CA_OPT_SPAN_TENSOR takes 0, 1 or 2");
+        c->opt_span_tensor = (int)value;
+        return CA_OK;
     } else if (option == CA_OPT_TRACE) {
         DeviceGuard guard(c->device);
         if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
@@ -341,6 +349,18 @@ int ca_context_set_option(ca_context* c, int option, int64_t value) {
 
 static int upload_plan(ca_context* c, const ca::Plan& pl, cudaStream_t stream);
 
+static std::string plan_for(const ca_context* c, ca::Plan& plan, const ca_chunk_info* infos, int n_infos, int n_seqs, int n_ctas) {
+    if (!c->shaped)
+        return ca::build_plan(plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold, n_ctas,
+                              c->max_chunks, c->opt_split, c->geo.d_head, c->geo.esize, c->fast, c->opt_sf_tensor, c->opt_wide,
+                              /*want_paths=*/!c->fast);
+    // items of up to 64 query rows (a sequence brings `group` of them), one partial per row; no kernel of their own for
+    // short tails or wide runs
+    return ca::build_plan(plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold, n_ctas, c->max_chunks,
+                          false, (c->geo.d_head + c->geo.d_value) / 2, c->geo.esize, c->items, /*seq_first_tensor=*/false,
+                          /*wide_mode=*/0, /*want_paths=*/!c->items, 64 / c->group, /*one_partial_per_row=*/true);
+}
+
 int ca_refresh_kernel_context(ca_context* c, const ca_chunk_info* infos, int n_infos, int n_seqs, ca_stream stream_) {
     if (!c) return fail(CA_ERR_INVALID, "context is null");
     cudaStream_t stream = static_cast<cudaStream_t>(stream_);
@@ -348,9 +368,7 @@ int ca_refresh_kernel_context(ca_context* c, const ca_chunk_info* infos, int n_i
     if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
     c->valid = false;
     const int n_ctas = c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * ca::FAST_CTAS_PER_SM;
-    std::string err = ca::build_plan(c->plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size,
-                                     c->tpp_threshold, n_ctas, c->max_chunks, c->opt_split, c->geo.d_head,
-                                     c->geo.esize, c->fast, c->opt_sf_tensor, c->opt_wide, /*want_paths=*/!c->fast);
+    std::string err = plan_for(c, c->plan, infos, n_infos, n_seqs, n_ctas);
     if (!err.empty()) return fail(CA_ERR_INVALID, "work list rejected: " + err);
     return upload_plan(c, c->plan, stream);
 }
@@ -361,16 +379,14 @@ int ca_plan_build_for_context(const ca_context* c, ca_plan** out, const ca_chunk
     if (!p) p = new (std::nothrow) ca_plan();
     if (!p) return fail(CA_ERR_INVALID, "out of host memory");
     const int n_ctas = c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * ca::FAST_CTAS_PER_SM;
-    std::string err = ca::build_plan(p->plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold,
-                                     n_ctas, c->max_chunks, c->opt_split, c->geo.d_head, c->geo.esize, c->fast,
-                                     c->opt_sf_tensor, c->opt_wide, /*want_paths=*/!c->fast);
+    std::string err = plan_for(c, p->plan, infos, n_infos, n_seqs, n_ctas);
     if (!err.empty()) {
         if (!*out) delete p;  // a caller-owned plan is left to the caller (its contents are unspecified now)
         return fail(CA_ERR_INVALID, "work list rejected: " + err);
     }
     p->max_chunks = c->max_chunks;
     p->wide_mode = c->opt_wide;
-    p->fast = c->fast;
+    p->fast = c->items;
     p->d_head = c->geo.d_head;
     p->esize = c->geo.esize;
     *out = p;
@@ -382,8 +398,8 @@ int ca_refresh_from_plan(ca_context* c, const ca_plan* plan, ca_stream stream_) 
     const ca::Plan& pl = plan->plan;
     const int n_ctas = c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * ca::FAST_CTAS_PER_SM;
     if (pl.n_heads != c->geo.n_heads || pl.chunk_size != c->geo.chunk_size || plan->d_head != c->geo.d_head ||
-        plan->esize != c->geo.esize || plan->fast != c->fast || plan->max_chunks > c->max_chunks ||
-        pl.split_phases != c->opt_split || pl.tpp_threshold != c->tpp_threshold || (c->fast && pl.n_ctas > n_ctas) ||
+        plan->esize != c->geo.esize || plan->fast != c->items || plan->max_chunks > c->max_chunks ||
+        pl.split_phases != c->opt_split || pl.tpp_threshold != c->tpp_threshold || (c->items && pl.n_ctas > n_ctas) ||
         plan->wide_mode != c->opt_wide)
         return fail(CA_ERR_INVALID, "the plan was built for a different geometry, pool size or set of options");
     DeviceGuard guard(c->device);
@@ -455,7 +471,8 @@ static int upload_plan(ca_context* c, const ca::Plan& pl, cudaStream_t stream) {
     }
 
     // partial-result scratch, grow-only
-    const size_t slots = (size_t)pl.stats.n_slots;
+    const size_t slots = (size_t)pl.stats.n_slots * c->group;
+    const size_t part_width = c->shaped ? (size_t)c->geo.d_value : (size_t)ca::FAST_D;
     if (slots > c->part_cap) {
         if (c->part_o) CA_CUDA(cudaFree(c->part_o));
         if (c->part_ml) CA_CUDA(cudaFree(c->part_ml));
@@ -463,7 +480,7 @@ static int upload_plan(ca_context* c, const ca::Plan& pl, cudaStream_t stream) {
         c->part_ml = nullptr;
         c->part_cap = 0;
         const size_t cap = slots * 3 / 2 + 64;
-        CA_CUDA(cudaMalloc(reinterpret_cast<void**>(&c->part_o), cap * ca::FAST_D * sizeof(float)));
+        CA_CUDA(cudaMalloc(reinterpret_cast<void**>(&c->part_o), cap * part_width * sizeof(float)));
         CA_CUDA(cudaMalloc(reinterpret_cast<void**>(&c->part_ml), cap * sizeof(float2)));
         c->part_cap = cap;
     }
@@ -940,6 +957,62 @@ int ca_attention_rows(ca_context* c, const ca_rows_args* a, ca_stream stream_) {
     DeviceGuard guard(c->device);
     if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
     cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+    if (c->dtype == CA_DTYPE_BF16) {
+        ca::RowsParams r{};
+        r.pool = c->pool;
+        r.geo = c->geo;
+        r.group = c->group;
+        r.q = a->q;
+        r.out = a->out;
+        r.out_width = c->shape.d_value;
+        r.n_rows = a->n_rows;
+        r.scale_log2 = c->shape.scale * 1.4426950408889634f;
+        r.sink = c->shape.sink;
+        r.positions = a->positions;
+        r.value_freq = a->value_freq;
+        if (decode) {
+            r.items = c->d_items;
+            r.n_items = c->meta.n_items;
+            r.delta_tokens = c->delta_tokens;
+            r.part_o = c->part_o;
+            r.part_ml = c->part_ml;
+            r.part_width = c->geo.d_value;
+            r.merge_off = c->d_merge_off;
+            r.merge_slots = c->d_merge_slots;
+            r.subs = c->group <= 64 ? 1 : (c->group + 63) / 64;
+        } else {
+            r.blocks = a->blocks;
+            r.n_blocks = a->n_blocks;
+            r.path_off = a->path_off;
+            r.path_chunks = a->path_chunks;
+            r.subs = (a->block_rows * c->group + 63) / 64;
+        }
+        if (!decode && c->opt_span_tensor && a->n_rows >= 32 && r.scale_log2 != 0.f &&
+            ca::span_attn_serves(c->geo, c->shape.d_value, a->block_rows * c->group)) {
+            ca::SpanAttnParams t{};
+            t.pool = c->pool;
+            t.n_kv_heads = c->geo.n_heads;
+            t.group = c->group;
+            t.q = a->q;
+            t.out = a->out;
+            t.scale_log2 = r.scale_log2;
+            t.sink = r.sink;
+            t.split_weights = c->opt_span_tensor == 1;
+            t.positions = a->positions;
+            t.value_freq = a->value_freq;
+            t.blocks = a->blocks;
+            t.n_blocks = a->n_blocks;
+            t.path_off = a->path_off;
+            t.path_chunks = a->path_chunks;
+            t.max_chunks = (int)c->max_chunks;
+            t.status = c->status;
+            t.wait_limit = c->opt_wait_limit;
+            CA_CUDA(ca::launch_span_attn(t, c->geo.d_head, c->geo.d_value, stream));
+            return CA_OK;
+        }
+        CA_CUDA(ca::launch_attn_rows(r, stream));
+        return CA_OK;
+    }
     if (decode) {
         const int rc = ensure_paths(c, stream);
         if (rc != CA_OK) return rc;

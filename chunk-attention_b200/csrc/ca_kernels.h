@@ -150,6 +150,59 @@ struct GenericParams {
 };
 cudaError_t launch_attn_seq_generic(const GenericParams& p, int dtype, cudaStream_t stream);
 
+// ---- grouped heads on tensor cores (ca_attn_rows.cu) -------------------------------------------------------
+struct RowsParams {
+    const void* pool;
+    Geometry geo;
+    int group;                   // query heads per key/value head
+    const void* q;               // bf16 [rows, n_heads * group, geo.d_head]
+    void* out;                   // bf16 [rows, n_heads * group, out_width]
+    int out_width;
+    int n_rows;
+    float scale_log2;            // scale * log2(e)
+    int sink;
+    const int32_t* positions;    // [n_rows]
+    const float* value_freq;     // null: values are not rotated
+    int subs;                    // 64-row sub-blocks of a block
+    // portions
+    const int32_t* blocks;       // [n_blocks][4]: span, first token, end token, 0; null: decode
+    int n_blocks;
+    const int32_t* path_off;
+    const int32_t* path_chunks;
+    // decode: the planner's items
+    const int4* items;
+    int n_items;
+    int delta_tokens;
+    float* part_o;               // [slots][part_width]
+    float2* part_ml;             // [slots]
+    int part_width;
+    const int32_t* merge_off;
+    const int32_t* merge_slots;
+};
+cudaError_t launch_attn_rows(const RowsParams& p, cudaStream_t stream);
+
+// ---- portions of prompts on tcgen05 (ca_attn_span.cu) -------------------------------------------------------
+struct SpanAttnParams {
+    const void* pool;
+    int n_kv_heads, group;
+    const void* q;               // bf16 [rows, n_kv_heads * group, d_key]
+    void* out;                   // bf16 [rows, n_kv_heads * group, d_value]
+    float scale_log2;
+    int sink;
+    int split_weights;           // 1: softmax weights enter the second product as two bf16 numbers
+    const int32_t* positions;
+    const float* value_freq;
+    const int32_t* blocks;       // [n_blocks][4]: span, first token, end token, 0
+    int n_blocks;
+    const int32_t* path_off;
+    const int32_t* path_chunks;
+    int max_chunks;
+    int* status;
+    long long wait_limit;
+};
+bool span_attn_serves(const Geometry& g, int d_value, int block_query_rows);
+cudaError_t launch_span_attn(const SpanAttnParams& p, int d_key, int d_value, cudaStream_t stream);
+
 // ---- projections to attention operands (ca_qkv.cu) ------------------------------------------------------
 struct QkvParams {
     void* pool;

@@ -87,7 +87,8 @@ void build_paths(Plan& plan) {
 std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int n_seqs, int n_heads,
                        int chunk_size, int tpp_threshold, int n_ctas, int64_t max_chunks,
                        bool split_phases, int d_head, int esize, bool fast_path, bool seq_first_tensor, int wide_mode,
-                       bool want_paths) {
+                       bool want_paths, int rows_per_item, bool one_partial_per_row) {
+    if (rows_per_item < 1) rows_per_item = 1;
     // the vectors keep their capacity from one rebuild to the next
     plan.items.clear();
     plan.wide_chunks.clear();
@@ -210,13 +211,13 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
         Run& r = runs[ri];
         if (run_wide[ri]) continue;
         const int n = r.e - r.b;
-        const int n_blocks = (n + MAX_ROWS_PER_ITEM - 1) / MAX_ROWS_PER_ITEM;
+        const int n_blocks = (n + rows_per_item - 1) / rows_per_item;
         const int rows_per_block = (n + n_blocks - 1) / n_blocks;
         for (int blk = 0; blk < n_blocks; blk++) {
             const int rb = r.b + blk * rows_per_block;
             const int rows = std::min(rows_per_block, r.e - rb);
             if (rows <= 0) continue;
-            const int splits = rows <= 16 ? 4 : (rows <= 32 ? 2 : 1);
+            const int splits = one_partial_per_row ? 1 : rows <= 16 ? 4 : (rows <= 32 ? 2 : 1);
             units.push_back(Unit{r.chunks.data(), (int32_t)r.chunks.size(), rb, rows, splits, chunk_size, false});
         }
     }

@@ -87,7 +87,9 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
                        int chunk_size, int tpp_threshold, int n_ctas, int64_t max_chunks,
                        bool split_phases, int d_head, int esize, bool fast_path, bool seq_first_tensor,
                        int wide_mode = 1,   // 0: never route runs to the tcgen05 kernel, 1: by cost, 2: every shared run
-                       bool want_paths = true);  // also build the per-row path lists of the any-geometry kernel
+                       bool want_paths = true,   // also build the per-row path lists of the any-geometry kernel
+                       int rows_per_item = MAX_ROWS_PER_ITEM,
+                       bool one_partial_per_row = false);  // items of shared runs do not emit a partial per token split
 // The per-row path lists (path_off / path_chunks / path_tokens) from plan.infos, for a plan built without them.
 void build_paths(Plan& plan);
 

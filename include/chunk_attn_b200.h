@@ -141,6 +141,9 @@ CA_API int ca_context_create_shaped(ca_context** out, int device, const ca_head_
  * stores the output rows itself: no merge launch, and the tails' partials never travel through memory.
  * 0: the tails are written as partial rows and the merge kernel combines them. */
 #define CA_OPT_FINISH_IN_TAILS 10
+/* Contexts with a head shape, portions of prompts in bf16 with 64-token chunks and heads of 64 or 128 elements: 1 (default)
+ * the tcgen05 kernel, softmax weights as two bf16 numbers; 2 the same with one bf16 number; 0 the mma.sync kernel. */
+#define CA_OPT_SPAN_TENSOR 11
 /* Failure-path tests only: the CTA that draws item `value` of the next launches stops feeding its consumer
  * warps, whose bounded wait then runs out (status 1).  -1 (default) switches it off. */
 #define CA_OPT_TEST_WITHHOLD_ITEM 8
