@@ -306,7 +306,7 @@ class GagoraxForCausalLM:
         for s, t in zip(slots, tokens):
             state.length[s] += len(t)
         step = Step(spans, attention, state, [t[0] for t in tokens] if decode else None, self.config.torch_dtype)
-        x = self.embed.index_select(0, spans.tokens).float()
+        x = ops.embed_rows(self.embed, spans)
         plain = shifted = None
         for i, layer in enumerate(self.layers):
             plain, shifted = layer(x, plain, shifted, step, self.layers[i + 1] if i + 1 < len(self.layers) else None)

@@ -970,6 +970,9 @@ int ca_attention_rows(ca_context* c, const ca_rows_args* a, ca_stream stream_) {
         r.sink = c->shape.sink;
         r.positions = a->positions;
         r.value_freq = a->value_freq;
+        r.max_chunks = (int)c->max_chunks;
+        r.status = c->status;
+        r.wait_limit = c->opt_wait_limit;
         if (decode) {
             r.items = c->d_items;
             r.n_items = c->meta.n_items;

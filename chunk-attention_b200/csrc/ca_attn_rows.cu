@@ -123,7 +123,9 @@ __device__ __forceinline__ void warp_tile(uint32_t k_tile, uint32_t v_tile, int 
     }
 }
 
-template <int DK, int DV, int STAGES, bool SPAN>
+// BULK: chunks of 64 tokens whose tiles are exactly DK and DV wide are staged verbatim (the pool's layout is the staged one)
+// by 1-D TMA bulk copies of one thread.
+template <int DK, int DV, int STAGES, bool SPAN, bool BULK>
 __global__ void __launch_bounds__(R_THREADS) rows_mma_kernel(const RowsParams p) {
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int K_BYTES = R_TILE * DK * 2, STAGE_BYTES = R_TILE * (DK + DV) * 2;
@@ -167,14 +169,39 @@ __global__ void __launch_bounds__(R_THREADS) rows_mma_kernel(const RowsParams p)
     // ---- staging
     const int gpr = p.geo.gpr, v_gpr = p.geo.v_gpr;
     const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(p.pool);
+    const int n_tiles = (n_ctx + R_TILE - 1) / R_TILE;
+    const uint32_t bars = sbase + STAGES * STAGE_BYTES;  // BULK: one barrier per stage
+    if (BULK) {
+        if (tid == 0) {
+            for (int i = 0; i < STAGES; i++) mbar_init(bars + 8 * i, 1);
+            asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        }
+        __syncthreads();
+    }
+    auto copy_tile = [&](int j) {  // one thread
+        const uint32_t dst = sbase + (j % STAGES) * STAGE_BYTES, bar = bars + 8 * (j % STAGES);
+        int chunk = __ldg(list + j);
+        if (chunk < 0 || chunk >= p.max_chunks) {
+            atomicCAS(p.status, STATUS_OK, STATUS_BAD_WORK_LIST);
+            chunk = 0;
+        }
+        const uint8_t* src = static_cast<const uint8_t*>(p.pool) + ((size_t)chunk * G + kvh) * (size_t)STAGE_BYTES;
+        const uint32_t lines = min(R_TILE, n_ctx - j * R_TILE);
+        mbar_arrive_expect_tx(bar, lines * (DK + DV) * 2);
+        if (lines == R_TILE) {
+            bulk_copy_g2s(dst, src, STAGE_BYTES, bar);
+        } else {
+#pragma unroll
+            for (int pn = 0; pn < (DK + DV) / 64; pn++) bulk_copy_g2s(dst + pn * (R_TILE * 128), src + pn * (R_TILE * 128), lines * 128, bar);
+        }
+    };
     // granules past the stored head size are zero in every stage
-    for (int i = tid; i < STAGES * R_TILE * (DK + DV) / 8; i += R_THREADS) {
+    if (!BULK) for (int i = tid; i < STAGES * R_TILE * (DK + DV) / 8; i += R_THREADS) {
         const int st = i / (R_TILE * (DK + DV) / 8), q = i % (R_TILE * (DK + DV) / 8);
         const bool is_k = q < R_TILE * DK / 8;
         const int qq = is_k ? q : q - R_TILE * DK / 8, t = qq % R_TILE, g = qq / R_TILE;
         if (g >= (is_k ? gpr : v_gpr)) sts128_zero(sbase + st * STAGE_BYTES + (is_k ? 0 : K_BYTES) + staged(t, g));
     }
-    const int n_tiles = (n_ctx + R_TILE - 1) / R_TILE;
     const int g_sub = tid & 7;
     auto load_tile = [&](int j) {
         const uint32_t dst = sbase + (j % STAGES) * STAGE_BYTES;
@@ -205,8 +232,12 @@ __global__ void __launch_bounds__(R_THREADS) rows_mma_kernel(const RowsParams p)
     };
 #pragma unroll
     for (int j = 0; j < STAGES - 1; j++) {
-        if (j < n_tiles) load_tile(j);
-        cp_async_commit();
+        if (BULK) {
+            if (tid == 0 && j < n_tiles) copy_tile(j);
+        } else {
+            if (j < n_tiles) load_tile(j);
+            cp_async_commit();
+        }
     }
 
     // ---- queries, straight into fragments
@@ -235,10 +266,33 @@ __global__ void __launch_bounds__(R_THREADS) rows_mma_kernel(const RowsParams p)
         for (int k = 0; k < 4; k++) o[i][k] = 0.f;
 
     for (int j = 0; j < n_tiles; j++) {
-        cp_async_wait<STAGES - 2>();
-        __syncthreads();
-        if (j + STAGES - 1 < n_tiles) load_tile(j + STAGES - 1);
-        cp_async_commit();
+        if (BULK) {
+            bool ok = mbar_wait_bounded(bars + 8 * (j % STAGES), (j / STAGES) & 1, p.wait_limit);
+            const int lines = n_ctx - j * R_TILE;
+            if (lines < R_TILE) {
+                // the rows of V behind the stored ones meet weights of zero and only have to be finite
+                const uint32_t v = sbase + (j % STAGES) * STAGE_BYTES + K_BYTES;
+                for (int i = tid; i < (DV / 64) * (R_TILE - lines) * 8; i += R_THREADS) {
+                    const int pn = i / ((R_TILE - lines) * 8), q = i % ((R_TILE - lines) * 8);
+                    sts128_zero(v + pn * (R_TILE * 128) + lines * 128 + q * 16);
+                }
+            }
+            if (!__syncthreads_and(ok)) {
+                // record it, wait (again with the limit) for the copies in flight, and leave the rows unwritten
+                if (tid == 0) {
+                    atomicCAS(p.status, STATUS_OK, STATUS_FULL_WAIT_TIMEOUT);
+                    for (int f = j; f < min(n_tiles, j + STAGES - 1); f++)
+                        mbar_wait_bounded(bars + 8 * (f % STAGES), (f / STAGES) & 1, p.wait_limit);
+                }
+                return;
+            }
+            if (tid == 0 && j + STAGES - 1 < n_tiles) copy_tile(j + STAGES - 1);
+        } else {
+            cp_async_wait<STAGES - 2>();
+            __syncthreads();
+            if (j + STAGES - 1 < n_tiles) load_tile(j + STAGES - 1);
+            cp_async_commit();
+        }
         const uint32_t kt = sbase + (j % STAGES) * STAGE_BYTES, vt = kt + K_BYTES;
         if (!busy) continue;
         if (splits == 4) warp_tile<DK, DV, 1>(kt, vt, my_s * 16, j * R_TILE, qf, limit, p.scale_log2, m, l, o, lane);
@@ -376,12 +430,12 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
     }
 }
 
-template <int DK, int DV, int STAGES>
+template <int DK, int DV, int STAGES, bool BULK>
 cudaError_t launch(const RowsParams& p, cudaStream_t stream) {
-    constexpr int ring = STAGES * R_TILE * (DK + DV) * 2, out = 4 * 16 * (DV + 4) * 4 + 64 * 8;
+    constexpr int ring = STAGES * R_TILE * (DK + DV) * 2 + (BULK ? STAGES * 8 : 0), out = 4 * 16 * (DV + 4) * 4 + 64 * 8;
     constexpr int smem = ring > out ? ring : out;
-    auto* span = rows_mma_kernel<DK, DV, STAGES, true>;
-    auto* items = rows_mma_kernel<DK, DV, STAGES, false>;
+    auto* span = rows_mma_kernel<DK, DV, STAGES, true, BULK>;
+    auto* items = rows_mma_kernel<DK, DV, STAGES, false, BULK>;
     auto* k = p.blocks ? span : items;
     cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return e;
@@ -403,14 +457,20 @@ cudaError_t launch(const RowsParams& p, cudaStream_t stream) {
 cudaError_t launch_attn_rows(const RowsParams& p, cudaStream_t stream) {
     const int dk = p.geo.d_head, dv = p.geo.d_value;
     if (dk > 256 || dv > 256) return cudaErrorInvalidValue;
-    if (dk <= 64) {
-        if (dv <= 64) return launch<64, 64, 4>(p, stream);
-        if (dv <= 128) return launch<64, 128, 3>(p, stream);
-    } else if (dk <= 128) {
-        if (dv <= 64) return launch<128, 64, 3>(p, stream);
-        if (dv <= 128) return launch<128, 128, 3>(p, stream);
+    if (p.geo.chunk_size == R_TILE) {  // tiles as the staged layout has them
+        if (dk == 64 && dv == 64) return launch<64, 64, 4, true>(p, stream);
+        if (dk == 64 && dv == 128) return launch<64, 128, 4, true>(p, stream);
+        if (dk == 128 && dv == 64) return launch<128, 64, 4, true>(p, stream);
+        if (dk == 128 && dv == 128) return launch<128, 128, 3, true>(p, stream);
     }
-    return launch<256, 256, 2>(p, stream);
+    if (dk <= 64) {
+        if (dv <= 64) return launch<64, 64, 4, false>(p, stream);
+        if (dv <= 128) return launch<64, 128, 3, false>(p, stream);
+    } else if (dk <= 128) {
+        if (dv <= 64) return launch<128, 64, 3, false>(p, stream);
+        if (dv <= 128) return launch<128, 128, 3, false>(p, stream);
+    }
+    return launch<256, 256, 2, false>(p, stream);
 }
 
 }  // namespace ca

@@ -72,7 +72,7 @@ __global__ void gated_norm_add_kernel(float* __restrict__ x, const T* __restrict
                                       T* __restrict__ plain, const float* __restrict__ next_mu, float* __restrict__ next_state,
                                       T* __restrict__ shifted, const ca_spans sp, int width) {
     const size_t t = blockIdx.x;
-    float g[STEPS][V];
+    float g[STEPS][V], xs[STEPS][V];
     float ss = 0.f;
     auto gated = [&](int c, float (&out)[V]) {
         float a[V], z[V], b[V];
@@ -87,6 +87,7 @@ __global__ void gated_norm_add_kernel(float* __restrict__ x, const T* __restrict
     for (int s = 0; s < STEPS; s++) {
         const int c = threadIdx.x * V + s * stride;
         if (c < width) {
+            load_f<float, V>(x + t * width + c, xs[s]);  // requested before the reduction
             gated(c, g[s]);
 #pragma unroll
             for (int i = 0; i < V; i++) ss = fmaf(g[s][i], g[s][i], ss);
@@ -99,9 +100,8 @@ __global__ void gated_norm_add_kernel(float* __restrict__ x, const T* __restrict
         for (int i = 0; i < V; i++) ss = fmaf(a[i], a[i], ss);
     }
     const float inv = 1.f / sqrtf(block_sum(ss) / width + eps);
-    auto finish = [&](int c, const float (&a)[V]) {
-        float h[V], ww[V];
-        load_f<float, V>(x + t * width + c, h);
+    auto finish = [&](int c, const float (&a)[V], float (&h)[V]) {
+        float ww[V];
         load_f<float, V>(w + c, ww);
 #pragma unroll
         for (int i = 0; i < V; i++) h[i] += a[i] * inv * ww[i];
@@ -126,12 +126,13 @@ __global__ void gated_norm_add_kernel(float* __restrict__ x, const T* __restrict
 #pragma unroll
     for (int s = 0; s < STEPS; s++) {
         const int c = threadIdx.x * V + s * stride;
-        if (c < width) finish(c, g[s]);
+        if (c < width) finish(c, g[s], xs[s]);
     }
     for (int c = threadIdx.x * V + STEPS * stride; c < width; c += stride) {
-        float a[V];
+        float a[V], h[V];
+        load_f<float, V>(x + t * width + c, h);
         gated(c, a);
-        finish(c, a);
+        finish(c, a, h);
     }
 }
 
@@ -142,32 +143,62 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const TI* __restrict__ x, 
                                  const float* __restrict__ w, const T* __restrict__ gate, int64_t gate_stride, float eps, int width) {
     const size_t t = blockIdx.x;
     const TI* src = x + (size_t)(rows ? rows[t] : t) * x_stride;
+    constexpr int STEPS = V == 1 ? 4 : 2;  // of the row a thread keeps in registers, gate included
+    float kept[STEPS][V], z[STEPS][V];
     float ss = 0.f;
-    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+    const int stride = blockDim.x * V;
+#pragma unroll
+    for (int s = 0; s < STEPS; s++) {
+        const int c = threadIdx.x * V + s * stride;
+        if (c < width) {
+            load_f<TI, V>(src + c, kept[s]);
+            if (gate) load_f<T, V>(gate + t * gate_stride + c, z[s]);
+#pragma unroll
+            for (int i = 0; i < V; i++) ss = fmaf(kept[s][i], kept[s][i], ss);
+        }
+    }
+    for (int c = threadIdx.x * V + STEPS * stride; c < width; c += stride) {
         float a[V];
         load_f<TI, V>(src + c, a);
 #pragma unroll
         for (int i = 0; i < V; i++) ss = fmaf(a[i], a[i], ss);
     }
     const float inv = 1.f / sqrtf(block_sum(ss) / width + eps);
-    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
-        float a[V], ww[V];
-        load_f<TI, V>(src + c, a);
+    auto finish = [&](int c, float (&a)[V], const float (&zz)[V]) {
+        float ww[V];
         load_f<float, V>(w + c, ww);
-        if (gate) {
-            float z[V];
-            load_f<T, V>(gate + t * gate_stride + c, z);
 #pragma unroll
-            for (int i = 0; i < V; i++) ww[i] *= sigmoid_f(z[i]);
-        }
-#pragma unroll
-        for (int i = 0; i < V; i++) a[i] *= inv * ww[i];
+        for (int i = 0; i < V; i++) a[i] *= inv * ww[i] * (gate ? sigmoid_f(zz[i]) : 1.f);
         store_f<T, V>(out + t * width + c, a);
+    };
+#pragma unroll
+    for (int s = 0; s < STEPS; s++) {
+        const int c = threadIdx.x * V + s * stride;
+        if (c < width) finish(c, kept[s], z[s]);
+    }
+    for (int c = threadIdx.x * V + STEPS * stride; c < width; c += stride) {
+        float a[V], zz[V];
+        load_f<TI, V>(src + c, a);
+        if (gate) load_f<T, V>(gate + t * gate_stride + c, zz);
+        finish(c, a, zz);
+    }
+}
+
+// x[t] = table[ids[t]] in fp32: the start of the residual stream
+template <typename T, int V>
+__global__ void embed_rows_kernel(float* __restrict__ x, const T* __restrict__ table, const int32_t* __restrict__ ids, int width) {
+    const T* src = table + (size_t)ids[blockIdx.x] * width;
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+        float a[V];
+        load_f<T, V>(src + c, a);
+        store_f<float, V>(x + (size_t)blockIdx.x * width + c, a);
     }
 }
 
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-    return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    // (1 + tanh u) / 2 = 1 / (1 + exp(-2u)); one exponential and one division
+    const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return __fdividef(z, 1.f + exp2f(-2.885390081777927f * u));
 }
 
 template <typename T, int V>
@@ -250,7 +281,7 @@ int ca_gated_norm_add(float* x, const void* r, int64_t r_stride, const void* gat
     return by_type(dtype, vec, [&](auto tv, auto vv) {
         using T = decltype(tv);
         constexpr int V = decltype(vv)::value;
-        gated_norm_add_kernel<T, V, 4><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
+        gated_norm_add_kernel<T, V, V == 1 ? 4 : 2><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
             x, static_cast<const T*>(r), r_stride, static_cast<const T*>(gate), gate_stride, bias, weight, eps, static_cast<T*>(plain),
             next_mu, next_state, static_cast<T*>(next_shifted), spans, width);
     });
@@ -273,6 +304,19 @@ int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const
         else
             norm_rows_kernel<T, T, V><<<(unsigned)n_rows, threads, 0, static_cast<cudaStream_t>(stream)>>>(
                 static_cast<T*>(out), static_cast<const T*>(x), x_stride, rows, weight, static_cast<const T*>(gate), gate_stride, eps, width);
+    });
+}
+
+int ca_embed_rows(float* x, const void* table, const int32_t* ids, int64_t n_tokens, int width, int dtype, ca_stream stream) {
+    if (n_tokens < 0 || width <= 0) return fail("embed_rows: bad shape");
+    if (n_tokens == 0) return CA_OK;
+    if (!x || !table || !ids) return fail("embed_rows: null pointer");
+    const bool vec = width % 4 == 0 && aligned16(x) && aligned16(table);
+    return by_type(dtype, vec, [&](auto tv, auto vv) {
+        using T = decltype(tv);
+        constexpr int V = decltype(vv)::value;
+        embed_rows_kernel<T, V><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
+            x, static_cast<const T*>(table), ids, width);
     });
 }
 

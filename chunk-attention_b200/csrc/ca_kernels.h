@@ -5,6 +5,7 @@
 
 #include <string>
 
+#include "../../include/chunk_attn_b200.h"
 #include "ca_layout.h"
 
 namespace ca {
@@ -178,6 +179,9 @@ struct RowsParams {
     int part_width;
     const int32_t* merge_off;
     const int32_t* merge_slots;
+    int max_chunks;
+    int* status;
+    long long wait_limit;
 };
 cudaError_t launch_attn_rows(const RowsParams& p, cudaStream_t stream);
 
@@ -202,6 +206,21 @@ struct SpanAttnParams {
 };
 bool span_attn_serves(const Geometry& g, int d_value, int block_query_rows);
 cudaError_t launch_span_attn(const SpanAttnParams& p, int d_key, int d_value, cudaStream_t stream);
+
+// ---- linear attention with decay on tensor cores (ca_decay_mma.cu) -------------------------------------------
+struct DecayMmaParams {
+    void* out;                   // bf16 [T, H * dv]
+    const void* qkv;             // bf16, row t: q heads | k heads | v heads, before SiLU
+    int64_t row_stride;
+    const float* decay;          // [H]
+    float* state;                // [slots, H, dk, dv]
+    float* piece_state;          // [pieces, H, dk, dv] (run > 0)
+    int H, dk, dv;
+    int run;                     // pieces per CTA; 0: a CTA takes a whole span
+    ca_spans sp;
+};
+bool decay_mma_serves(int dk, int dv, int64_t row_stride, const void* qkv, int work_len);
+cudaError_t launch_decay_mma(const DecayMmaParams& p, cudaStream_t stream);
 
 // ---- projections to attention operands (ca_qkv.cu) ------------------------------------------------------
 struct QkvParams {

@@ -4,9 +4,11 @@
 // s of the batch into the next free row of sequence s's tail chunk; a portion of a prompt names the pool row of
 // every token, and tokens whose chunk an earlier sequence already filled are not written.
 //
-// One CTA per token: its angles go to shared memory once, then a warp takes a head at a time, 2 elements (one
-// rotation pair) per lane and step.  All arithmetic in fp32, one rounding at the store.  Heads are padded with zeros
+// One CTA per token: its angles go to shared memory once; then a group of lanes takes a head at a time, one 16-byte granule
+// per lane (heads whose size or alignment does not allow that: a warp per head, one rotation pair per lane and step).  All arithmetic in fp32, one rounding at the store.  Heads are padded with zeros
 // to whole 16-byte granules in the pool and in q, so that the attention kernels read granules for every head size.
+#include <algorithm>
+
 #include "ca_kernels.h"
 #include "ca_types.cuh"
 
@@ -99,14 +101,115 @@ __global__ void __launch_bounds__(QKV_WARPS * 32) store_qkv_kernel(const QkvPara
     }
 }
 
+// Heads of whole granules, up to `lanes` of them (a power of two, at most 32).
+constexpr int QKV_VEC_THREADS = 256;
+template <typename T>
+__global__ void __launch_bounds__(QKV_VEC_THREADS) store_qkv_vec_kernel(const QkvParams p, int lanes) {
+    constexpr int EPG = 16 / sizeof(T), PPG = EPG / 2;
+    __shared__ float2 turn_k[QKV_MAX_D / 2], turn_v[QKV_MAX_D / 2];  // (cos, sin) of every pair
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const float pos = (float)p.positions[t];
+    const int kp = p.key_freq ? p.rot_dims / 2 : 0, vp = p.value_freq ? p.d_value / 2 : 0;
+    int chunk, slot;
+    if (p.tok_slot) {
+        const int s = p.tok_slot[t];
+        chunk = s < 0 ? -1 : s / p.geo.chunk_size;
+        slot = s - chunk * p.geo.chunk_size;
+    } else {
+        chunk = p.tail_chunk[t];
+        slot = p.tail_tokens[t] + p.delta_tokens;
+        if (slot >= p.geo.chunk_size) chunk = -1;  // rejected on the host; never write past the tile
+    }
+    const int G = p.geo.n_heads, H = G * p.group, units = H + 2 * G;
+    const int g = tid & (lanes - 1), per_pass = QKV_VEC_THREADS / lanes;
+    const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.row_stride;
+    T* pool = reinterpret_cast<T*>(p.pool);
+    const Geometry v_side = tile_side(p.geo, 1);
+    Pack<T, EPG> in;
+    auto source = [&](int u) { return row + (u < H + G ? u * p.d_key : (H + G) * p.d_key + (u - H - G) * p.d_value) + g * EPG; };
+    auto size_of = [&](int u) { return u < H + G ? p.d_key : p.d_value; };
+    int u = tid / lanes;
+    if (u < units && g * EPG < size_of(u)) in = *reinterpret_cast<const Pack<T, EPG>*>(source(u));
+    for (int i = tid; i < kp + vp; i += QKV_VEC_THREADS) {
+        float sn, cs;
+        sincosf(pos * (i < kp ? p.key_freq[i] : p.value_freq[i - kp]), &sn, &cs);
+        (i < kp ? turn_k[i] : turn_v[i - kp]) = make_float2(cs, sn);
+    }
+    __syncthreads();
+    for (int u0 = 0; u0 < units; u0 += per_pass, u += per_pass) {
+        const bool on = u < units && g * EPG < size_of(min(u, units - 1));
+        const int kind = u < H ? 0 : (u < H + G ? 1 : 2);  // q, k, v
+        float x[EPG];
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < EPG; i++) {
+            x[i] = on ? to_f32(in.v[i]) : 0.f;
+            ss = fmaf(x[i], x[i], ss);
+        }
+        // the next head's granule is requested before this one is worked on
+        if (u + per_pass < units && g * EPG < size_of(u + per_pass)) in = *reinterpret_cast<const Pack<T, EPG>*>(source(u + per_pass));
+        for (int off = lanes >> 1; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+        if (!on || (kind > 0 && chunk < 0)) continue;
+        const float* w = kind == 0 ? p.q_norm : (kind == 1 ? p.k_norm : nullptr);
+        if (w) {
+            const float inv = 1.f / sqrtf(ss / p.d_key + p.eps);
+#pragma unroll
+            for (int i = 0; i < EPG; i += 4) {
+                const float4 ww = *reinterpret_cast<const float4*>(w + g * EPG + i);
+                x[i] *= inv * ww.x;
+                x[i + 1] *= inv * ww.y;
+                x[i + 2] *= inv * ww.z;
+                x[i + 3] *= inv * ww.w;
+            }
+        }
+        const float2* turn = (kind == 2 ? turn_v : turn_k) + g * PPG;
+        const int pairs = (kind == 2 ? vp : kp) - g * PPG;
+#pragma unroll
+        for (int i = 0; i < PPG; i++)
+            if (i < pairs) {
+                const float2 cs = turn[i];
+                const float a = x[2 * i], b = x[2 * i + 1];
+                x[2 * i] = a * cs.x - b * cs.y;
+                x[2 * i + 1] = b * cs.x + a * cs.y;
+            }
+        Pack<T, EPG> o;
+#pragma unroll
+        for (int i = 0; i < EPG; i++) o.v[i] = from_f32<T>(x[i]);
+        Pack<T, EPG>* dst;
+        if (kind == 0) {
+            dst = reinterpret_cast<Pack<T, EPG>*>(reinterpret_cast<T*>(p.q_out) + ((size_t)t * H + u) * p.geo.d_head) + g;
+        } else {
+            const int h = u - (kind == 1 ? H : H + G);
+            dst = reinterpret_cast<Pack<T, EPG>*>(pool + tile_base_elems(p.geo, chunk, h, kind - 1)) +
+                  tile_granule_index(kind == 2 ? v_side : p.geo, slot, g);
+        }
+        *dst = o;
+    }
+}
+
+template <typename T>
+void run_store_qkv(const QkvParams& p, cudaStream_t stream) {
+    constexpr int EPG = 16 / sizeof(T);
+    auto aligned = [](const void* q) { return reinterpret_cast<uintptr_t>(q) % 16 == 0; };
+    const int granules = std::max(p.d_key, p.d_value) / EPG;
+    if (p.d_key % EPG == 0 && p.d_value % EPG == 0 && p.row_stride % EPG == 0 && aligned(p.qkv) && aligned(p.q_norm) && aligned(p.k_norm) &&
+        granules <= 32) {
+        int lanes = 1;
+        while (lanes < granules) lanes *= 2;
+        store_qkv_vec_kernel<T><<<p.n_tokens, QKV_VEC_THREADS, 0, stream>>>(p, lanes);
+    } else {
+        store_qkv_kernel<T><<<p.n_tokens, QKV_WARPS * 32, 0, stream>>>(p);
+    }
+}
+
 }  // namespace
 
 cudaError_t launch_store_qkv(const QkvParams& p, int dtype, cudaStream_t stream) {
     if (p.n_tokens <= 0) return cudaSuccess;
     if (p.geo.d_head > QKV_MAX_D || p.geo.d_value > QKV_MAX_D || p.geo.epg < 2) return cudaErrorInvalidValue;
-    if (dtype == 2) store_qkv_kernel<__nv_bfloat16><<<p.n_tokens, QKV_WARPS * 32, 0, stream>>>(p);
-    else if (dtype == 1) store_qkv_kernel<float><<<p.n_tokens, QKV_WARPS * 32, 0, stream>>>(p);
-    else store_qkv_kernel<__half><<<p.n_tokens, QKV_WARPS * 32, 0, stream>>>(p);
+    if (dtype == 2) run_store_qkv<__nv_bfloat16>(p, stream);
+    else if (dtype == 1) run_store_qkv<float>(p, stream);
+    else run_store_qkv<__half>(p, stream);
     return cudaGetLastError();
 }
 

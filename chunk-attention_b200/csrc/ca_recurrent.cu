@@ -6,6 +6,7 @@
 // The work of a step is listed as PIECES of at most `work_len` tokens of one span (ca_spans).  A step whose spans are
 // all single pieces runs a recurrence in one launch; otherwise the scan takes three: local end state of every piece
 // from zero, a sweep over the pieces of each sequence that turns them into initial states, and the outputs.
+#include <algorithm>
 #include <type_traits>
 
 #include "../../include/chunk_attn_b200.h"
@@ -79,21 +80,29 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(T* __restrict__ out, con
 #pragma unroll
                 for (int v = 0; v < V; v++) st[(size_t)(j - (KMAX - K)) * channels + v] = keep[j][v];
     }
-    for (int t = t0; t < t1; t++) {
-        const Pack<T, V> a = *reinterpret_cast<const Pack<T, V>*>(x + (size_t)t * x_stride + c);
-        Pack<T, V> o;
+    constexpr int GROUP = 4;  // tokens requested together
+    for (int tg = t0; tg < t1; tg += GROUP) {
+        Pack<T, V> in[GROUP];
 #pragma unroll
-        for (int v = 0; v < V; v++) {
-            const float xv = to_f32(a.v[v]);
-            float acc = fmaf(xv, tap[KMAX - 1][v], b[v]);
+        for (int k = 0; k < GROUP; k++) in[k] = *reinterpret_cast<const Pack<T, V>*>(x + (size_t)min(tg + k, t1 - 1) * x_stride + c);
 #pragma unroll
-            for (int j = 0; j < KMAX - 1; j++) acc = fmaf(hist[j][v], tap[j][v], acc);
+        for (int k = 0; k < GROUP; k++) {
+            if (tg + k < t1) {
+                Pack<T, V> o;
 #pragma unroll
-            for (int j = 0; j < KMAX - 2; j++) hist[j][v] = hist[j + 1][v];
-            if (KMAX > 1) hist[KMAX > 1 ? KMAX - 2 : 0][v] = xv;
-            o.v[v] = from_f32<T>(silu_f(acc));
+                for (int v = 0; v < V; v++) {
+                    const float xv = to_f32(in[k].v[v]);
+                    float acc = fmaf(xv, tap[KMAX - 1][v], b[v]);
+#pragma unroll
+                    for (int j = 0; j < KMAX - 1; j++) acc = fmaf(hist[j][v], tap[j][v], acc);
+#pragma unroll
+                    for (int j = 0; j < KMAX - 2; j++) hist[j][v] = hist[j + 1][v];
+                    if (KMAX > 1) hist[KMAX > 1 ? KMAX - 2 : 0][v] = xv;
+                    o.v[v] = from_f32<T>(silu_f(acc));
+                }
+                *reinterpret_cast<Pack<T, V>*>(out + (size_t)(tg + k) * channels + c) = o;
+            }
         }
-        *reinterpret_cast<Pack<T, V>*>(out + (size_t)t * channels + c) = o;
     }
 }
 
@@ -112,7 +121,8 @@ struct ScanParams {
     float* state;            // [slots, C, N]
     float* piece_state;      // [pieces, C, N]
     float* piece_dt;         // [pieces, C]: sum of dt over the piece
-    int C, N, lane_shift;    // 1 << lane_shift lanes share a channel, NS states each
+    int C, N;
+    int run;                 // pieces a CTA takes (0: whole spans)
     ca_spans sp;
 };
 constexpr int SCAN_THREADS = 128;
@@ -120,91 +130,154 @@ constexpr int SCAN_TOKENS = 16;  // tokens whose B and C are staged at a time
 constexpr int SCAN_GROUP = 8;    // tokens whose x, dt, z are requested together
 
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// 2^x for x <= 0: one MUFU operation; results below 2^-126 are 0
+__device__ __forceinline__ float decay_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
-// PHASE 0: the span is one piece: state in, outputs, state out.  1: end state of the piece from zero, and sum of dt.
-// 2: outputs from the piece's initial state.
-template <typename T, int NS, int PHASE>
+// L lanes share a channel, NS states each.  Of a group of tokens, lane i of a channel reads the inputs of tokens i, i + L,
+// ... and evaluates their step size and, at the end, their output; dt and dt x travel by shuffles.
+// PHASE 0: whole spans: state in, outputs, state out (spans in turn per CTA column).  1: end state of the run from zero, and
+// sum of dt.  2: outputs from the run's initial state.
+template <typename T, int L, int NS, int PHASE>
 __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) {
-    extern __shared__ float bc_s[];  // [SCAN_TOKENS][2 N]
-    const int4 wk = reinterpret_cast<const int4*>(p.sp.work)[blockIdx.y];
-    const int e = wk.x, t0 = wk.y, t1 = wk.z;
-    const int L = 1 << p.lane_shift;
-    const int c = blockIdx.x * (SCAN_THREADS >> p.lane_shift) + (threadIdx.x >> p.lane_shift);
-    const int n0 = (threadIdx.x & (L - 1)) * NS, N = p.N, N2 = 2 * N;
+    extern __shared__ __align__(16) float bc_s[];  // [SCAN_TOKENS][B: L * NS | C: L * NS], zero past N
+    constexpr int NP = L * NS, OWN = (SCAN_GROUP + L - 1) / L;
+    const int c = blockIdx.x * (SCAN_THREADS / L) + threadIdx.x / L;
+    const int ln = threadIdx.x & (L - 1), base = (threadIdx.x & 31) & ~(L - 1), n0 = ln * NS, N = p.N;
     const bool on = c < p.C;
     const int cc = on ? c : p.C - 1;
-    float S[NS], A2[NS];
-    float* slot = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N;
-    float* piece = p.piece_state + ((size_t)blockIdx.y * p.C + cc) * N;
-    const bool live = p.sp.start[e] > 0;
+    float A2[NS];
 #pragma unroll
-    for (int i = 0; i < NS; i++) {
-        const int n = n0 + i;
-        A2[i] = n < N ? p.A[(size_t)cc * N + n] * LOG2E : 0.f;
-        S[i] = 0.f;
-        if (n < N) {
-            if (PHASE == 0 && live) S[i] = slot[n];
-            if (PHASE == 2) S[i] = piece[n];
-        }
-    }
+    for (int i = 0; i < NS; i++) A2[i] = n0 + i < N ? p.A[(size_t)cc * N + n0 + i] * LOG2E : 0.f;
     const float bias = p.dt_bias[cc], D = PHASE == 1 ? 0.f : p.D[cc];
     const T* X = static_cast<const T*>(p.x) + cc;
     const T* Z = static_cast<const T*>(p.z) + cc;
     T* Y = static_cast<T*>(p.y) + cc;
     const float* DT = p.dt + cc;
-    float sum_dt = 0.f;
-    for (int tb = t0; tb < t1; tb += SCAN_TOKENS) {
-        const int nt = min(SCAN_TOKENS, t1 - tb);
-        __syncthreads();
-        for (int i = threadIdx.x; i < nt * N2; i += SCAN_THREADS) {
-            const int tt = i / N2;
-            bc_s[i] = p.bc[(size_t)(tb + tt) * p.bc_stride + (i - tt * N2)];
+    for (int unit = blockIdx.y; unit < (PHASE == 0 ? p.sp.n_entries : p.sp.n_work); unit += gridDim.y) {
+        int e = unit, t0, t1;
+        if (PHASE == 0) {
+            t0 = p.sp.cu[e];
+            t1 = p.sp.cu[e + 1];
+        } else {
+            const int4 wk = reinterpret_cast<const int4*>(p.sp.work)[unit];
+            if (wk.w % p.run) continue;  // a run starts at every run-th piece
+            e = wk.x;
+            t0 = wk.y;
+            t1 = min(p.sp.cu[e + 1], t0 + p.run * p.sp.work_len);
         }
-        __syncthreads();
-        for (int g = 0; g < nt; g += SCAN_GROUP) {
-            float xs[SCAN_GROUP], ds[SCAN_GROUP], zs[SCAN_GROUP];
+        float S[NS];
+        float* slot = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N + n0;
+        float* piece = PHASE == 0 ? nullptr : p.piece_state + ((size_t)unit * p.C + cc) * N + n0;
+        const bool live = p.sp.start[e] > 0;
+        const bool vec = NS == 4 && N % 4 == 0;
+        const float* from = PHASE == 0 ? slot : piece;
 #pragma unroll
-            for (int k = 0; k < SCAN_GROUP; k++) {
-                const size_t t = (size_t)min(tb + g + k, t1 - 1);
-                xs[k] = to_f32(X[t * p.C]);
-                ds[k] = DT[t * p.C];
-                if (PHASE != 1) zs[k] = to_f32(Z[t * p.z_stride]);
+        for (int i = 0; i < NS; i++) S[i] = 0.f;
+        if (PHASE == 2 || (PHASE == 0 && live)) {
+            if (vec) {
+                if (n0 < N) {
+                    const float4 v = *reinterpret_cast<const float4*>(from);
+                    S[0] = v.x; S[1 % NS] = v.y; S[2 % NS] = v.z; S[3 % NS] = v.w;
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < NS; i++)
+                    if (n0 + i < N) S[i] = from[i];
             }
+        }
+        float sum_dt = 0.f;
+        for (int tb = t0; tb < t1; tb += SCAN_TOKENS) {
+            const int nt = min(SCAN_TOKENS, t1 - tb);
+            __syncthreads();
+            for (int i = threadIdx.x; i < nt * 2 * NP; i += SCAN_THREADS) {
+                const int tt = i / (2 * NP), r = i - tt * 2 * NP, n = r < NP ? r : r - NP;
+                bc_s[i] = n < N ? p.bc[(size_t)(tb + tt) * p.bc_stride + n + (r < NP ? 0 : N)] : 0.f;
+            }
+            __syncthreads();
+            for (int g = 0; g < nt; g += SCAN_GROUP) {
+                float xs[OWN], ds[OWN], zs[OWN], ys[OWN];
 #pragma unroll
-            for (int k = 0; k < SCAN_GROUP; k++) {
-                if (g + k < nt) {
-                    const float dt = softplus_f(ds[k] + bias);
-                    const float u = dt * xs[k];
-                    const float* B = bc_s + (g + k) * N2 + n0;
-                    float y = 0.f;
+                for (int k = 0; k < OWN; k++) {
+                    const int tk = ln + k * L;
+                    const size_t t = (size_t)min(tb + g + tk, t1 - 1);
+                    if (tk < SCAN_GROUP) {
+                        xs[k] = to_f32(X[t * p.C]);
+                        ds[k] = DT[t * p.C];
+                        if (PHASE != 1) zs[k] = to_f32(Z[t * p.z_stride]);
+                    } else {
+                        xs[k] = ds[k] = zs[k] = 0.f;
+                    }
+                }
+                float us[OWN];
 #pragma unroll
-                    for (int i = 0; i < NS; i++) {
-                        if (NS * L == N || n0 + i < N) {
-                            S[i] = fmaf(exp2f(dt * A2[i]), S[i], u * B[i]);
-                            if (PHASE != 1) y = fmaf(S[i], B[N + i], y);
+                for (int k = 0; k < OWN; k++) {
+                    ds[k] = softplus_f(ds[k] + bias);
+                    us[k] = ds[k] * xs[k];
+                    ys[k] = 0.f;
+                }
+#pragma unroll
+                for (int k = 0; k < SCAN_GROUP; k++) {
+                    if (g + k < nt) {
+                        const int own = k % L;
+                        float dt = ds[k / L], u = us[k / L];
+                        if (L > 1) {
+                            dt = __shfl_sync(0xffffffffu, dt, base + own);
+                            u = __shfl_sync(0xffffffffu, u, base + own);
+                        }
+                        const float* B = bc_s + (g + k) * 2 * NP + n0;
+                        float bv[NS], cv[NS];
+                        if (NS % 4 == 0) {
+#pragma unroll
+                            for (int i = 0; i < NS; i += 4) {
+                                const float4 b4 = *reinterpret_cast<const float4*>(B + i), c4 = *reinterpret_cast<const float4*>(B + NP + i);
+                                bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
+                                cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
+                            }
+                        }
+                        float y = 0.f;
+#pragma unroll
+                        for (int i = 0; i < NS; i++) {
+                            S[i] = fmaf(decay_exp2(dt * A2[i]), S[i], u * bv[i]);
+                            if (PHASE != 1) y = fmaf(S[i], cv[i], y);
+                        }
+                        if (PHASE == 1) {
+                            sum_dt += dt;
+                        } else {
+#pragma unroll
+                            for (int off = L >> 1; off >= 1; off >>= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
+                            if (own == ln) ys[k / L] = y;
                         }
                     }
-                    if (PHASE == 1) {
-                        sum_dt += dt;
-                    } else {
-                        for (int off = L >> 1; off >= 1; off >>= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
-                        if (on && n0 == 0) Y[(size_t)(tb + g + k) * p.C] = from_f32<T>(fmaf(D, xs[k], y) * silu_f(zs[k]));
+                }
+                if (PHASE != 1) {
+#pragma unroll
+                    for (int k = 0; k < OWN; k++) {
+                        const int tk = ln + k * L;
+                        if (on && tk < SCAN_GROUP && g + tk < nt)
+                            Y[(size_t)(tb + g + tk) * p.C] = from_f32<T>(fmaf(D, xs[k], ys[k]) * silu_f(zs[k]));
                     }
                 }
             }
         }
-    }
-    if (!on) return;
-    float* dst = PHASE == 0 ? slot : piece;
-    if (PHASE != 2) {
+        if (PHASE != 2 && on) {
+            float* dst = PHASE == 0 ? slot : piece;
+            if (vec) {
+                if (n0 < N) *reinterpret_cast<float4*>(dst) = make_float4(S[0], S[1 % NS], S[2 % NS], S[3 % NS]);
+            } else {
 #pragma unroll
-        for (int i = 0; i < NS; i++)
-            if (n0 + i < N) dst[n0 + i] = S[i];
-        if (PHASE == 1 && n0 == 0) p.piece_dt[(size_t)blockIdx.y * p.C + c] = sum_dt;
+                for (int i = 0; i < NS; i++)
+                    if (n0 + i < N) dst[i] = S[i];
+            }
+            if (PHASE == 1 && ln == 0) p.piece_dt[(size_t)unit * p.C + c] = sum_dt;
+        }
     }
 }
 
-// per (span, channel, state): end states of the pieces -> initial states, and the span's end state to its slot
+// per (span, channel, state): end states of the runs -> initial states, and the span's end state to its slot
 __global__ void scan_sweep_kernel(const ScanParams p) {
     const int e = blockIdx.y;
     const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x, CN = (int64_t)p.C * p.N;
@@ -213,37 +286,44 @@ __global__ void scan_sweep_kernel(const ScanParams p) {
     const float A2 = p.A[i] * LOG2E;
     float* slot = p.state + (size_t)p.sp.slot[e] * CN + i;
     float S = p.sp.start[e] > 0 ? *slot : 0.f;
-    for (int w = p.sp.work_off[e]; w < p.sp.work_off[e + 1]; w++) {
+    for (int w = p.sp.work_off[e]; w < p.sp.work_off[e + 1]; w += p.run) {
         float* piece = p.piece_state + (size_t)w * CN + i;
         const float local = *piece;
         *piece = S;
-        S = fmaf(exp2f(A2 * p.piece_dt[(size_t)w * p.C + c]), S, local);
+        S = fmaf(decay_exp2(A2 * p.piece_dt[(size_t)w * p.C + c]), S, local);
     }
     *slot = S;
 }
 
-template <typename T, int NS>
-void launch_scan(const ScanParams& p, int phase, cudaStream_t stream) {
-    const int per_block = SCAN_THREADS >> p.lane_shift;
-    const dim3 grid((p.C + per_block - 1) / per_block, p.sp.n_work);
-    const size_t smem = (size_t)SCAN_TOKENS * 2 * p.N * sizeof(float);
-    if (phase == 0) scan_kernel<T, NS, 0><<<grid, SCAN_THREADS, smem, stream>>>(p);
-    else if (phase == 1) scan_kernel<T, NS, 1><<<grid, SCAN_THREADS, smem, stream>>>(p);
-    else scan_kernel<T, NS, 2><<<grid, SCAN_THREADS, smem, stream>>>(p);
+int scan_lanes(int n_states) {
+    int lanes = 1;
+    while (lanes < 32 && lanes * 4 < n_states) lanes *= 2;
+    return lanes;
 }
-template <typename T>
-void dispatch_scan(ScanParams& p, int phase, cudaStream_t stream) {
-    // decode-like pieces: many lanes per channel, few states each (coalesced state traffic); long pieces: the fewest
-    // lanes that keep a channel's states in registers
-    const int max_ns = phase == 0 && p.sp.max_tokens <= 4 ? 4 : 16;
-    int shift = 0;
-    while (shift < 5 && (p.N + (1 << shift) - 1) / (1 << shift) > max_ns) shift++;
-    const int ns = (p.N + (1 << shift) - 1) / (1 << shift);
-    p.lane_shift = shift;
-    if (ns <= 4) launch_scan<T, 4>(p, phase, stream);
-    else if (ns <= 8) launch_scan<T, 8>(p, phase, stream);
-    else if (ns <= 12) launch_scan<T, 12>(p, phase, stream);
-    else launch_scan<T, 16>(p, phase, stream);
+// Pieces per CTA.  Sequential over whole spans (0) when spans and channels alone fill the GPU; else runs that do.
+int scan_run(const ca_spans& sp, int channels, int n_states) {
+    const int per_block = SCAN_THREADS / scan_lanes(n_states);
+    const int64_t blocks = (channels + per_block - 1) / per_block;
+    if (sp.n_work == sp.n_entries || blocks * sp.n_entries >= 256) return 0;
+    const int64_t run = std::max<int64_t>(1, blocks * sp.n_work / 592);  // about four CTAs per SM
+    const int longest = (sp.max_tokens + sp.work_len - 1) / sp.work_len;
+    return run >= longest ? 0 : (int)run;
+}
+
+template <typename T, int L, int NS>
+void launch_scan(const ScanParams& p, cudaStream_t stream) {
+    const int per_block = SCAN_THREADS / L;
+    const int blocks = (p.C + per_block - 1) / per_block;
+    const size_t smem = (size_t)SCAN_TOKENS * 2 * L * NS * sizeof(float);
+    if (p.run == 0) {
+        // decode steps: a CTA takes several spans, so that its rows of A are read once
+        const int rows = p.sp.max_tokens > 1 ? p.sp.n_entries : std::min(p.sp.n_entries, std::max(1, 148 * 16 / blocks));
+        scan_kernel<T, L, NS, 0><<<dim3(blocks, rows), SCAN_THREADS, smem, stream>>>(p);
+    } else {
+        scan_kernel<T, L, NS, 1><<<dim3(blocks, p.sp.n_work), SCAN_THREADS, smem, stream>>>(p);
+        scan_sweep_kernel<<<dim3((unsigned)(((int64_t)p.C * p.N + 255) / 256), p.sp.n_entries), 256, 0, stream>>>(p);
+        scan_kernel<T, L, NS, 2><<<dim3(blocks, p.sp.n_work), SCAN_THREADS, smem, stream>>>(p);
+    }
 }
 
 // ---- linear attention with decay --------------------------------------------------------------------------------
@@ -253,6 +333,7 @@ struct DecayParams {
     int64_t row_stride;
     const float* decay;      // [H]
     float* state;            // [slots, H, dk, dv]
+    float* scratch;          // [pieces, H, dk, dv] or null
     int H, dk, dv;
     ca_spans sp;
 };
@@ -389,13 +470,16 @@ bool aligned16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0;
 template <typename T>
 int conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, const float* bias, float* state, const ca_spans& sp,
               int channels, int K, cudaStream_t stream) {
-    const bool v2 = channels % 2 == 0 && x_stride % 2 == 0 && reinterpret_cast<uintptr_t>(x) % (2 * sizeof(T)) == 0;
-    const int per = 128 * (v2 ? 2 : 1);
+    auto packs = [&](int v) { return channels % v == 0 && x_stride % v == 0 && reinterpret_cast<uintptr_t>(x) % (v * sizeof(T)) == 0; };
+    const int v = packs(4) && K <= 4 ? 4 : (packs(2) ? 2 : 1);
+    const int per = 128 * v;
     const dim3 grid((channels + per - 1) / per, sp.n_work);
     T* o = static_cast<T*>(out);
     const T* in = static_cast<const T*>(x);
 #define CA_CONV(V, KM) conv_silu_kernel<T, V, KM><<<grid, 128, 0, stream>>>(o, in, x_stride, taps, bias, state, sp, channels, K)
-    if (v2) {
+    if (v == 4) {
+        CA_CONV(4, 4);
+    } else if (v == 2) {
         if (K <= 4) CA_CONV(2, 4); else CA_CONV(2, 16);
     } else {
         if (K <= 4) CA_CONV(1, 4); else CA_CONV(1, 16);
@@ -405,16 +489,37 @@ int conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, con
 }
 
 template <typename T>
-int selective_scan(ScanParams& p, cudaStream_t stream) {
-    if (p.sp.n_work == p.sp.n_entries) {
-        dispatch_scan<T>(p, 0, stream);
-    } else {
-        dispatch_scan<T>(p, 1, stream);
-        const dim3 grid((unsigned)(((int64_t)p.C * p.N + 255) / 256), p.sp.n_entries);
-        scan_sweep_kernel<<<grid, 256, 0, stream>>>(p);
-        dispatch_scan<T>(p, 2, stream);
+int selective_scan(const ScanParams& p, cudaStream_t stream) {
+    switch (scan_lanes(p.N)) {
+        case 1: launch_scan<T, 1, 4>(p, stream); break;
+        case 2: launch_scan<T, 2, 4>(p, stream); break;
+        case 4: launch_scan<T, 4, 4>(p, stream); break;
+        case 8: launch_scan<T, 8, 4>(p, stream); break;
+        case 16: launch_scan<T, 16, 4>(p, stream); break;
+        default:
+            if (p.N <= 128) launch_scan<T, 32, 4>(p, stream);
+            else launch_scan<T, 32, 8>(p, stream);
     }
     return done();
+}
+
+// Pieces per CTA of the tensor-core kernel (one CTA per SM): the run length that needs the fewest block times, counting two
+// passes for runs and one for whole spans (0).
+int decay_run(const ca_spans& sp, int heads) {
+    const int longest = (sp.max_tokens + sp.work_len - 1) / sp.work_len;
+    if (longest <= 1) return 0;
+    auto waves = [](int64_t ctas) { return (double)((ctas + 147) / 148); };
+    double best = waves((int64_t)sp.n_entries * heads) * longest;
+    int best_run = 0;
+    for (int run = 1; run < longest; run++) {
+        const int64_t runs = (sp.n_work + (int64_t)(run - 1) * sp.n_entries) / run;  // at most
+        const double cost = waves(runs * heads) * run * 1.4 + 2.0 + 0.1 * runs / sp.n_entries;
+        if (cost < best) {
+            best = cost;
+            best_run = run;
+        }
+    }
+    return best_run;
 }
 
 template <typename T>
@@ -427,6 +532,12 @@ int decay_attention(const DecayParams& p, cudaStream_t stream) {
         if (v4) decay_step_kernel<T, 4><<<grid, DECAY_STEP_THREADS, smem, stream>>>(p);
         else decay_step_kernel<T, 1><<<grid, DECAY_STEP_THREADS, smem, stream>>>(p);
         return done();
+    }
+    if (std::is_same<T, __nv_bfloat16>::value && decay_mma_serves(p.dk, p.dv, p.row_stride, p.qkv, p.sp.work_len)) {
+        DecayMmaParams m{p.out, p.qkv, p.row_stride, p.decay, p.state, p.scratch, p.H, p.dk, p.dv, decay_run(p.sp, p.H), p.sp};
+        if (m.run > 0 && !p.scratch) return fail("decay_attention: this batch needs scratch");
+        const cudaError_t e = launch_decay_mma(m, stream);
+        return e == cudaSuccess ? CA_OK : fail(cudaGetErrorString(e), CA_ERR_CUDA);
     }
     const size_t smem = (size_t)(2 * DS_TOK * (p.dk + 1) + p.dk * (DS_COL + 1) + 2 * DS_TOK * (DS_COL + 1) + DS_TOK + 1) * sizeof(float);
     const cudaError_t e = cudaFuncSetAttribute(decay_span_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -456,12 +567,11 @@ int ca_conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, 
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (dtype == CA_DTYPE_BF16) return conv_silu<__nv_bfloat16>(out, x, x_stride, taps, bias, state, *sp, channels, n_taps, s);
     if (dtype == CA_DTYPE_F32) return conv_silu<float>(out, x, x_stride, taps, bias, state, *sp, channels, n_taps, s);
-    if (dtype == CA_DTYPE_F16) return conv_silu<__half>(out, x, x_stride, taps, bias, state, *sp, channels, n_taps, s);
     return fail("conv_silu: unknown element type");
 }
 
 int64_t ca_scan_scratch_floats(const ca_spans* sp, int channels, int n_states) {
-    if (!sp || sp->n_work == sp->n_entries) return 0;
+    if (!sp || channels <= 0 || n_states <= 0 || scan_run(*sp, channels, n_states) == 0) return 0;
     return (int64_t)sp->n_work * channels * ((int64_t)n_states + 1);
 }
 
@@ -471,31 +581,35 @@ int ca_selective_scan(void* y, const void* x, const void* z, int64_t z_stride, c
     if (!spans_ok(sp)) return fail("selective_scan: bad spans");
     if (channels <= 0 || n_states < 1 || n_states > 256) return fail("selective_scan: 1 to 256 states per channel");
     if (!y || !x || !z || !dt || !dt_bias || !A || !bc || !D || !state) return fail("selective_scan: null pointer");
-    if (sp->n_work != sp->n_entries && !scratch) return fail("selective_scan: spans of several pieces need scratch");
     ScanParams p;
+    p.run = scan_run(*sp, channels, n_states);
+    if (p.run > 0 && !scratch) return fail("selective_scan: this batch needs scratch");
     p.y = y; p.x = x; p.z = z; p.z_stride = z_stride; p.dt = dt; p.dt_bias = dt_bias; p.A = A; p.bc = bc; p.bc_stride = bc_stride;
     p.D = D; p.state = state; p.piece_state = scratch;
     p.piece_dt = scratch ? scratch + (size_t)sp->n_work * channels * n_states : nullptr;
-    p.C = channels; p.N = n_states; p.lane_shift = 0; p.sp = *sp;
+    p.C = channels; p.N = n_states; p.sp = *sp;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (dtype == CA_DTYPE_BF16) return selective_scan<__nv_bfloat16>(p, s);
     if (dtype == CA_DTYPE_F32) return selective_scan<float>(p, s);
-    if (dtype == CA_DTYPE_F16) return selective_scan<__half>(p, s);
     return fail("selective_scan: unknown element type");
 }
 
-int ca_decay_attention(void* out, const void* qkv, int64_t row_stride, const float* decay, float* state, const ca_spans* sp,
+int64_t ca_decay_scratch_floats(const ca_spans* sp, int n_heads, int d_key, int d_value, int dtype) {
+    if (!sp || dtype != CA_DTYPE_BF16 || sp->max_tokens <= 1 || n_heads <= 0 || decay_run(*sp, n_heads) == 0) return 0;
+    return (int64_t)sp->n_work * n_heads * d_key * d_value;
+}
+
+int ca_decay_attention(void* out, const void* qkv, int64_t row_stride, const float* decay, float* state, float* scratch, const ca_spans* sp,
                        int n_heads, int d_key, int d_value, int dtype, ca_stream stream) {
     if (!spans_ok(sp)) return fail("decay_attention: bad spans");
     if (n_heads <= 0 || d_key <= 0 || d_key > 256 || d_value <= 0 || d_value > 1024) return fail("decay_attention: head sizes out of range");
     if (!out || !qkv || !decay || !state) return fail("decay_attention: null pointer");
     DecayParams p;
-    p.out = out; p.qkv = qkv; p.row_stride = row_stride; p.decay = decay; p.state = state;
+    p.out = out; p.qkv = qkv; p.row_stride = row_stride; p.decay = decay; p.state = state; p.scratch = scratch;
     p.H = n_heads; p.dk = d_key; p.dv = d_value; p.sp = *sp;
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (dtype == CA_DTYPE_BF16) return decay_attention<__nv_bfloat16>(p, s);
     if (dtype == CA_DTYPE_F32) return decay_attention<float>(p, s);
-    if (dtype == CA_DTYPE_F16) return decay_attention<__half>(p, s);
     return fail("decay_attention: unknown element type");
 }
 

@@ -95,6 +95,18 @@ Tensor norm_rows(Tensor x, Tensor weight, double eps, py::object dtype, c10::opt
     return out;
 }
 
+// fp32 rows of the embedding table for a batch's tokens; a token outside the table raises before anything runs
+Tensor embed_rows(Tensor table, const SpanBatch& sp) {
+    need(table.is_cuda() && table.dim() == 2 && table.is_contiguous() && table.device() == sp.device(), "embed_rows: a contiguous [vocab, width] table on the spans' CUDA device is required");
+    need(sp.min_token() >= 0 && sp.max_token() < table.size(0), "embed_rows: a token id lies outside the vocabulary");
+    c10::cuda::CUDAGuard guard(table.device());
+    Tensor x = torch::empty({sp.n_tokens(), table.size(1)}, table.options().dtype(torch::kFloat32));
+    check_rc(ca_embed_rows(x.data_ptr<float>(), table.data_ptr(), sp.tokens.data_ptr<int32_t>(), sp.n_tokens(), (int)table.size(1),
+                           dtype_code(table, "embed_rows"), stream_of(table)),
+             "embed_rows");
+    return x;
+}
+
 Tensor gelu_tanh(Tensor x) {
     need(rows_of(x, x.size(0), x.size(-1)), "gelu_tanh: [rows, width] on a CUDA device is required");
     c10::cuda::CUDAGuard guard(x.device());
@@ -141,7 +153,11 @@ Tensor decay_attention(Tensor qkv, Tensor decay, int64_t d_key, int64_t d_value,
     need(f32_vec(decay, H) && state_ok(state, sp, H * d_key * d_value), "decay_attention: decay fp32 [heads], state fp32 [slots, heads, d_key, d_value]");
     c10::cuda::CUDAGuard guard(qkv.device());
     Tensor out = torch::empty({T, H * d_value}, qkv.options());
-    check_rc(ca_decay_attention(out.data_ptr(), qkv.data_ptr(), qkv.stride(0), decay.data_ptr<float>(), state.data_ptr<float>(), sp.view(),
+    const int64_t n = ca_decay_scratch_floats(sp.view(), (int)H, (int)d_key, (int)d_value, dtype_code(qkv, "decay_attention"));
+    Tensor scratch;
+    if (n > 0) scratch = torch::empty({n}, qkv.options().dtype(torch::kFloat32));
+    check_rc(ca_decay_attention(out.data_ptr(), qkv.data_ptr(), qkv.stride(0), decay.data_ptr<float>(), state.data_ptr<float>(),
+                                n > 0 ? scratch.data_ptr<float>() : nullptr, sp.view(),
                                 (int)H, (int)d_key, (int)d_value, dtype_code(qkv, "decay_attention"), stream_of(qkv)),
              "decay_attention");
     return out;
@@ -170,6 +186,7 @@ void init_block_ops(py::module& m, py::module& ops) {
             "x += rms_norm(r * sigmoid(gate + bias)) * weight on an fp32 stream, in place");
     ops.def("norm_rows", &norm_rows, py::arg("x"), py::arg("weight"), py::arg("eps"), py::arg("dtype"), py::arg("rows") = py::none(),
             py::arg("gate") = py::none(), "RMS norm of (selected) rows, optionally times sigmoid(gate)");
+    ops.def("embed_rows", &embed_rows, py::arg("table"), py::arg("spans"), "fp32 embedding rows of a batch's tokens");
     ops.def("gelu_tanh", &gelu_tanh, py::arg("x"), "tanh form of GELU");
     ops.def("conv_silu", &conv_silu, py::arg("x"), py::arg("taps"), py::arg("bias"), py::arg("state"), py::arg("spans"),
             "causal depthwise convolution + SiLU over spans");

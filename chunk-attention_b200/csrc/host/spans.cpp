@@ -50,6 +50,8 @@ SpanBatch::SpanBatch(const std::vector<std::vector<int>>& toks, const std::vecto
         }
         for (int i = 0; i < n; i++) {
             d[o_tok + t + i] = toks[e][i];
+            min_token_ = std::min(min_token_, toks[e][i]);
+            max_token_ = std::max(max_token_, toks[e][i]);
             d[o_pos + t + i] = starts[e] + i;
             d[o_ent + t + i] = (int32_t)e;
         }

@@ -22,11 +22,13 @@ class SpanBatch {
     torch::Tensor tokens, positions, entry_of, last;        // int32 views of the uploaded buffer; last: row of each entry's last token
     torch::Device device() const { return buffer_.device(); }
     int max_slot() const { return max_slot_; }
+    int min_token() const { return min_token_; }
+    int max_token() const { return max_token_; }
 
   private:
     torch::Tensor buffer_;
     ca_spans spans_{};
-    int max_slot_ = -1;
+    int max_slot_ = -1, min_token_ = 0, max_token_ = 0;
 };
 
 }  // namespace ca_host

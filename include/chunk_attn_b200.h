@@ -381,12 +381,14 @@ CA_API int ca_attention_rows(ca_context* ctx, const ca_rows_args* args, ca_strea
  *   next_mu (one token per span only) also the token shift of the result.
  * ca_norm_rows: out[i] = row rows[i] (NULL: i) of x, RMS-normed, times weight, times sigmoid(gate[i]) if given.
  * ca_gelu_tanh: the tanh form.
+ * ca_embed_rows: x[t] = table[ids[t]] (rows of `dtype`) as fp32; the caller has checked the ids.
  * ca_conv_silu: depthwise causal convolution with bias (taps [channels, n_taps], last tap = current token), then
  *   SiLU; state [slots, n_taps - 1, channels], oldest first.
  * ca_selective_scan: dt = softplus(dt + dt_bias); S[c, n] = exp(dt A) S + dt x B_n; y = (S . C + D x) * silu(z);
  *   bc row: B then C; state [slots, channels, n_states]; scratch of ca_scan_scratch_floats() floats.
  * ca_decay_attention: q, k, v = silu of the heads of qkv; S = decay_h S + k v^T, out = S^T q; state
- *   [slots, heads, d_key, d_value]. */
+ *   [slots, heads, d_key, d_value]; scratch of ca_decay_scratch_floats() floats.
+ * The recurrences come in bf16 and fp32. */
 CA_API int ca_token_shift(const float* x, const float* mu, float* state, void* plain, void* shifted, const ca_spans* spans,
                           int width, int dtype, ca_stream stream);
 CA_API int ca_gated_norm_add(float* x, const void* r, int64_t r_stride, const void* gate, int64_t gate_stride,
@@ -396,6 +398,8 @@ CA_API int ca_gated_norm_add(float* x, const void* r, int64_t r_stride, const vo
 CA_API int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const int32_t* rows, const float* weight,
                         const void* gate, int64_t gate_stride, float eps, int64_t n_rows, int width, int dtype,
                         ca_stream stream);
+CA_API int ca_embed_rows(float* x, const void* table, const int32_t* ids, int64_t n_tokens, int width, int dtype,
+                         ca_stream stream);
 CA_API int ca_gelu_tanh(void* out, const void* in, int64_t in_stride, int64_t n_rows, int width, int dtype, ca_stream stream);
 CA_API int ca_conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, const float* bias, float* state,
                         const ca_spans* spans, int channels, int n_taps, int dtype, ca_stream stream);
@@ -403,7 +407,8 @@ CA_API int64_t ca_scan_scratch_floats(const ca_spans* spans, int channels, int n
 CA_API int ca_selective_scan(void* y, const void* x, const void* z, int64_t z_stride, const float* dt, const float* dt_bias,
                              const float* A, const float* bc, int64_t bc_stride, const float* D, float* state, float* scratch,
                              const ca_spans* spans, int channels, int n_states, int dtype, ca_stream stream);
-CA_API int ca_decay_attention(void* out, const void* qkv, int64_t row_stride, const float* decay, float* state,
+CA_API int64_t ca_decay_scratch_floats(const ca_spans* spans, int n_heads, int d_key, int d_value, int dtype);
+CA_API int ca_decay_attention(void* out, const void* qkv, int64_t row_stride, const float* decay, float* state, float* scratch,
                               const ca_spans* spans, int n_heads, int d_key, int d_value, int dtype, ca_stream stream);
 
 /* ---- allocation-free decode step ---------------------------------------------------------------
