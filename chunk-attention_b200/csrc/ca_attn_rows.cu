@@ -345,7 +345,7 @@ __global__ void __launch_bounds__(R_THREADS) rows_mma_kernel(const RowsParams p)
                 b *= inv;
                 if (p.value_freq) {
                     float sn, cs;
-                    sincosf(pos * p.value_freq[i], &sn, &cs);
+                    fast_sincos(pos * p.value_freq[i], &sn, &cs);
                     const float t = a * cs + b * sn;
                     b = b * cs - a * sn;
                     a = t;
@@ -420,7 +420,7 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
         float a = acc[k][0] * inv, c = acc[k][1] * inv;
         if (p.value_freq) {
             float sn, cs;
-            sincosf(pos * p.value_freq[i], &sn, &cs);
+            fast_sincos(pos * p.value_freq[i], &sn, &cs);
             const float t = a * cs + c * sn;
             c = c * cs - a * sn;
             a = t;

@@ -196,16 +196,21 @@ __global__ void __launch_bounds__(A_THREADS, 2) span_attn_kernel(const SpanAttnP
         // moved into the queries, so that the largest score is the largest product.
         const uint32_t flip = p.scale_log2 < 0.f ? 0x80008000u : 0u;
         constexpr int GR = DK / 8;
-        for (int i = threadIdx.x; i < A_ROWS * GR; i += 4 * 32) {
-            const int r = i / GR, g = i % GR;
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        uint4 v[GR];  // all loads of a thread in flight together
+#pragma unroll
+        for (int u = 0; u < GR; u++) {
+            const int i = threadIdx.x + u * (4 * 32), r = i / GR, g = i % GR;
+            v[u] = make_uint4(0u, 0u, 0u, 0u);
             if (r < n_rows) {
                 const int token = token0 + r / group, head = kvh * group + r % group;
-                v = __ldg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) + ((size_t)token * H + head) * DK) + g);
-                v.x ^= flip; v.y ^= flip; v.z ^= flip; v.w ^= flip;
+                v[u] = __ldg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) + ((size_t)token * H + head) * DK) + g);
             }
+        }
+#pragma unroll
+        for (int u = 0; u < GR; u++) {
+            const int i = threadIdx.x + u * (4 * 32), r = i / GR, g = i % GR;
             const uint32_t dst = sbase + (g >> 3) * Z::Q_PANEL + r * 128 + (((g & 7) ^ (r & 7)) << 4);
-            asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(dst), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
+            sts128(dst, (int)(v[u].x ^ flip), (int)(v[u].y ^ flip), (int)(v[u].z ^ flip), (int)(v[u].w ^ flip));
         }
         fence_proxy_async();
         mbar_arrive(q_ready);
@@ -338,7 +343,7 @@ __global__ void __launch_bounds__(A_THREADS, 2) span_attn_kernel(const SpanAttnP
                     float a = __uint_as_float(o[2 * i]) * inv, bb = __uint_as_float(o[2 * i + 1]) * inv;
                     if (p.value_freq) {
                         float sn, cs;
-                        sincosf(pos * __ldg(p.value_freq + c * 16 + i), &sn, &cs);
+                        fast_sincos(pos * __ldg(p.value_freq + c * 16 + i), &sn, &cs);
                         const float t = a * cs + bb * sn;
                         bb = bb * cs - a * sn;
                         a = t;

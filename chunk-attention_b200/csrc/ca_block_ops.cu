@@ -80,7 +80,7 @@ __global__ void gated_norm_add_kernel(float* __restrict__ x, const T* __restrict
         load_f<T, V>(gate + t * gate_stride + c, z);
         load_f<float, V>(bias + c, b);
 #pragma unroll
-        for (int i = 0; i < V; i++) out[i] = a[i] * sigmoid_f(z[i] + b[i]);
+        for (int i = 0; i < V; i++) out[i] = a[i] * sigmoid_for<T>(z[i] + b[i]);
     };
     const int stride = blockDim.x * V;
 #pragma unroll
@@ -143,7 +143,7 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const TI* __restrict__ x, 
                                  const float* __restrict__ w, const T* __restrict__ gate, int64_t gate_stride, float eps, int width) {
     const size_t t = blockIdx.x;
     const TI* src = x + (size_t)(rows ? rows[t] : t) * x_stride;
-    constexpr int STEPS = V == 1 ? 4 : 2;  // of the row a thread keeps in registers, gate included
+    constexpr int STEPS = V == 1 ? 4 : (V == 8 ? 1 : 2);  // of the row a thread keeps in registers, gate included
     float kept[STEPS][V], z[STEPS][V];
     float ss = 0.f;
     const int stride = blockDim.x * V;
@@ -168,7 +168,7 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const TI* __restrict__ x, 
         float ww[V];
         load_f<float, V>(w + c, ww);
 #pragma unroll
-        for (int i = 0; i < V; i++) a[i] *= inv * ww[i] * (gate ? sigmoid_f(zz[i]) : 1.f);
+        for (int i = 0; i < V; i++) a[i] *= inv * ww[i] * (gate ? sigmoid_for<T>(zz[i]) : 1.f);
         store_f<T, V>(out + t * width + c, a);
     };
 #pragma unroll
@@ -202,16 +202,15 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 }
 
 template <typename T, int V>
-__global__ void gelu_rows_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t in_stride, int width, int64_t total) {
-    const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
-    if (i >= total) return;
-    const int64_t t = i / width;
-    const int c = (int)(i - t * width);
-    float a[V];
-    load_f<T, V>(in + t * in_stride + c, a);
+__global__ void gelu_rows_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t in_stride, int width) {
+    const size_t t = blockIdx.x;
+    for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
+        float a[V];
+        load_f<T, V>(in + t * in_stride + c, a);
 #pragma unroll
-    for (int k = 0; k < V; k++) a[k] = gelu_tanh_f(a[k]);
-    store_f<T, V>(out + i, a);
+        for (int k = 0; k < V; k++) a[k] = gelu_tanh_f(a[k]);
+        store_f<T, V>(out + t * width + c, a);
+    }
 }
 
 int row_threads(int units) {
@@ -228,10 +227,13 @@ int done() {
     return e == cudaSuccess ? CA_OK : fail(cudaGetErrorString(e), CA_ERR_CUDA);
 }
 
-// calls f(T value, integral_constant V): V elements per access
-template <typename F> int by_type(int dtype, bool vec, F&& f) {
+bool aligned32(const void* p) { return reinterpret_cast<uintptr_t>(p) % 32 == 0; }
+
+// calls f(T value, integral_constant V): V elements per access (wide: 8 of a 16-bit type)
+template <typename F> int by_type(int dtype, bool vec, F&& f, bool wide = false) {
     if (dtype == CA_DTYPE_BF16) {
-        if (vec) f(__nv_bfloat16(), std::integral_constant<int, 4>());
+        if (vec && wide) f(__nv_bfloat16(), std::integral_constant<int, 8>());
+        else if (vec) f(__nv_bfloat16(), std::integral_constant<int, 4>());
         else f(__nv_bfloat16(), std::integral_constant<int, 1>());
     } else if (dtype == CA_DTYPE_F16) {
         if (vec) f(__half(), std::integral_constant<int, 4>());
@@ -281,10 +283,11 @@ int ca_gated_norm_add(float* x, const void* r, int64_t r_stride, const void* gat
     return by_type(dtype, vec, [&](auto tv, auto vv) {
         using T = decltype(tv);
         constexpr int V = decltype(vv)::value;
-        gated_norm_add_kernel<T, V, V == 1 ? 4 : 2><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
+        gated_norm_add_kernel<T, V, V == 1 ? 4 : (V == 8 ? 1 : 2)><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
             x, static_cast<const T*>(r), r_stride, static_cast<const T*>(gate), gate_stride, bias, weight, eps, static_cast<T*>(plain),
             next_mu, next_state, static_cast<T*>(next_shifted), spans, width);
-    });
+    }, n_tokens <= 512 && width % 8 == 0 && r_stride % 8 == 0 && gate_stride % 8 == 0 && aligned32(x) && aligned32(bias) && aligned32(weight) &&
+           aligned32(next_mu) && aligned32(next_state));
 }
 
 int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const int32_t* rows, const float* weight,
@@ -304,7 +307,7 @@ int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const
         else
             norm_rows_kernel<T, T, V><<<(unsigned)n_rows, threads, 0, static_cast<cudaStream_t>(stream)>>>(
                 static_cast<T*>(out), static_cast<const T*>(x), x_stride, rows, weight, static_cast<const T*>(gate), gate_stride, eps, width);
-    });
+    }, width % 8 == 0 && x_stride % 8 == 0 && (!gate || gate_stride % 8 == 0) && aligned32(x) && aligned32(weight));
 }
 
 int ca_embed_rows(float* x, const void* table, const int32_t* ids, int64_t n_tokens, int width, int dtype, ca_stream stream) {
@@ -328,10 +331,9 @@ int ca_gelu_tanh(void* out, const void* in, int64_t in_stride, int64_t n_rows, i
     return by_type(dtype, vec, [&](auto tv, auto vv) {
         using T = decltype(tv);
         constexpr int V = decltype(vv)::value;
-        const int64_t total = n_rows * width;
-        gelu_rows_kernel<T, V><<<(unsigned)((total / V + 255) / 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(
-            static_cast<T*>(out), static_cast<const T*>(in), in_stride, width, total);
-    });
+        gelu_rows_kernel<T, V><<<(unsigned)n_rows, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
+            static_cast<T*>(out), static_cast<const T*>(in), in_stride, width);
+    }, width % 8 == 0 && in_stride % 8 == 0);
 }
 
 }  // extern "C"

@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(D_THREADS, 1) decay_mma_kernel(const DecayMmaP
                 const uint4 v = __ldg(reinterpret_cast<const uint4*>(qkv + (size_t)(t0 + t) * p.row_stride + offset) + g);
                 const uint32_t x[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-                for (int k = 0; k < 4; k++) o[k] = pack_bf16(silu_f(lo_f(x[k])), silu_f(hi_f(x[k])));
+                for (int k = 0; k < 4; k++) o[k] = pack_bf16(silu_for<__nv_bfloat16>(lo_f(x[k])), silu_for<__nv_bfloat16>(hi_f(x[k])));
             }
             sts128(dst + at<D_TOK>(t, g), (int)o[0], (int)o[1], (int)o[2], (int)o[3]);
         }
@@ -278,14 +278,18 @@ cudaError_t launch(const DecayMmaParams& p, cudaStream_t stream) {
     if (p.run == 0) return launch_phase<DK, DV, 0>(p, p.sp.n_entries, stream);
     cudaError_t e = launch_phase<DK, DV, 1>(p, p.sp.n_work, stream);
     if (e != cudaSuccess) return e;
-    const int64_t quads = (int64_t)p.H * p.dk * p.dv / 4;
-    decay_sweep_kernel<<<dim3((unsigned)((quads + 255) / 256), p.sp.n_entries), 256, 0, stream>>>(p);
-    e = cudaGetLastError();
+    e = launch_decay_sweep(p, stream);
     if (e != cudaSuccess) return e;
     return launch_phase<DK, DV, 2>(p, p.sp.n_work, stream);
 }
 
 }  // namespace
+
+cudaError_t launch_decay_sweep(const DecayMmaParams& p, cudaStream_t stream) {
+    const int64_t quads = (int64_t)p.H * p.dk * p.dv / 4;
+    decay_sweep_kernel<<<dim3((unsigned)((quads + 255) / 256), p.sp.n_entries), 256, 0, stream>>>(p);
+    return cudaGetLastError();
+}
 
 bool decay_mma_serves(int dk, int dv, int64_t row_stride, const void* qkv, int work_len) {
     return dk % 16 == 0 && dv % 16 == 0 && dk <= 128 && dv <= 128 && row_stride % 8 == 0 && reinterpret_cast<uintptr_t>(qkv) % 16 == 0 &&

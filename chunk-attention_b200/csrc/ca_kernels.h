@@ -221,6 +221,11 @@ struct DecayMmaParams {
 };
 bool decay_mma_serves(int dk, int dv, int64_t row_stride, const void* qkv, int work_len);
 cudaError_t launch_decay_mma(const DecayMmaParams& p, cudaStream_t stream);
+cudaError_t launch_decay_sweep(const DecayMmaParams& p, cudaStream_t stream);
+// the same on tcgen05 (ca_decay_tc.cu), for sizes where its 128-token blocks pay; what decay_mma_serves refuses it refuses too
+bool decay_tc_serves(int dk, int dv);
+cudaError_t launch_decay_tc(const DecayMmaParams& p, cudaStream_t stream);
+cudaError_t read_decay_status(int* status, cudaStream_t stream);  // 0, or STATUS_* of the first wait that ran out
 
 // ---- projections to attention operands (ca_qkv.cu) ------------------------------------------------------
 struct QkvParams {

@@ -27,7 +27,7 @@ __global__ void __launch_bounds__(QKV_WARPS * 32) store_qkv_kernel(const QkvPara
     const int kp = p.key_freq ? p.rot_dims / 2 : 0, vp = p.value_freq ? p.d_value / 2 : 0;
     for (int i = threadIdx.x; i < kp + vp; i += blockDim.x) {
         float sn, cs;
-        sincosf(pos * (i < kp ? p.key_freq[i] : p.value_freq[i - kp]), &sn, &cs);
+        sincos_for<T>(pos * (i < kp ? p.key_freq[i] : p.value_freq[i - kp]), &sn, &cs);
         (i < kp ? turn_k[i] : turn_v[i - kp]) = make_float2(cs, sn);
     }
     int chunk, slot;
@@ -125,18 +125,26 @@ __global__ void __launch_bounds__(QKV_VEC_THREADS) store_qkv_vec_kernel(const Qk
     const T* row = reinterpret_cast<const T*>(p.qkv) + (size_t)t * p.row_stride;
     T* pool = reinterpret_cast<T*>(p.pool);
     const Geometry v_side = tile_side(p.geo, 1);
-    Pack<T, EPG> in;
+    constexpr int AHEAD = 1;  // heads whose granules are requested together
+    Pack<T, EPG> in[AHEAD];
     auto source = [&](int u) { return row + (u < H + G ? u * p.d_key : (H + G) * p.d_key + (u - H - G) * p.d_value) + g * EPG; };
     auto size_of = [&](int u) { return u < H + G ? p.d_key : p.d_value; };
     int u = tid / lanes;
-    if (u < units && g * EPG < size_of(u)) in = *reinterpret_cast<const Pack<T, EPG>*>(source(u));
+    auto request = [&](int u) {
+#pragma unroll
+        for (int a = 0; a < AHEAD; a++) {
+            const int ua = u + a * per_pass;
+            if (ua < units && g * EPG < size_of(ua)) in[a] = *reinterpret_cast<const Pack<T, EPG>*>(source(ua));
+        }
+    };
+    request(u);
     for (int i = tid; i < kp + vp; i += QKV_VEC_THREADS) {
         float sn, cs;
-        sincosf(pos * (i < kp ? p.key_freq[i] : p.value_freq[i - kp]), &sn, &cs);
+        sincos_for<T>(pos * (i < kp ? p.key_freq[i] : p.value_freq[i - kp]), &sn, &cs);
         (i < kp ? turn_k[i] : turn_v[i - kp]) = make_float2(cs, sn);
     }
     __syncthreads();
-    for (int u0 = 0; u0 < units; u0 += per_pass, u += per_pass) {
+    auto one_head = [&](int u, const Pack<T, EPG>& in) {
         const bool on = u < units && g * EPG < size_of(min(u, units - 1));
         const int kind = u < H ? 0 : (u < H + G ? 1 : 2);  // q, k, v
         float x[EPG];
@@ -146,10 +154,8 @@ __global__ void __launch_bounds__(QKV_VEC_THREADS) store_qkv_vec_kernel(const Qk
             x[i] = on ? to_f32(in.v[i]) : 0.f;
             ss = fmaf(x[i], x[i], ss);
         }
-        // the next head's granule is requested before this one is worked on
-        if (u + per_pass < units && g * EPG < size_of(u + per_pass)) in = *reinterpret_cast<const Pack<T, EPG>*>(source(u + per_pass));
         for (int off = lanes >> 1; off >= 1; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
-        if (!on || (kind > 0 && chunk < 0)) continue;
+        if (!on || (kind > 0 && chunk < 0)) return;
         const float* w = kind == 0 ? p.q_norm : (kind == 1 ? p.k_norm : nullptr);
         if (w) {
             const float inv = 1.f / sqrtf(ss / p.d_key + p.eps);
@@ -184,9 +190,13 @@ __global__ void __launch_bounds__(QKV_VEC_THREADS) store_qkv_vec_kernel(const Qk
                   tile_granule_index(kind == 2 ? v_side : p.geo, slot, g);
         }
         *dst = o;
+    };
+    for (int u0 = 0; u0 < units; u0 += AHEAD * per_pass, u += AHEAD * per_pass) {
+        if (u0 > 0) request(u);
+#pragma unroll
+        for (int a = 0; a < AHEAD; a++) one_head(u + a * per_pass, in[a]);
     }
 }
-
 template <typename T>
 void run_store_qkv(const QkvParams& p, cudaStream_t stream) {
     constexpr int EPG = 16 / sizeof(T);

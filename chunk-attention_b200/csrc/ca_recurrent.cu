@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(T* __restrict__ out, con
 #pragma unroll
                     for (int j = 0; j < KMAX - 2; j++) hist[j][v] = hist[j + 1][v];
                     if (KMAX > 1) hist[KMAX > 1 ? KMAX - 2 : 0][v] = xv;
-                    o.v[v] = from_f32<T>(silu_f(acc));
+                    o.v[v] = from_f32<T>(silu_for<T>(acc));
                 }
                 *reinterpret_cast<Pack<T, V>*>(out + (size_t)(tg + k) * channels + c) = o;
             }
@@ -126,16 +126,8 @@ struct ScanParams {
     ca_spans sp;
 };
 constexpr int SCAN_THREADS = 128;
-constexpr int SCAN_TOKENS = 16;  // tokens whose B and C are staged at a time
-constexpr int SCAN_GROUP = 8;    // tokens whose x, dt, z are requested together
+constexpr int SCAN_TOKENS = 32;  // tokens whose B and C are staged at a time (two buffers)
 
-__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-// 2^x for x <= 0: one MUFU operation; results below 2^-126 are 0
-__device__ __forceinline__ float decay_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 
 // L lanes share a channel, NS states each.  Of a group of tokens, lane i of a channel reads the inputs of tokens i, i + L,
 // ... and evaluates their step size and, at the end, their output; dt and dt x travel by shuffles.
@@ -143,8 +135,9 @@ __device__ __forceinline__ float decay_exp2(float x) {
 // sum of dt.  2: outputs from the run's initial state.
 template <typename T, int L, int NS, int PHASE>
 __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) {
-    extern __shared__ __align__(16) float bc_s[];  // [SCAN_TOKENS][B: L * NS | C: L * NS], zero past N
-    constexpr int NP = L * NS, OWN = (SCAN_GROUP + L - 1) / L;
+    extern __shared__ __align__(16) float bc_s[];  // 2 x [SCAN_TOKENS][B: L * NS | C: L * NS], zero past N
+    constexpr int GROUP = L <= 8 ? 8 : L;  // tokens whose x, dt, z are requested together, one group ahead
+    constexpr int NP = L * NS, OWN = (GROUP + L - 1) / L, BUF = SCAN_TOKENS * 2 * NP;
     const int c = blockIdx.x * (SCAN_THREADS / L) + threadIdx.x / L;
     const int ln = threadIdx.x & (L - 1), base = (threadIdx.x & 31) & ~(L - 1), n0 = ln * NS, N = p.N;
     const bool on = c < p.C;
@@ -157,6 +150,9 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) 
     const T* Z = static_cast<const T*>(p.z) + cc;
     T* Y = static_cast<T*>(p.y) + cc;
     const float* DT = p.dt + cc;
+    // the padding past N is never copied into
+    for (int i = threadIdx.x; i < 2 * BUF; i += SCAN_THREADS)
+        if (i % NP >= N) bc_s[i] = 0.f;
     for (int unit = blockIdx.y; unit < (PHASE == 0 ? p.sp.n_entries : p.sp.n_work); unit += gridDim.y) {
         int e = unit, t0, t1;
         if (PHASE == 0) {
@@ -173,16 +169,18 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) 
         float* slot = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N + n0;
         float* piece = PHASE == 0 ? nullptr : p.piece_state + ((size_t)unit * p.C + cc) * N + n0;
         const bool live = p.sp.start[e] > 0;
-        const bool vec = NS == 4 && N % 4 == 0;
+        const bool vec = N % 4 == 0;
         const float* from = PHASE == 0 ? slot : piece;
 #pragma unroll
         for (int i = 0; i < NS; i++) S[i] = 0.f;
         if (PHASE == 2 || (PHASE == 0 && live)) {
             if (vec) {
-                if (n0 < N) {
-                    const float4 v = *reinterpret_cast<const float4*>(from);
-                    S[0] = v.x; S[1 % NS] = v.y; S[2 % NS] = v.z; S[3 % NS] = v.w;
-                }
+#pragma unroll
+                for (int i = 0; i < NS; i += 4)
+                    if (n0 + i < N) {
+                        const float4 v = *reinterpret_cast<const float4*>(from + i);
+                        S[i] = v.x; S[i + 1] = v.y; S[i + 2] = v.z; S[i + 3] = v.w;
+                    }
             } else {
 #pragma unroll
                 for (int i = 0; i < NS; i++)
@@ -190,75 +188,93 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) 
             }
         }
         float sum_dt = 0.f;
-        for (int tb = t0; tb < t1; tb += SCAN_TOKENS) {
+        auto stage = [&](int tb, int buf) {  // B and C of the next tokens, asynchronously
             const int nt = min(SCAN_TOKENS, t1 - tb);
-            __syncthreads();
-            for (int i = threadIdx.x; i < nt * 2 * NP; i += SCAN_THREADS) {
-                const int tt = i / (2 * NP), r = i - tt * 2 * NP, n = r < NP ? r : r - NP;
-                bc_s[i] = n < N ? p.bc[(size_t)(tb + tt) * p.bc_stride + n + (r < NP ? 0 : N)] : 0.f;
+            for (int i = threadIdx.x; i < nt * 2 * N; i += SCAN_THREADS) {
+                const int tt = i / (2 * N), r = i - tt * 2 * N;
+                const uint32_t dst = (uint32_t)__cvta_generic_to_shared(bc_s + buf * BUF + tt * 2 * NP + (r < N ? r : r - N + NP));
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(p.bc + (size_t)(tb + tt) * p.bc_stride + r) : "memory");
             }
-            __syncthreads();
-            for (int g = 0; g < nt; g += SCAN_GROUP) {
-                float xs[OWN], ds[OWN], zs[OWN], ys[OWN];
+        };
+        float xs[OWN], ds[OWN], zs[OWN], nx[OWN], nd[OWN], nz[OWN];
+        auto request = [&](int t) {  // this lane's tokens of the group that starts at t
 #pragma unroll
-                for (int k = 0; k < OWN; k++) {
-                    const int tk = ln + k * L;
-                    const size_t t = (size_t)min(tb + g + tk, t1 - 1);
-                    if (tk < SCAN_GROUP) {
-                        xs[k] = to_f32(X[t * p.C]);
-                        ds[k] = DT[t * p.C];
-                        if (PHASE != 1) zs[k] = to_f32(Z[t * p.z_stride]);
-                    } else {
-                        xs[k] = ds[k] = zs[k] = 0.f;
-                    }
+            for (int k = 0; k < OWN; k++) {
+                const int tk = ln + k * L;
+                nx[k] = nd[k] = nz[k] = 0.f;
+                if (tk < GROUP && t + tk < t1) {
+                    nx[k] = to_f32(X[(size_t)(t + tk) * p.C]);
+                    nd[k] = DT[(size_t)(t + tk) * p.C];
+                    if (PHASE != 1) nz[k] = to_f32(Z[(size_t)(t + tk) * p.z_stride]);
                 }
-                float us[OWN];
+            }
+        };
+        __syncthreads();  // nobody reads the buffers of the span before any more
+        stage(t0, 0);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        request(t0);
+        int buf = 0;
+        for (int tb = t0; tb < t1; tb += SCAN_TOKENS, buf ^= 1) {
+            const int nt = min(SCAN_TOKENS, t1 - tb);
+            if (tb > t0) __syncthreads();  // the other buffer is free
+            if (tb + SCAN_TOKENS < t1) stage(tb + SCAN_TOKENS, buf ^ 1);
+            asm volatile("cp.async.commit_group;" ::: "memory");
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+            __syncthreads();
+            for (int g = 0; g < nt; g += GROUP) {
+                float us[OWN], ys[OWN];
 #pragma unroll
                 for (int k = 0; k < OWN; k++) {
-                    ds[k] = softplus_f(ds[k] + bias);
+                    xs[k] = nx[k];
+                    zs[k] = nz[k];
+                    ds[k] = softplus_f(nd[k] + bias);
                     us[k] = ds[k] * xs[k];
                     ys[k] = 0.f;
                 }
-#pragma unroll
-                for (int k = 0; k < SCAN_GROUP; k++) {
-                    if (g + k < nt) {
-                        const int own = k % L;
-                        float dt = ds[k / L], u = us[k / L];
-                        if (L > 1) {
-                            dt = __shfl_sync(0xffffffffu, dt, base + own);
-                            u = __shfl_sync(0xffffffffu, u, base + own);
-                        }
-                        const float* B = bc_s + (g + k) * 2 * NP + n0;
-                        float bv[NS], cv[NS];
-                        if (NS % 4 == 0) {
-#pragma unroll
-                            for (int i = 0; i < NS; i += 4) {
-                                const float4 b4 = *reinterpret_cast<const float4*>(B + i), c4 = *reinterpret_cast<const float4*>(B + NP + i);
-                                bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
-                                cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
-                            }
-                        }
-                        float y = 0.f;
-#pragma unroll
-                        for (int i = 0; i < NS; i++) {
-                            S[i] = fmaf(decay_exp2(dt * A2[i]), S[i], u * bv[i]);
-                            if (PHASE != 1) y = fmaf(S[i], cv[i], y);
-                        }
-                        if (PHASE == 1) {
-                            sum_dt += dt;
-                        } else {
-#pragma unroll
-                            for (int off = L >> 1; off >= 1; off >>= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
-                            if (own == ln) ys[k / L] = y;
-                        }
+                if (tb + g + GROUP < t1) request(tb + g + GROUP);
+                auto token = [&](int k) {
+                    const int own = k % L;
+                    float dt = ds[k / L], u = us[k / L];
+                    if (L > 1) {
+                        dt = __shfl_sync(0xffffffffu, dt, base + own);
+                        u = __shfl_sync(0xffffffffu, u, base + own);
                     }
+                    const float* B = bc_s + buf * BUF + (g + k) * 2 * NP + n0;
+                    float bv[NS], cv[NS];
+#pragma unroll
+                    for (int i = 0; i < NS; i += 4) {
+                        const float4 b4 = *reinterpret_cast<const float4*>(B + i), c4 = *reinterpret_cast<const float4*>(B + NP + i);
+                        bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
+                        cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
+                    }
+                    float y = 0.f;
+#pragma unroll
+                    for (int i = 0; i < NS; i++) {
+                        S[i] = fmaf(exp2_approx(dt * A2[i]), S[i], u * bv[i]);
+                        if (PHASE != 1) y = fmaf(S[i], cv[i], y);
+                    }
+                    if (PHASE == 1) {
+                        sum_dt += dt;
+                    } else {
+#pragma unroll
+                        for (int off = L >> 1; off >= 1; off >>= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
+                        if (own == ln) ys[k / L] = y;
+                    }
+                };
+                if (nt - g >= GROUP) {
+#pragma unroll
+                    for (int k = 0; k < GROUP; k++) token(k);
+                } else {
+#pragma unroll
+                    for (int k = 0; k < GROUP; k++)
+                        if (g + k < nt) token(k);
                 }
                 if (PHASE != 1) {
 #pragma unroll
                     for (int k = 0; k < OWN; k++) {
                         const int tk = ln + k * L;
-                        if (on && tk < SCAN_GROUP && g + tk < nt)
-                            Y[(size_t)(tb + g + tk) * p.C] = from_f32<T>(fmaf(D, xs[k], ys[k]) * silu_f(zs[k]));
+                        if (on && tk < GROUP && g + tk < nt)
+                            Y[(size_t)(tb + g + tk) * p.C] = from_f32<T>(fmaf(D, xs[k], ys[k]) * silu_for<T>(zs[k]));
                     }
                 }
             }
@@ -266,13 +282,80 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) 
         if (PHASE != 2 && on) {
             float* dst = PHASE == 0 ? slot : piece;
             if (vec) {
-                if (n0 < N) *reinterpret_cast<float4*>(dst) = make_float4(S[0], S[1 % NS], S[2 % NS], S[3 % NS]);
+#pragma unroll
+                for (int i = 0; i < NS; i += 4)
+                    if (n0 + i < N) *reinterpret_cast<float4*>(dst + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
             } else {
 #pragma unroll
                 for (int i = 0; i < NS; i++)
                     if (n0 + i < N) dst[i] = S[i];
             }
             if (PHASE == 1 && ln == 0) p.piece_dt[(size_t)unit * p.C + c] = sum_dt;
+        }
+    }
+}
+
+// One token per span: four states per lane straight from and to memory, spans in turn per CTA column so that A is read
+// once, the next span's state requested before this one's is worked on.
+template <typename T, int L, bool VEC>
+__global__ void __launch_bounds__(SCAN_THREADS) scan_step_kernel(const ScanParams p) {
+    const int c = blockIdx.x * (SCAN_THREADS / L) + threadIdx.x / L;
+    const int ln = threadIdx.x & (L - 1), N = p.N;
+    const bool on = c < p.C;
+    const int cc = on ? c : p.C - 1;
+    constexpr int NS = 4;
+    const int n0 = ln * NS;
+    float A2[NS], S[NS], nxt[NS];
+#pragma unroll
+    for (int i = 0; i < NS; i++) A2[i] = n0 + i < N ? p.A[(size_t)cc * N + n0 + i] * LOG2E : 0.f;
+    const float bias = p.dt_bias[cc], D = p.D[cc];
+    auto request = [&](int e) {
+#pragma unroll
+        for (int i = 0; i < NS; i++) nxt[i] = 0.f;
+        if (e >= p.sp.n_entries || p.sp.start[e] == 0) return;
+        const float* s = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N + n0;
+        if (VEC) {
+            if (n0 < N) {
+                const float4 v = *reinterpret_cast<const float4*>(s);
+                nxt[0] = v.x; nxt[1] = v.y; nxt[2] = v.z; nxt[3] = v.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < NS; i++)
+                if (n0 + i < N) nxt[i] = s[i];
+        }
+    };
+    request(blockIdx.y);
+    for (int e = blockIdx.y; e < p.sp.n_entries; e += gridDim.y) {
+#pragma unroll
+        for (int i = 0; i < NS; i++) S[i] = nxt[i];
+        request(e + gridDim.y);
+        const size_t t = p.sp.cu[e];
+        const float x = to_f32(static_cast<const T*>(p.x)[t * p.C + cc]);
+        const float dt = softplus_f(p.dt[t * p.C + cc] + bias), u = dt * x;
+        const float* B = p.bc + t * p.bc_stride + n0;
+        float y = 0.f;
+#pragma unroll
+        for (int i = 0; i < NS; i++)
+            if (n0 + i < N) {
+                S[i] = fmaf(exp2_approx(dt * A2[i]), S[i], u * __ldg(B + i));
+                y = fmaf(S[i], __ldg(B + N + i), y);
+            }
+#pragma unroll
+        for (int off = L >> 1; off >= 1; off >>= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
+        float* s = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N + n0;
+        if (on) {
+            if (VEC) {
+                if (n0 < N) *reinterpret_cast<float4*>(s) = make_float4(S[0], S[1], S[2], S[3]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < NS; i++)
+                    if (n0 + i < N) s[i] = S[i];
+            }
+            if (ln == 0) {
+                y = fmaf(D, x, y);
+                static_cast<T*>(p.y)[t * p.C + c] = from_f32<T>(y * silu_for<T>(to_f32(static_cast<const T*>(p.z)[t * p.z_stride + c])));
+            }
         }
     }
 }
@@ -290,39 +373,63 @@ __global__ void scan_sweep_kernel(const ScanParams p) {
         float* piece = p.piece_state + (size_t)w * CN + i;
         const float local = *piece;
         *piece = S;
-        S = fmaf(decay_exp2(A2 * p.piece_dt[(size_t)w * p.C + c]), S, local);
+        S = fmaf(exp2_approx(A2 * p.piece_dt[(size_t)w * p.C + c]), S, local);
     }
     *slot = S;
 }
 
-int scan_lanes(int n_states) {
+// Lanes per channel: eight states each in the scan, whose inner loop then is bound by the exponentials and not by shuffles
+// and shared memory; four in the decode step, where the state's way through memory is what counts.
+int scan_lanes(int n_states, int per_lane) {
     int lanes = 1;
-    while (lanes < 32 && lanes * 4 < n_states) lanes *= 2;
+    while (lanes < 32 && lanes * per_lane < n_states) lanes *= 2;
     return lanes;
 }
 // Pieces per CTA.  Sequential over whole spans (0) when spans and channels alone fill the GPU; else runs that do.
 int scan_run(const ca_spans& sp, int channels, int n_states) {
-    const int per_block = SCAN_THREADS / scan_lanes(n_states);
+    const int per_block = SCAN_THREADS / scan_lanes(n_states, 8);
     const int64_t blocks = (channels + per_block - 1) / per_block;
-    if (sp.n_work == sp.n_entries || blocks * sp.n_entries >= 256) return 0;
-    const int64_t run = std::max<int64_t>(1, blocks * sp.n_work / 592);  // about four CTAs per SM
+    if (sp.n_work == sp.n_entries || blocks * sp.n_entries >= 444) return 0;
+    const int64_t run = std::max<int64_t>(1, blocks * sp.n_work / 740);  // about five CTAs per SM
     const int longest = (sp.max_tokens + sp.work_len - 1) / sp.work_len;
     return run >= longest ? 0 : (int)run;
 }
 
-template <typename T, int L, int NS>
+template <typename T, int L>
 void launch_scan(const ScanParams& p, cudaStream_t stream) {
-    const int per_block = SCAN_THREADS / L;
+    constexpr int NS = 8, per_block = SCAN_THREADS / L;
     const int blocks = (p.C + per_block - 1) / per_block;
-    const size_t smem = (size_t)SCAN_TOKENS * 2 * L * NS * sizeof(float);
+    const size_t smem = (size_t)2 * SCAN_TOKENS * 2 * L * NS * sizeof(float);  // at most 128 KiB (256 states)
+    if (smem > 48 * 1024) {
+        cudaFuncSetAttribute(scan_kernel<T, L, NS, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(scan_kernel<T, L, NS, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(scan_kernel<T, L, NS, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    }
     if (p.run == 0) {
-        // decode steps: a CTA takes several spans, so that its rows of A are read once
-        const int rows = p.sp.max_tokens > 1 ? p.sp.n_entries : std::min(p.sp.n_entries, std::max(1, 148 * 16 / blocks));
-        scan_kernel<T, L, NS, 0><<<dim3(blocks, rows), SCAN_THREADS, smem, stream>>>(p);
+        scan_kernel<T, L, NS, 0><<<dim3(blocks, p.sp.n_entries), SCAN_THREADS, smem, stream>>>(p);
     } else {
         scan_kernel<T, L, NS, 1><<<dim3(blocks, p.sp.n_work), SCAN_THREADS, smem, stream>>>(p);
         scan_sweep_kernel<<<dim3((unsigned)(((int64_t)p.C * p.N + 255) / 256), p.sp.n_entries), 256, 0, stream>>>(p);
         scan_kernel<T, L, NS, 2><<<dim3(blocks, p.sp.n_work), SCAN_THREADS, smem, stream>>>(p);
+    }
+}
+template <typename T, int L>
+void launch_scan_step(const ScanParams& p, cudaStream_t stream) {
+    constexpr int per_block = SCAN_THREADS / L;
+    const int blocks = (p.C + per_block - 1) / per_block;
+    const dim3 grid(blocks, std::min(p.sp.n_entries, std::max(1, 148 * 16 / blocks)));
+    if (p.N % 4 == 0) scan_step_kernel<T, L, true><<<grid, SCAN_THREADS, 0, stream>>>(p);
+    else scan_step_kernel<T, L, false><<<grid, SCAN_THREADS, 0, stream>>>(p);
+}
+// f(integral_constant L)
+template <typename F> void by_lanes(int lanes, F&& f) {
+    switch (lanes) {
+        case 1: f(std::integral_constant<int, 1>()); break;
+        case 2: f(std::integral_constant<int, 2>()); break;
+        case 4: f(std::integral_constant<int, 4>()); break;
+        case 8: f(std::integral_constant<int, 8>()); break;
+        case 16: f(std::integral_constant<int, 16>()); break;
+        default: f(std::integral_constant<int, 32>());
     }
 }
 
@@ -490,20 +597,14 @@ int conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, con
 
 template <typename T>
 int selective_scan(const ScanParams& p, cudaStream_t stream) {
-    switch (scan_lanes(p.N)) {
-        case 1: launch_scan<T, 1, 4>(p, stream); break;
-        case 2: launch_scan<T, 2, 4>(p, stream); break;
-        case 4: launch_scan<T, 4, 4>(p, stream); break;
-        case 8: launch_scan<T, 8, 4>(p, stream); break;
-        case 16: launch_scan<T, 16, 4>(p, stream); break;
-        default:
-            if (p.N <= 128) launch_scan<T, 32, 4>(p, stream);
-            else launch_scan<T, 32, 8>(p, stream);
-    }
+    if (p.sp.max_tokens == 1 && p.N <= 128)
+        by_lanes(scan_lanes(p.N, 4), [&](auto l) { launch_scan_step<T, decltype(l)::value>(p, stream); });
+    else
+        by_lanes(scan_lanes(p.N, 8), [&](auto l) { launch_scan<T, decltype(l)::value>(p, stream); });
     return done();
 }
 
-// Pieces per CTA of the tensor-core kernel (one CTA per SM): the run length that needs the fewest block times, counting two
+// Pieces per CTA of the tensor-core kernels (one CTA per SM; an even number, for blocks of 128 tokens): the run length that needs the fewest block times, counting two
 // passes for runs and one for whole spans (0).
 int decay_run(const ca_spans& sp, int heads) {
     const int longest = (sp.max_tokens + sp.work_len - 1) / sp.work_len;
@@ -511,7 +612,7 @@ int decay_run(const ca_spans& sp, int heads) {
     auto waves = [](int64_t ctas) { return (double)((ctas + 147) / 148); };
     double best = waves((int64_t)sp.n_entries * heads) * longest;
     int best_run = 0;
-    for (int run = 1; run < longest; run++) {
+    for (int run = 2; run < longest; run += 2) {
         const int64_t runs = (sp.n_work + (int64_t)(run - 1) * sp.n_entries) / run;  // at most
         const double cost = waves(runs * heads) * run * 1.4 + 2.0 + 0.1 * runs / sp.n_entries;
         if (cost < best) {
@@ -536,7 +637,9 @@ int decay_attention(const DecayParams& p, cudaStream_t stream) {
     if (std::is_same<T, __nv_bfloat16>::value && decay_mma_serves(p.dk, p.dv, p.row_stride, p.qkv, p.sp.work_len)) {
         DecayMmaParams m{p.out, p.qkv, p.row_stride, p.decay, p.state, p.scratch, p.H, p.dk, p.dv, decay_run(p.sp, p.H), p.sp};
         if (m.run > 0 && !p.scratch) return fail("decay_attention: this batch needs scratch");
-        const cudaError_t e = launch_decay_mma(m, stream);
+        // short portions leave most of a 128-token block empty
+        const bool tc = decay_tc_serves(p.dk, p.dv) && p.sp.max_tokens > 32;
+        const cudaError_t e = tc ? launch_decay_tc(m, stream) : launch_decay_mma(m, stream);
         return e == cudaSuccess ? CA_OK : fail(cudaGetErrorString(e), CA_ERR_CUDA);
     }
     const size_t smem = (size_t)(2 * DS_TOK * (p.dk + 1) + p.dk * (DS_COL + 1) + 2 * DS_TOK * (DS_COL + 1) + DS_TOK + 1) * sizeof(float);
@@ -592,6 +695,12 @@ int ca_selective_scan(void* y, const void* x, const void* z, int64_t z_stride, c
     if (dtype == CA_DTYPE_BF16) return selective_scan<__nv_bfloat16>(p, s);
     if (dtype == CA_DTYPE_F32) return selective_scan<float>(p, s);
     return fail("selective_scan: unknown element type");
+}
+
+int ca_block_status(int32_t* status, ca_stream stream) {
+    if (!status) return fail("block_status: null pointer");
+    const cudaError_t e = read_decay_status(status, static_cast<cudaStream_t>(stream));
+    return e == cudaSuccess ? CA_OK : fail(cudaGetErrorString(e), CA_ERR_CUDA);
 }
 
 int64_t ca_decay_scratch_floats(const ca_spans* sp, int n_heads, int d_key, int d_value, int dtype) {

@@ -38,7 +38,50 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 
+// sine and cosine for 16-bit kernels: the angle is brought into [-pi, pi] in two fp32 steps, then the hardware
+// functions (absolute error below 2^-20)
+__device__ __forceinline__ void fast_sincos(float a, float* sn, float* cs) {
+    const float k = rintf(a * 0.15915494309189535f);
+    float r = fmaf(k, -6.2831854820251465f, a);   // 2 pi rounded to fp32 ...
+    r = fmaf(k, 1.7484556e-7f, r);                // ... and what the rounding added
+    *sn = __sinf(r);
+    *cs = __cosf(r);
+}
+template <typename T> __device__ __forceinline__ void sincos_for(float a, float* sn, float* cs) { fast_sincos(a, sn, cs); }
+template <> __device__ __forceinline__ void sincos_for<float>(float a, float* sn, float* cs) { sincosf(a, sn, cs); }
+
+// one MUFU operation; results below 2^-126 are 0
+__device__ __forceinline__ float exp2_approx(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// for results that are rounded to T: kernels of 16-bit types use the hardware approximations (relative error about 2^-21)
+template <typename T> __device__ __forceinline__ float sigmoid_for(float z) { return rcp_approx(1.f + exp2_approx(-1.4426950408889634f * z)); }
+template <> __device__ __forceinline__ float sigmoid_for<float>(float z) { return sigmoid_f(z); }
+template <typename T> __device__ __forceinline__ float silu_for(float z) { return z * sigmoid_for<T>(z); }
+template <> __device__ __forceinline__ float silu_for<float>(float z) { return silu_f(z); }
+
+// log(1 + exp(z)) = max(z, 0) + log(1 + e), e = exp(-|z|) in (0, 1], with log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3,
+// by its power series up to s^13 (the rest is below 2^-25 of the sum)
+__device__ __forceinline__ float softplus_f(float z) {
+    const float e = exp2f(-1.4426950408889634f * fabsf(z));
+    const float s = __fdividef(e, 2.f + e), q = s * s;
+    float a = fmaf(q, 1.f / 13.f, 1.f / 11.f);
+    a = fmaf(q, a, 1.f / 9.f);
+    a = fmaf(q, a, 1.f / 7.f);
+    a = fmaf(q, a, 1.f / 5.f);
+    a = fmaf(q, a, 1.f / 3.f);
+    a = fmaf(q, a, 1.f);
+    return fmaf(2.f * s, a, fmaxf(z, 0.f));
+}
 
 }  // namespace ca

@@ -192,6 +192,13 @@ void init_block_ops(py::module& m, py::module& ops) {
             "causal depthwise convolution + SiLU over spans");
     ops.def("selective_scan", &selective_scan, py::arg("x"), py::arg("z"), py::arg("dt"), py::arg("dt_bias"), py::arg("A"), py::arg("bc"),
             py::arg("D"), py::arg("state"), py::arg("spans"), "selective scan over spans, gated by silu(z)");
+    ops.def("block_status", [](py::object device) {
+                const torch::Device d = torch::python::detail::py_object_to_device(device);
+                c10::cuda::CUDAGuard guard(d);
+                int32_t st = 0;
+                check_rc(ca_block_status(&st, c10::cuda::getCurrentCUDAStream(d.index()).stream()), "block_status");
+                return st;
+            }, py::arg("device"), "0, or 1 when a bounded wait inside a block kernel has run out");
     ops.def("decay_attention", &decay_attention, py::arg("qkv"), py::arg("decay"), py::arg("d_key"), py::arg("d_value"), py::arg("state"),
             py::arg("spans"), "linear attention with a per-head decay over spans");
 }

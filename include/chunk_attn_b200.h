@@ -407,6 +407,8 @@ CA_API int64_t ca_scan_scratch_floats(const ca_spans* spans, int channels, int n
 CA_API int ca_selective_scan(void* y, const void* x, const void* z, int64_t z_stride, const float* dt, const float* dt_bias,
                              const float* A, const float* bc, int64_t bc_stride, const float* D, float* state, float* scratch,
                              const ca_spans* spans, int channels, int n_states, int dtype, ca_stream stream);
+/* 0, or 1 when a bounded wait inside a block kernel of the current device has run out (synchronises the stream) */
+CA_API int ca_block_status(int32_t* status, ca_stream stream);
 CA_API int64_t ca_decay_scratch_floats(const ca_spans* spans, int n_heads, int d_key, int d_value, int dtype);
 CA_API int ca_decay_attention(void* out, const void* qkv, int64_t row_stride, const float* decay, float* state, float* scratch,
                               const ca_spans* spans, int n_heads, int d_key, int d_value, int dtype, ca_stream stream);
