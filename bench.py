@@ -18,7 +18,8 @@ Workloads (synthetic, seeded; synthetic_workloads.py):
          is recorded in `config.workload_choice`.
 `--workload` overrides the choice (cfg2, cfg5, cfg3_s<shared>, cfg4, short<n_seqs>: a 1024-token common
 prompt with 20-token private suffixes, sys<n_seqs>: a 2048-token system prompt with 8-token suffixes, llama: the
-decoder loop).
+decoder loop, gagorax: prefill and decode of the Gagorax decoder's layers beside a Llama layer of equal width, with the
+time of every kernel against its roofline).
 
 Every line carries `parity`: sampled (row, head) outputs of the very tensors that are timed, compared with dense
 fp64 attention computed from the seeded inputs (on N > 1 including heads owned by other ranks, regenerated from
@@ -1241,6 +1242,204 @@ def run_llama(args):
 
 
 
+# ---- the Gagorax decoder beside the Llama decoder -------------------------------------------------------------------
+BF16_PEAK = 1.59e15  # of fallback: cuBLAS bf16 burst on this pool
+
+
+def gagorax_layers():
+    """One layer of each kind at width 4096, sized like a 7B model's."""
+    ff = {"kind": "dense", "ff": 11008}
+    rot = {"base": 10000.0, "dims": 128}
+    att = lambda kv: {"type": "attention", "mlp": ff, "mixer": {"heads": 32, "kv_heads": kv, "dim": 128, "vdim": 128, "rot": rot, "scale": 128 ** -0.5}}
+    mamba = {"type": "mamba1", "mlp": None, "mixer": {"inner": 8192, "state": 16, "dt_rank": 256, "conv": 4}}
+    light = {"type": "lightning", "mlp": None, "mixer": {"heads": 32, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - i / 4) for i in range(32)]}}
+    return {"attention": [att(32)], "attention_8kv": [att(8)], "mamba1": [mamba], "lightning": [light], "mixed": [mamba, att(8), light, mamba]}
+
+
+def run_gagorax(args):
+    """Tokens per second of whole steps (the model's own step function, device time by CUDA events) for prefill and decode,
+    and the device time of each kernel alone, L2 flushed before every call, against its roofline: the larger of bytes over the
+    HBM copy peak and FLOPs over the bf16 GEMM peak."""
+    import torch
+    import chunk_attn
+    from chunk_attn import SpanBatch, ops
+    from chunk_attn.models.gagorax import GagoraxConfig, GagoraxForCausalLM
+    from chunk_attn.models.gagorax.modeling_gagorax import random_weights
+    from chunk_attn.models.llama_hf import LlamaConfig, LlamaForCausalLM
+    from chunk_attn.models.sequence import Sequence
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(0)
+    hbm = measured_peak()[0] * 1e9
+    steps, warm = min(args.steps, 30), max(3, min(args.warmup, 10))
+    prefills, decodes = ([4096], [1024] * 8), ((64, 1024), (16, 4096))
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)  # 256 MB, twice the L2
+
+    def timed(fn, n, before=None):
+        """Median device time of fn in microseconds; `before` runs untimed ahead of every call."""
+        us = []
+        for i in range(warm + n):
+            if before is not None:
+                before()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            if i >= warm:
+                us.append(a.elapsed_time(b) * 1e3)
+        return statistics.median(us)
+
+    def prompt(i, n):
+        return [(7 * i + 13 * j) % 1000 for j in range(n)]
+
+    out = {"layers": {}, "kernels": {}}
+    with torch.inference_mode():
+        for name, layers in gagorax_layers().items():
+            cfg = GagoraxConfig.from_dict({"vocab": 32000, "width": 4096, "layers": layers, "norm": {"eps": 1e-5}}, kvcache_gb=12.0, state_slots=128)
+            model = GagoraxForCausalLM(cfg, random_weights(cfg, 0, device=dev))
+            caches = model.create_kv_caches()
+
+            def clear():
+                for c in caches:
+                    c.clear()
+
+            r = {}
+            for lens in prefills:
+                toks = [prompt(i, n) for i, n in enumerate(lens)]
+                us = timed(lambda: model.step([None] * len(lens), toks, caches), steps, before=clear)
+                r["prefill_%dx%d" % (len(lens), lens[0])] = {"us": round(us, 1), "tokens_per_s": round(sum(lens) / us * 1e6)}
+            for batch, ctx in decodes:
+                clear()
+                for i in range(batch):
+                    model.step([None], [prompt(i, ctx)], caches)
+
+                def decode():
+                    x, sp, _ = model.step(list(range(batch)), [[5]] * batch, caches)
+                    return model.head_logits(x, sp.last)
+
+                us = timed(decode, steps)
+                r["decode_%d_at_%d" % (batch, ctx)] = {"us": round(us, 1), "tokens_per_s": round(batch / us * 1e6)}
+            out["layers"][name] = r
+            bad = [c.device_status() for c in caches[:-1] if c.device_status()]
+            if bad or ops.block_status(dev):
+                raise RuntimeError("device status %s" % (bad or "block"))
+            del model, caches
+        lcfg = LlamaConfig(num_hidden_layers=1, chunk_attn_kvcache_gb=12.0, torch_dtype=torch.float16, torch_device="cuda:0")
+        llama = LlamaForCausalLM(lcfg, seed=0).to(device=dev, dtype=torch.float16).eval()
+        kv = llama.create_kv_caches()
+        r = {}
+        for lens in prefills:
+            seqs = [prompt(i, n) for i, n in enumerate(lens)]
+            us = timed(lambda: llama.model([Sequence(p) for p in seqs], kv, True), steps, before=lambda: [c.clear() for c in kv])
+            r["prefill_%dx%d" % (len(lens), lens[0])] = {"us": round(us, 1), "tokens_per_s": round(sum(lens) / us * 1e6)}
+        for batch, ctx in decodes:
+            for c in kv:
+                c.clear()
+            live = []
+            for i in range(batch):
+                live.append(Sequence(prompt(i, ctx)))
+                llama([live[-1]], kv, True)
+
+            def decode():
+                for s in live:
+                    s.append(5)
+                return llama.logits(live, kv, False)
+
+            us = timed(decode, steps)
+            r["decode_%d_at_%d" % (batch, ctx)] = {"us": round(us, 1), "tokens_per_s": round(batch / us * 1e6)}
+        out["layers"]["llama"] = r
+        del llama, kv
+
+        def kernel(name, fn, nbytes, flops=0.0, like=None):
+            us = timed(fn, steps, before=flush.zero_)
+            least = max(nbytes / hbm, flops / BF16_PEAK) * 1e6
+            out["kernels"][name] = {"us": round(us, 1), "roofline_us": round(least, 1), "fraction": round(least / us, 3), "like": like}
+
+        bf, f32, f16 = torch.bfloat16, torch.float32, torch.float16
+        g = torch.Generator(device=dev).manual_seed(0)
+        rnd = lambda *s, dtype=bf: torch.randn(s, generator=g, device=dev).to(dtype)
+        W, H, d, C, N = 4096, 32, 128, 8192, 16
+        for lens in prefills:
+            E, T = len(lens), sum(lens)
+            tag = "%dx%d" % (E, lens[0])
+            sp = SpanBatch([prompt(i, n) for i, n in enumerate(lens)], [0] * E, list(range(E)), dev)
+            x, r_, gate, w, b = rnd(T, W, dtype=f32), rnd(T, W), rnd(T, W), rnd(W, dtype=f32), rnd(W, dtype=f32)
+            shift = torch.zeros(E, W, device=dev)
+            half = rnd(T, W, dtype=f16)
+            half2, hw = half.clone(), rnd(W, dtype=f16)
+            kernel("fused_add_rms_norm " + tag, lambda: ops.fused_add_rms_norm(half, half2, hw, 1e-5), 8.0 * T * W)
+            kernel("gated_norm_add " + tag, lambda: ops.gated_norm_add(x, r_, gate, b, w, 1e-5), 14.0 * T * W, like="fused_add_rms_norm")
+            kernel("token_shift " + tag, lambda: ops.token_shift(x, w, shift, sp, bf), 8.0 * T * W, like="fused_add_rms_norm")
+            kernel("norm_rows_gate " + tag, lambda: ops.norm_rows(r_, w, 1e-5, bf, gate=gate), 6.0 * T * W, like="fused_add_rms_norm")
+            u = rnd(T, 11008)
+            kernel("silu_mul (torch) " + tag, lambda: torch.nn.functional.silu(u) * u, 10.0 * T * 11008)
+            kernel("gelu_tanh " + tag, lambda: ops.gelu_tanh(u), 4.0 * T * 11008, like="silu_mul")
+            xz, taps, cb = rnd(T, 2 * C), rnd(C, 4, dtype=f32), rnd(C, dtype=f32)
+            cs = torch.zeros(E, 3, C, device=dev)
+            kernel("conv_silu " + tag, lambda: ops.conv_silu(xz[:, :C], taps, cb, cs, sp), 4.0 * T * C, like="fused_add_rms_norm")
+            xc, dt, bc = rnd(T, C), rnd(T, C, dtype=f32), rnd(T, 2 * N, dtype=f32)
+            A, D, ss = -torch.exp(rnd(C, N, dtype=f32)), rnd(C, dtype=f32), torch.zeros(E, C, N, device=dev)
+            kernel("selective_scan " + tag, lambda: ops.selective_scan(xc, xz[:, C:], dt, cb, A, bc, D, ss, sp), 10.0 * T * C)
+            qkvg, dec, ls = rnd(T, 4 * W), torch.full((H,), 0.99, device=dev), torch.zeros(E, H, d, d, device=dev)
+            # per token and head, 128-token blocks: scores and P V (half of them above the diagonal), Q S, K^T V
+            kernel("decay_attention " + tag, lambda: ops.decay_attention(qkvg, dec, d, d, ls, sp), 8.0 * T * W, flops=T * H * (2 * 128 * d + 4.0 * d * d), like="sdpa")
+            pos, q16 = torch.arange(T, device=dev) % lens[0], rnd(T, W, dtype=f16)
+            k16, table = q16.clone(), rnd(4096, d, dtype=f16)
+            kernel("rotary " + tag, lambda: ops.rotary_embedding(pos, q16, k16, d, table, True), 8.0 * T * W)
+            plain = chunk_attn.Attention(n_heads=H, d_head=d, chunk_size=64, memory_mb=4096, dtype=f16, device=dev)
+            k3, ids = q16.view(E, lens[0], H, d), [prompt(i, n) for i, n in enumerate(lens)]
+            kernel("scatter_prefill " + tag, lambda: (plain.clear(), [plain.add_seq(tokens=ids[i], k=k3[i], v=k3[i]) for i in range(E)]), 8.0 * T * W)
+            sh = (E, lens[0], H, d)
+            kernel("sdpa (torch) " + tag, lambda: torch.nn.functional.scaled_dot_product_attention(
+                q16.view(sh).transpose(1, 2), k16.view(sh).transpose(1, 2), half.view(sh).transpose(1, 2), is_causal=True),
+                8.0 * T * W, flops=sum(2.0 * n * n for n in lens) * H * d)
+            for kvh in (32, 8):
+                cache = chunk_attn.Attention.shaped(n_heads=H, n_kv_heads=kvh, d_key=d, d_value=d, scale=d ** -0.5, sink=True, memory_mb=4096, dtype=bf, device=dev)
+                cache.extend([-1] * E, ids)
+                qkv, qn = rnd(T, (H + 2 * kvh) * d), rnd(d, dtype=f32)
+                freq = (10000.0 ** (-torch.arange(64, device=dev) / 64.0)).float()
+                kernel("store_qkv kv%d %s" % (kvh, tag), lambda: cache.store_qkv(qkv, sp.positions, qn, qn, 1e-5, d, freq, freq), 4.0 * T * (H + 2 * kvh) * d, like="rotary + scatter_prefill")
+                q = cache.store_qkv(qkv, sp.positions, qn, qn, 1e-5, d, freq, freq)
+                kernel("attention_rows kv%d %s" % (kvh, tag), lambda: cache.forward_rows(q, sp.positions, freq, sp.entry_of),
+                       4.0 * T * (H + kvh) * d, flops=sum(2.0 * n * n for n in lens) * H * d, like="sdpa")
+                del cache, qkv, q
+            del x, r_, gate, half, half2, u, xz, xc, dt, qkvg, plain, q16, k16
+        for batch, ctx in decodes:
+            tag = "%d_at_%d" % (batch, ctx)
+            ids = [prompt(i, ctx) for i in range(batch)]
+            plain = chunk_attn.Attention(n_heads=H, d_head=d, chunk_size=64, memory_mb=4096, dtype=f16, device=dev)
+            k3 = rnd(ctx, H, d, dtype=f16)
+            for p in ids:
+                plain.add_seq(tokens=p, k=k3, v=k3)
+            qd = rnd(batch, H, d, dtype=f16)
+            kernel("attention (fp16) " + tag, lambda: plain.forward(q=qd), 4.0 * batch * ctx * H * d)
+            sp = SpanBatch([[5]] * batch, [ctx] * batch, list(range(batch)), dev)
+            for kvh in (32, 8):
+                cache = chunk_attn.Attention.shaped(n_heads=H, n_kv_heads=kvh, d_key=d, d_value=d, scale=d ** -0.5, sink=True, memory_mb=4096, dtype=bf, device=dev)
+                k3 = rnd(ctx, kvh, d)
+                for p in ids:
+                    cache.add_seq(tokens=p, k=k3, v=k3)
+                qkv, qn = rnd(batch, (H + 2 * kvh) * d), rnd(d, dtype=f32)
+                q = cache.store_qkv(qkv, sp.positions, qn, qn, 1e-5, append_tokens=[5] * batch)
+                kernel("attention_rows decode kv%d %s" % (kvh, tag), lambda: cache.forward_rows(q, sp.positions), 4.0 * batch * ctx * kvh * d, like="attention (fp16)")
+                del cache
+            A, D, cb = -torch.exp(rnd(C, N, dtype=f32)), rnd(C, dtype=f32), rnd(C, dtype=f32)
+            ss, xc, xz = torch.zeros(batch, C, N, device=dev), rnd(batch, C), rnd(batch, 2 * C)
+            dt, bc = rnd(batch, C, dtype=f32), rnd(batch, 2 * N, dtype=f32)
+            kernel("selective_scan decode " + tag, lambda: ops.selective_scan(xc, xz[:, C:], dt, cb, A, bc, D, ss, sp), 8.0 * batch * C * N + 10.0 * batch * C, like="attention (fp16)")
+            qkvg, dec, ls = rnd(batch, 4 * W), torch.full((H,), 0.99, device=dev), torch.zeros(batch, H, d, d, device=dev)
+            kernel("decay_attention decode " + tag, lambda: ops.decay_attention(qkvg, dec, d, d, ls, sp), 8.0 * batch * H * d * d, like="attention (fp16)")
+            del plain, ss, ls
+    value = out["layers"]["mixed"]["decode_64_at_1024"]
+    line = {"metric": "gagorax_mixed_decode_tokens_per_s", "value": value["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": steps,
+            "warmup": warm, "ms_per_step": value["us"] * 1e-3, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
+            "data": "synthetic", "config": {"workload": "gagorax: layers of width 4096 (random bf16 weights), prefill 1 x 4096 and 8 x 1024 tokens, decode 64 rows "
+            "at 1024 and 16 at 4096; value: decode of a four-layer model (mamba1, attention, lightning, mamba1) with head, 64 rows at 1024; kernels "
+            "alone with a 256 MB L2 flush before each call"}}
+    line.update(out)
+    emit(line)
+
+
 def emit(line):
     """The one JSON line goes to the process's original stdout; everything else any library prints
     (NCCL's version banner, the reference's logger) was diverted to stderr in main()."""
@@ -1262,6 +1461,8 @@ def main():
         run_cfg4(args)
     elif args.workload == "llama":
         run_llama(args)
+    elif args.workload == "gagorax":
+        run_gagorax(args)
     else:
         run_b200(args)
 

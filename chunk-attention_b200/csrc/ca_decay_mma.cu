@@ -253,12 +253,22 @@ __global__ void decay_sweep_kernel(const DecayMmaParams p) {
     float4 S = p.sp.start[e] > 0 ? *slot : make_float4(0.f, 0.f, 0.f, 0.f);
     const int end = p.sp.cu[e + 1], full = p.run * p.sp.work_len;
     const float d_full = powf(d, (float)full);
-    for (int w = p.sp.work_off[e], t = p.sp.cu[e]; w < p.sp.work_off[e + 1]; w += p.run, t += full) {
-        float4* piece = reinterpret_cast<float4*>(p.piece_state + (size_t)w * all + i);
-        const float4 local = *piece;
-        const float f = end - t >= full ? d_full : powf(d, (float)(end - t));
-        *piece = S;
-        S = make_float4(fmaf(f, S.x, local.x), fmaf(f, S.y, local.y), fmaf(f, S.z, local.z), fmaf(f, S.w, local.w));
+    constexpr int AHEAD = 8;  // runs requested together
+    const int w_end = p.sp.work_off[e + 1];
+    int t = p.sp.cu[e];
+    for (int w0 = p.sp.work_off[e]; w0 < w_end; w0 += AHEAD * p.run) {
+        float4 local[AHEAD];
+#pragma unroll
+        for (int k = 0; k < AHEAD; k++)
+            if (w0 + k * p.run < w_end) local[k] = *reinterpret_cast<const float4*>(p.piece_state + (size_t)(w0 + k * p.run) * all + i);
+#pragma unroll
+        for (int k = 0; k < AHEAD; k++) {
+            if (w0 + k * p.run >= w_end) break;
+            const float f = end - t >= full ? d_full : powf(d, (float)(end - t));
+            *reinterpret_cast<float4*>(p.piece_state + (size_t)(w0 + k * p.run) * all + i) = S;
+            S = make_float4(fmaf(f, S.x, local[k].x), fmaf(f, S.y, local[k].y), fmaf(f, S.z, local[k].z), fmaf(f, S.w, local[k].w));
+            t += full;
+        }
     }
     *slot = S;
 }

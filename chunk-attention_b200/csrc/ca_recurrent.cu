@@ -134,7 +134,7 @@ constexpr int SCAN_TOKENS = 32;  // tokens whose B and C are staged at a time (t
 // PHASE 0: whole spans: state in, outputs, state out (spans in turn per CTA column).  1: end state of the run from zero, and
 // sum of dt.  2: outputs from the run's initial state.
 template <typename T, int L, int NS, int PHASE>
-__global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) {
+__global__ void __launch_bounds__(SCAN_THREADS, 8) scan_kernel(const ScanParams p) {
     extern __shared__ __align__(16) float bc_s[];  // 2 x [SCAN_TOKENS][B: L * NS | C: L * NS], zero past N
     constexpr int GROUP = L <= 8 ? 8 : L;  // tokens whose x, dt, z are requested together, one group ahead
     constexpr int NP = L * NS, OWN = (GROUP + L - 1) / L, BUF = SCAN_TOKENS * 2 * NP;
@@ -196,16 +196,18 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) 
                 asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(p.bc + (size_t)(tb + tt) * p.bc_stride + r) : "memory");
             }
         };
-        float xs[OWN], ds[OWN], zs[OWN], nx[OWN], nd[OWN], nz[OWN];
+        float xs[OWN], ds[OWN], zs[OWN], nd[OWN];
+        T nx[OWN], nz[OWN];  // as they come: a conversion here would wait for the loads
         auto request = [&](int t) {  // this lane's tokens of the group that starts at t
 #pragma unroll
             for (int k = 0; k < OWN; k++) {
                 const int tk = ln + k * L;
-                nx[k] = nd[k] = nz[k] = 0.f;
+                nd[k] = 0.f;
+                nx[k] = nz[k] = from_f32<T>(0.f);
                 if (tk < GROUP && t + tk < t1) {
-                    nx[k] = to_f32(X[(size_t)(t + tk) * p.C]);
+                    nx[k] = X[(size_t)(t + tk) * p.C];
                     nd[k] = DT[(size_t)(t + tk) * p.C];
-                    if (PHASE != 1) nz[k] = to_f32(Z[(size_t)(t + tk) * p.z_stride]);
+                    if (PHASE != 1) nz[k] = Z[(size_t)(t + tk) * p.z_stride];
                 }
             }
         };
@@ -225,8 +227,8 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_kernel(const ScanParams p) 
                 float us[OWN], ys[OWN];
 #pragma unroll
                 for (int k = 0; k < OWN; k++) {
-                    xs[k] = nx[k];
-                    zs[k] = nz[k];
+                    xs[k] = to_f32(nx[k]);
+                    zs[k] = to_f32(nz[k]);
                     ds[k] = softplus_f(nd[k] + bias);
                     us[k] = ds[k] * xs[k];
                     ys[k] = 0.f;
@@ -614,7 +616,8 @@ int decay_run(const ca_spans& sp, int heads) {
     int best_run = 0;
     for (int run = 2; run < longest; run += 2) {
         const int64_t runs = (sp.n_work + (int64_t)(run - 1) * sp.n_entries) / run;  // at most
-        const double cost = waves(runs * heads) * run * 1.4 + 2.0 + 0.1 * runs / sp.n_entries;
+        // in times of a piece: a run's two passes with their start, and the sweep over the runs
+        const double cost = waves(runs * heads) * (run + 1.0) * 1.75 + 2.0 + 0.2 * runs;
         if (cost < best) {
             best = cost;
             best_run = run;
