@@ -1244,6 +1244,7 @@ def run_llama(args):
 
 # ---- the Gagorax decoder beside the Llama decoder -------------------------------------------------------------------
 BF16_PEAK = 1.59e15  # of fallback: cuBLAS bf16 burst on this pool
+MUFU_PEAK = 16 * 148 * 1.965e9  # exponentials per second: 16 per clock and SM at the highest clock
 
 
 def gagorax_layers():
@@ -1259,7 +1260,7 @@ def gagorax_layers():
 def run_gagorax(args):
     """Tokens per second of whole steps (the model's own step function, device time by CUDA events) for prefill and decode,
     and the device time of each kernel alone, L2 flushed before every call, against its roofline: the larger of bytes over the
-    HBM copy peak and FLOPs over the bf16 GEMM peak."""
+    HBM copy peak, FLOPs over the bf16 GEMM peak, and exponentials over the special-function rate (the scan)."""
     import torch
     import chunk_attn
     from chunk_attn import SpanBatch, ops
@@ -1350,9 +1351,9 @@ def run_gagorax(args):
         out["layers"]["llama"] = r
         del llama, kv
 
-        def kernel(name, fn, nbytes, flops=0.0, like=None):
+        def kernel(name, fn, nbytes, flops=0.0, like=None, exps=0.0):
             us = timed(fn, steps, before=flush.zero_)
-            least = max(nbytes / hbm, flops / BF16_PEAK) * 1e6
+            least = max(nbytes / hbm, flops / BF16_PEAK, exps / MUFU_PEAK) * 1e6
             out["kernels"][name] = {"us": round(us, 1), "roofline_us": round(least, 1), "fraction": round(least / us, 3), "like": like}
 
         bf, f32, f16 = torch.bfloat16, torch.float32, torch.float16
@@ -1379,7 +1380,7 @@ def run_gagorax(args):
             kernel("conv_silu " + tag, lambda: ops.conv_silu(xz[:, :C], taps, cb, cs, sp), 4.0 * T * C, like="fused_add_rms_norm")
             xc, dt, bc = rnd(T, C), rnd(T, C, dtype=f32), rnd(T, 2 * N, dtype=f32)
             A, D, ss = -torch.exp(rnd(C, N, dtype=f32)), rnd(C, dtype=f32), torch.zeros(E, C, N, device=dev)
-            kernel("selective_scan " + tag, lambda: ops.selective_scan(xc, xz[:, C:], dt, cb, A, bc, D, ss, sp), 10.0 * T * C)
+            kernel("selective_scan " + tag, lambda: ops.selective_scan(xc, xz[:, C:], dt, cb, A, bc, D, ss, sp), 10.0 * T * C, exps=float(T) * C * N)
             qkvg, dec, ls = rnd(T, 4 * W), torch.full((H,), 0.99, device=dev), torch.zeros(E, H, d, d, device=dev)
             # per token and head, 128-token blocks: scores and P V (half of them above the diagonal), Q S, K^T V
             kernel("decay_attention " + tag, lambda: ops.decay_attention(qkvg, dec, d, d, ls, sp), 8.0 * T * W, flops=T * H * (2 * 128 * d + 4.0 * d * d), like="sdpa")

@@ -371,6 +371,7 @@ __global__ void __launch_bounds__(R_THREADS) rows_mma_kernel(const RowsParams p)
 }
 
 // One warp per (row, query head): combine the row's partials, add the sink, turn the result back, store.
+template <int K>  // pairs of value elements per lane
 __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
     const int H = p.geo.n_heads * p.group;
     const int pair = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -380,9 +381,9 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
     float M = p.sink ? 0.f : R_NEG_BIG;
     for (int i = lane; i < n; i += 32) M = fmaxf(M, p.part_ml[(size_t)p.merge_slots[b + i] * H + head].x);
     M = warp_max(M);
-    float acc[4][2], L = p.sink && lane == 0 ? fast_exp2(-M) : 0.f;  // pairs lane + 32 k
+    float acc[K][2], L = p.sink && lane == 0 ? fast_exp2(-M) : 0.f;  // pairs lane + 32 k
 #pragma unroll
-    for (int k = 0; k < 4; k++) acc[k][0] = acc[k][1] = 0.f;
+    for (int k = 0; k < K; k++) acc[k][0] = acc[k][1] = 0.f;
     const int pairs = p.part_width / 2;
     for (int i0 = 0; i0 < n; i0 += 32) {
         size_t slot = 0;
@@ -394,17 +395,25 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
             L = fmaf(w, ml.y, L);
         }
         const int m = min(32, n - i0);
-#pragma unroll 4
-        for (int i = 0; i < m; i++) {
-            const float wi = __shfl_sync(0xffffffffu, w, i);
-            const float* src = p.part_o + __shfl_sync(0xffffffffu, (unsigned long long)slot, i) * p.part_width;
+        constexpr int AHEAD = 8;  // partial rows requested together
+        for (int ib = 0; ib < m; ib += AHEAD) {
+            float2 x[AHEAD][K];
 #pragma unroll
-            for (int k = 0; k < 4; k++) {
-                const int q = lane + 32 * k;
-                if (q < pairs) {
-                    const float2 x = *reinterpret_cast<const float2*>(src + 2 * q);
-                    acc[k][0] = fmaf(wi, x.x, acc[k][0]);
-                    acc[k][1] = fmaf(wi, x.y, acc[k][1]);
+            for (int i = 0; i < AHEAD; i++) {
+                const float* src = p.part_o + __shfl_sync(0xffffffffu, (unsigned long long)slot, (ib + i) & 31) * p.part_width;
+#pragma unroll
+                for (int k = 0; k < K; k++) {
+                    const int q = lane + 32 * k;
+                    x[i][k] = ib + i < m && q < pairs ? *reinterpret_cast<const float2*>(src + 2 * q) : make_float2(0.f, 0.f);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < AHEAD; i++) {
+                const float wi = __shfl_sync(0xffffffffu, w, (ib + i) & 31);
+#pragma unroll
+                for (int k = 0; k < K; k++) {
+                    acc[k][0] = fmaf(wi, x[i][k].x, acc[k][0]);
+                    acc[k][1] = fmaf(wi, x[i][k].y, acc[k][1]);
                 }
             }
         }
@@ -414,7 +423,7 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t)pair * p.out_width;
     const float pos = p.positions ? (float)p.positions[row] : 0.f;
 #pragma unroll
-    for (int k = 0; k < 4; k++) {
+    for (int k = 0; k < K; k++) {
         const int i = lane + 32 * k;
         if (2 * i >= p.out_width) break;
         float a = acc[k][0] * inv, c = acc[k][1] * inv;
@@ -447,7 +456,10 @@ cudaError_t launch(const RowsParams& p, cudaStream_t stream) {
         e = cudaGetLastError();
         if (e != cudaSuccess) return e;
         const int64_t pairs = (int64_t)p.n_rows * p.geo.n_heads * p.group;
-        rows_merge_kernel<<<(unsigned)((pairs + 7) / 8), 256, 0, stream>>>(p);
+        const unsigned grid = (unsigned)((pairs + 7) / 8);
+        if (p.part_width <= 64) rows_merge_kernel<1><<<grid, 256, 0, stream>>>(p);
+        else if (p.part_width <= 128) rows_merge_kernel<2><<<grid, 256, 0, stream>>>(p);
+        else rows_merge_kernel<4><<<grid, 256, 0, stream>>>(p);
     }
     return cudaGetLastError();
 }

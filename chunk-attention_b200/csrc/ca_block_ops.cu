@@ -144,15 +144,24 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const TI* __restrict__ x, 
     const size_t t = blockIdx.x;
     const TI* src = x + (size_t)(rows ? rows[t] : t) * x_stride;
     constexpr int STEPS = V == 1 ? 4 : (V == 8 ? 1 : 2);  // of the row a thread keeps in registers, gate included
-    float kept[STEPS][V], z[STEPS][V];
+    float kept[STEPS][V], f[STEPS][V];  // the factor (weight and gate) is ready before the reduction
     float ss = 0.f;
+    auto factor = [&](int c, float (&out)[V]) {
+        load_f<float, V>(w + c, out);
+        if (gate) {
+            float z[V];
+            load_f<T, V>(gate + t * gate_stride + c, z);
+#pragma unroll
+            for (int i = 0; i < V; i++) out[i] *= sigmoid_for<T>(z[i]);
+        }
+    };
     const int stride = blockDim.x * V;
 #pragma unroll
     for (int s = 0; s < STEPS; s++) {
         const int c = threadIdx.x * V + s * stride;
         if (c < width) {
             load_f<TI, V>(src + c, kept[s]);
-            if (gate) load_f<T, V>(gate + t * gate_stride + c, z[s]);
+            factor(c, f[s]);
 #pragma unroll
             for (int i = 0; i < V; i++) ss = fmaf(kept[s][i], kept[s][i], ss);
         }
@@ -164,23 +173,21 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const TI* __restrict__ x, 
         for (int i = 0; i < V; i++) ss = fmaf(a[i], a[i], ss);
     }
     const float inv = 1.f / sqrtf(block_sum(ss) / width + eps);
-    auto finish = [&](int c, float (&a)[V], const float (&zz)[V]) {
-        float ww[V];
-        load_f<float, V>(w + c, ww);
+    auto finish = [&](int c, float (&a)[V], const float (&ff)[V]) {
 #pragma unroll
-        for (int i = 0; i < V; i++) a[i] *= inv * ww[i] * (gate ? sigmoid_for<T>(zz[i]) : 1.f);
+        for (int i = 0; i < V; i++) a[i] *= inv * ff[i];
         store_f<T, V>(out + t * width + c, a);
     };
 #pragma unroll
     for (int s = 0; s < STEPS; s++) {
         const int c = threadIdx.x * V + s * stride;
-        if (c < width) finish(c, kept[s], z[s]);
+        if (c < width) finish(c, kept[s], f[s]);
     }
     for (int c = threadIdx.x * V + STEPS * stride; c < width; c += stride) {
-        float a[V], zz[V];
+        float a[V], ff[V];
         load_f<TI, V>(src + c, a);
-        if (gate) load_f<T, V>(gate + t * gate_stride + c, zz);
-        finish(c, a, zz);
+        factor(c, ff);
+        finish(c, a, ff);
     }
 }
 

@@ -142,9 +142,12 @@ __global__ void __launch_bounds__(SCAN_THREADS, 8) scan_kernel(const ScanParams 
     const int ln = threadIdx.x & (L - 1), base = (threadIdx.x & 31) & ~(L - 1), n0 = ln * NS, N = p.N;
     const bool on = c < p.C;
     const int cc = on ? c : p.C - 1;
-    float A2[NS];
+    uint64_t A2[NS / 2];  // pairs of states
 #pragma unroll
-    for (int i = 0; i < NS; i++) A2[i] = n0 + i < N ? p.A[(size_t)cc * N + n0 + i] * LOG2E : 0.f;
+    for (int i = 0; i < NS; i += 2) {
+        const float* a = p.A + (size_t)cc * N + n0 + i;
+        A2[i / 2] = pair_f32(n0 + i < N ? a[0] * LOG2E : 0.f, n0 + i + 1 < N ? a[1] * LOG2E : 0.f);
+    }
     const float bias = p.dt_bias[cc], D = PHASE == 1 ? 0.f : p.D[cc];
     const T* X = static_cast<const T*>(p.x) + cc;
     const T* Z = static_cast<const T*>(p.z) + cc;
@@ -187,6 +190,9 @@ __global__ void __launch_bounds__(SCAN_THREADS, 8) scan_kernel(const ScanParams 
                     if (n0 + i < N) S[i] = from[i];
             }
         }
+        uint64_t S2[NS / 2];
+#pragma unroll
+        for (int i = 0; i < NS; i += 2) S2[i / 2] = pair_f32(S[i], S[i + 1]);
         float sum_dt = 0.f;
         auto stage = [&](int tb, int buf) {  // B and C of the next tokens, asynchronously
             const int nt = min(SCAN_TOKENS, t1 - tb);
@@ -242,19 +248,24 @@ __global__ void __launch_bounds__(SCAN_THREADS, 8) scan_kernel(const ScanParams 
                         u = __shfl_sync(0xffffffffu, u, base + own);
                     }
                     const float* B = bc_s + buf * BUF + (g + k) * 2 * NP + n0;
-                    float bv[NS], cv[NS];
+                    const uint64_t dt2 = pair_f32(dt, dt), u2 = pair_f32(u, u);
+                    uint64_t y2 = 0;
 #pragma unroll
                     for (int i = 0; i < NS; i += 4) {
-                        const float4 b4 = *reinterpret_cast<const float4*>(B + i), c4 = *reinterpret_cast<const float4*>(B + NP + i);
-                        bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
-                        cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
-                    }
-                    float y = 0.f;
+                        const ulonglong2 b4 = *reinterpret_cast<const ulonglong2*>(B + i), c4 = *reinterpret_cast<const ulonglong2*>(B + NP + i);
+                        const uint64_t bb[2] = {b4.x, b4.y}, cc2[2] = {c4.x, c4.y};
 #pragma unroll
-                    for (int i = 0; i < NS; i++) {
-                        S[i] = fmaf(exp2_approx(dt * A2[i]), S[i], u * bv[i]);
-                        if (PHASE != 1) y = fmaf(S[i], cv[i], y);
+                        for (int j = 0; j < 2; j++) {
+                            uint64_t& s2 = S2[i / 2 + j];
+                            float lo, hi;
+                            unpair_f32(mul_f32x2(dt2, A2[i / 2 + j]), lo, hi);
+                            s2 = fma_f32x2(pair_f32(exp2_approx(lo), exp2_approx(hi)), s2, mul_f32x2(u2, bb[j]));
+                            if (PHASE != 1) y2 = fma_f32x2(s2, cc2[j], y2);
+                        }
                     }
+                    float y, y_hi;
+                    unpair_f32(y2, y, y_hi);
+                    y += y_hi;
                     if (PHASE == 1) {
                         sum_dt += dt;
                     } else {
@@ -281,6 +292,8 @@ __global__ void __launch_bounds__(SCAN_THREADS, 8) scan_kernel(const ScanParams 
                 }
             }
         }
+#pragma unroll
+        for (int i = 0; i < NS; i += 2) unpair_f32(S2[i / 2], S[i], S[i + 1]);
         if (PHASE != 2 && on) {
             float* dst = PHASE == 0 ? slot : piece;
             if (vec) {
@@ -297,8 +310,8 @@ __global__ void __launch_bounds__(SCAN_THREADS, 8) scan_kernel(const ScanParams 
     }
 }
 
-// One token per span: four states per lane straight from and to memory, spans in turn per CTA column so that A is read
-// once, the next span's state requested before this one's is worked on.
+// One token per span: four states per lane straight from and to memory, a few spans in turn per CTA so that A is read
+// once for them, everything of the next span requested before this one is worked on.
 template <typename T, int L, bool VEC>
 __global__ void __launch_bounds__(SCAN_THREADS) scan_step_kernel(const ScanParams p) {
     const int c = blockIdx.x * (SCAN_THREADS / L) + threadIdx.x / L;
@@ -307,57 +320,65 @@ __global__ void __launch_bounds__(SCAN_THREADS) scan_step_kernel(const ScanParam
     const int cc = on ? c : p.C - 1;
     constexpr int NS = 4;
     const int n0 = ln * NS;
-    float A2[NS], S[NS], nxt[NS];
+    float A2[NS];
 #pragma unroll
     for (int i = 0; i < NS; i++) A2[i] = n0 + i < N ? p.A[(size_t)cc * N + n0 + i] * LOG2E : 0.f;
     const float bias = p.dt_bias[cc], D = p.D[cc];
+    struct Inputs {  // of one span, as they come
+        float S[NS], B[NS], C[NS], dt;
+        T x, z;
+    } in;
     auto request = [&](int e) {
 #pragma unroll
-        for (int i = 0; i < NS; i++) nxt[i] = 0.f;
-        if (e >= p.sp.n_entries || p.sp.start[e] == 0) return;
+        for (int i = 0; i < NS; i++) in.S[i] = in.B[i] = in.C[i] = 0.f;
+        if (e >= p.sp.n_entries) return;
+        const size_t t = p.sp.cu[e];
+        in.x = static_cast<const T*>(p.x)[t * p.C + cc];
+        in.z = static_cast<const T*>(p.z)[t * p.z_stride + cc];
+        in.dt = p.dt[t * p.C + cc];
+        const float* B = p.bc + t * p.bc_stride + n0;
+#pragma unroll
+        for (int i = 0; i < NS; i++)
+            if (n0 + i < N) {
+                in.B[i] = __ldg(B + i);
+                in.C[i] = __ldg(B + N + i);
+            }
+        if (p.sp.start[e] == 0) return;
         const float* s = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N + n0;
         if (VEC) {
             if (n0 < N) {
                 const float4 v = *reinterpret_cast<const float4*>(s);
-                nxt[0] = v.x; nxt[1] = v.y; nxt[2] = v.z; nxt[3] = v.w;
+                in.S[0] = v.x; in.S[1] = v.y; in.S[2] = v.z; in.S[3] = v.w;
             }
         } else {
 #pragma unroll
             for (int i = 0; i < NS; i++)
-                if (n0 + i < N) nxt[i] = s[i];
+                if (n0 + i < N) in.S[i] = s[i];
         }
     };
     request(blockIdx.y);
     for (int e = blockIdx.y; e < p.sp.n_entries; e += gridDim.y) {
-#pragma unroll
-        for (int i = 0; i < NS; i++) S[i] = nxt[i];
+        Inputs now = in;
         request(e + gridDim.y);
-        const size_t t = p.sp.cu[e];
-        const float x = to_f32(static_cast<const T*>(p.x)[t * p.C + cc]);
-        const float dt = softplus_f(p.dt[t * p.C + cc] + bias), u = dt * x;
-        const float* B = p.bc + t * p.bc_stride + n0;
+        const float x = to_f32(now.x), dt = softplus_f(now.dt + bias), u = dt * x;
         float y = 0.f;
 #pragma unroll
-        for (int i = 0; i < NS; i++)
-            if (n0 + i < N) {
-                S[i] = fmaf(exp2_approx(dt * A2[i]), S[i], u * __ldg(B + i));
-                y = fmaf(S[i], __ldg(B + N + i), y);
-            }
+        for (int i = 0; i < NS; i++) {
+            now.S[i] = fmaf(exp2_approx(dt * A2[i]), now.S[i], u * now.B[i]);
+            y = fmaf(now.S[i], now.C[i], y);
+        }
 #pragma unroll
         for (int off = L >> 1; off >= 1; off >>= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
         float* s = p.state + ((size_t)p.sp.slot[e] * p.C + cc) * N + n0;
         if (on) {
             if (VEC) {
-                if (n0 < N) *reinterpret_cast<float4*>(s) = make_float4(S[0], S[1], S[2], S[3]);
+                if (n0 < N) *reinterpret_cast<float4*>(s) = make_float4(now.S[0], now.S[1], now.S[2], now.S[3]);
             } else {
 #pragma unroll
                 for (int i = 0; i < NS; i++)
-                    if (n0 + i < N) s[i] = S[i];
+                    if (n0 + i < N) s[i] = now.S[i];
             }
-            if (ln == 0) {
-                y = fmaf(D, x, y);
-                static_cast<T*>(p.y)[t * p.C + c] = from_f32<T>(y * silu_for<T>(to_f32(static_cast<const T*>(p.z)[t * p.z_stride + c])));
-            }
+            if (ln == 0) static_cast<T*>(p.y)[(size_t)p.sp.cu[e] * p.C + c] = from_f32<T>(fmaf(D, x, y) * silu_for<T>(to_f32(now.z)));
         }
     }
 }
@@ -392,7 +413,7 @@ int scan_run(const ca_spans& sp, int channels, int n_states) {
     const int per_block = SCAN_THREADS / scan_lanes(n_states, 8);
     const int64_t blocks = (channels + per_block - 1) / per_block;
     if (sp.n_work == sp.n_entries || blocks * sp.n_entries >= 444) return 0;
-    const int64_t run = std::max<int64_t>(1, blocks * sp.n_work / 740);  // about five CTAs per SM
+    const int64_t run = (blocks * sp.n_work + 148 * 7 - 1) / (148 * 7);  // one wave of about seven CTAs per SM
     const int longest = (sp.max_tokens + sp.work_len - 1) / sp.work_len;
     return run >= longest ? 0 : (int)run;
 }
@@ -419,7 +440,7 @@ template <typename T, int L>
 void launch_scan_step(const ScanParams& p, cudaStream_t stream) {
     constexpr int per_block = SCAN_THREADS / L;
     const int blocks = (p.C + per_block - 1) / per_block;
-    const dim3 grid(blocks, std::min(p.sp.n_entries, std::max(1, 148 * 16 / blocks)));
+    const dim3 grid(blocks, std::min(p.sp.n_entries, std::max(1, 148 * 64 / blocks)));
     if (p.N % 4 == 0) scan_step_kernel<T, L, true><<<grid, SCAN_THREADS, 0, stream>>>(p);
     else scan_step_kernel<T, L, false><<<grid, SCAN_THREADS, 0, stream>>>(p);
 }
@@ -478,17 +499,30 @@ __global__ void __launch_bounds__(DECAY_STEP_THREADS) decay_step_kernel(const De
                 v[i] = silu_f(to_f32(row[2 * Hk + h * p.dv + cg * V + i]));
                 acc[i] = 0.f;
             }
-#pragma unroll 8
-            for (int r = rg; r < p.dk; r += groups) {
-                Pack<float, V>* cell = reinterpret_cast<Pack<float, V>*>(S + (size_t)r * p.dv + cg * V);
-                Pack<float, V> s;
-                if (live) s = *cell;
+            constexpr int AHEAD = 8;  // rows requested together
+            for (int r0 = rg; r0 < p.dk; r0 += AHEAD * groups) {
+                Pack<float, V> s[AHEAD];
 #pragma unroll
-                for (int i = 0; i < V; i++) {
-                    s.v[i] = fmaf(k[r], v[i], live ? d * s.v[i] : 0.f);
-                    acc[i] = fmaf(q[r], s.v[i], acc[i]);
+                for (int x = 0; x < AHEAD; x++) {
+                    const int r = r0 + x * groups;
+                    if (live && r < p.dk) {
+                        s[x] = *reinterpret_cast<const Pack<float, V>*>(S + (size_t)r * p.dv + cg * V);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < V; i++) s[x].v[i] = 0.f;
+                    }
                 }
-                *cell = s;
+#pragma unroll
+                for (int x = 0; x < AHEAD; x++) {
+                    const int r = r0 + x * groups;
+                    if (r >= p.dk) break;
+#pragma unroll
+                    for (int i = 0; i < V; i++) {
+                        s[x].v[i] = fmaf(k[r], v[i], d * s[x].v[i]);
+                        acc[i] = fmaf(q[r], s[x].v[i], acc[i]);
+                    }
+                    *reinterpret_cast<Pack<float, V>*>(S + (size_t)r * p.dv + cg * V) = s[x];
+                }
             }
 #pragma unroll
             for (int i = 0; i < V; i++) red[rg * p.dv + cg * V + i] = acc[i];
