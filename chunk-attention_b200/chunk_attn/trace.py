@@ -1,17 +1,16 @@
-"""Replays a trace through a model: token ids come in step by step, logits go out.  Nothing is sampled.
+"""Feeds recorded token ids to a model and writes the logits it gives them, without sampling.
 
     trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N
 
-Steps are read from standard input, one JSON object a line:
+Every line of standard input is a JSON object, one step:
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "x", "tokens": [11, 4], "want": [1]}], "end": ["x"]}
 
-`entries` are the next tokens of each request and the places among them whose logits are wanted; `end` names the
-requests that are finished after the step.  A step that wants something writes <out>/<step>.f32, the logits in the order
-of the entries, as little-endian fp32; after every step the line "done <step>" is printed.
+An entry continues the request of that id (or starts it) by its tokens and asks for logits at the given indexes into them;
+requests named in `end` leave the caches once the step has run.  Where anything is asked for, <out>/<step>.f32 receives
+little-endian fp32 rows [asked, vocab], entry by entry; "done <step>" on standard output follows each step.
 
-It drives the model's own step function and caches: each entry is a span of the step, continued from what earlier steps
-left.
+The work is the model's step function on its own caches: each entry is a span of the step.
 """
 import argparse
 import json
@@ -30,7 +29,7 @@ class TraceRunner:
         self.order = []  # request ids in the caches' row order
 
     def step(self, entries, end):
-        """entries: [(id, tokens, wanted places)].  Returns the wanted logits, fp32 [n, vocab] on the CPU, or None."""
+        """entries: [(id, tokens, indexes to return)].  Returns fp32 logits [n, vocab] on the CPU, or None."""
         logits = None
         if entries:
             rows = [self.order.index(i) if i in self.order else None for i, _, _ in entries]
@@ -58,7 +57,7 @@ def main(argv=None):
     ap.add_argument("--model", required=True, help="folder with config.json and model.safetensors")
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="folder for <step>.f32")
-    ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
+    ap.add_argument("--max-tokens", type=int, required=True, help="upper bound of the tokens alive at once: sizes the KV pools")
     a = ap.parse_args(argv)
     runner = TraceRunner(load_model(a.model, dtype=getattr(torch, a.dtype)), a.max_tokens)
     for line in sys.stdin:
