@@ -121,7 +121,7 @@ def test_convolution(channels, taps, dtype, schedule):
         close(y, oracle.silu(oracle.causal_conv(x.double().numpy(), f.double().numpy(), b.double().numpy())), dtype)
 
 
-@pytest.mark.parametrize("schedule", SCHEDULES)
+@pytest.mark.parametrize("schedule", SCHEDULES + [[[700, 0, 129], [333, 3, 1]]])
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("channels,states", [(64, 16), (33, 5), (130, 40), (40, 1), (128, 64), (24, 100)])
 def test_selective_scan(channels, states, dtype, schedule):
@@ -148,7 +148,7 @@ def test_selective_scan(channels, states, dtype, schedule):
             close(state[[4, 0, 2][e]], S, torch.float32, "state")
 
 
-@pytest.mark.parametrize("schedule", SCHEDULES)
+@pytest.mark.parametrize("schedule", SCHEDULES + [[[700, 0, 129], [333, 3, 1]]])  # the last one takes runs of blocks in two passes
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("dk,dv,decay", [(16, 16, [0.9, 0.5]), (20, 36, [1.0]), (64, 64, [0.999, 0.0, 0.7]), (128, 128, [0.98, 0.9999]),
                                          (128, 64, [0.99]), (48, 80, [0.95, 0.3])])
