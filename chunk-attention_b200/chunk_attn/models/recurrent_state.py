@@ -19,6 +19,7 @@ class RecurrentState:
         self.rows = []       # slot of each live sequence, in row order
         self.length = {}     # slot -> tokens the sequence has run
         self.free = list(range(self.capacity))
+        self.views = []      # per-layer handles into the caches, where a model's layers share caches
 
     def register(self, name, shape):
         """An array of per-sequence state; read it back with state[name] (it moves when the slots grow)."""

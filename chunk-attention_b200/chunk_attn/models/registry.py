@@ -13,6 +13,12 @@ def _gagorax(folder, config, dtype, device, engine):
     return GagoraxForCausalLM(cfg, read_model_weights(folder))
 
 
+def _bikelix(folder, config, dtype, device, engine):
+    from .bikelix import BikelixConfig, BikelixForCausalLM
+    cfg = BikelixConfig.from_dict(config, torch_dtype=dtype or torch.bfloat16, torch_device=str(device), **engine)
+    return BikelixForCausalLM(cfg, read_model_weights(folder))
+
+
 def _llama(folder, config, dtype, device, engine):
     from .llama_hf import LlamaConfig, LlamaForCausalLM
     dtype = dtype or torch.float16
@@ -26,7 +32,7 @@ def _llama(folder, config, dtype, device, engine):
     return model.to(device=device, dtype=dtype).eval()
 
 
-MODELS = {"Gagorax": _gagorax, "LlamaForCausalLM": _llama}
+MODELS = {"Bikelix": _bikelix, "Gagorax": _gagorax, "LlamaForCausalLM": _llama}
 
 
 def architecture_of(config):

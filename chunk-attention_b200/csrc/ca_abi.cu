@@ -3,6 +3,7 @@
 // decode step.  No torch, no exceptions across the boundary.
 #include <cuda_runtime.h>
 
+#include <algorithm>
 #include <cmath>
 #include <cstring>
 #include <new>
@@ -52,12 +53,16 @@ int shaped_esize_of(int dtype) { return dtype == CA_DTYPE_BF16 ? 2 : esize_of(dt
 
 // pool geometry of a head shape: heads padded to whole 16-byte granules
 ca::Geometry shaped_geometry(const ca_head_shape& sh, int chunk_size, int esize) {
+    if (sh.latent) return ca::make_latent_geometry(sh.d_key, sh.d_value, chunk_size, esize);
     const int per16 = 16 / esize;
     auto pad = [&](int d) { return (d + per16 - 1) / per16 * per16; };
     return ca::make_geometry(sh.n_kv_heads, pad(sh.d_key), chunk_size, esize, pad(sh.d_value));
 }
 bool shape_ok(const ca_head_shape* sh) {
-    return sh && sh->n_heads > 0 && sh->n_kv_heads > 0 && sh->n_heads % sh->n_kv_heads == 0 && sh->d_key > 0 && sh->d_value > 0 &&
+    if (sh && sh->latent)
+        return sh->n_heads > 0 && sh->n_kv_heads == 1 && sh->d_value > 0 && sh->d_value <= 1024 && sh->d_key >= sh->d_value &&
+               sh->d_key <= 1152 && (sh->d_key - sh->d_value) % 2 == 0 && sh->window >= 0;
+    return sh && sh->window == 0 && sh->n_heads > 0 && sh->n_kv_heads > 0 && sh->n_heads % sh->n_kv_heads == 0 && sh->d_key > 0 && sh->d_value > 0 &&
            sh->d_key <= 256 && sh->d_value <= 256;
 }
 
@@ -78,6 +83,7 @@ struct ca_plan {
     int wide_mode = 1;
     int d_head = ca::FAST_D;
     int esize = 2;
+    int window = 0, group = 1;
 };
 
 namespace {
@@ -206,7 +212,7 @@ static int make_context(ca_context** out, int device, const ca_head_shape* shape
         c->shaped = true;
         c->shape = *shape;
         c->group = shape->n_heads / shape->n_kv_heads;
-        c->items = dtype == CA_DTYPE_BF16;
+        c->items = dtype == CA_DTYPE_BF16 && (!shape->latent || ca::latent_rows_serves(geo));
     }
     c->pool = pool;
     c->max_chunks = max_chunks;
@@ -354,11 +360,12 @@ static std::string plan_for(const ca_context* c, ca::Plan& plan, const ca_chunk_
         return ca::build_plan(plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold, n_ctas,
                               c->max_chunks, c->opt_split, c->geo.d_head, c->geo.esize, c->fast, c->opt_sf_tensor, c->opt_wide,
                               /*want_paths=*/!c->fast);
+    const int d_mean = c->shape.latent ? c->geo.d_head / 2 : (c->geo.d_head + c->geo.d_value) / 2;
     // items of up to 64 query rows (a sequence brings `group` of them), one partial per row; no kernel of their own for
     // short tails or wide runs
     return ca::build_plan(plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold, n_ctas, c->max_chunks,
-                          false, (c->geo.d_head + c->geo.d_value) / 2, c->geo.esize, c->items, /*seq_first_tensor=*/false,
-                          /*wide_mode=*/0, /*want_paths=*/!c->items, 64 / c->group, /*one_partial_per_row=*/true);
+                          false, d_mean, c->geo.esize, c->items, /*seq_first_tensor=*/false,
+                          /*wide_mode=*/0, /*want_paths=*/!c->items, 64 / c->group, /*one_partial_per_row=*/true, c->shape.window);
 }
 
 int ca_refresh_kernel_context(ca_context* c, const ca_chunk_info* infos, int n_infos, int n_seqs, ca_stream stream_) {
@@ -389,6 +396,8 @@ int ca_plan_build_for_context(const ca_context* c, ca_plan** out, const ca_chunk
     p->fast = c->items;
     p->d_head = c->geo.d_head;
     p->esize = c->geo.esize;
+    p->window = c->shape.window;
+    p->group = c->group;
     *out = p;
     return CA_OK;
 }
@@ -400,7 +409,7 @@ int ca_refresh_from_plan(ca_context* c, const ca_plan* plan, ca_stream stream_) 
     if (pl.n_heads != c->geo.n_heads || pl.chunk_size != c->geo.chunk_size || plan->d_head != c->geo.d_head ||
         plan->esize != c->geo.esize || plan->fast != c->items || plan->max_chunks > c->max_chunks ||
         pl.split_phases != c->opt_split || pl.tpp_threshold != c->tpp_threshold || (c->items && pl.n_ctas > n_ctas) ||
-        plan->wide_mode != c->opt_wide)
+        plan->wide_mode != c->opt_wide || plan->window != c->shape.window || plan->group != c->group)
         return fail(CA_ERR_INVALID, "the plan was built for a different geometry, pool size or set of options");
     DeviceGuard guard(c->device);
     if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
@@ -515,6 +524,7 @@ int ca_context_delta_tokens(const ca_context* c) { return c ? c->delta_tokens : 
 
 int ca_append_kv(ca_context* c, const void* k, const void* v, int n_seqs, ca_stream stream_) {
     if (!c) return fail(CA_ERR_INVALID, "context is null");
+    if (c->shape.latent) return fail(CA_ERR_INVALID, "a latent cache takes no separate keys and values");
     if (!c->valid) return fail(CA_ERR_STATE, "work list is stale: call ca_refresh_kernel_context first");
     if (n_seqs != c->meta.n_seqs) return fail(CA_ERR_INVALID, "n_seqs differs from the refreshed work list");
     if (n_seqs == 0) return CA_OK;
@@ -892,7 +902,7 @@ int ca_attention(ca_context* c, const void* q, void* out, int n_seqs, int partit
 
 int ca_store_qkv(ca_context* c, const ca_qkv_args* a, ca_stream stream_) {
     if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
-    if (!c->shaped) return fail(CA_ERR_INVALID, "store_qkv needs a context with a head shape");
+    if (!c->shaped || c->shape.latent) return fail(CA_ERR_INVALID, "store_qkv needs a context with a head shape that is not latent");
     if (a->n_tokens < 0) return fail(CA_ERR_INVALID, "negative token count");
     if (a->n_tokens == 0) return CA_OK;
     if (!a->qkv || !a->q_out || !a->positions) return fail(CA_ERR_INVALID, "qkv, q_out or positions is null");
@@ -941,7 +951,7 @@ int ca_rows_block(const ca_head_shape* shape) {
 
 int ca_attention_rows(ca_context* c, const ca_rows_args* a, ca_stream stream_) {
     if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
-    if (!c->shaped) return fail(CA_ERR_INVALID, "attention_rows needs a context with a head shape");
+    if (!c->shaped || c->shape.latent) return fail(CA_ERR_INVALID, "attention_rows needs a context with a head shape that is not latent");
     if (a->n_rows < 0) return fail(CA_ERR_INVALID, "negative row count");
     if (a->n_rows == 0) return CA_OK;
     if (!a->q || !a->out) return fail(CA_ERR_INVALID, "q or out is null");
@@ -1041,9 +1051,151 @@ int ca_attention_rows(ca_context* c, const ca_rows_args* a, ca_stream stream_) {
     return CA_OK;
 }
 
+int ca_latent_decodes(const ca_context* c) { return c && c->shape.latent && c->items; }
+
+int ca_latent_block(const ca_head_shape* shape) {
+    if (!shape_ok(shape) || shape->n_heads >= 64) return 1;
+    return 64 / shape->n_heads;  // the query heads of the block's tokens are 64 rows
+}
+
+int ca_latent_store(ca_context* c, const ca_latent_store_args* a, ca_stream stream_) {
+    if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
+    if (!c->shape.latent) return fail(CA_ERR_INVALID, "latent_store needs a latent context");
+    if (a->n_tokens < 0 || a->q_rank < 0) return fail(CA_ERR_INVALID, "negative count");
+    if (a->n_tokens == 0) return CA_OK;
+    const int rot = c->shape.d_key - c->shape.d_value;
+    if (!a->in || !a->kv_norm || !a->positions || (a->q_rank > 0 && (!a->q_out || !a->q_norm)) || (rot > 0 && !a->freq))
+        return fail(CA_ERR_INVALID, "an operand is null");
+    const bool append = a->tok_slot == nullptr;
+    if (append) {
+        if (!c->valid) return fail(CA_ERR_STATE, "work list is stale: call ca_refresh_kernel_context first");
+        if (a->n_tokens != c->meta.n_seqs) return fail(CA_ERR_INVALID, "one token per row of the refreshed work list is required");
+        if (c->max_tail_tokens + c->delta_tokens >= c->geo.chunk_size)
+            return fail(CA_ERR_STATE, "a tail chunk is full: reserve a new tail and refresh before appending");
+    }
+    DeviceGuard guard(c->device);
+    if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
+    ca::LatentStoreParams p{};
+    p.pool = c->pool;
+    p.geo = c->geo;
+    p.q_rank = a->q_rank;
+    p.kv_rank = c->shape.d_value;
+    p.rot = rot;
+    p.in = a->in;
+    p.row_stride = a->row_stride;
+    p.q_out = a->q_out;
+    p.q_norm = a->q_norm;
+    p.kv_norm = a->kv_norm;
+    p.eps = a->eps;
+    p.freq = a->freq;
+    p.positions = a->positions;
+    p.tok_slot = a->tok_slot;
+    p.tail_chunk = c->d_tail_chunk;
+    p.tail_tokens = c->d_tail_tokens;
+    p.delta_tokens = c->delta_tokens;
+    p.n_tokens = a->n_tokens;
+    CA_CUDA(ca::launch_latent_store(p, c->dtype, static_cast<cudaStream_t>(stream_)));
+    if (append) c->delta_tokens += 1;
+    return CA_OK;
+}
+
+int ca_latent_attention(ca_context* c, const ca_latent_args* a, ca_stream stream_) {
+    if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
+    if (!c->shape.latent) return fail(CA_ERR_INVALID, "latent_attention needs a latent context");
+    if (a->n_rows < 0) return fail(CA_ERR_INVALID, "negative row count");
+    if (a->n_rows == 0) return CA_OK;
+    const int rot = c->shape.d_key - c->shape.d_value;
+    if (!a->q_lat || !a->out || !a->positions || (rot > 0 && (!a->q_rot || !a->freq))) return fail(CA_ERR_INVALID, "an operand is null");
+    const bool decode = a->path_off == nullptr;
+    if (decode) {
+        if (!c->items) return fail(CA_ERR_STATE, "decode steps of this geometry are given as portions");
+        if (!c->valid) return fail(CA_ERR_STATE, "work list is stale: call ca_refresh_kernel_context first");
+        if (a->n_rows != c->meta.n_seqs) return fail(CA_ERR_INVALID, "n_rows differs from the refreshed work list");
+    } else if (!a->row_entry || !a->path_chunks || !a->blocks || a->block_rows < 1) {
+        return fail(CA_ERR_INVALID, "portions need row_entry, path_chunks and blocks");
+    }
+    DeviceGuard guard(c->device);
+    if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
+    ca::LatentParams p{};
+    p.pool = c->pool;
+    p.geo = c->geo;
+    p.n_heads = c->shape.n_heads;
+    p.kv_rank = c->shape.d_value;
+    p.rot = rot;
+    p.window = c->shape.window;
+    p.q_lat = a->q_lat;
+    p.q_rot = a->q_rot;
+    p.q_rot_row = a->q_rot_row;
+    p.q_rot_head = a->q_rot_head;
+    p.out = a->out;
+    p.n_rows = a->n_rows;
+    p.scale = c->shape.scale;
+    p.scale_log2 = c->shape.scale * 1.4426950408889634f;
+    p.sink = a->sink;
+    p.positions = a->positions;
+    p.freq = a->freq;
+    p.row_entry = a->row_entry;
+    p.path_off = a->path_off;
+    p.path_chunks = a->path_chunks;
+    p.blocks = a->blocks;
+    p.n_blocks = a->n_blocks;
+    p.block_rows = a->block_rows;
+    p.max_chunks = (int)c->max_chunks;
+    p.status = c->status;
+    p.wait_limit = c->opt_wait_limit;
+    if (decode) {
+        p.items = c->d_items;
+        p.n_items = c->meta.n_items;
+        p.item_rows = c->meta.n_items_cf > 0 ? std::max(1, 64 / c->group) * c->group : c->group;
+        p.delta_tokens = a->delta_tokens >= 0 ? a->delta_tokens : c->delta_tokens;
+        p.part_o = c->part_o;
+        p.part_ml = c->part_ml;
+        p.part_width = c->geo.d_value;
+        p.merge_off = c->d_merge_off;
+        p.merge_slots = c->d_merge_slots;
+    }
+    cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+    if (c->items) CA_CUDA(ca::launch_latent_rows(p, stream));
+    else CA_CUDA(ca::launch_latent_generic(p, c->dtype, stream));
+    return CA_OK;
+}
+
+int ca_latent_gather(ca_context* c, const ca_latent_gather_args* a, ca_stream stream_) {
+    if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
+    if (!c->shape.latent) return fail(CA_ERR_INVALID, "latent_gather needs a latent context");
+    if (a->n_rows < 0) return fail(CA_ERR_INVALID, "negative row count");
+    if (a->n_rows == 0) return CA_OK;
+    if (!a->lat || !a->rot || !a->row_span || !a->base || !a->first || !a->path_off || !a->path_chunks)
+        return fail(CA_ERR_INVALID, "an operand is null");
+    if (a->rot_stride < c->shape.d_key - c->shape.d_value || a->rot_stride % 8 || reinterpret_cast<uintptr_t>(a->lat) % 16 ||
+        reinterpret_cast<uintptr_t>(a->rot) % 16)
+        return fail(CA_ERR_INVALID, "rot_stride must be a multiple of 8 that holds the rotated elements, outputs 16-byte aligned");
+    DeviceGuard guard(c->device);
+    if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
+    ca::LatentGatherParams p{};
+    p.pool = c->pool;
+    p.geo = c->geo;
+    p.kv_rank = c->shape.d_value;
+    p.rot_dims = c->shape.d_key - c->shape.d_value;
+    p.lat = a->lat;
+    p.rot = a->rot;
+    p.rot_stride = a->rot_stride;
+    p.n_rows = a->n_rows;
+    p.row_span = a->row_span;
+    p.base = a->base;
+    p.first = a->first;
+    p.path_off = a->path_off;
+    p.path_chunks = a->path_chunks;
+    p.max_chunks = (int)c->max_chunks;
+    p.status = c->status;
+    CA_CUDA(ca::launch_latent_gather(p, c->dtype, static_cast<cudaStream_t>(stream_)));
+    return CA_OK;
+}
+
 int ca_scatter_prefill(ca_context* c, const void* k, const void* v, int64_t stride_token, int64_t stride_head,
                        int first_token, int n_tokens, const int32_t* chunk_ids, ca_stream stream_) {
     if (!c) return fail(CA_ERR_INVALID, "context is null");
+    if (c->shape.latent) return fail(CA_ERR_INVALID, "a latent cache takes no separate keys and values");
     if (n_tokens < 0 || first_token < 0) return fail(CA_ERR_INVALID, "negative token range");
     if (n_tokens == 0) return CA_OK;
     if (!k || !v || !chunk_ids) return fail(CA_ERR_INVALID, "k, v or chunk_ids is null");
@@ -1085,6 +1237,7 @@ int ca_scatter_prefill(ca_context* c, const void* k, const void* v, int64_t stri
 int ca_scatter_rows(ca_context* c, const void* k, const void* v, int64_t stride_token, int64_t stride_head,
                     int n_tokens, const int32_t* chunk_ids, const int32_t* rows, ca_stream stream_) {
     if (!c) return fail(CA_ERR_INVALID, "context is null");
+    if (c->shape.latent) return fail(CA_ERR_INVALID, "a latent cache takes no separate keys and values");
     if (n_tokens < 0) return fail(CA_ERR_INVALID, "negative token count");
     if (n_tokens == 0) return CA_OK;
     if (!k || !v || !chunk_ids || !rows) return fail(CA_ERR_INVALID, "k, v, chunk_ids or rows is null");

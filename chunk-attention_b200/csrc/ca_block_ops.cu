@@ -1,5 +1,6 @@
 // Element-wise and row-wise kernels of decoder blocks whose residual stream is kept in fp32: token shift, gated
-// sublayer output + RMS norm + residual sum, RMS norm of an fp32 row, gated RMS norm, tanh-GELU.  HBM / latency
+// sublayer output + RMS norm + residual sum, scaled residual sum + RMS norm, RMS norm of an fp32 row, gated RMS norm,
+// tanh-GELU, clamped gated linear unit, soft cap of logits.  HBM / latency
 // bound: one CTA per token (or a flat grid), fp32 arithmetic, 16-byte accesses where rows allow.
 #include "../../include/chunk_attn_b200.h"
 #include "ca_kernels.h"
@@ -191,15 +192,106 @@ __global__ void norm_rows_kernel(T* __restrict__ out, const TI* __restrict__ x, 
     }
 }
 
-// x[t] = table[ids[t]] in fp32: the start of the residual stream
+// x = y / rms(y) * w with y = alpha * x + r + bias (in place, fp32); plain = x rounded to T.  A thread keeps its part of y
+// in registers (STEPS vectors); longer rows are recomputed in the second pass.
+template <typename T, int V, int STEPS>
+__global__ void scaled_norm_kernel(float* __restrict__ x, const T* __restrict__ r, int64_t r_stride, const float* __restrict__ bias,
+                                   float alpha, const float* __restrict__ w, float eps, T* __restrict__ plain, int width) {
+    const size_t t = blockIdx.x;
+    float y[STEPS][V], ws[STEPS][V];
+    float ss = 0.f;
+    auto sum = [&](int c, float (&out)[V]) {
+        float a[V];
+        load_f<float, V>(x + t * width + c, out);
+        load_f<T, V>(r + t * r_stride + c, a);
+#pragma unroll
+        for (int i = 0; i < V; i++) out[i] = fmaf(alpha, out[i], a[i]);
+        if (bias) {
+            load_f<float, V>(bias + c, a);
+#pragma unroll
+            for (int i = 0; i < V; i++) out[i] += a[i];
+        }
+    };
+    const int stride = blockDim.x * V;
+#pragma unroll
+    for (int s = 0; s < STEPS; s++) {
+        const int c = threadIdx.x * V + s * stride;
+        if (c < width) {
+            load_f<float, V>(w + c, ws[s]);  // requested before the reduction
+            sum(c, y[s]);
+#pragma unroll
+            for (int i = 0; i < V; i++) ss = fmaf(y[s][i], y[s][i], ss);
+        }
+    }
+    for (int c = threadIdx.x * V + STEPS * stride; c < width; c += stride) {
+        float a[V];
+        sum(c, a);
+#pragma unroll
+        for (int i = 0; i < V; i++) ss = fmaf(a[i], a[i], ss);
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss) / width + eps);
+    auto finish = [&](int c, float (&a)[V], const float (&ww)[V]) {
+#pragma unroll
+        for (int i = 0; i < V; i++) a[i] *= inv * ww[i];
+        store_f<float, V>(x + t * width + c, a);
+        if (plain) store_f<T, V>(plain + t * width + c, a);
+    };
+#pragma unroll
+    for (int s = 0; s < STEPS; s++) {
+        const int c = threadIdx.x * V + s * stride;
+        if (c < width) finish(c, y[s], ws[s]);
+    }
+    for (int c = threadIdx.x * V + STEPS * stride; c < width; c += stride) {
+        float a[V], ww[V];
+        sum(c, a);
+        load_f<float, V>(w + c, ww);
+        finish(c, a, ww);
+    }
+}
+
+// x[t] = table[ids[t]] * scale in fp32: the start of the residual stream; plain = x rounded to T
 template <typename T, int V>
-__global__ void embed_rows_kernel(float* __restrict__ x, const T* __restrict__ table, const int32_t* __restrict__ ids, int width) {
+__global__ void embed_rows_kernel(float* __restrict__ x, T* __restrict__ plain, const T* __restrict__ table, const int32_t* __restrict__ ids,
+                                  float scale, int width) {
     const T* src = table + (size_t)ids[blockIdx.x] * width;
     for (int c = threadIdx.x * V; c < width; c += blockDim.x * V) {
         float a[V];
         load_f<T, V>(src + c, a);
+#pragma unroll
+        for (int i = 0; i < V; i++) a[i] *= scale;
         store_f<float, V>(x + (size_t)blockIdx.x * width + c, a);
+        if (plain) store_f<T, V>(plain + (size_t)blockIdx.x * width + c, a);
     }
+}
+
+// out = g sigmoid(slope g) (u + 1), g = min(gate + bias, limit), u = clamp(up + bias, -limit, limit); a row of `in` is gate | up
+template <typename T, int V>
+__global__ void clamped_glu_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t in_stride, const float* __restrict__ bias,
+                                   float limit, float slope, int width) {
+    const size_t t = blockIdx.x;
+    const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+    if (c >= width) return;
+    float g[V], u[V], bg[V], bu[V];
+    load_f<T, V>(in + t * in_stride + c, g);
+    load_f<T, V>(in + t * in_stride + width + c, u);
+    load_f<float, V>(bias + c, bg);
+    load_f<float, V>(bias + width + c, bu);
+#pragma unroll
+    for (int k = 0; k < V; k++) {
+        const float a = fminf(g[k] + bg[k], limit), b = fminf(fmaxf(u[k] + bu[k], -limit), limit);
+        g[k] = a * sigmoid_for<T>(slope * a) * (b + 1.f);
+    }
+    store_f<T, V>(out + t * width + c, g);
+}
+
+template <int V> __global__ void softcap_kernel(float* __restrict__ z, float cap, int64_t n) {
+    const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= n) return;
+    float a[V];
+    load_f<float, V>(z + i, a);
+#pragma unroll
+    for (int k = 0; k < V; k++) a[k] = cap * tanhf(a[k] / cap);
+    store_f<float, V>(z + i, a);
 }
 
 __device__ __forceinline__ float gelu_tanh_f(float z) {
@@ -317,17 +409,59 @@ int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const
     }, width % 8 == 0 && x_stride % 8 == 0 && (!gate || gate_stride % 8 == 0) && aligned32(x) && aligned32(weight));
 }
 
-int ca_embed_rows(float* x, const void* table, const int32_t* ids, int64_t n_tokens, int width, int dtype, ca_stream stream) {
+int ca_embed_rows(float* x, void* plain, const void* table, const int32_t* ids, float scale, int64_t n_tokens, int width, int dtype,
+                  ca_stream stream) {
     if (n_tokens < 0 || width <= 0) return fail("embed_rows: bad shape");
     if (n_tokens == 0) return CA_OK;
     if (!x || !table || !ids) return fail("embed_rows: null pointer");
-    const bool vec = width % 4 == 0 && aligned16(x) && aligned16(table);
+    const bool vec = width % 4 == 0 && aligned16(x) && aligned16(table) && aligned16(plain);
     return by_type(dtype, vec, [&](auto tv, auto vv) {
         using T = decltype(tv);
         constexpr int V = decltype(vv)::value;
         embed_rows_kernel<T, V><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
-            x, static_cast<const T*>(table), ids, width);
+            x, static_cast<T*>(plain), static_cast<const T*>(table), ids, scale, width);
     });
+}
+
+int ca_scaled_norm(float* x, const void* r, int64_t r_stride, const float* bias, float alpha, const float* weight, float eps, void* plain,
+                   int64_t n_tokens, int width, int dtype, ca_stream stream) {
+    if (n_tokens < 0 || width <= 0) return fail("scaled_norm: bad shape");
+    if (n_tokens == 0) return CA_OK;
+    if (!x || !r || !weight) return fail("scaled_norm: null pointer");
+    const bool vec = width % 4 == 0 && r_stride % 4 == 0 && aligned16(x) && aligned16(r) && aligned16(bias) && aligned16(weight) && aligned16(plain);
+    return by_type(dtype, vec, [&](auto tv, auto vv) {
+        using T = decltype(tv);
+        constexpr int V = decltype(vv)::value;
+        scaled_norm_kernel<T, V, V == 1 ? 4 : (V == 8 ? 1 : 2)><<<(unsigned)n_tokens, row_threads(width / V), 0, static_cast<cudaStream_t>(stream)>>>(
+            x, static_cast<const T*>(r), r_stride, bias, alpha, weight, eps, static_cast<T*>(plain), width);
+    }, width % 8 == 0 && r_stride % 8 == 0 && aligned32(x) && aligned32(bias) && aligned32(weight));
+}
+
+int ca_clamped_glu(void* out, const void* in, int64_t in_stride, const float* bias, float limit, float slope, int64_t n_rows, int width,
+                   int dtype, ca_stream stream) {
+    if (n_rows < 0 || width <= 0) return fail("clamped_glu: bad shape");
+    if (n_rows == 0) return CA_OK;
+    if (!out || !in || !bias) return fail("clamped_glu: null pointer");
+    const bool vec = width % 4 == 0 && in_stride % 4 == 0 && aligned16(out) && aligned16(in) && aligned16(bias);
+    return by_type(dtype, vec, [&](auto tv, auto vv) {
+        using T = decltype(tv);
+        constexpr int V = decltype(vv)::value;
+        const int units = (width + V - 1) / V, threads = units >= 256 ? 256 : row_threads(units);
+        clamped_glu_kernel<T, V><<<dim3((unsigned)n_rows, (units + threads - 1) / threads), threads, 0, static_cast<cudaStream_t>(stream)>>>(
+            static_cast<T*>(out), static_cast<const T*>(in), in_stride, bias, limit, slope, width);
+    }, width % 8 == 0 && in_stride % 8 == 0 && aligned32(bias));
+}
+
+int ca_softcap(float* z, float cap, int64_t n, ca_stream stream) {
+    if (n < 0 || !(cap > 0.f)) return fail("softcap: bad size or cap");
+    if (n == 0) return CA_OK;
+    if (!z) return fail("softcap: null pointer");
+    const int V = n % 4 == 0 && aligned16(z) ? 4 : 1;
+    const int64_t blocks = (n / V + 255) / 256;
+    if (blocks > 0x7fffffff) return fail("softcap: too many elements");
+    if (V == 4) softcap_kernel<4><<<(unsigned)blocks, 256, 0, static_cast<cudaStream_t>(stream)>>>(z, cap, n);
+    else softcap_kernel<1><<<(unsigned)blocks, 256, 0, static_cast<cudaStream_t>(stream)>>>(z, cap, n);
+    return done();
 }
 
 int ca_gelu_tanh(void* out, const void* in, int64_t in_stride, int64_t n_rows, int width, int dtype, ca_stream stream) {

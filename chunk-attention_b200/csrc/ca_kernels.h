@@ -162,6 +162,7 @@ struct RowsParams {
     int n_rows;
     float scale_log2;            // scale * log2(e)
     int sink;
+    const float* sink_scores = nullptr;  // [query heads]: a score per head instead of the sink's 0 (merge kernel only)
     const int32_t* positions;    // [n_rows]
     const float* value_freq;     // null: values are not rotated
     int subs;                    // 64-row sub-blocks of a block
@@ -184,6 +185,85 @@ struct RowsParams {
     long long wait_limit;
 };
 cudaError_t launch_attn_rows(const RowsParams& p, cudaStream_t stream);
+// one warp per (row, query head): combines the row's partials
+cudaError_t launch_rows_merge(const RowsParams& p, cudaStream_t stream);
+
+// ---- latent caches (ca_latent.cu, ca_latent_rows.cu) -----------------------------------------------------------
+struct LatentStoreParams {
+    void* pool;
+    Geometry geo;
+    int q_rank, kv_rank, rot;
+    const void* in;              // [n_tokens, row_stride]: query latent | key/value latent | shared key part
+    int64_t row_stride;
+    void* q_out;                 // [n_tokens, q_rank]
+    const float* q_norm;
+    const float* kv_norm;
+    float eps;
+    const float* freq;           // [rot / 2]
+    const int32_t* positions;
+    const int32_t* tok_slot;     // as in QkvParams
+    const int32_t* tail_chunk;
+    const int32_t* tail_tokens;
+    int delta_tokens;
+    int n_tokens;
+};
+cudaError_t launch_latent_store(const LatentStoreParams& p, int dtype, cudaStream_t stream);
+
+struct LatentParams {
+    const void* pool;
+    Geometry geo;
+    int n_heads, kv_rank, rot;
+    int window;                  // 0: none
+    const void* q_lat;           // [n_rows, n_heads, kv_rank]
+    const void* q_rot;           // not rotated yet; strides in elements
+    int64_t q_rot_row, q_rot_head;
+    void* out;                   // [n_rows, n_heads, kv_rank]
+    int n_rows;
+    float scale, scale_log2;     // scale and scale * log2(e)
+    const float* sink;           // [n_heads] or null
+    const int32_t* positions;    // [n_rows]
+    const float* freq;           // [rot / 2]
+    // portions
+    const int32_t* row_entry;
+    const int32_t* path_off;     // null: decode
+    const int32_t* path_chunks;
+    const int32_t* blocks;       // [n_blocks][4]: span, first token, end token, 0
+    int n_blocks, block_rows;
+    // decode: the planner's items
+    const int4* items;
+    int n_items;
+    int item_rows;               // most query rows (tokens x heads) of an item
+    int delta_tokens;
+    float* part_o;               // [slots][part_width]
+    float2* part_ml;
+    int part_width;
+    const int32_t* merge_off;
+    const int32_t* merge_slots;
+    int max_chunks;
+    int* status;
+    long long wait_limit;
+};
+cudaError_t launch_latent_generic(const LatentParams& p, int dtype, cudaStream_t stream);  // portions, any geometry
+bool latent_rows_serves(const Geometry& g);
+cudaError_t launch_latent_rows(const LatentParams& p, cudaStream_t stream);                // bf16, 64-token chunks
+
+struct LatentGatherParams {
+    const void* pool;
+    Geometry geo;
+    int kv_rank, rot_dims;
+    void* lat;                   // [n_rows, kv_rank]
+    void* rot;                   // [n_rows, rot_stride]
+    int rot_stride;
+    int n_rows;
+    const int32_t* row_span;
+    const int32_t* base;
+    const int32_t* first;
+    const int32_t* path_off;
+    const int32_t* path_chunks;
+    int max_chunks;
+    int* status;
+};
+cudaError_t launch_latent_gather(const LatentGatherParams& p, int dtype, cudaStream_t stream);
 
 // ---- portions of prompts on tcgen05 (ca_attn_span.cu) -------------------------------------------------------
 struct SpanAttnParams {

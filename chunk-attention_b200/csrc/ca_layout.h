@@ -65,6 +65,18 @@ CA_HD Geometry make_geometry(int n_heads, int d_head, int chunk_size, int esize,
     return g;
 }
 
+// A latent cache: one row per token, padded to whole 128-byte lines, whose leading elements are also the value; d_value
+// (a multiple of 64) is how many of them the attention kernels accumulate.
+CA_HD Geometry make_latent_geometry(int d_key, int d_value, int chunk_size, int esize) {
+    const int line = 128 / esize;
+    Geometry g = make_geometry(1, (d_key + line - 1) / line * line, chunk_size, esize);
+    g.d_value = (d_value + 63) / 64 * 64;
+    g.v_gpr = g.d_value / g.epg;
+    g.v_tile_elems = 0;
+    g.chunk_elems = g.tile_elems;
+    return g;
+}
+
 // the geometry as seen by code that handles "a tile": the K side (kv = 0) or the V side (kv = 1)
 CA_HD Geometry tile_side(const Geometry& g, int kv) {
     Geometry s = g;

@@ -15,6 +15,7 @@ struct Unit {
     int32_t n_chunks;
     int32_t row_begin, n_rows, splits, last_tokens;
     bool tail;                    // last tile is a sequence's tail chunk
+    int32_t first = 0;            // position of the first token (plans with a window)
 };
 
 std::string fmt(const char* f, long a = 0, long b = 0, long c = 0) {
@@ -47,7 +48,7 @@ void cut_units(Plan& plan, const std::vector<Unit>& units, size_t ubegin, size_t
             plan.items.emplace_back();
             PlanItem& it = plan.items.back();
             it.n_tiles = len;
-            it.head = 0;
+            it.first = plan.window > 0 ? un.first + j * plan.chunk_size : 0;
             it.row_begin = un.row_begin;
             it.n_rows = un.n_rows;
             it.slot_base = n_slots;
@@ -60,6 +61,20 @@ void cut_units(Plan& plan, const std::vector<Unit>& units, size_t ubegin, size_t
             remaining -= (int64_t)len * n_heads;
         }
     }
+}
+
+// Position of the first token of every entry of a depth-first chunk list.
+std::vector<int32_t> first_positions(const ca_chunk_info* infos, int n_infos) {
+    struct Open { int32_t b, e, end; };
+    std::vector<Open> above;  // entries on the path to the current one
+    std::vector<int32_t> first((size_t)n_infos);
+    for (int i = 0; i < n_infos; i++) {
+        const ca_chunk_info& ci = infos[i];
+        while (!above.empty() && !(above.back().b <= ci.seq_begin && ci.seq_end <= above.back().e)) above.pop_back();
+        first[i] = above.empty() ? 0 : above.back().end;
+        above.push_back(Open{ci.seq_begin, ci.seq_end, first[i] + ci.n_tokens});
+    }
+    return first;
 }
 
 }  // namespace
@@ -87,8 +102,9 @@ void build_paths(Plan& plan) {
 std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int n_seqs, int n_heads,
                        int chunk_size, int tpp_threshold, int n_ctas, int64_t max_chunks,
                        bool split_phases, int d_head, int esize, bool fast_path, bool seq_first_tensor, int wide_mode,
-                       bool want_paths, int rows_per_item, bool one_partial_per_row) {
+                       bool want_paths, int rows_per_item, bool one_partial_per_row, int window) {
     if (rows_per_item < 1) rows_per_item = 1;
+    plan.window = window;
     // the vectors keep their capacity from one rebuild to the next
     plan.items.clear();
     plan.wide_chunks.clear();
@@ -154,6 +170,24 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
         plan.tail_tokens[s] = infos[leaf[s]].n_tokens;
     }
 
+    // ---- a window: entries that end before the window of every row they serve are not part of the work.  Tokens that are
+    // appended later only move the windows on, so what is left out stays out; along a path the entries left out come
+    // first, so that the chunks of a run keep consecutive positions.
+    std::vector<int32_t> first;
+    std::vector<char> dropped((size_t)n_infos, 0);
+    if (window > 0) {
+        first = first_positions(infos, n_infos);
+        for (int i = 0; i < n_infos; i++) {
+            const ca_chunk_info& ci = infos[i];
+            int32_t shortest = INT32_MAX;
+            for (int s = ci.seq_begin; s < ci.seq_end; s++) shortest = std::min(shortest, first[leaf[s]] + infos[leaf[s]].n_tokens);
+            if (leaf[ci.seq_begin] != i && first[i] + ci.n_tokens <= (int64_t)shortest - window) {
+                dropped[i] = 1;
+                unique_tokens -= ci.n_tokens;
+            }
+        }
+    }
+
     plan.stats.unique_kv_bytes = unique_tokens * (int64_t)n_heads * d_head * 2 * esize;
     plan.stats.n_chunks = n_infos;
     plan.stats.fast_path = fast_path ? 1 : 0;
@@ -166,13 +200,14 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
     }
 
     // ---- classify chunks, group shared ones into runs ----------------------------------------------
-    struct Run { int32_t b, e; std::vector<int32_t> chunks; };
+    struct Run { int32_t b, e; std::vector<int32_t> chunks; int32_t first; };
     std::vector<Run> runs;
     std::unordered_map<uint64_t, int> run_of;
     std::vector<char> shared(n_infos, 0);
     for (int i = 0; i < n_infos; i++) {
         const ca_chunk_info& ci = infos[i];
         const int n = ci.seq_end - ci.seq_begin;
+        if (dropped[i]) continue;
         if (n > tpp_threshold && ci.n_tokens == chunk_size) {
             shared[i] = 1;
             plan.stats.n_shared_chunks++;
@@ -182,7 +217,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
             if (f == run_of.end()) {
                 r = (int)runs.size();
                 run_of.emplace(key, r);
-                runs.push_back(Run{ci.seq_begin, ci.seq_end, {}});
+                runs.push_back(Run{ci.seq_begin, ci.seq_end, {}, window > 0 ? first[i] : 0});
             } else {
                 r = f->second;
             }
@@ -218,7 +253,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
             const int rows = std::min(rows_per_block, r.e - rb);
             if (rows <= 0) continue;
             const int splits = one_partial_per_row ? 1 : rows <= 16 ? 4 : (rows <= 32 ? 2 : 1);
-            units.push_back(Unit{r.chunks.data(), (int32_t)r.chunks.size(), rb, rows, splits, chunk_size, false});
+            units.push_back(Unit{r.chunks.data(), (int32_t)r.chunks.size(), rb, rows, splits, chunk_size, false, r.first});
         }
     }
     const size_t n_units_cf = units.size();
@@ -226,7 +261,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
     // their rows, and those serve a single row unless tpp_threshold was raised.
     std::vector<int32_t> priv_off((size_t)n_seqs + 1, 0);
     for (int i = 0; i < n_infos; i++)
-        if (!shared[i])
+        if (!shared[i] && !dropped[i])
             for (int s = infos[i].seq_begin; s < infos[i].seq_end; s++) {
                 // a non-final private tile must be full: only the tail may be partially filled
                 if (i != leaf[s] && infos[i].n_tokens != chunk_size)
@@ -234,12 +269,15 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
                 priv_off[s + 1]++;
             }
     for (int s = 0; s < n_seqs; s++) priv_off[s + 1] += priv_off[s];
-    std::vector<int32_t> priv_arena((size_t)priv_off[n_seqs]);
+    std::vector<int32_t> priv_arena((size_t)priv_off[n_seqs]), priv_first((size_t)n_seqs, -1);
     {
         std::vector<int32_t> cursor(priv_off.begin(), priv_off.end() - 1);
         for (int i = 0; i < n_infos; i++)
-            if (!shared[i])
-                for (int s = infos[i].seq_begin; s < infos[i].seq_end; s++) priv_arena[cursor[s]++] = infos[i].chunk_id;
+            if (!shared[i] && !dropped[i])
+                for (int s = infos[i].seq_begin; s < infos[i].seq_end; s++) {
+                    if (window > 0 && priv_first[s] < 0) priv_first[s] = first[i];
+                    priv_arena[cursor[s]++] = infos[i].chunk_id;
+                }
     }
     // Sequences whose private part is a single chunk (a short tail).  When there are many of them they
     // are not walked by the persistent kernel, where an item costs the same whatever its size, but by
@@ -255,7 +293,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
     for (int s = 0; s < n_seqs; s++) {
         const int32_t n_priv = priv_off[s + 1] - priv_off[s];
         std::vector<Unit>& dst = (route_short && n_priv == 1) ? short_units : units;
-        dst.push_back(Unit{priv_arena.data() + priv_off[s], n_priv, s, 1, seq_first_tensor ? 4 : 0, plan.tail_tokens[s], true});
+        dst.push_back(Unit{priv_arena.data() + priv_off[s], n_priv, s, 1, seq_first_tensor ? 4 : 0, plan.tail_tokens[s], true, priv_first[s]});
     }
 
     // ---- items ---------------------------------------------------------------------------------------------
@@ -286,7 +324,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
         plan.items.emplace_back();
         PlanItem& it = plan.items.back();
         it.n_tiles = 1;
-        it.head = 0;
+        it.first = 0;
         it.row_begin = un.row_begin;
         it.n_rows = 1;
         it.slot_base = n_slots++;
@@ -321,7 +359,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
                     plan.items.emplace_back();
                     PlanItem& it = plan.items.back();
                     it.n_tiles = c1 - c0;
-                    it.head = 0;
+                    it.first = 0;
                     it.row_begin = rb;
                     it.n_rows = rows;
                     it.slot_base = n_slots;

@@ -49,7 +49,7 @@ constexpr double WIDE_HBM_BYTES_PER_S = 6.4e12;
 
 struct PlanItem {
     int32_t n_tiles;      // 1 .. MAX_TILES_PER_ITEM
-    int32_t head;
+    int32_t first;        // position of the item's first token (plans with a window; else 0)
     int32_t row_begin;    // first row of q / out this item serves
     int32_t n_rows;       // 1: sequence-first item; >= 2: chunk-first item
     int32_t slot_base;    // first partial slot
@@ -73,6 +73,7 @@ struct Plan {
     int max_merge_len = 0;                // pieces of the row that has most
     std::vector<ca_chunk_info> infos;     // the input, kept so that the path lists can be built later
     bool has_paths = false;               // path_* are filled (build_paths)
+    int window = 0;
     std::vector<int32_t> path_off, path_chunks, path_tokens;
     std::vector<int32_t> tail_chunk, tail_tokens;
     ca_plan_stats stats{};
@@ -89,7 +90,8 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
                        int wide_mode = 1,   // 0: never route runs to the tcgen05 kernel, 1: by cost, 2: every shared run
                        bool want_paths = true,   // also build the per-row path lists of the any-geometry kernel
                        int rows_per_item = MAX_ROWS_PER_ITEM,
-                       bool one_partial_per_row = false);  // items of shared runs do not emit a partial per token split
+                       bool one_partial_per_row = false,   // items of shared runs do not emit a partial per token split
+                       int window = 0);  // > 0: chunks that lie before the window of every row they serve are left out
 // The per-row path lists (path_off / path_chunks / path_tokens) from plan.infos, for a plan built without them.
 void build_paths(Plan& plan);
 

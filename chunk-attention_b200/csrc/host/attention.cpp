@@ -36,6 +36,28 @@ Attention::Attention(Attention& other)
     shared_tables_ = other.shared_tables_;
 }
 
+Attention::Attention(Attention& source, int n_heads, double scale, int window, Attention* sibling)
+  : n_heads_(n_heads), d_head_(source.d_head_), chunk_size_(source.chunk_size_), memory_mb_(source.memory_mb_),
+    tpp_threshold_(source.tpp_threshold_), shaped_(true), shape_(source.shape_), share_prefix_(source.share_prefix_),
+    options_(source.options_) {
+    source.need_latent("reader");
+    if (n_heads <= 0 || window < 0) throw std::runtime_error("reader: n_heads must be positive, window not negative");
+    shape_.n_heads = n_heads;
+    shape_.scale = (float)scale;
+    shape_.window = window;
+    reader_ = true;
+    pool_ = source.pool_;
+    tree_ = source.tree_;
+    tables_ = source.tables_;
+    init();
+    shared_tables_ = source.shared_tables_;
+    if (sibling) {
+        if (!sibling->reader_ || sibling->shape_.n_heads != n_heads || sibling->shape_.window != window || sibling->d_head_ != d_head_)
+            throw std::runtime_error("reader: the sibling has other sizes");
+        shared_plan_ = sibling->shared_plan_;
+    }
+}
+
 Attention::Attention(const ca_head_shape& shape, int chunk_size, int memory_mb, bool share_prefix, int tpp_threshold,
                      torch::Dtype dtype, torch::Device device)
   : n_heads_(shape.n_heads), d_head_(shape.d_key), chunk_size_(chunk_size), memory_mb_(memory_mb),
@@ -76,8 +98,11 @@ void Attention::init() {
     // same sizing rule as the reference's allocator: as many whole chunks as memory_mb holds
     max_chunks_ = (int64_t)((double)memory_mb_ * 1024.0 * 1024.0 / (double)chunk_bytes_);
     c10::cuda::CUDAGuard guard(options_.device());
-    pool_ = torch::empty({std::max<int64_t>(max_chunks_, 1) * chunk_bytes_}, options_.dtype(torch::kUInt8));
-    tree_.reset(new PrefixTree(chunk_size_, max_chunks_, chunk_bytes_, share_prefix_));
+    if (!reader_) {
+        pool_ = torch::empty({std::max<int64_t>(max_chunks_, 1) * chunk_bytes_}, options_.dtype(torch::kUInt8));
+        tree_ = std::make_shared<PrefixTree>(chunk_size_, max_chunks_, chunk_bytes_, share_prefix_);
+        tables_ = std::make_shared<Tables>();
+    }
     check_rc(shaped_ ? ca_context_create_shaped(&ctx_, options_.device().index(), &shape_, chunk_size_, ca_dtype_,
                                                 pool_.data_ptr(), max_chunks_, tpp_threshold_)
                      : ca_context_create(&ctx_, options_.device().index(), n_heads_, d_head_, chunk_size_, ca_dtype_,
@@ -130,6 +155,7 @@ torch::Tensor Attention::to_cache(torch::Tensor t) const {
 }
 
 void Attention::check_kv(const torch::Tensor& k, const torch::Tensor& v, int64_t n, const char* what) const {
+    if (shape_.latent) throw std::runtime_error("a latent cache takes no separate keys and values");
     const int dv = shaped_ ? shape_.d_value : d_head_;
     if (k.dim() != 3 || v.dim() != 3 || k.size(0) != n || v.size(0) != n || k.size(1) != kv_heads() || v.size(1) != kv_heads() ||
         k.size(2) != d_head_ || v.size(2) != dv)
@@ -141,6 +167,7 @@ torch::Tensor Attention::pad_heads(torch::Tensor t, int padded) const {
 }
 
 int Attention::add_seq(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v) {
+    need_owner();
     check_kv(k, v, k.dim() > 0 ? k.size(0) : 0, "add_seq: k and v must be [n_tokens, n_heads, d_head]");
     // rows past the last token (a right-padded prompt) are ignored, as the reference's slices do
     if (k.size(0) < (int64_t)tokens.size()) throw std::runtime_error("add_seq: one K/V row per token is required");
@@ -197,6 +224,7 @@ std::shared_ptr<std::future<int>> Attention::add_seq_async(const std::vector<int
 }
 
 int Attention::append_completion(int seq_idx, const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v) {
+    need_owner();
     const int64_t n = (int64_t)tokens.size();
     check_kv(k, v, n, "append_completion: k and v must be [n_tokens, n_heads, d_head]");
     std::vector<std::pair<Chunk*, Chunk*>> pairs;
@@ -230,11 +258,13 @@ int Attention::append_completion(int seq_idx, const std::vector<int>& tokens, to
 }
 
 void Attention::remove_seq(int seq_idx) {
+    need_owner();
     tree_->remove_seq(seq_idx);
     valid_ = false;
 }
 
 std::vector<Chunk*> Attention::reserve() {
+    need_owner();
     std::vector<Chunk*> fresh = tree_->reserve();
     if (!fresh.empty()) valid_ = false;
     return fresh;
@@ -247,7 +277,7 @@ inline int64_t now_ns() {
 }  // namespace
 
 void Attention::refresh_kernel_context(bool force) {
-    if (!force && valid_) return;
+    if (!force && valid_ && planned_version_ == tree_->version()) return;
     const int64_t t0 = now_ns();
     std::vector<ca_chunk_info> infos = tree_->get_chunks();
     const int64_t t1 = now_ns();
@@ -268,6 +298,8 @@ void Attention::refresh_kernel_context(bool force) {
     const int64_t t2 = now_ns();
     check_rc(ca_refresh_from_plan(ctx_, sp.plan, stream()), "refresh_kernel_context");
     valid_ = true;
+    planned_version_ = tree_->version();
+    planned_appended_ = tree_->appended();
     const int64_t t3 = now_ns();
     host_times_.refreshes++;
     host_times_.walk_ns += t1 - t0;
@@ -290,11 +322,13 @@ std::vector<Chunk*> Attention::append_token(const std::vector<int>& tokens, torc
 }
 
 void Attention::clear() {
+    need_owner();
     tree_->clear();
     valid_ = false;
 }
 
 void Attention::duplicate(int seq_idx, int copies) {
+    need_owner();
     std::vector<std::pair<Chunk*, Chunk*>> pairs;
     tree_->duplicate(seq_idx, copies, pairs);
     if (pairs.empty()) return;
@@ -361,6 +395,7 @@ void Attention::forward_to_peers(torch::Tensor q, const std::vector<int64_t>& pe
 }
 
 std::vector<int> Attention::extend(const std::vector<int>& rows, const std::vector<std::vector<int>>& tokens) {
+    need_owner();
     const size_t n = rows.size();
     if (tokens.size() != n) throw std::runtime_error("extend: one token list per row is required");
     // everything that can be refused is refused before anything changes
@@ -377,7 +412,7 @@ std::vector<int> Attention::extend(const std::vector<int>& rows, const std::vect
     }
     if (tree_->pool().max_chunks() - tree_->pool().in_use() < need) throw std::runtime_error("ChunkAllocator: capacity reached");
     valid_ = false;
-    tables_.n_tokens = -1;
+    tables_->n_tokens = -1;
 
     std::vector<int> out(rows);
     std::vector<std::vector<int32_t>> slot_of(n);
@@ -402,32 +437,40 @@ std::vector<int> Attention::extend(const std::vector<int>& rows, const std::vect
     // tables: tok_slot | path_off | path_chunks | blocks (16-byte aligned)
     std::vector<int32_t> data;
     for (const auto& s : slot_of) data.insert(data.end(), s.begin(), s.end());
-    tables_.path_off = (int64_t)data.size();
+    tables_->path_off = (int64_t)data.size();
     std::vector<int32_t> off{0}, chunks;
+    tables_->starts.assign(n, 0);
+    tables_->lens.assign(n, 0);
     for (size_t i = 0; i < n; i++) {
         const size_t b = chunks.size();
-        for (Chunk* c = tail[i]; c->parent != nullptr; c = c->parent) chunks.push_back(c->id);
+        tables_->lens[i] = (int)tokens[i].size();
+        tables_->starts[i] = -tables_->lens[i];
+        for (Chunk* c = tail[i]; c->parent != nullptr; c = c->parent) {
+            chunks.push_back(c->id);
+            tables_->starts[i] += c->n_tokens();
+        }
         std::reverse(chunks.begin() + b, chunks.end());
         off.push_back((int32_t)chunks.size());
     }
     data.insert(data.end(), off.begin(), off.end());
-    tables_.path_chunks = (int64_t)data.size();
+    tables_->path_chunks = (int64_t)data.size();
     data.insert(data.end(), chunks.begin(), chunks.end());
     while (data.size() % 4) data.push_back(0);
-    tables_.blocks = (int64_t)data.size();
-    tables_.block_rows = ca_rows_block(&shape_);
-    tables_.n_blocks = 0;
+    tables_->blocks = (int64_t)data.size();
+    tables_->block_rows = shape_.latent ? ca_latent_block(&shape_) : ca_rows_block(&shape_);
+    tables_->n_blocks = 0;
     int32_t base = 0;
     for (size_t i = 0; i < n; i++) {
         const int len = (int)tokens[i].size();
         // the last blocks of a portion see the most context: they go first
-        for (int b = (len - 1) / tables_.block_rows; b >= 0; b--) {
-            const int lo = b * tables_.block_rows, hi = std::min(len, lo + tables_.block_rows);
+        for (int b = (len - 1) / tables_->block_rows; b >= 0; b--) {
+            const int lo = b * tables_->block_rows, hi = std::min(len, lo + tables_->block_rows);
             data.insert(data.end(), {(int32_t)i, base + lo, base + hi, 0});
-            tables_.n_blocks++;
+            tables_->n_blocks++;
         }
         base += len;
     }
+    data.insert(data.end(), tables_->starts.begin(), tables_->starts.end());
     c10::cuda::CUDAGuard guard(options_.device());
     SharedTables& st = *shared_tables_;
     if (!st.device.defined() || st.data != data) {
@@ -435,9 +478,11 @@ std::vector<int> Attention::extend(const std::vector<int>& rows, const std::vect
         std::memcpy(host.data_ptr(), data.data(), data.size() * sizeof(int32_t));
         st.device = host.to(options_.device(), torch::kInt32, /*non_blocking=*/true);
         st.data.swap(data);
+        st.blocks.clear();
+        st.windows.clear();
     }
-    tables_.device = st.device;
-    tables_.n_tokens = base;
+    tables_->device = st.device;
+    tables_->n_tokens = base;
     return out;
 }
 
@@ -484,8 +529,8 @@ torch::Tensor Attention::store_qkv(torch::Tensor qkv, torch::Tensor positions, c
         check_rc(ca_store_qkv(ctx_, &a, stream()), "store_qkv");
         tree_->append_token_ids(*append_tokens);
     } else {
-        if (tables_.n_tokens != n) throw std::runtime_error("store_qkv: extend must have described these tokens");
-        a.tok_slot = tables_.device.data_ptr<int32_t>();
+        if (tables_->n_tokens != n) throw std::runtime_error("store_qkv: extend must have described these tokens");
+        a.tok_slot = tables_->device.data_ptr<int32_t>();
         check_rc(ca_store_qkv(ctx_, &a, stream()), "store_qkv");
     }
     return q;
@@ -507,19 +552,183 @@ torch::Tensor Attention::forward_rows(torch::Tensor q, torch::Tensor positions, 
     a.positions = i32_ptr(positions, n, "forward_rows: positions must be int32 [n_rows]");
     a.value_freq = f32_ptr(value_freq, shape_.d_value / 2, "forward_rows: value_freq must be fp32 [d_value / 2]");
     if (row_entry.has_value()) {
-        if (tables_.n_tokens != n) throw std::runtime_error("forward_rows: extend must have described these tokens");
-        const int32_t* t = tables_.device.data_ptr<int32_t>();
+        if (tables_->n_tokens != n) throw std::runtime_error("forward_rows: extend must have described these tokens");
+        const int32_t* t = tables_->device.data_ptr<int32_t>();
         a.row_entry = i32_ptr(*row_entry, n, "forward_rows: row_entry must be int32 [n_rows]");
-        a.path_off = t + tables_.path_off;
-        a.path_chunks = t + tables_.path_chunks;
-        a.blocks = t + tables_.blocks;
-        a.n_blocks = tables_.n_blocks;
-        a.block_rows = tables_.block_rows;
+        a.path_off = t + tables_->path_off;
+        a.path_chunks = t + tables_->path_chunks;
+        a.blocks = t + tables_->blocks;
+        a.n_blocks = tables_->n_blocks;
+        a.block_rows = tables_->block_rows;
     } else {
         refresh_kernel_context(false);
     }
     check_rc(ca_attention_rows(ctx_, &a, stream()), "forward_rows");
     return out;
+}
+
+// ---- latent caches ------------------------------------------------------------------------------------------------------
+
+void Attention::need_latent(const char* what) const {
+    if (!shape_.latent) throw std::runtime_error(std::string(what) + " needs a latent cache");
+}
+void Attention::need_owner() const {
+    if (reader_) throw std::runtime_error("a reader does not change the cache it reads");
+}
+
+namespace {
+torch::Tensor upload(const std::vector<int32_t>& data, torch::Device device) {
+    torch::Tensor host = torch::empty({(int64_t)data.size()}, torch::TensorOptions().dtype(torch::kInt32).pinned_memory(true));
+    std::memcpy(host.data_ptr(), data.data(), data.size() * sizeof(int32_t));
+    return host.to(device, torch::kInt32, /*non_blocking=*/true);
+}
+}  // namespace
+
+// {entry, first row, end row, 0} of runs of at most block_rows rows
+const std::pair<torch::Tensor, int>& Attention::blocks_of(int block_rows) {
+    auto& all = shared_tables_->blocks;
+    auto f = all.find(block_rows);
+    if (f != all.end()) return f->second;
+    std::vector<int32_t> data;
+    int32_t base = 0;
+    for (size_t i = 0; i < tables_->lens.size(); i++) {
+        const int len = tables_->lens[i];
+        for (int b = 0; b < len; b += block_rows) data.insert(data.end(), {(int32_t)i, base + b, base + std::min(len, b + block_rows), 0});
+        base += len;
+    }
+    return all.emplace(block_rows, std::make_pair(upload(data, options_.device()), (int)(data.size() / 4))).first->second;
+}
+
+const Attention::WindowTables& Attention::window_tables() {
+    auto& all = shared_tables_->windows;
+    auto f = all.find(shape_.window);
+    if (f != all.end()) return f->second;
+    const size_t E = tables_->lens.size();
+    WindowTables w;
+    std::vector<int32_t> span, base{0}, first;
+    for (size_t i = 0; i < E; i++) {
+        const int64_t start = tables_->starts[i], len = tables_->lens[i], win = shape_.window > 0 ? shape_.window : start + len;
+        first.push_back((int32_t)std::max<int64_t>(0, start - win + 1));
+        base.push_back(base.back() + (int32_t)(start + len - first.back()));
+        // positions start .. start + len - 1 see min(position + 1, win) tokens each
+        const int64_t growing = std::min(len, std::max<int64_t>(0, win - start));
+        w.pairs += growing * (2 * start + growing + 1) / 2 + (len - growing) * win;
+        span.insert(span.end(), base[i + 1] - base[i], (int32_t)i);
+    }
+    w.rows = base.back();
+    span.insert(span.end(), base.begin(), base.end());
+    span.insert(span.end(), first.begin(), first.end());
+    w.device = upload(span, options_.device());
+    return all.emplace(shape_.window, w).first->second;
+}
+
+std::pair<int64_t, int64_t> Attention::window_load() {
+    need_latent("window_load");
+    if (tables_->n_tokens < 0) throw std::runtime_error("window_load: extend must have described the tokens");
+    const WindowTables& w = window_tables();
+    return {w.rows, w.pairs};
+}
+
+torch::Tensor Attention::store_latent(torch::Tensor in, torch::Tensor positions, torch::Tensor q_norm, torch::Tensor kv_norm, double eps,
+                                      c10::optional<torch::Tensor> freq, c10::optional<std::vector<int>> append_tokens) {
+    need_latent("store_latent");
+    need_owner();
+    const int64_t q_rank = q_norm.numel(), rot = shape_.d_key - shape_.d_value;
+    const int64_t n = in.dim() == 2 ? in.size(0) : -1;
+    if (n < 1 || in.size(1) < q_rank + shape_.d_key || in.stride(1) != 1 || in.device() != options_.device() ||
+        in.scalar_type() != c10::typeMetaToScalarType(options_.dtype()))
+        throw std::runtime_error("store_latent: [n_tokens, query latent | latent | shared key part] with the dtype and device of the cache is required");
+    ca_latent_store_args a{};
+    a.in = in.data_ptr();
+    a.row_stride = in.stride(0);
+    a.q_rank = (int32_t)q_rank;
+    a.q_norm = f32_ptr(q_norm, q_rank, "store_latent: q_norm must be fp32 [q_rank]");
+    a.kv_norm = f32_ptr(kv_norm, shape_.d_value, "store_latent: kv_norm must be fp32 [latent size]");
+    a.eps = (float)eps;
+    a.freq = f32_ptr(freq, rot / 2, "store_latent: freq must be fp32 [rotated / 2]");
+    a.positions = i32_ptr(positions, n, "store_latent: positions must be int32 [n_tokens]");
+    a.n_tokens = (int32_t)n;
+    c10::cuda::CUDAGuard guard(options_.device());
+    torch::Tensor q = torch::empty({n, q_rank}, options_);
+    a.q_out = q.data_ptr();
+    if (append_tokens.has_value()) {
+        if (tree_->tails().size() != append_tokens->size() || (int64_t)append_tokens->size() != n)
+            throw std::runtime_error("num of seqs is not equal to num of tokens");
+        reserve();
+        refresh_kernel_context(false);
+        check_rc(ca_latent_store(ctx_, &a, stream()), "store_latent");
+        tree_->append_token_ids(*append_tokens);
+    } else {
+        if (tables_->n_tokens != n) throw std::runtime_error("store_latent: extend must have described these tokens");
+        a.tok_slot = tables_->device.data_ptr<int32_t>();
+        check_rc(ca_latent_store(ctx_, &a, stream()), "store_latent");
+    }
+    return q;
+}
+
+torch::Tensor Attention::forward_latent(torch::Tensor q_lat, torch::Tensor q, torch::Tensor positions, c10::optional<torch::Tensor> freq,
+                                        c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> row_entry) {
+    need_latent("forward_latent");
+    const int64_t rot = shape_.d_key - shape_.d_value;
+    const auto st = c10::typeMetaToScalarType(options_.dtype());
+    if (q_lat.dim() != 3 || q_lat.size(1) != n_heads_ || q_lat.size(2) != shape_.d_value || !q_lat.is_contiguous() ||
+        q_lat.device() != options_.device() || q_lat.scalar_type() != st)
+        throw std::runtime_error("forward_latent: q_lat must be contiguous [n_rows, n_heads, latent size] with the dtype and device of the cache");
+    const int64_t n = q_lat.size(0);
+    if (q.dim() != 3 || q.size(0) != n || q.size(1) != n_heads_ || q.size(2) < rot || q.stride(2) != 1 || q.device() != options_.device() ||
+        q.scalar_type() != st)
+        throw std::runtime_error("forward_latent: q must be [n_rows, n_heads, unrotated + rotated] like q_lat");
+    c10::cuda::CUDAGuard guard(options_.device());
+    torch::Tensor out = torch::empty_like(q_lat);
+    ca_latent_args a{};
+    a.q_lat = q_lat.data_ptr();
+    a.q_rot = static_cast<const char*>(q.data_ptr()) + (q.size(2) - rot) * q.element_size();
+    a.q_rot_row = q.stride(0);
+    a.q_rot_head = q.stride(1);
+    a.out = out.data_ptr();
+    a.n_rows = (int32_t)n;
+    a.positions = i32_ptr(positions, n, "forward_latent: positions must be int32 [n_rows]");
+    a.freq = f32_ptr(freq, rot / 2, "forward_latent: freq must be fp32 [rotated / 2]");
+    a.sink = f32_ptr(sink, n_heads_, "forward_latent: sink must be fp32 [n_heads]");
+    a.delta_tokens = -1;
+    if (row_entry.has_value()) {
+        if (tables_->n_tokens != n) throw std::runtime_error("forward_latent: extend must have described these tokens");
+        const int32_t* t = tables_->device.data_ptr<int32_t>();
+        a.block_rows = ca_latent_block(&shape_);
+        const auto& blocks = blocks_of(a.block_rows);
+        a.row_entry = i32_ptr(*row_entry, n, "forward_latent: row_entry must be int32 [n_rows]");
+        a.path_off = t + tables_->path_off;
+        a.path_chunks = t + tables_->path_chunks;
+        a.blocks = blocks.first.data_ptr<int32_t>();
+        a.n_blocks = blocks.second;
+    } else {
+        refresh_kernel_context(false);
+        a.delta_tokens = (int32_t)(tree_->appended() - planned_appended_);
+    }
+    check_rc(ca_latent_attention(ctx_, &a, stream()), "forward_latent");
+    return out;
+}
+
+std::pair<torch::Tensor, torch::Tensor> Attention::gather_latents() {
+    need_latent("gather_latents");
+    if (tables_->n_tokens < 0) throw std::runtime_error("gather_latents: extend must have described the tokens");
+    c10::cuda::CUDAGuard guard(options_.device());
+    const WindowTables& w = window_tables();
+    const int64_t E = (int64_t)tables_->lens.size(), pad = (shape_.d_key - shape_.d_value + 63) / 64 * 64;
+    torch::Tensor lat = torch::empty({w.rows, shape_.d_value}, options_), rot = torch::empty({w.rows, std::max<int64_t>(pad, 64)}, options_);
+    const int32_t* t = w.device.data_ptr<int32_t>();
+    ca_latent_gather_args a{};
+    a.lat = lat.data_ptr();
+    a.rot = rot.data_ptr();
+    a.rot_stride = (int32_t)rot.size(1);
+    a.n_rows = (int32_t)w.rows;
+    a.row_span = t;
+    a.base = t + w.rows;
+    a.first = t + w.rows + E + 1;
+    a.path_off = tables_->device.data_ptr<int32_t>() + tables_->path_off;
+    a.path_chunks = tables_->device.data_ptr<int32_t>() + tables_->path_chunks;
+    check_rc(ca_latent_gather(ctx_, &a, stream()), "gather_latents");
+    return {lat, rot};
 }
 
 void Attention::print(Chunk* root, int level) {

@@ -14,6 +14,7 @@
 #include <deque>
 #include <functional>
 #include <future>
+#include <map>
 #include <memory>
 #include <mutex>
 #include <thread>
@@ -35,6 +36,10 @@ class Attention {
               torch::Dtype dtype, torch::Device device);
     // same configuration, fresh empty cache (one per transformer layer in the reference's model)
     Attention(Attention& other);
+    // A second view of a latent cache for a layer that reads what `source` stores, with query heads, a scale and a window of
+    // its own: pool, tree and the tables of the current portions are the source's, and only the source changes them.
+    // `sibling`: a reader of the same sizes whose work lists are shared.
+    Attention(Attention& source, int n_heads, double scale, int window, Attention* sibling);
     ~Attention();
     Attention& operator=(const Attention&) = delete;
 
@@ -58,6 +63,21 @@ class Attention {
     // [n_rows, n_heads, d_value]: decode over every row (row_entry not given), or the tokens of the last extend
     torch::Tensor forward_rows(torch::Tensor q, torch::Tensor positions, c10::optional<torch::Tensor> value_freq,
                                c10::optional<torch::Tensor> row_entry);
+    // ---- latent caches ----
+    // Projections [n_tokens, query latent | key/value latent | shared key part] to the pool; returns the normalised query
+    // latents [n_tokens, q_rank].  append_tokens as in store_qkv.
+    torch::Tensor store_latent(torch::Tensor in, torch::Tensor positions, torch::Tensor q_norm, torch::Tensor kv_norm, double eps,
+                               c10::optional<torch::Tensor> freq, c10::optional<std::vector<int>> append_tokens);
+    // q_lat [n_rows, n_heads, latent size]: queries in the latent space; q [n_rows, n_heads, unrotated + rotated], whose last
+    // part is used.  Returns [n_rows, n_heads, latent size].  row_entry as in forward_rows.
+    torch::Tensor forward_latent(torch::Tensor q_lat, torch::Tensor q, torch::Tensor positions, c10::optional<torch::Tensor> freq,
+                                 c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> row_entry);
+    // whether decode steps may leave row_entry out (bf16, 64-token chunks); otherwise every step is given by extend
+    bool latent_decodes() const { return ca_latent_decodes(ctx_) != 0; }
+    // What the current portions read: (rows of their windows in the cache, (query, key) pairs inside the windows)
+    std::pair<int64_t, int64_t> window_load();
+    // Those rows, laid out densely: latents [rows, latent size] and shared key parts [rows, padded to 64]
+    std::pair<torch::Tensor, torch::Tensor> gather_latents();
     std::vector<Chunk*> append_token(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v, bool fused = true);
     void refresh_kernel_context(bool force = false);
     std::vector<Chunk*> reserve();
@@ -118,9 +138,11 @@ class Attention {
     int64_t max_chunks_ = 0;
     int64_t chunk_bytes_ = 0;
     torch::Tensor pool_;  // one uint8 tensor: [max_chunks][n_heads][K|V][chunk_size][d_head]
-    std::unique_ptr<PrefixTree> tree_;
+    std::shared_ptr<PrefixTree> tree_;
+    bool reader_ = false;  // pool and tree belong to another cache
     ca_context* ctx_ = nullptr;
     bool valid_ = false;
+    int64_t planned_version_ = -1, planned_appended_ = 0;  // of the tree, at the last refresh
     HostTimes host_times_;
 
     // The work list of the current tree, shared by the caches made from one another with
@@ -136,16 +158,29 @@ class Attention {
     std::shared_ptr<SharedPlan> shared_plan_;
 
     // The device tables of the current portions (extend), shared the same way: equal tables are uploaded once.
+    struct WindowTables {
+        torch::Tensor device;  // row_span [rows] | base [entries + 1] | first [entries]
+        int64_t rows = 0, pairs = 0;
+    };
     struct SharedTables {
         std::vector<int32_t> data;
         torch::Tensor device;
+        // made from the portions on demand, by block size and by window
+        std::map<int, std::pair<torch::Tensor, int>> blocks;
+        std::map<int, WindowTables> windows;
     };
     std::shared_ptr<SharedTables> shared_tables_;
-    struct {
-        torch::Tensor device;      // tok_slot | path_off | path_chunks | blocks
+    struct Tables {
+        torch::Tensor device;      // tok_slot | path_off | path_chunks | blocks | starts
         int64_t n_tokens = -1, path_off = 0, path_chunks = 0, blocks = 0;
         int n_blocks = 0, block_rows = 1;
-    } tables_;
+        std::vector<int> starts, lens;  // first position and tokens of every entry
+    };
+    std::shared_ptr<Tables> tables_;
+    const std::pair<torch::Tensor, int>& blocks_of(int block_rows);
+    const WindowTables& window_tables();
+    void need_latent(const char* what) const;
+    void need_owner() const;
 
     // add_seq_async: one worker thread, started on first use, runs the queued insertions in order
     void worker_loop();

@@ -94,6 +94,39 @@ PYBIND11_MODULE(chunk_attn_c, m) {
            py::arg("n_heads"), py::arg("n_kv_heads"), py::arg("d_key"), py::arg("d_value"), py::arg("scale"),
            py::arg("sink") = false, py::arg("chunk_size") = 64, py::arg("memory_mb") = 1024, py::arg("share_prefix") = true,
            py::arg("tpp_threshold") = 1, py::arg("dtype"), py::arg("device"))
+      // a cache of one row per token for all heads: a latent vector (the value, and the leading part of the key) and a
+      // rotated key part; window: how many tokens a position sees, itself included (0: all)
+      .def_static("latent",
+           [](int n_heads, int latent, int rotated, double scale, int window, int chunk_size, int memory_mb, bool share_prefix,
+              int tpp_threshold, py::object dtype, py::object device) {
+               ca_head_shape sh{};
+               sh.n_heads = n_heads;
+               sh.n_kv_heads = 1;
+               sh.d_key = latent + rotated;
+               sh.d_value = latent;
+               sh.scale = (float)scale;
+               sh.latent = 1;
+               sh.window = window;
+               if (py::isinstance<py::str>(device)) device = py::module_::import("torch").attr("device")(device);
+               return std::make_shared<Attention>(sh, chunk_size, memory_mb, share_prefix, tpp_threshold,
+                                                  torch::python::detail::py_object_to_dtype(dtype),
+                                                  torch::python::detail::py_object_to_device(device));
+           },
+           py::arg("n_heads"), py::arg("latent"), py::arg("rotated"), py::arg("scale"), py::arg("window") = 0,
+           py::arg("chunk_size") = 64, py::arg("memory_mb") = 1024, py::arg("share_prefix") = true, py::arg("tpp_threshold") = 1,
+           py::arg("dtype"), py::arg("device"))
+      .def("reader",
+           [](Attention& self, int n_heads, double scale, int window, Attention* sibling) {
+               return std::make_shared<Attention>(self, n_heads, scale, window, sibling);
+           },
+           py::arg("n_heads"), py::arg("scale"), py::arg("window") = 0, py::arg("sibling") = nullptr)
+      .def("store_latent", &Attention::store_latent, py::arg("x"), py::arg("positions"), py::arg("q_norm"), py::arg("kv_norm"),
+           py::arg("eps"), py::arg("freq") = py::none(), py::arg("append_tokens") = py::none())
+      .def("forward_latent", &Attention::forward_latent, py::arg("q_lat"), py::arg("q"), py::arg("positions"),
+           py::arg("freq") = py::none(), py::arg("sink") = py::none(), py::arg("row_entry") = py::none())
+      .def_property_readonly("latent_decodes", &Attention::latent_decodes)
+      .def("window_load", &Attention::window_load)
+      .def("gather_latents", &Attention::gather_latents)
       .def("extend", &Attention::extend, py::arg("rows"), py::arg("tokens"))
       .def("store_qkv", &Attention::store_qkv, py::arg("qkv"), py::arg("positions"), py::arg("q_norm") = py::none(),
            py::arg("k_norm") = py::none(), py::arg("eps") = 0.0, py::arg("rot_dims") = 0, py::arg("key_freq") = py::none(),

@@ -95,16 +95,52 @@ Tensor norm_rows(Tensor x, Tensor weight, double eps, py::object dtype, c10::opt
     return out;
 }
 
-// fp32 rows of the embedding table for a batch's tokens; a token outside the table raises before anything runs
-Tensor embed_rows(Tensor table, const SpanBatch& sp) {
+// fp32 rows of the embedding table for a batch's tokens, times scale, and with want_plain the same rounded; a token outside
+// the table raises before anything runs
+py::object embed_rows(Tensor table, const SpanBatch& sp, double scale, bool want_plain) {
     need(table.is_cuda() && table.dim() == 2 && table.is_contiguous() && table.device() == sp.device(), "embed_rows: a contiguous [vocab, width] table on the spans' CUDA device is required");
     need(sp.min_token() >= 0 && sp.max_token() < table.size(0), "embed_rows: a token id lies outside the vocabulary");
     c10::cuda::CUDAGuard guard(table.device());
-    Tensor x = torch::empty({sp.n_tokens(), table.size(1)}, table.options().dtype(torch::kFloat32));
-    check_rc(ca_embed_rows(x.data_ptr<float>(), table.data_ptr(), sp.tokens.data_ptr<int32_t>(), sp.n_tokens(), (int)table.size(1),
-                           dtype_code(table, "embed_rows"), stream_of(table)),
+    Tensor x = torch::empty({sp.n_tokens(), table.size(1)}, table.options().dtype(torch::kFloat32)), plain;
+    if (want_plain) plain = torch::empty({sp.n_tokens(), table.size(1)}, table.options());
+    check_rc(ca_embed_rows(x.data_ptr<float>(), want_plain ? plain.data_ptr() : nullptr, table.data_ptr(), sp.tokens.data_ptr<int32_t>(),
+                           (float)scale, sp.n_tokens(), (int)table.size(1), dtype_code(table, "embed_rows"), stream_of(table)),
              "embed_rows");
-    return x;
+    if (!want_plain) return py::cast(x);
+    return py::make_tuple(x, plain);
+}
+
+// x (fp32, in place) = rms_norm(alpha * x + r + bias) * weight.  Returns x rounded to r's type, or x itself in fp32.
+Tensor scaled_norm(Tensor x, Tensor r, double alpha, Tensor weight, double eps, c10::optional<Tensor> bias) {
+    const int64_t T = x.size(0), W = x.size(-1);
+    need(rows_of(x, T, W) && x.is_contiguous() && x.scalar_type() == torch::kFloat32, "scaled_norm: x must be contiguous fp32 [n_tokens, width] on a CUDA device (there is no CPU path)");
+    need(rows_of(r, T, W) && f32_vec(weight, W) && (!bias.has_value() || f32_vec(*bias, W)), "scaled_norm: r must be [n_tokens, width], weight and bias fp32 [width]");
+    c10::cuda::CUDAGuard guard(x.device());
+    const bool rounded = r.scalar_type() != torch::kFloat32;
+    Tensor plain = rounded ? torch::empty({T, W}, r.options()) : x;
+    check_rc(ca_scaled_norm(x.data_ptr<float>(), r.data_ptr(), r.stride(0), bias.has_value() ? bias->data_ptr<float>() : nullptr, (float)alpha,
+                            weight.data_ptr<float>(), (float)eps, rounded ? plain.data_ptr() : nullptr, T, (int)W, dtype_code(r, "scaled_norm"),
+                            stream_of(x)),
+             "scaled_norm");
+    return plain;
+}
+
+Tensor clamped_glu(Tensor x, Tensor bias, double limit, double slope) {
+    const int64_t T = x.size(0), F = x.size(-1) / 2;
+    need(rows_of(x, T, 2 * F) && f32_vec(bias, 2 * F), "clamped_glu: [rows, gate | up] on a CUDA device and an fp32 bias [gate | up] are required");
+    c10::cuda::CUDAGuard guard(x.device());
+    Tensor out = torch::empty({T, F}, x.options());
+    check_rc(ca_clamped_glu(out.data_ptr(), x.data_ptr(), x.stride(0), bias.data_ptr<float>(), (float)limit, (float)slope, T, (int)F,
+                            dtype_code(x, "clamped_glu"), stream_of(x)),
+             "clamped_glu");
+    return out;
+}
+
+Tensor softcap(Tensor z, double cap) {
+    need(z.is_cuda() && z.scalar_type() == torch::kFloat32 && z.is_contiguous(), "softcap: a contiguous fp32 tensor on a CUDA device is required");
+    c10::cuda::CUDAGuard guard(z.device());
+    check_rc(ca_softcap(z.data_ptr<float>(), (float)cap, z.numel(), stream_of(z)), "softcap");
+    return z;
 }
 
 Tensor gelu_tanh(Tensor x) {
@@ -186,7 +222,13 @@ void init_block_ops(py::module& m, py::module& ops) {
             "x += rms_norm(r * sigmoid(gate + bias)) * weight on an fp32 stream, in place");
     ops.def("norm_rows", &norm_rows, py::arg("x"), py::arg("weight"), py::arg("eps"), py::arg("dtype"), py::arg("rows") = py::none(),
             py::arg("gate") = py::none(), "RMS norm of (selected) rows, optionally times sigmoid(gate)");
-    ops.def("embed_rows", &embed_rows, py::arg("table"), py::arg("spans"), "fp32 embedding rows of a batch's tokens");
+    ops.def("embed_rows", &embed_rows, py::arg("table"), py::arg("spans"), py::arg("scale") = 1.0, py::arg("want_plain") = false,
+            "fp32 embedding rows of a batch's tokens, times scale; with want_plain also rounded");
+    ops.def("scaled_norm", &scaled_norm, py::arg("x"), py::arg("r"), py::arg("alpha"), py::arg("weight"), py::arg("eps"), py::arg("bias") = py::none(),
+            "x = rms_norm(alpha x + r + bias) * weight on an fp32 stream, in place; returns it rounded to r's type");
+    ops.def("clamped_glu", &clamped_glu, py::arg("x"), py::arg("bias"), py::arg("limit"), py::arg("slope") = 1.702,
+            "gated linear unit of clamped halves: g sigmoid(slope g) (u + 1)");
+    ops.def("softcap", &softcap, py::arg("z"), py::arg("cap"), "cap * tanh(z / cap) in place");
     ops.def("gelu_tanh", &gelu_tanh, py::arg("x"), "tanh form of GELU");
     ops.def("conv_silu", &conv_silu, py::arg("x"), py::arg("taps"), py::arg("bias"), py::arg("state"), py::arg("spans"),
             "causal depthwise convolution + SiLU over spans");

@@ -52,6 +52,7 @@ int PrefixTree::add_seq(const std::vector<int>& tokens, std::vector<NewChunk>& c
     if (pool_.max_chunks() - pool_.in_use() < need) throw std::runtime_error("ChunkAllocator: capacity reached");
 
     // Pass 2: mutate.  Cannot fail any more.
+    version_++;
     root_->n_seqs += 1;
     for (Chunk* m : matched) m->n_seqs += 1;
     for (; start < total; start += chunk_size_) {
@@ -68,6 +69,7 @@ int PrefixTree::add_seq(const std::vector<int>& tokens, std::vector<NewChunk>& c
 
 void PrefixTree::remove_seq(int seq_idx) {
     if (seq_idx < 0 || seq_idx >= (int)tails_.size()) throw std::runtime_error("seq_idx out of range");
+    version_++;
     Chunk* node = tails_[seq_idx];
     while (node != nullptr) {
         node->n_seqs -= 1;
@@ -96,6 +98,7 @@ void PrefixTree::extend_seq(int seq_idx, const std::vector<int>& tokens, std::ve
     const int need = extend_need(seq_idx, total);
     if (total == 0) return;
     if (pool_.max_chunks() - pool_.in_use() < need) throw std::runtime_error("ChunkAllocator: capacity reached");
+    version_++;
     slots.reserve(total);
     Chunk* tail = tails_[seq_idx];
     for (int i = 0; i < total;) {
@@ -117,6 +120,7 @@ std::vector<Chunk*> PrefixTree::reserve() {
     for (size_t i = 0; i < tails_.size(); i++) {
         if (tails_[i]->full()) {
             Chunk* child = pool_.allocate();
+            version_++;
             fresh.push_back(child);
             tails_[i] = tails_[i]->add_child(child);
         }
@@ -125,6 +129,7 @@ std::vector<Chunk*> PrefixTree::reserve() {
 }
 
 void PrefixTree::append_token_ids(const std::vector<int>& tokens) {
+    appended_++;
     for (size_t i = 0; i < tails_.size(); i++) tails_[i]->append_tokens(tokens, (int)i, (int)i + 1);
 }
 
@@ -133,6 +138,7 @@ void PrefixTree::duplicate(int seq_idx, int copies, std::vector<std::pair<Chunk*
     if (copies < 1) return;
     if (seq_idx < 0 || seq_idx >= (int)tails_.size()) throw std::runtime_error("seq_idx out of range");
     if (pool_.max_chunks() - pool_.in_use() < copies) throw std::runtime_error("ChunkAllocator: capacity reached");
+    version_++;
     Chunk* leaf = tails_[seq_idx];
     for (Chunk* node = leaf->parent; node != nullptr; node = node->parent) node->n_seqs += copies;
     Chunk* parent = leaf->parent;
@@ -165,6 +171,7 @@ void PrefixTree::append_completion(int seq_idx, const std::vector<int>& tokens,
     if (pool_.max_chunks() - pool_.in_use() < need) throw std::runtime_error("ChunkAllocator: capacity reached");
     reserve();
     duplicate(seq_idx, n - 1, pairs);
+    version_++;
     for (int i = 0; i < n; i++) {
         Chunk* tail = tails_[seq_idx + i];
         slots.emplace_back(tail, tail->n_tokens());

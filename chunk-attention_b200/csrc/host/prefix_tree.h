@@ -57,10 +57,15 @@ class PrefixTree {
     ChunkPool& pool() { return pool_; }
     const ChunkPool& pool() const { return pool_; }
     int chunk_size() const { return chunk_size_; }
+    // changes whenever the chunk list does (chunks or rows come or go, a portion is added); append_token_ids is counted
+    // apart: what was planned from the chunk list stays valid then
+    int64_t version() const { return version_; }
+    int64_t appended() const { return appended_; }
 
   private:
     int chunk_size_;
     bool share_prefix_;
+    int64_t version_ = 0, appended_ = 0;
     ChunkPool pool_;
     std::unique_ptr<Chunk> root_;
     std::vector<Chunk*> tails_;

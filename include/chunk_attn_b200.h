@@ -93,14 +93,21 @@ CA_API void ca_context_destroy(ca_context* ctx);
  * whole 16-byte granules in the pool and in q ([rows, n_heads, padded d_key]); outputs are not padded.
  * score = (q . k) * scale; with `sink` the softmax denominator has one added (a score of 0 without a value).
  * fp32, fp16 and bf16.  Served by ca_store_qkv, ca_attention_rows and the pool functions; the counterpart of the
- * fixed-geometry calls for models with grouped heads. */
+ * fixed-geometry calls for models with grouped heads.
+ * With `latent` the pool has ONE row per token for all heads (n_kv_heads 1): a latent vector of d_value elements followed
+ * by d_key - d_value rotated ones, padded with zeros to whole 128-byte lines.  The row is the key, its leading d_value
+ * elements are also the value, and there are no value tiles.  Served by the ca_latent_* calls (fp32 and bf16); several
+ * contexts of different n_heads and window may read one pool.
+ * window > 0 (latent contexts): position i sees the positions j with 0 <= i - j < window. */
 typedef struct ca_head_shape {
     int32_t n_heads;     /* query heads                                   */
     int32_t n_kv_heads;  /* divides n_heads                               */
-    int32_t d_key;       /* <= 256                                        */
-    int32_t d_value;     /* <= 256                                        */
+    int32_t d_key;       /* <= 256; latent: <= 1152                       */
+    int32_t d_value;     /* <= 256; latent: <= 1024                       */
     int32_t sink;        /* 1: unit term in the softmax denominator       */
     float scale;
+    int32_t latent;
+    int32_t window;
 } ca_head_shape;
 CA_API int64_t ca_chunk_bytes_shaped(const ca_head_shape* shape, int chunk_size, int dtype);
 CA_API int ca_context_create_shaped(ca_context** out, int device, const ca_head_shape* shape, int chunk_size, int dtype,
@@ -375,13 +382,84 @@ typedef struct ca_rows_args {
 CA_API int ca_rows_block(const ca_head_shape* shape);
 CA_API int ca_attention_rows(ca_context* ctx, const ca_rows_args* args, ca_stream stream);
 
+/* Latent caches.  in: [n_tokens, row_stride] of the context's type, q_rank elements of the query latent | d_value of the
+ * key/value latent | d_key - d_value of the shared key part.  The query latent is RMS-normed (q_norm, fp32 [q_rank]) into
+ * q_out [n_tokens, q_rank] (q_rank 0: there is none); the key/value latent is RMS-normed (kv_norm, fp32 [d_value]), the
+ * shared key part rotated (element i with element i + half, by position * freq[i], fp32 [half]), both go to the pool.
+ * tok_slot as in ca_store_qkv. */
+typedef struct ca_latent_store_args {
+    const void* in;
+    int64_t row_stride;
+    int32_t q_rank;
+    const float* q_norm;
+    void* q_out;
+    const float* kv_norm;
+    float eps;
+    const float* freq;
+    const int32_t* positions;
+    const int32_t* tok_slot;
+    int32_t n_tokens;
+} ca_latent_store_args;
+CA_API int ca_latent_store(ca_context* ctx, const ca_latent_store_args* args, ca_stream stream);
+
+/* Attention over a latent cache, queries already brought into the latent space: score = (q_lat . latent + rotated q_rot .
+ * shared part) * scale, out = softmax-weighted sum of the latents.  q_lat, out: [n_rows, n_heads, d_value] contiguous;
+ * q_rot: head h of row t at q_rot + t * q_rot_row + h * q_rot_head, not yet rotated.  sink: fp32 [n_heads], one more score
+ * per head (not scaled) in the softmax denominator, or NULL.  Decode and portions as in ca_attention_rows; blocks cut the
+ * rows of every span into runs of at most block_rows (ca_latent_block).  delta_tokens (decode): tokens appended to every
+ * row since the work list was built, -1: as the context has counted them. */
+typedef struct ca_latent_args {
+    const void* q_lat;
+    const void* q_rot;
+    int64_t q_rot_row, q_rot_head;
+    void* out;
+    int32_t n_rows;
+    const int32_t* positions;   /* [n_rows]                         */
+    const float* freq;
+    const float* sink;
+    const int32_t* row_entry;   /* [n_rows]                         */
+    const int32_t* path_off;    /* [n_entries + 1]; NULL: decode    */
+    const int32_t* path_chunks;
+    const int32_t* blocks;
+    int32_t n_blocks;
+    int32_t block_rows;
+    int32_t delta_tokens;
+} ca_latent_args;
+CA_API int ca_latent_block(const ca_head_shape* shape);
+CA_API int ca_latent_attention(ca_context* ctx, const ca_latent_args* args, ca_stream stream);
+/* 1 when decode steps of the context read the work list (bf16 rows of 64-token chunks); 0 when every step has to be given
+ * as portions */
+CA_API int ca_latent_decodes(const ca_context* ctx);
+
+/* The cached rows a step of portions reads, laid out densely: workspace row base[e] + i is position first[e] + i of span
+ * e, for i < base[e + 1] - base[e].  lat: [base[n], d_value], rot: [base[n], rot_stride] (zeros behind the rotated
+ * elements; rot_stride a multiple of 8). */
+typedef struct ca_latent_gather_args {
+    void* lat;
+    void* rot;
+    int32_t rot_stride;
+    int32_t n_rows;             /* base[n_entries]                  */
+    const int32_t* row_span;    /* [n_rows]: span of each row       */
+    const int32_t* base;        /* [n_entries + 1]                  */
+    const int32_t* first;       /* [n_entries]                      */
+    const int32_t* path_off;
+    const int32_t* path_chunks;
+} ca_latent_gather_args;
+CA_API int ca_latent_gather(ca_context* ctx, const ca_latent_gather_args* args, ca_stream stream);
+
 /* Block kernels (fp32 residual stream x, activations of `dtype`).  Vectors of weights are fp32.
  * ca_token_shift: plain = x, shifted = x + (previous token's x - x) * mu; state [slots, width].
  * ca_gated_norm_add: g = r * sigmoid(gate + bias); x += g / sqrt(mean(g^2) + eps) * weight; plain (optional) = x.  With
  *   next_mu (one token per span only) also the token shift of the result.
  * ca_norm_rows: out[i] = row rows[i] (NULL: i) of x, RMS-normed, times weight, times sigmoid(gate[i]) if given.
  * ca_gelu_tanh: the tanh form.
- * ca_embed_rows: x[t] = table[ids[t]] (rows of `dtype`) as fp32; the caller has checked the ids.
+ * ca_scaled_norm: x = y / sqrt(mean(y^2) + eps) * weight with y = alpha * x + r + bias (bias may be NULL); plain
+ *   (optional) = x.
+ * ca_clamped_glu: in [n_rows, 2 width], gate | up, each plus its part of bias [2 width]; g = min(gate, limit),
+ *   u = clamp(up, -limit, limit); out = g * sigmoid(slope * g) * (u + 1).
+ * ca_softcap: z = cap * tanh(z / cap), fp32, in place.
+ * ca_embed_rows: x[t] = table[ids[t]] * scale (rows of `dtype`) as fp32, plain (optional) the same rounded; the caller has
+ *   checked the ids.
  * ca_conv_silu: depthwise causal convolution with bias (taps [channels, n_taps], last tap = current token), then
  *   SiLU; state [slots, n_taps - 1, channels], oldest first.
  * ca_selective_scan: dt = softplus(dt + dt_bias); S[c, n] = exp(dt A) S + dt x B_n; y = (S . C + D x) * silu(z);
@@ -398,8 +476,13 @@ CA_API int ca_gated_norm_add(float* x, const void* r, int64_t r_stride, const vo
 CA_API int ca_norm_rows(void* out, const void* x, int x_is_f32, int64_t x_stride, const int32_t* rows, const float* weight,
                         const void* gate, int64_t gate_stride, float eps, int64_t n_rows, int width, int dtype,
                         ca_stream stream);
-CA_API int ca_embed_rows(float* x, const void* table, const int32_t* ids, int64_t n_tokens, int width, int dtype,
-                         ca_stream stream);
+CA_API int ca_embed_rows(float* x, void* plain, const void* table, const int32_t* ids, float scale, int64_t n_tokens, int width,
+                         int dtype, ca_stream stream);
+CA_API int ca_scaled_norm(float* x, const void* r, int64_t r_stride, const float* bias, float alpha, const float* weight,
+                          float eps, void* plain, int64_t n_tokens, int width, int dtype, ca_stream stream);
+CA_API int ca_clamped_glu(void* out, const void* in, int64_t in_stride, const float* bias, float limit, float slope,
+                          int64_t n_rows, int width, int dtype, ca_stream stream);
+CA_API int ca_softcap(float* z, float cap, int64_t n, ca_stream stream);
 CA_API int ca_gelu_tanh(void* out, const void* in, int64_t in_stride, int64_t n_rows, int width, int dtype, ca_stream stream);
 CA_API int ca_conv_silu(void* out, const void* x, int64_t x_stride, const float* taps, const float* bias, float* state,
                         const ca_spans* spans, int channels, int n_taps, int dtype, ca_stream stream);
