@@ -27,7 +27,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "-I", INCLUDE]
 CU_SOURCES = ["ca_attn_fast.cu", "ca_attn_wide.cu", "ca_attn_generic.cu", "ca_pool_ops.cu", "ca_abi.cu", "ca_noalloc.cu", "ca_ops.cu",
               "ca_qkv.cu", "ca_attn_rows.cu", "ca_attn_span.cu", "ca_block_ops.cu", "ca_recurrent.cu", "ca_decay_mma.cu", "ca_decay_tc.cu",
-              "ca_latent.cu", "ca_latent_rows.cu"]
+              "ca_latent.cu", "ca_latent_rows.cu", "ca_latent_span.cu"]
 CPP_SOURCES = ["ca_plan.cpp"]
 HOST_SOURCES = ["host/chunk.cpp", "host/prefix_tree.cpp", "host/attention.cpp", "host/ops.cpp", "host/spans.cpp",
                 "host/block_ops.cpp", "host/bindings.cpp"]

@@ -35,6 +35,7 @@ EXPORTED = [
     "ca_chunk_bytes_shaped", "ca_context_create_shaped", "ca_store_qkv", "ca_attention_rows", "ca_rows_block", "ca_token_shift", "ca_gated_norm_add",
     "ca_norm_rows", "ca_embed_rows", "ca_gelu_tanh", "ca_conv_silu", "ca_scan_scratch_floats", "ca_selective_scan", "ca_decay_scratch_floats", "ca_block_status", "ca_decay_attention",
     "ca_scaled_norm", "ca_clamped_glu", "ca_softcap", "ca_latent_store", "ca_latent_block", "ca_latent_attention", "ca_latent_decodes", "ca_latent_gather",
+    "ca_latent_expands", "ca_latent_expanded_block", "ca_latent_expanded",
 ]
 CA_STATIC_MAX_SLOTS = 16384
 

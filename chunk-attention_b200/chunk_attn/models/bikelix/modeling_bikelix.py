@@ -26,6 +26,8 @@ from ..span_decoder import SpanDecoder, Weights, linear_f32, pair_frequencies
 from .configuration_bikelix import BikelixConfig
 
 GATE_SLOPE = 1.702
+EXPAND_MIN_TOKENS = 32   # of a step
+ABSORBED_COST = 3        # of a product in the latent space, in units of one between expanded heads
 
 
 class LatentAttentionMixer:
@@ -69,9 +71,25 @@ class LatentAttentionMixer:
         torch.bmm(c.transpose(0, 1), self.w_uv.transpose(1, 2), out=o.transpose(0, 1))
         return o
 
+    def expanded(self, q, step, cache):
+        lat, rot = cache.gather_latents()
+        return cache.forward_expanded(q, linear(lat, self.w_ukv), rot, step.spans.positions, self.freq, self.sink, self.vdim)
+
+    def expands(self, tokens, step, cache):
+        """Whether making keys and values of the step's windows is less work than bringing its queries into the latent
+        space and attending there, on whose longer rows the tensor cores also run slower."""
+        if step.append_tokens is not None or tokens < EXPAND_MIN_TOKENS or not cache.latent_expands(self.dim, self.vdim):
+            return False
+        rows, pairs = cache.window_load()
+        per_row = self.m["kv_rank"] * (self.dim + self.vdim)
+        there = ABSORBED_COST * pairs * (2 * self.m["kv_rank"] + self.rot)
+        return rows * per_row + pairs * (self.dim + self.rot + self.vdim) < tokens * per_row + there
+
     def __call__(self, h, step):
         cache = step.state.views[self.layer]
-        o = self.absorbed(self.queries(h, step, cache), step, cache)
+        q = self.queries(h, step, cache)
+        attend = self.expanded if self.expands(q.shape[0], step, cache) else self.absorbed
+        o = attend(q, step, cache)
         return linear(o.view(o.shape[0], -1), self.w_o)
 
 

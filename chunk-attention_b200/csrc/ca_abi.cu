@@ -1160,6 +1160,53 @@ int ca_latent_attention(ca_context* c, const ca_latent_args* a, ca_stream stream
     return CA_OK;
 }
 
+int ca_latent_expands(const ca_context* c, int dim, int vdim) {
+    return c && c->shape.latent && c->dtype == CA_DTYPE_BF16 && c->shape.scale > 0.f &&
+           ca::latent_span_serves(dim, c->shape.d_key - c->shape.d_value, vdim);
+}
+
+int ca_latent_expanded(ca_context* c, const ca_latent_expanded_args* a, ca_stream stream_) {
+    if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
+    if (!ca_latent_expands(c, a->dim, a->vdim)) return fail(CA_ERR_INVALID, "latent_expanded does not serve these sizes");
+    if (a->n_rows < 0 || a->kv_rows < 0 || a->n_blocks < 0) return fail(CA_ERR_INVALID, "negative count");
+    if (a->n_rows == 0 || a->n_blocks == 0) return CA_OK;
+    const int rot = c->shape.d_key - c->shape.d_value;
+    if (!a->q || !a->kv || !a->rot || !a->out || !a->positions || !a->base || !a->first || !a->blocks || (rot > 0 && !a->freq))
+        return fail(CA_ERR_INVALID, "an operand is null");
+    auto aligned = [](const void* q) { return reinterpret_cast<uintptr_t>(q) % 16 == 0; };
+    if (!aligned(a->q) || !aligned(a->kv) || !aligned(a->rot) || !aligned(a->out) || a->kv_stride % 8 || a->rot_stride % 8 ||
+        a->kv_stride < (int64_t)c->shape.n_heads * (a->dim + a->vdim) || a->rot_stride < 64 * ca::latent_span_rot_panels(rot))
+        return fail(CA_ERR_INVALID, "operands must be 16-byte aligned, strides multiples of 8 that hold a row");
+    DeviceGuard guard(c->device);
+    if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
+    ca::LatentSpanParams p{};
+    p.n_heads = c->shape.n_heads;
+    p.dim = a->dim;
+    p.rot = rot;
+    p.vdim = a->vdim;
+    p.window = c->shape.window;
+    p.q = a->q;
+    p.kv = a->kv;
+    p.kv_rows = a->kv_rows;
+    p.kv_stride = a->kv_stride;
+    p.rot_keys = a->rot;
+    p.rot_stride = a->rot_stride;
+    p.out = a->out;
+    p.scale_log2 = c->shape.scale * 1.4426950408889634f;
+    p.sink = a->sink;
+    p.positions = a->positions;
+    p.freq = a->freq;
+    p.base = a->base;
+    p.first = a->first;
+    p.blocks = a->blocks;
+    p.n_blocks = a->n_blocks;
+    p.status = c->status;
+    p.wait_limit = c->opt_wait_limit;
+    CA_CUDA(ca::launch_latent_span(p, static_cast<cudaStream_t>(stream_)));
+    return CA_OK;
+}
+int ca_latent_expanded_block(void) { return ca::LATENT_SPAN_BLOCK; }
+
 int ca_latent_gather(ca_context* c, const ca_latent_gather_args* a, ca_stream stream_) {
     if (!c || !a) return fail(CA_ERR_INVALID, "null argument");
     if (!c->shape.latent) return fail(CA_ERR_INVALID, "latent_gather needs a latent context");

@@ -247,6 +247,32 @@ cudaError_t launch_latent_generic(const LatentParams& p, int dtype, cudaStream_t
 bool latent_rows_serves(const Geometry& g);
 cudaError_t launch_latent_rows(const LatentParams& p, cudaStream_t stream);                // bf16, 64-token chunks
 
+// portions of prompts on tcgen05, keys and values expanded (ca_latent_span.cu)
+struct LatentSpanParams {
+    int n_heads, dim, rot, vdim;
+    int window;                  // 0: none
+    const void* q;               // bf16 [rows, n_heads, dim + rot], the last part not rotated yet
+    const void* kv;              // bf16 [kv_rows, kv_stride]: unrotated keys of all heads | values of all heads
+    int64_t kv_rows, kv_stride;
+    const void* rot_keys;        // bf16 [kv_rows, rot_stride], rotated
+    int rot_stride;
+    void* out;                   // bf16 [rows, n_heads, vdim]
+    float scale_log2;            // > 0
+    const float* sink;           // [n_heads] or null
+    const int32_t* positions;
+    const float* freq;           // [rot / 2]
+    const int32_t* base;         // workspace row of position first[e] of span e
+    const int32_t* first;
+    const int32_t* blocks;       // [n_blocks][4]: span, first token, end token, 0; at most 256 tokens each
+    int n_blocks;
+    int* status;
+    long long wait_limit;
+};
+constexpr int LATENT_SPAN_BLOCK = 256;
+bool latent_span_serves(int dim, int rot, int vdim);
+int latent_span_rot_panels(int rot);  // 64-element panels of the rotated part
+cudaError_t launch_latent_span(const LatentSpanParams& p, cudaStream_t stream);
+
 struct LatentGatherParams {
     const void* pool;
     Geometry geo;

@@ -731,6 +731,45 @@ std::pair<torch::Tensor, torch::Tensor> Attention::gather_latents() {
     return {lat, rot};
 }
 
+torch::Tensor Attention::forward_expanded(torch::Tensor q, torch::Tensor kv, torch::Tensor rot, torch::Tensor positions,
+                                          c10::optional<torch::Tensor> freq, c10::optional<torch::Tensor> sink, int vdim) {
+    need_latent("forward_expanded");
+    const int64_t rotated = shape_.d_key - shape_.d_value, n = q.size(0);
+    const auto st = c10::typeMetaToScalarType(options_.dtype());
+    if (q.dim() != 3 || q.size(1) != n_heads_ || q.size(2) <= rotated || !q.is_contiguous() || q.device() != options_.device() || q.scalar_type() != st)
+        throw std::runtime_error("forward_expanded: q must be contiguous [n_rows, n_heads, unrotated + rotated] with the dtype and device of the cache");
+    if (tables_->n_tokens != n) throw std::runtime_error("forward_expanded: extend must have described these tokens");
+    const int dim = (int)(q.size(2) - rotated);
+    c10::cuda::CUDAGuard guard(options_.device());
+    const WindowTables& w = window_tables();
+    if (kv.dim() != 2 || kv.size(0) != w.rows || kv.size(1) != (int64_t)n_heads_ * (dim + vdim) || kv.stride(1) != 1 || kv.device() != options_.device() ||
+        kv.scalar_type() != st || rot.dim() != 2 || rot.size(0) != w.rows || !rot.is_contiguous() || rot.device() != options_.device() || rot.scalar_type() != st)
+        throw std::runtime_error("forward_expanded: kv must be [window rows, n_heads * (dim + vdim)], rot what gather_latents returned");
+    torch::Tensor out = torch::empty({n, n_heads_, vdim}, options_);
+    const auto& blocks = blocks_of(ca_latent_expanded_block());
+    const int32_t* t = w.device.data_ptr<int32_t>();
+    ca_latent_expanded_args a{};
+    a.q = q.data_ptr();
+    a.kv = kv.data_ptr();
+    a.kv_rows = w.rows;
+    a.kv_stride = kv.stride(0);
+    a.rot = rot.data_ptr();
+    a.rot_stride = (int32_t)rot.size(1);
+    a.out = out.data_ptr();
+    a.n_rows = (int32_t)n;
+    a.dim = dim;
+    a.vdim = vdim;
+    a.positions = i32_ptr(positions, n, "forward_expanded: positions must be int32 [n_rows]");
+    a.freq = f32_ptr(freq, rotated / 2, "forward_expanded: freq must be fp32 [rotated / 2]");
+    a.sink = f32_ptr(sink, n_heads_, "forward_expanded: sink must be fp32 [n_heads]");
+    a.base = t + w.rows;
+    a.first = t + w.rows + (int64_t)tables_->lens.size() + 1;
+    a.blocks = blocks.first.data_ptr<int32_t>();
+    a.n_blocks = blocks.second;
+    check_rc(ca_latent_expanded(ctx_, &a, stream()), "forward_expanded");
+    return out;
+}
+
 void Attention::print(Chunk* root, int level) {
     if (root == nullptr) root = tree_->root();
     std::string indent(4 * level, ' ');

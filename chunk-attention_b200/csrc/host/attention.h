@@ -78,6 +78,12 @@ class Attention {
     std::pair<int64_t, int64_t> window_load();
     // Those rows, laid out densely: latents [rows, latent size] and shared key parts [rows, padded to 64]
     std::pair<torch::Tensor, torch::Tensor> gather_latents();
+    // whether forward_expanded serves heads of these sizes
+    bool latent_expands(int dim, int vdim) const { return ca_latent_expands(ctx_, dim, vdim) != 0; }
+    // Attention of the current portions over keys and values expanded from the gathered rows: kv [rows, n_heads * (dim +
+    // vdim)], keys of all heads, then values; rot as gather_latents returns it.  Returns [n_rows, n_heads, vdim].
+    torch::Tensor forward_expanded(torch::Tensor q, torch::Tensor kv, torch::Tensor rot, torch::Tensor positions,
+                                   c10::optional<torch::Tensor> freq, c10::optional<torch::Tensor> sink, int vdim);
     std::vector<Chunk*> append_token(const std::vector<int>& tokens, torch::Tensor k, torch::Tensor v, bool fused = true);
     void refresh_kernel_context(bool force = false);
     std::vector<Chunk*> reserve();

@@ -127,6 +127,9 @@ PYBIND11_MODULE(chunk_attn_c, m) {
       .def_property_readonly("latent_decodes", &Attention::latent_decodes)
       .def("window_load", &Attention::window_load)
       .def("gather_latents", &Attention::gather_latents)
+      .def("latent_expands", &Attention::latent_expands, py::arg("dim"), py::arg("vdim"))
+      .def("forward_expanded", &Attention::forward_expanded, py::arg("q"), py::arg("kv"), py::arg("rot"), py::arg("positions"),
+           py::arg("freq") = py::none(), py::arg("sink") = py::none(), py::arg("vdim"))
       .def("extend", &Attention::extend, py::arg("rows"), py::arg("tokens"))
       .def("store_qkv", &Attention::store_qkv, py::arg("qkv"), py::arg("positions"), py::arg("q_norm") = py::none(),
            py::arg("k_norm") = py::none(), py::arg("eps") = 0.0, py::arg("rot_dims") = 0, py::arg("key_freq") = py::none(),

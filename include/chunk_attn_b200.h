@@ -447,6 +447,31 @@ typedef struct ca_latent_gather_args {
 } ca_latent_gather_args;
 CA_API int ca_latent_gather(ca_context* ctx, const ca_latent_gather_args* args, ca_stream stream);
 
+/* Attention of portions over keys and values expanded from gathered rows (bf16, head sizes of whole granules up to 128, a
+ * positive scale: ca_latent_expands).  kv: [kv_rows, kv_stride], per workspace row the unrotated keys of all heads (dim
+ * each), then their values (vdim each); rot: the gathered shared key parts, [kv_rows, rot_stride], at least 64 (128 for more
+ * than 64 rotated elements) wide; q: [n_rows, n_heads, dim + rotated], not yet rotated; out: [n_rows, n_heads, vdim].  base and
+ * first as in ca_latent_gather, blocks of at most ca_latent_expanded_block() rows. */
+typedef struct ca_latent_expanded_args {
+    const void* q;
+    const void* kv;
+    int64_t kv_rows, kv_stride;
+    const void* rot;
+    int32_t rot_stride;
+    void* out;
+    int32_t n_rows, dim, vdim;
+    const int32_t* positions;
+    const float* freq;
+    const float* sink;
+    const int32_t* base;
+    const int32_t* first;
+    const int32_t* blocks;
+    int32_t n_blocks;
+} ca_latent_expanded_args;
+CA_API int ca_latent_expands(const ca_context* ctx, int dim, int vdim);
+CA_API int ca_latent_expanded_block(void);
+CA_API int ca_latent_expanded(ca_context* ctx, const ca_latent_expanded_args* args, ca_stream stream);
+
 /* Block kernels (fp32 residual stream x, activations of `dtype`).  Vectors of weights are fp32.
  * ca_token_shift: plain = x, shifted = x + (previous token's x - x) * mu; state [slots, width].
  * ca_gated_norm_add: g = r * sigmoid(gate + bias); x += g / sqrt(mean(g^2) + eps) * weight; plain (optional) = x.  With
