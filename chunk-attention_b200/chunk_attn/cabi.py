@@ -36,6 +36,7 @@ EXPORTED = [
     "ca_norm_rows", "ca_embed_rows", "ca_gelu_tanh", "ca_conv_silu", "ca_scan_scratch_floats", "ca_selective_scan", "ca_decay_scratch_floats", "ca_block_status", "ca_decay_attention",
     "ca_scaled_norm", "ca_clamped_glu", "ca_softcap", "ca_latent_store", "ca_latent_block", "ca_latent_attention", "ca_latent_decodes", "ca_latent_gather",
     "ca_latent_expands", "ca_latent_expanded_block", "ca_latent_expanded",
+    "ca_plan_build_windowed",
 ]
 CA_STATIC_MAX_SLOTS = 16384
 
@@ -92,6 +93,7 @@ def _load():
         "ca_context_stats": (i32, [vp, C.POINTER(PlanStats)]),
         "ca_context_read_trace": (i32, [vp, C.POINTER(C.c_uint64), i32, C.POINTER(i32), vp]),
         "ca_plan_build": (i32, [C.POINTER(vp), C.POINTER(ChunkInfo), i32, i32, i32, i32, i32, i32, i64, i32, i32, i32]),
+        "ca_plan_build_windowed": (i32, [C.POINTER(vp), C.POINTER(ChunkInfo), i32, i32, i32, i32, i32, i64, i32, i32]),
         "ca_plan_build_for_context": (i32, [vp, C.POINTER(vp), C.POINTER(ChunkInfo), i32, i32]),
         "ca_refresh_from_plan": (i32, [vp, vp, vp]),
         "ca_plan_array": (i32, [vp, i32, C.POINTER(C.POINTER(C.c_int32)), C.POINTER(i64)]),
@@ -144,6 +146,15 @@ class Plan:
         self._h = C.c_void_p()
         check(lib.ca_plan_build(C.byref(self._h), arr, n, n_seqs, n_heads, chunk_size, tpp_threshold,
                                 n_ctas, max_chunks, int(split_phases), int(seq_first_tensor), int(wide_runs)))
+
+    @classmethod
+    def windowed(cls, infos, n_seqs, window, chunk_size=64, tpp_threshold=1, n_ctas=296, max_chunks=1 << 30, rows_per_item=64):
+        """The work list of a latent cache's decode step."""
+        self = cls.__new__(cls)
+        arr, n = make_infos(infos)
+        self._h = C.c_void_p()
+        check(lib.ca_plan_build_windowed(C.byref(self._h), arr, n, n_seqs, chunk_size, tpp_threshold, n_ctas, max_chunks, rows_per_item, window))
+        return self
 
     def array(self, which):
         ptr, cnt = C.POINTER(C.c_int32)(), C.c_int64()

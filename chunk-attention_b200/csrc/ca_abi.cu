@@ -1426,6 +1426,24 @@ int ca_plan_build(ca_plan** out, const ca_chunk_info* infos, int n_infos, int n_
     return CA_OK;
 }
 
+int ca_plan_build_windowed(ca_plan** out, const ca_chunk_info* infos, int n_infos, int n_seqs, int chunk_size, int tpp_threshold,
+                           int n_ctas, int64_t max_chunks, int rows_per_item, int window) {
+    if (!out) return fail(CA_ERR_INVALID, "out is null");
+    *out = nullptr;
+    if (window < 0) return fail(CA_ERR_INVALID, "negative window");
+    ca_plan* p = new (std::nothrow) ca_plan();
+    if (!p) return fail(CA_ERR_INVALID, "out of host memory");
+    std::string err = ca::build_plan(p->plan, infos, n_infos, n_seqs, 1, chunk_size, tpp_threshold, n_ctas, max_chunks, false, ca::FAST_D, 2,
+                                     true, false, /*wide_mode=*/0, /*want_paths=*/false, rows_per_item, /*one_partial_per_row=*/true, window);
+    if (!err.empty()) {
+        delete p;
+        return fail(CA_ERR_INVALID, "work list rejected: " + err);
+    }
+    p->window = window;
+    *out = p;
+    return CA_OK;
+}
+
 int ca_plan_array(const ca_plan* plan, int which, const int32_t** data, int64_t* count) {
     if (!plan || !data || !count) return fail(CA_ERR_INVALID, "null argument");
     const ca::Plan& pl = plan->plan;

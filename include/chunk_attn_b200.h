@@ -598,6 +598,11 @@ CA_API int ca_attention_static_status(int32_t* status, ca_stream stream);
 CA_API int ca_plan_build(ca_plan** out, const ca_chunk_info* infos, int n_infos, int n_seqs,
                          int n_heads, int chunk_size, int tpp_threshold, int n_ctas,
                          int64_t max_chunks, int split_phases, int seq_first_tensor, int wide_runs);
+/* The work list of a latent cache's decode step: items of up to rows_per_item rows, one partial per row of an item; chunks
+ * that end before the window of every row they serve are left out (window 0: none).  Word 1 of an item is then the
+ * position of its first token. */
+CA_API int ca_plan_build_windowed(ca_plan** out, const ca_chunk_info* infos, int n_infos, int n_seqs, int chunk_size,
+                                  int tpp_threshold, int n_ctas, int64_t max_chunks, int rows_per_item, int window);
 CA_API int ca_plan_array(const ca_plan* plan, int which, const int32_t** data, int64_t* count);
 CA_API int ca_plan_stats_get(const ca_plan* plan, ca_plan_stats* out);
 /* One work list for several contexts.  The caches of a model's layers see the same tree at every step, so

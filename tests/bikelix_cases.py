@@ -42,7 +42,7 @@ def make(cfg, dtype, seed=0, weights=None, **engine):
     return BikelixForCausalLM(c, w), {k: v.double().numpy() for k, v in w.items()}
 
 
-TOL = {torch.float32: 3e-5, torch.bfloat16: 0.1}
+TOL = {torch.float32: 3e-5, torch.bfloat16: 0.03}
 
 
 def reference(cfg, weights, tokens):
