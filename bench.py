@@ -19,7 +19,7 @@ Workloads (synthetic, seeded; synthetic_workloads.py):
 `--workload` overrides the choice (cfg2, cfg5, cfg3_s<shared>, cfg4, short<n_seqs>: a 1024-token common
 prompt with 20-token private suffixes, sys<n_seqs>: a 2048-token system prompt with 8-token suffixes, llama: the
 decoder loop, gagorax: prefill and decode of the Gagorax decoder's layers beside a Llama layer of equal width, with the
-time of every kernel against its roofline).
+time of every kernel against its roofline, bikelix: the same for the Bikelix decoder, beside both).
 
 Every line carries `parity`: sampled (row, head) outputs of the very tensors that are timed, compared with dense
 fp64 attention computed from the seeded inputs (on N > 1 including heads owned by other ranks, regenerated from
@@ -1242,9 +1242,114 @@ def run_llama(args):
 
 
 
-# ---- the Gagorax decoder beside the Llama decoder -------------------------------------------------------------------
+# ---- decoders that run steps, beside the Llama decoder ---------------------------------------------------------------
 BF16_PEAK = 1.59e15  # of fallback: cuBLAS bf16 burst on this pool
 MUFU_PEAK = 16 * 148 * 1.965e9  # exponentials per second: 16 per clock and SM at the highest clock
+
+
+def measured_bf16_peak():
+    path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        with open(path) as f:
+            return float(json.load(f)["bf16_tflops"]) * 1e12
+    return BF16_PEAK
+
+
+class LayerBench:
+    """Device times (CUDA events, medians) of whole steps of a decoder and of single kernels, the latter with the L2 flushed
+    before every call and against their roofline: the larger of bytes over the HBM copy peak, FLOPs over the bf16 GEMM peak,
+    and exponentials over the special-function rate."""
+    PREFILLS, DECODES = ([4096], [1024] * 8), ((64, 1024), (16, 4096))
+
+    def __init__(self, args, bf16_peak):
+        import torch
+        self.torch, self.dev, self.bf16_peak = torch, torch.device("cuda", 0), bf16_peak
+        torch.cuda.set_device(0)
+        self.hbm = measured_peak()[0] * 1e9
+        self.steps, self.warm = min(args.steps, 30), max(3, min(args.warmup, 10))
+        self.flush = torch.empty(64 << 20, dtype=torch.float32, device=self.dev)  # 256 MB, twice the L2
+        self.layers, self.kernels = {}, {}
+
+    def timed(self, fn, n=None, before=None):
+        """Median device time of fn in microseconds; `before` runs untimed ahead of every call."""
+        us = []
+        for i in range(self.warm + (n or self.steps)):
+            if before is not None:
+                before()
+            a, b = self.torch.cuda.Event(enable_timing=True), self.torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            self.torch.cuda.synchronize()
+            if i >= self.warm:
+                us.append(a.elapsed_time(b) * 1e3)
+        return statistics.median(us)
+
+    @staticmethod
+    def prompt(i, n):
+        return [(7 * i + 13 * j) % 1000 for j in range(n)]
+
+    def record(self, r, what, us, tokens):
+        r[what] = {"us": round(us, 1), "tokens_per_s": round(tokens / us * 1e6)}
+
+    def decoder(self, name, model):
+        """Prefill and decode of a model with a step function."""
+        caches, r = model.create_kv_caches(), {}
+
+        def clear():
+            for c in caches:
+                c.clear()
+
+        for lens in self.PREFILLS:
+            toks = [self.prompt(i, n) for i, n in enumerate(lens)]
+            us = self.timed(lambda: model.step([None] * len(lens), toks, caches), before=clear)
+            self.record(r, "prefill_%dx%d" % (len(lens), lens[0]), us, sum(lens))
+        for batch, ctx in self.DECODES:
+            clear()
+            for i in range(batch):
+                model.step([None], [self.prompt(i, ctx)], caches)
+
+            def decode():
+                x, sp, _ = model.step(list(range(batch)), [[5]] * batch, caches)
+                return model.head_logits(x, sp.last)
+
+            self.record(r, "decode_%d_at_%d" % (batch, ctx), self.timed(decode), batch)
+        self.layers[name] = r
+        bad = [c.device_status() for c in list(caches[:-1]) + caches[-1].views if c.device_status()]
+        if bad:
+            raise RuntimeError("device status %s" % bad)
+
+    def llama(self):
+        torch = self.torch
+        from chunk_attn.models.llama_hf import LlamaConfig, LlamaForCausalLM
+        from chunk_attn.models.sequence import Sequence
+        lcfg = LlamaConfig(num_hidden_layers=1, chunk_attn_kvcache_gb=12.0, torch_dtype=torch.float16, torch_device="cuda:0")
+        llama = LlamaForCausalLM(lcfg, seed=0).to(device=self.dev, dtype=torch.float16).eval()
+        kv, r = llama.create_kv_caches(), {}
+        for lens in self.PREFILLS:
+            seqs = [self.prompt(i, n) for i, n in enumerate(lens)]
+            us = self.timed(lambda: llama.model([Sequence(p) for p in seqs], kv, True), before=lambda: [c.clear() for c in kv])
+            self.record(r, "prefill_%dx%d" % (len(lens), lens[0]), us, sum(lens))
+        for batch, ctx in self.DECODES:
+            for c in kv:
+                c.clear()
+            live = []
+            for i in range(batch):
+                live.append(Sequence(self.prompt(i, ctx)))
+                llama([live[-1]], kv, True)
+
+            def decode():
+                for s in live:
+                    s.append(5)
+                return llama.logits(live, kv, False)
+
+            self.record(r, "decode_%d_at_%d" % (batch, ctx), self.timed(decode), batch)
+        self.layers["llama"] = r
+
+    def kernel(self, name, fn, nbytes, flops=0.0, like=None, exps=0.0):
+        us = self.timed(fn, before=self.flush.zero_)
+        least = max(nbytes / self.hbm, flops / self.bf16_peak, exps / MUFU_PEAK) * 1e6
+        self.kernels[name] = {"us": round(us, 1), "roofline_us": round(least, 1), "fraction": round(least / us, 3), "like": like}
 
 
 def gagorax_layers():
@@ -1258,103 +1363,22 @@ def gagorax_layers():
 
 
 def run_gagorax(args):
-    """Tokens per second of whole steps (the model's own step function, device time by CUDA events) for prefill and decode,
-    and the device time of each kernel alone, L2 flushed before every call, against its roofline: the larger of bytes over the
-    HBM copy peak, FLOPs over the bf16 GEMM peak, and exponentials over the special-function rate (the scan)."""
+    """Tokens per second of whole steps (the model's own step function) for prefill and decode, and every kernel alone."""
     import torch
     import chunk_attn
     from chunk_attn import SpanBatch, ops
     from chunk_attn.models.gagorax import GagoraxConfig, GagoraxForCausalLM
     from chunk_attn.models.gagorax.modeling_gagorax import random_weights
-    from chunk_attn.models.llama_hf import LlamaConfig, LlamaForCausalLM
-    from chunk_attn.models.sequence import Sequence
-    dev = torch.device("cuda", 0)
-    torch.cuda.set_device(0)
-    hbm = measured_peak()[0] * 1e9
-    steps, warm = min(args.steps, 30), max(3, min(args.warmup, 10))
-    prefills, decodes = ([4096], [1024] * 8), ((64, 1024), (16, 4096))
-    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)  # 256 MB, twice the L2
-
-    def timed(fn, n, before=None):
-        """Median device time of fn in microseconds; `before` runs untimed ahead of every call."""
-        us = []
-        for i in range(warm + n):
-            if before is not None:
-                before()
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            a.record()
-            fn()
-            b.record()
-            torch.cuda.synchronize()
-            if i >= warm:
-                us.append(a.elapsed_time(b) * 1e3)
-        return statistics.median(us)
-
-    def prompt(i, n):
-        return [(7 * i + 13 * j) % 1000 for j in range(n)]
-
-    out = {"layers": {}, "kernels": {}}
+    bench = LayerBench(args, BF16_PEAK)
+    dev, steps, warm, prompt, kernel, prefills, decodes = bench.dev, bench.steps, bench.warm, bench.prompt, bench.kernel, bench.PREFILLS, bench.DECODES
+    out = {"layers": bench.layers, "kernels": bench.kernels}
     with torch.inference_mode():
         for name, layers in gagorax_layers().items():
             cfg = GagoraxConfig.from_dict({"vocab": 32000, "width": 4096, "layers": layers, "norm": {"eps": 1e-5}}, kvcache_gb=12.0, state_slots=128)
-            model = GagoraxForCausalLM(cfg, random_weights(cfg, 0, device=dev))
-            caches = model.create_kv_caches()
-
-            def clear():
-                for c in caches:
-                    c.clear()
-
-            r = {}
-            for lens in prefills:
-                toks = [prompt(i, n) for i, n in enumerate(lens)]
-                us = timed(lambda: model.step([None] * len(lens), toks, caches), steps, before=clear)
-                r["prefill_%dx%d" % (len(lens), lens[0])] = {"us": round(us, 1), "tokens_per_s": round(sum(lens) / us * 1e6)}
-            for batch, ctx in decodes:
-                clear()
-                for i in range(batch):
-                    model.step([None], [prompt(i, ctx)], caches)
-
-                def decode():
-                    x, sp, _ = model.step(list(range(batch)), [[5]] * batch, caches)
-                    return model.head_logits(x, sp.last)
-
-                us = timed(decode, steps)
-                r["decode_%d_at_%d" % (batch, ctx)] = {"us": round(us, 1), "tokens_per_s": round(batch / us * 1e6)}
-            out["layers"][name] = r
-            bad = [c.device_status() for c in caches[:-1] if c.device_status()]
-            if bad or ops.block_status(dev):
-                raise RuntimeError("device status %s" % (bad or "block"))
-            del model, caches
-        lcfg = LlamaConfig(num_hidden_layers=1, chunk_attn_kvcache_gb=12.0, torch_dtype=torch.float16, torch_device="cuda:0")
-        llama = LlamaForCausalLM(lcfg, seed=0).to(device=dev, dtype=torch.float16).eval()
-        kv = llama.create_kv_caches()
-        r = {}
-        for lens in prefills:
-            seqs = [prompt(i, n) for i, n in enumerate(lens)]
-            us = timed(lambda: llama.model([Sequence(p) for p in seqs], kv, True), steps, before=lambda: [c.clear() for c in kv])
-            r["prefill_%dx%d" % (len(lens), lens[0])] = {"us": round(us, 1), "tokens_per_s": round(sum(lens) / us * 1e6)}
-        for batch, ctx in decodes:
-            for c in kv:
-                c.clear()
-            live = []
-            for i in range(batch):
-                live.append(Sequence(prompt(i, ctx)))
-                llama([live[-1]], kv, True)
-
-            def decode():
-                for s in live:
-                    s.append(5)
-                return llama.logits(live, kv, False)
-
-            us = timed(decode, steps)
-            r["decode_%d_at_%d" % (batch, ctx)] = {"us": round(us, 1), "tokens_per_s": round(batch / us * 1e6)}
-        out["layers"]["llama"] = r
-        del llama, kv
-
-        def kernel(name, fn, nbytes, flops=0.0, like=None, exps=0.0):
-            us = timed(fn, steps, before=flush.zero_)
-            least = max(nbytes / hbm, flops / BF16_PEAK, exps / MUFU_PEAK) * 1e6
-            out["kernels"][name] = {"us": round(us, 1), "roofline_us": round(least, 1), "fraction": round(least / us, 3), "like": like}
+            bench.decoder(name, GagoraxForCausalLM(cfg, random_weights(cfg, 0, device=dev)))
+            if ops.block_status(dev):
+                raise RuntimeError("a bounded wait of a block kernel has run out")
+        bench.llama()
 
         bf, f32, f16 = torch.bfloat16, torch.float32, torch.float16
         g = torch.Generator(device=dev).manual_seed(0)
@@ -1441,6 +1465,132 @@ def run_gagorax(args):
     emit(line)
 
 
+# ---- the Bikelix decoder beside Gagorax's attention layers and the Llama decoder ----------------------------------------
+def bikelix_layers():
+    """Layers at width 4096, sized like a 7B model's: 32 heads of 128 + 64, latents of 512."""
+    def layer(window, **more):
+        m = {"heads": 32, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 1536, "kv_rank": 512, "scale": 192 ** -0.5, "mask": {"size": window},
+             "rot": {"base": 10000.0, "dims": 64}}
+        return {"type": "latent_attention", "mixer": dict(m, **more), "mlp": {"kind": "dense", "ff": 11008, "limit": 7.0}}
+    return {"window 1024": [layer(1024)], "window 4096": [layer(4096)], "owner + reader, window 1024": [layer(1024), layer(1024, kv_from=0)]}
+
+
+def run_bikelix(args):
+    """Tokens per second of whole steps (the model's own step function) for prefill and decode, beside Gagorax's attention
+    layers and a Llama layer of equal width, and every kernel alone beside the like kernel."""
+    import torch
+    import chunk_attn
+    from chunk_attn import SpanBatch, ops
+    from chunk_attn.models.bikelix import BikelixConfig, BikelixForCausalLM
+    from chunk_attn.models.bikelix.modeling_bikelix import random_weights
+    from chunk_attn.models.gagorax import GagoraxConfig, GagoraxForCausalLM
+    from chunk_attn.models.gagorax.modeling_gagorax import random_weights as gagorax_weights
+    bench = LayerBench(args, measured_bf16_peak())
+    dev, prompt, kernel = bench.dev, bench.prompt, bench.kernel
+    bf, f32, f16 = torch.bfloat16, torch.float32, torch.float16
+    g = torch.Generator(device=dev).manual_seed(0)
+
+    def rnd(*s, dtype=bf):
+        return torch.randn(s, generator=g, device=dev).to(dtype)
+
+    def pairs_of(starts, lens, window):
+        return sum(min(p + 1, window) for s, n in zip(starts, lens) for p in range(s, s + n))
+
+    with torch.inference_mode():
+        for name, layers in bikelix_layers().items():
+            cfg = BikelixConfig.from_dict({"vocab": 32000, "width": 4096, "layers": layers, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+                                           "postln_alpha": 1.0, "logit_softcap": 30.0}, kvcache_gb=12.0, state_slots=128)
+            bench.decoder(name, BikelixForCausalLM(cfg, random_weights(cfg, 0, device=dev)))
+        for name in ("attention", "attention_8kv"):
+            cfg = GagoraxConfig.from_dict({"vocab": 32000, "width": 4096, "layers": gagorax_layers()[name], "norm": {"eps": 1e-5}}, kvcache_gb=12.0, state_slots=128)
+            bench.decoder("gagorax " + name, GagoraxForCausalLM(cfg, gagorax_weights(cfg, 0, device=dev)))
+        bench.llama()
+
+        W, F, H, d, r, dv, QR, R = 4096, 11008, 32, 128, 64, 128, 1536, 512
+        scale = (d + r) ** -0.5
+        freq = (10000.0 ** (-torch.arange(r // 2, device=dev) * 2.0 / r)).float()
+        qn, kn, sink = 1 + 0.1 * rnd(QR, dtype=f32), 1 + 0.1 * rnd(R, dtype=f32), rnd(H, dtype=f32)
+        w_ukv = rnd(H * (d + dv), R) * R ** -0.5
+
+        def latent_cache(window):
+            return chunk_attn.Attention.latent(n_heads=H, latent=R, rotated=r, scale=scale, window=window, memory_mb=1024, dtype=bf, device=dev)
+
+        for lens in bench.PREFILLS:
+            E, T = len(lens), sum(lens)
+            tag, ids = "%dx%d" % (E, lens[0]), [prompt(i, n) for i, n in enumerate(lens)]
+            sp = SpanBatch(ids, [0] * E, list(range(E)), dev)
+            x, r_, gate, w, b = rnd(T, W, dtype=f32), rnd(T, W), rnd(T, W), rnd(W, dtype=f32), rnd(W, dtype=f32)
+            kernel("gated_norm_add " + tag, lambda: ops.gated_norm_add(x, r_, gate, b, w, 1e-5), 14.0 * T * W)
+            kernel("scaled_norm " + tag, lambda: ops.scaled_norm(x, r_, 1.0, w, 1e-5, bias=b), 12.0 * T * W, like="gated_norm_add")
+            u, gu, gb = rnd(T, F), rnd(T, 2 * F), rnd(2 * F, dtype=f32)
+            kernel("gelu_tanh " + tag, lambda: ops.gelu_tanh(u), 4.0 * T * F)
+            kernel("clamped_glu " + tag, lambda: ops.clamped_glu(gu, gb, 7.0), 6.0 * T * F, like="gelu_tanh")
+            z = rnd(64, 32000, dtype=f32)
+            kernel("softcap 64x32000 " + tag, lambda: ops.softcap(z, 30.0), 8.0 * z.numel(), like="gelu_tanh")
+            grouped = chunk_attn.Attention.shaped(n_heads=H, n_kv_heads=H, d_key=d, d_value=d, scale=d ** -0.5, sink=True, memory_mb=4096, dtype=bf, device=dev)
+            grouped.extend([-1] * E, ids)
+            qkv, hn = rnd(T, 3 * H * d), rnd(d, dtype=f32)
+            gfreq = (10000.0 ** (-torch.arange(64, device=dev) / 64.0)).float()
+            kernel("store_qkv kv32 " + tag, lambda: grouped.store_qkv(qkv, sp.positions, hn, hn, 1e-5, d, gfreq, gfreq), 12.0 * T * H * d)
+            q = grouped.store_qkv(qkv, sp.positions, hn, hn, 1e-5, d, gfreq, gfreq)
+            kernel("attention_rows kv32 " + tag, lambda: grouped.forward_rows(q, sp.positions, gfreq, sp.entry_of), 8.0 * T * H * d,
+                   flops=4.0 * pairs_of([0] * E, lens, 1 << 30) * H * d)
+            del grouped, qkv, q
+            proj = rnd(T, QR + R + r)
+            for window in (1024, 4096):
+                cache = latent_cache(window)
+                cache.extend([-1] * E, ids)
+                store = lambda: cache.store_latent(proj, sp.positions, qn, kn, 1e-5, freq)
+                if window == 1024:
+                    kernel("store_latent " + tag, store, 4.0 * T * (QR + R + r), like="store_qkv")
+                    kernel("gather_latents " + tag, cache.gather_latents, 4.0 * T * (R + r), like="store_qkv")
+                store()
+                lat, rot = cache.gather_latents()
+                kv, q = lat @ w_ukv.t(), rnd(T, H, d + r)
+                pairs = pairs_of([0] * E, lens, window)
+                kernel("forward_expanded window %d %s" % (window, tag), lambda: cache.forward_expanded(q, kv, rot, sp.positions, freq, sink, dv),
+                       2.0 * T * H * (d + r + dv + d + dv) + 2.0 * T * r, flops=2.0 * pairs * H * (d + r + dv), like="attention_rows kv32")
+                if window == 1024:
+                    ql = rnd(T, H, R)
+                    kernel("forward_latent portions window %d %s" % (window, tag), lambda: cache.forward_latent(ql, q, sp.positions, freq, sink, sp.entry_of),
+                           2.0 * T * H * (2 * R + r) + 2.0 * T * (R + r), flops=2.0 * pairs * H * (2 * R + r), like="attention_rows kv32")
+                    del ql
+                del cache, lat, rot, kv, q
+            del x, r_, gate, u, gu, proj
+        for batch, ctx in bench.DECODES:
+            tag, ids = "%d_at_%d" % (batch, ctx), [prompt(i, ctx) for i in range(batch)]
+            sp = SpanBatch([[5]] * batch, [ctx] * batch, list(range(batch)), dev)
+            for kvh in (32, 8):
+                cache = chunk_attn.Attention.shaped(n_heads=H, n_kv_heads=kvh, d_key=d, d_value=d, scale=d ** -0.5, sink=True, memory_mb=4096, dtype=bf, device=dev)
+                k3 = rnd(ctx, kvh, d)
+                for p in ids:
+                    cache.add_seq(tokens=p, k=k3, v=k3)
+                qkv, hn = rnd(batch, (H + 2 * kvh) * d), rnd(d, dtype=f32)
+                q = cache.store_qkv(qkv, sp.positions, hn, hn, 1e-5, append_tokens=[5] * batch)
+                kernel("attention_rows decode kv%d %s" % (kvh, tag), lambda: cache.forward_rows(q, sp.positions), 4.0 * batch * ctx * kvh * d,
+                       flops=4.0 * batch * ctx * H * d)
+                del cache
+            for window in (1024, 4096):
+                cache = latent_cache(window)
+                for i, p in enumerate(ids):
+                    cache.extend([-1], [p])
+                    one = SpanBatch([p], [0], [i], dev)
+                    cache.store_latent(rnd(ctx, QR + R + r), one.positions, qn, kn, 1e-5, freq)
+                cache.store_latent(rnd(batch, QR + R + r), sp.positions, qn, kn, 1e-5, freq, append_tokens=[5] * batch)
+                ql, q, seen = rnd(batch, H, R), rnd(batch, H, d + r), min(window, ctx + 1)
+                kernel("forward_latent decode window %d %s" % (window, tag), lambda: cache.forward_latent(ql, q, sp.positions, freq, sink),
+                       2.0 * batch * seen * (R + r) + 4.0 * batch * H * R, flops=2.0 * batch * seen * H * (2 * R + r), like="attention_rows decode kv8 / kv32")
+                del cache
+    value = bench.layers["window 1024"]["decode_64_at_1024"]
+    line = {"metric": "bikelix_decode_tokens_per_s", "value": value["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": bench.steps,
+            "warmup": bench.warm, "ms_per_step": value["us"] * 1e-3, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
+            "data": "synthetic", "config": {"workload": "bikelix: layers of width 4096 (random bf16 weights), prefill 1 x 4096 and 8 x 1024 tokens, decode 64 rows "
+            "at 1024 and 16 at 4096; value: decode of one layer with head, window 1024, 64 rows at 1024; kernels alone with a 256 MB L2 flush before each call",
+            "bf16_peak_tflops": round(bench.bf16_peak * 1e-12, 1)}}
+    line.update({"layers": bench.layers, "kernels": bench.kernels})
+    emit(line)
+
+
 def emit(line):
     """The one JSON line goes to the process's original stdout; everything else any library prints
     (NCCL's version banner, the reference's logger) was diverted to stderr in main()."""
@@ -1464,6 +1614,8 @@ def main():
         run_llama(args)
     elif args.workload == "gagorax":
         run_gagorax(args)
+    elif args.workload == "bikelix":
+        run_bikelix(args)
     else:
         run_b200(args)
 

@@ -355,6 +355,9 @@ int ca_context_set_option(ca_context* c, int option, int64_t value) {
 
 static int upload_plan(ca_context* c, const ca::Plan& pl, cudaStream_t stream);
 
+// CTAs the work list is cut for: the latent kernel's fill an SM each
+static int ctas_of(const ca_context* c) { return c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * (c->shape.latent ? 1 : ca::FAST_CTAS_PER_SM); }
+
 static std::string plan_for(const ca_context* c, ca::Plan& plan, const ca_chunk_info* infos, int n_infos, int n_seqs, int n_ctas) {
     if (!c->shaped)
         return ca::build_plan(plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold, n_ctas,
@@ -365,7 +368,8 @@ static std::string plan_for(const ca_context* c, ca::Plan& plan, const ca_chunk_
     // short tails or wide runs
     return ca::build_plan(plan, infos, n_infos, n_seqs, c->geo.n_heads, c->geo.chunk_size, c->tpp_threshold, n_ctas, c->max_chunks,
                           false, d_mean, c->geo.esize, c->items, /*seq_first_tensor=*/false,
-                          /*wide_mode=*/0, /*want_paths=*/!c->items, 64 / c->group, /*one_partial_per_row=*/true, c->shape.window);
+                          /*wide_mode=*/0, /*want_paths=*/!c->items, 64 / c->group, /*one_partial_per_row=*/true, c->shape.window,
+                          /*even_items=*/c->shape.latent != 0);
 }
 
 int ca_refresh_kernel_context(ca_context* c, const ca_chunk_info* infos, int n_infos, int n_seqs, ca_stream stream_) {
@@ -374,7 +378,7 @@ int ca_refresh_kernel_context(ca_context* c, const ca_chunk_info* infos, int n_i
     DeviceGuard guard(c->device);
     if (guard.err != cudaSuccess) return fail_cuda(guard.err, "cudaSetDevice");
     c->valid = false;
-    const int n_ctas = c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * ca::FAST_CTAS_PER_SM;
+    const int n_ctas = ctas_of(c);
     std::string err = plan_for(c, c->plan, infos, n_infos, n_seqs, n_ctas);
     if (!err.empty()) return fail(CA_ERR_INVALID, "work list rejected: " + err);
     return upload_plan(c, c->plan, stream);
@@ -385,7 +389,7 @@ int ca_plan_build_for_context(const ca_context* c, ca_plan** out, const ca_chunk
     ca_plan* p = *out;  // an existing plan is rebuilt in place and keeps its buffers
     if (!p) p = new (std::nothrow) ca_plan();
     if (!p) return fail(CA_ERR_INVALID, "out of host memory");
-    const int n_ctas = c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * ca::FAST_CTAS_PER_SM;
+    const int n_ctas = ctas_of(c);
     std::string err = plan_for(c, p->plan, infos, n_infos, n_seqs, n_ctas);
     if (!err.empty()) {
         if (!*out) delete p;  // a caller-owned plan is left to the caller (its contents are unspecified now)
@@ -405,7 +409,7 @@ int ca_plan_build_for_context(const ca_context* c, ca_plan** out, const ca_chunk
 int ca_refresh_from_plan(ca_context* c, const ca_plan* plan, ca_stream stream_) {
     if (!c || !plan) return fail(CA_ERR_INVALID, "null argument");
     const ca::Plan& pl = plan->plan;
-    const int n_ctas = c->opt_ctas > 0 ? c->opt_ctas : c->num_sms * ca::FAST_CTAS_PER_SM;
+    const int n_ctas = ctas_of(c);
     if (pl.n_heads != c->geo.n_heads || pl.chunk_size != c->geo.chunk_size || plan->d_head != c->geo.d_head ||
         plan->esize != c->geo.esize || plan->fast != c->items || plan->max_chunks > c->max_chunks ||
         pl.split_phases != c->opt_split || pl.tpp_threshold != c->tpp_threshold || (c->items && pl.n_ctas > n_ctas) ||
@@ -1434,7 +1438,7 @@ int ca_plan_build_windowed(ca_plan** out, const ca_chunk_info* infos, int n_info
     ca_plan* p = new (std::nothrow) ca_plan();
     if (!p) return fail(CA_ERR_INVALID, "out of host memory");
     std::string err = ca::build_plan(p->plan, infos, n_infos, n_seqs, 1, chunk_size, tpp_threshold, n_ctas, max_chunks, false, ca::FAST_D, 2,
-                                     true, false, /*wide_mode=*/0, /*want_paths=*/false, rows_per_item, /*one_partial_per_row=*/true, window);
+                                     true, false, /*wide_mode=*/0, /*want_paths=*/false, rows_per_item, /*one_partial_per_row=*/true, window, /*even_items=*/true);
     if (!err.empty()) {
         delete p;
         return fail(CA_ERR_INVALID, "work list rejected: " + err);

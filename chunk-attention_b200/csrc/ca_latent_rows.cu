@@ -1,17 +1,22 @@
-// Attention over a latent cache on tensor cores (bf16, mma.sync): decode items of the planner's work list, and portions of
-// prompts where expanding the latents into per-head keys and values (ca_latent_span.cu) does not pay.
+// Attention over a latent cache on the Blackwell tensor path (bf16, tcgen05): decode items of the planner's work list, and
+// portions of prompts where expanding the latents into per-head keys and values (ca_latent_span.cu) does not pay.
 //
 // A token's pool row is key and value of every head at once, so the query heads of a token, and the tokens of a block, are
-// rows of ONE product against the rows staged in shared memory: row r is head r % H of token r / H.
-//   S = Q K^T   the eight warps share the tile: MT 16-row groups x 8 / MT runs of tokens
-//   softmax     fp32, log2 units, online; the runs of a row meet in shared memory.  Every row has a window: positions from
-//               its own minus (window - 1) on
-//   O += P V    V is the leading part of the same staged rows; a warp owns d_value / 8 columns of every row.  The weights
-//               enter as a sum of two bf16 numbers, which keeps 16 bits of them
-// Tiles are half or whole chunks, copied verbatim (the pool's lines are the swizzled layout ldmatrix reads without
-// conflicts) by 1-D TMA bulk copies into a ring.  Decode emits one partial per row and item, combined by the merge kernel of
-// ca_attn_rows.cu; portions emit finished rows.  Every wait is bounded: when one runs out a status is recorded, the copies in
-// flight are waited for (again with the limit) and the rows stay unwritten.
+// rows of ONE product against the rows staged in shared memory: row r is head r % H of token r / H.  There are few of them
+// (up to 64) and the values are long, so the products are formed transposed, cache rows and value elements on the M side:
+//   S^T = K Q^T   M = 64 tokens, N = query rows; D in TMEM, two buffers, so that the scores of tile j + 1 are computed under
+//                 the softmax of tile j
+//   softmax       the scores go through shared memory once, so that 128 / N threads share a query row; fp32, log2 units;
+//                 every row has a window.  O is rescaled only when a row's maximum has grown by more than 8.  The
+//                 weights go back to shared memory as bf16 hi + lo parts, whose sum has 16 bits of the fp32 weight
+//   O^T += V^T P^T  M = 128 value elements (one TMEM block each), N = query rows; A = the same staged rows read the other way
+// Cache rows arrive by 1-D TMA bulk copies, verbatim (the pool's lines are the swizzled operand layout), in a ring of
+// 16 KiB units: two 64-element panels of a 64-token chunk, released one by one as the second product has used them.  Decode
+// emits one partial per row and item, combined by the merge kernel of ca_attn_rows.cu; portions emit finished rows.
+// Warp roles: 0-3 softmax and epilogue, 4 TMA producer, 5 TMEM and the MMA issue.
+//
+// Every wait is bounded: on expiry a status code is recorded, every role runs out without waiting further, nothing is
+// stored, and the TMEM columns are freed at the common exit.
 #include <algorithm>
 
 #include "ca_kernels.h"
@@ -23,117 +28,254 @@ namespace ca {
 namespace {
 using namespace ptx;
 
-constexpr int L_THREADS = 256, L_WARPS = 8, L_CHUNK = 64, L_MAX_STAGES = 6;
-constexpr float L_NEG_BIG = -1.0e30f, L_LOG2E = 1.4426950408889634f;
+constexpr int L_THREADS = 192, L_TOK = 64, L_PANEL = L_TOK * 128, L_UNIT = 2 * L_PANEL, L_MAX_UNITS = 16, L_MAX_ROWS = 64;
+constexpr float L_NEG_BIG = -1.0e30f, L_LOG2E = 1.4426950408889634f, L_RESCALE_STEP = 8.f;
 
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile(
-        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
+__host__ __device__ constexpr uint32_t idesc_bf16(int m, int n, bool a_mn_major) { return umma_idesc_f16(m, n, a_mn_major, false) | (1u << 7) | (1u << 10); }
+__device__ __forceinline__ void report(int* status, int code) { atomicCAS(status, STATUS_OK, code); }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&h);
 }
-__device__ __forceinline__ void sts32(uint32_t addr, uint32_t v) { asm volatile("st.shared.u32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
+__device__ __forceinline__ void softmax_warps_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void sts64(uint32_t addr, uint32_t x, uint32_t y) { asm volatile("st.shared.v2.u32 [%0], {%1,%2};" ::"r"(addr), "r"(x), "r"(y) : "memory"); }
 
-// tokens of a tile, and byte offset of granule g of line t in panels of `lines` 128-byte lines
-template <int MT> __host__ __device__ constexpr int tile_tokens() { return MT == 4 ? 32 : 64; }
-template <int LINES> __device__ __forceinline__ uint32_t staged(int t, int g) {
-    return (g >> 3) * (LINES * 128) + t * 128 + (((g & 7) ^ (t & 7)) << 4);
-}
-// hi (part 0) and lo (part 1) weights: granule g of row r.  A row of 32 tokens holds both parts in one line.
-template <int MT> __device__ __forceinline__ uint32_t weight_at(int part, int r, int g) {
-    if (MT == 4) return r * 128 + (((g + 4 * part) ^ (r & 7)) << 4);
-    return part * (16 * MT * 128) + r * 128 + ((g ^ (r & 7)) << 4);
-}
-template <int MT> constexpr int weight_bytes() { return MT == 4 ? 64 * 128 : 2 * 16 * MT * 128; }
+template <int N> __device__ __forceinline__ void tmem_ld(uint32_t taddr, uint32_t (&r)[N]);
+template <> __device__ __forceinline__ void tmem_ld<16>(uint32_t taddr, uint32_t (&r)[16]) { tmem_ld16(taddr, r); }
+template <> __device__ __forceinline__ void tmem_ld<32>(uint32_t taddr, uint32_t (&r)[32]) { tmem_ld32(taddr, r); }
 
-template <int MT, int NV, bool SPAN>
-__global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentParams p, int stages) {
+// byte offsets of the parts of shared memory behind the ring
+struct Layout {
+    int units, q, weights, scores, end;
+};
+template <int N> __host__ __device__ inline Layout layout_of(int gpr, int units) {
+    Layout l;
+    l.units = units;
+    l.q = units * L_UNIT;                        // queries: [gpr / 8 panels][N lines of 128 bytes]
+    l.weights = l.q + N * gpr * 16;              // weights: hi and lo, [N lines of 64 tokens] each
+    l.scores = l.weights + 2 * N * 128;          // fp32 [N][L_TOK + 4]
+    l.end = l.scores + N * (L_TOK + 4) * 4;
+    return l;
+}
+
+template <int N, bool SPAN>
+__global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentParams p, int units) {
     extern __shared__ __align__(1024) uint8_t smem[];
-    constexpr int NT = tile_tokens<MT>(), ROWS = 16 * MT, TS = L_WARPS / MT, RUN = NT / TS, NB = RUN / 8;
-    __shared__ float red[TS][ROWS], alpha_s[ROWS], m_s[ROWS];
-    __shared__ __align__(8) uint64_t full[L_MAX_STAGES];
+    constexpr int TPR = 128 / N, PER = L_TOK / TPR;  // threads of a row, tokens of a thread
+    constexpr int CH = N < 32 ? N : 32;              // TMEM columns read at a time
+    constexpr int S_COLS = N;
+    const int gpr = p.geo.gpr, panels = gpr >> 3, tile_units = (panels + 1) >> 1, blocks = (p.geo.d_value + 127) >> 7;
+    const Layout lay = layout_of<N>(gpr, units);
+    const uint32_t sbase = smem_u32(smem);
+    const uint32_t q_base = sbase + lay.q, w_base = sbase + lay.weights;
+    float* const sc = reinterpret_cast<float*>(smem + lay.scores);
+    uint64_t* const bar_mem = reinterpret_cast<uint64_t*>(smem + lay.end);
+    const uint32_t full = smem_u32(bar_mem), empty = full + 8 * L_MAX_UNITS, s_full = empty + 8 * L_MAX_UNITS, p_full = s_full + 16,
+                   o_done = p_full + 8, q_ready = o_done + 8;
+    float* const alpha_s = reinterpret_cast<float*>(bar_mem + 2 * L_MAX_UNITS + 5);  // [N]
+    int* const flag_s = reinterpret_cast<int*>(alpha_s + L_MAX_ROWS);                 // [2]
+    uint32_t* const tmem_slot = reinterpret_cast<uint32_t*>(flag_s + 2);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int H = p.n_heads, gpr = p.geo.gpr, panels = gpr >> 3;
-    const int q_bytes = ROWS * gpr * 16, stage_bytes = NT * gpr * 16;
-    const uint32_t q_base = smem_u32(smem), ring = q_base + q_bytes, w_base = ring + stages * stage_bytes;
-    const uint32_t bars = smem_u32(full);
+    const int H = p.n_heads;
 
     // ---- the block of rows and its tokens: [start, end) relative to position `first` of list[0]
-    int token0, n_rows, first, end, low, row_lo = 0, slot_base = 0;
+    int token0, n_rows, first, end, low, row_lo = (int)blockIdx.y * N, slot_base = 0;
     const int32_t* list;
     if (SPAN) {
         const int4 b = reinterpret_cast<const int4*>(p.blocks)[blockIdx.x];
         token0 = b.y;
         n_rows = (b.z - b.y) * H;
+        if (row_lo >= n_rows) return;
+        n_rows = min(N, n_rows - row_lo);
         first = 0;
         list = p.path_chunks + p.path_off[b.x];
-        row_lo = (int)blockIdx.y * ROWS;
-        if (row_lo >= n_rows) return;
-        n_rows = min(ROWS, n_rows - row_lo);
         end = p.positions[token0 + (row_lo + n_rows - 1) / H] + 1;
         low = p.positions[token0 + row_lo / H];
     } else {
-        const int* it = reinterpret_cast<const int*>(p.items) + 16 * blockIdx.x;
-        const int n_tiles = it[0], flags = it[5], last = it[6];
-        first = it[1];
-        token0 = it[2];
-        n_rows = it[3] * H;
-        slot_base = it[4];
-        list = it + 7;
-        end = (n_tiles - 1) * L_CHUNK + min(L_CHUNK, last + ((flags & ITEM_FLAG_TAIL) ? p.delta_tokens : 0));
-        low = p.positions[token0];
-        for (int i = 1; i < it[3]; i++) low = min(low, p.positions[token0 + i]);
-        row_lo = (int)blockIdx.y * ROWS;
+        const int4* it = p.items + 4 * blockIdx.x;
+        const int4 a = __ldg(it), b = __ldg(it + 1);  // tiles, first, row, rows | slot, flags, last, chunks ...
+        token0 = a.z;
+        n_rows = a.w * H;
         if (row_lo >= n_rows) return;
-        n_rows = min(ROWS, n_rows - row_lo);
+        n_rows = min(N, n_rows - row_lo);
+        first = a.y;
+        slot_base = b.x;
+        list = reinterpret_cast<const int32_t*>(it) + 7;
+        end = (a.x - 1) * L_TOK + min(L_TOK, b.z + ((b.y & ITEM_FLAG_TAIL) ? p.delta_tokens : 0));
+        low = p.positions[token0];
+        for (int i = 1; i < a.w; i++) low = min(low, p.positions[token0 + i]);
     }
-    const int start = p.window > 0 ? max(0, low - p.window + 1 - first) / NT * NT : 0;
-    const int n_tiles = end > start ? (end - start + NT - 1) / NT : 0;
-    const int m_tiles = (n_rows + 15) >> 4;
+    const int start = p.window > 0 ? max(0, low - p.window + 1 - first) / L_TOK * L_TOK : 0;
+    const int n_tiles = end > start ? (end - start + L_TOK - 1) / L_TOK : 0;
+    const int tail = end - start - (n_tiles - 1) * L_TOK;  // tokens of the last tile
 
     if (tid == 0) {
-        for (int i = 0; i < stages; i++) mbar_init(bars + 8 * i, 1);
+        for (int i = 0; i < units; i++) {
+            mbar_init(full + 8 * i, 1);
+            mbar_init(empty + 8 * i, 1);
+        }
+        mbar_init(s_full, 1);
+        mbar_init(s_full + 8, 1);
+        mbar_init(p_full, 128);
+        mbar_init(o_done, 1);
+        mbar_init(q_ready, 128);
+        flag_s[0] = flag_s[1] = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
+    // Only the stored tokens of the last tile are copied.  The lines behind them meet weights of zero, so they only have to be
+    // finite: they are cleared in the units that tile will use (what earlier tiles bring there is finite, too).
+    if (n_tiles > 0 && tail < L_TOK) {
+        const int lines = L_TOK - tail;
+        for (int i = tid; i < tile_units * 2 * lines * 8; i += L_THREADS) {
+            const int pn = i / (lines * 8), q = i % (lines * 8);
+            const int unit = ((n_tiles - 1) * tile_units + (pn >> 1)) % units;
+            sts128_zero(sbase + unit * L_UNIT + (pn & 1) * L_PANEL + tail * 128 + q * 16);
+        }
+        fence_proxy_async();
+    }
+    constexpr uint32_t COLS = 2 * S_COLS + 4 * N <= 128 ? 128 : (2 * S_COLS + 4 * N <= 256 ? 256 : 512);
+    constexpr uint32_t COL_S = 4 * N;  // O blocks at columns 0, N, 2 N, 3 N
+    if (warp == 5) {  // the warp that allocates is the warp that frees
+        tmem_alloc(smem_u32(tmem_slot), COLS);
+        tmem_relinquish_alloc_permit();
+    }
+    tc_fence_before_thread_sync();
     __syncthreads();
-    auto copy_tile = [&](int j) {  // one thread
-        const int at = start + j * NT, lines = min(NT, end - at);
-        const uint32_t dst = ring + (j % stages) * stage_bytes, bar = bars + 8 * (j % stages);
-        int chunk = __ldg(list + at / L_CHUNK);
-        if (chunk < 0 || chunk >= p.max_chunks) {
-            atomicCAS(p.status, STATUS_OK, STATUS_BAD_WORK_LIST);
-            chunk = 0;
-        }
-        const uint8_t* src = static_cast<const uint8_t*>(p.pool) + (size_t)chunk * (L_CHUNK * 16) * gpr + (at % L_CHUNK) * 128;
-        mbar_arrive_expect_tx(bar, lines * gpr * 16);
-        if (lines == L_CHUNK) {
-            bulk_copy_g2s(dst, src, stage_bytes, bar);
-        } else {
-            for (int pn = 0; pn < panels; pn++) bulk_copy_g2s(dst + pn * (NT * 128), src + pn * (L_CHUNK * 128), lines * 128, bar);
-        }
-    };
-    if (tid == 0)
-        for (int j = 0; j < min(stages - 1, n_tiles); j++) copy_tile(j);
+    tc_fence_after_thread_sync();
+    const uint32_t tmem_base = *tmem_slot;
 
-    // ---- queries: latent part as it comes, shared part turned by the row's position, zeros up to the pool's row
-    {
-        const bool whole = p.kv_rank % 8 == 0 && reinterpret_cast<uintptr_t>(p.q_lat) % 16 == 0;
-        const __nv_bfloat16* q_lat = static_cast<const __nv_bfloat16*>(p.q_lat);
-        const __nv_bfloat16* q_rot = static_cast<const __nv_bfloat16*>(p.q_rot);
-        const int half = p.rot / 2;
-        for (int i = tid; i < ROWS * gpr; i += L_THREADS) {
-            const int r = i / gpr, g = i % gpr, rr = row_lo + r, token = token0 + rr / H, head = rr % H;
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (r < n_rows) {
-                const __nv_bfloat16* src = q_lat + ((size_t)token * H + head) * p.kv_rank;
-                if (whole && 8 * g < p.kv_rank) {
-                    v = *reinterpret_cast<const uint4*>(src + 8 * g);
-                } else if (8 * g < p.kv_rank + p.rot) {
+    if (warp == 4) {
+        // ---- producer
+        if (lane == 0) {
+            int issued = 0;
+            bool live = true;
+            for (int j = 0; j < n_tiles && live; j++) {
+                const int at = start + j * L_TOK;
+                const uint32_t bytes = min(L_TOK, end - at) * 128;
+                int chunk = __ldg(list + at / L_TOK);
+                if (chunk < 0 || chunk >= p.max_chunks) {
+                    report(p.status, STATUS_BAD_WORK_LIST);
+                    chunk = 0;
+                }
+                const uint8_t* src = static_cast<const uint8_t*>(p.pool) + (size_t)chunk * (L_TOK * 16) * gpr;
+                for (int u = 0; u < tile_units; u++, issued++) {
+                    const int slot = issued % units;
+                    if (!mbar_wait_bounded(empty + 8 * slot, ((issued / units) & 1) ^ 1, p.wait_limit)) {
+                        report(p.status, STATUS_EMPTY_WAIT_TIMEOUT);
+                        live = false;
+                        break;
+                    }
+                    const bool two = 2 * u + 1 < panels;
+                    const uint32_t dst = sbase + slot * L_UNIT, bar = full + 8 * slot;
+                    mbar_arrive_expect_tx(bar, two ? 2 * bytes : bytes);
+                    if (two && bytes == L_PANEL) {
+                        bulk_copy_g2s(dst, src + 2 * u * L_PANEL, 2 * L_PANEL, bar);
+                    } else {
+                        bulk_copy_g2s(dst, src + 2 * u * L_PANEL, bytes, bar);
+                        if (two) bulk_copy_g2s(dst + L_PANEL, src + (2 * u + 1) * L_PANEL, bytes, bar);
+                    }
+                }
+            }
+            for (int f = issued > units ? issued - units : 0; f < issued; f++) {
+                if (!mbar_wait_bounded(full + 8 * (f % units), (f / units) & 1, p.wait_limit)) {
+                    report(p.status, STATUS_DRAIN_TIMEOUT);
+                    break;
+                }
+            }
+        }
+    } else if (warp == 5) {
+        // ---- MMA issuer: one thread.  Whatever is ready goes first: the scores of the next tile when its rows have
+        // arrived (at most one tile ahead of the second product: there are two score buffers), or the second product
+        if (elect_one() && n_tiles > 0) {
+            constexpr uint32_t DESC_HI = umma_desc_sw128_hi(1024);
+            constexpr uint32_t IDESC_QK = idesc_bf16(L_TOK, N, false), IDESC_PV = idesc_bf16(128, N, true);
+            bool live = mbar_wait_bounded(q_ready, 0, p.wait_limit);
+            if (!live) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
+            const uint32_t q_lo = umma_desc_sw128_lo(q_base, 16);
+            int jq = 0, jv = 0;
+            long long since = clock64();
+            while (live && jv < n_tiles) {
+                if (jq < n_tiles && jq <= jv + 1) {
+                    const int last = jq * tile_units + tile_units - 1;
+                    if (mbar_test_wait(full + 8 * (last % units), (last / units) & 1)) {
+                        const uint32_t d = tmem_base + COL_S + (jq & 1) * S_COLS;
+                        for (int u = 0; u < tile_units && live; u++) {
+                            const int g = jq * tile_units + u, slot = g % units;
+                            live = mbar_wait_bounded(full + 8 * slot, (g / units) & 1, p.wait_limit);
+                            if (!live) break;
+                            tc_fence_after_thread_sync();
+                            const uint32_t a_lo = umma_desc_sw128_lo(sbase + slot * L_UNIT, 16);
+                            const int n_pan = 2 * u + 1 < panels ? 2 : 1;
+                            for (int pn = 0; pn < n_pan; pn++)
+#pragma unroll
+                                for (int ks = 0; ks < 4; ks++) {
+                                    const uint64_t a = umma_desc_pack(a_lo + ((pn * L_PANEL + ks * 32) >> 4), DESC_HI);
+                                    const uint64_t b = umma_desc_pack(q_lo + (((2 * u + pn) * (N * 128) + ks * 32) >> 4), DESC_HI);
+                                    umma_ss_f16(d, a, b, IDESC_QK, (u > 0 || pn > 0 || ks > 0) ? 1u : 0u);
+                                }
+                            if (u >= blocks) umma_commit(empty + 8 * slot);  // holds no values
+                        }
+                        if (!live) {
+                            report(p.status, STATUS_FULL_WAIT_TIMEOUT);
+                            break;
+                        }
+                        umma_commit(s_full + 8 * (jq & 1));
+                        jq++;
+                        since = clock64();
+                        continue;
+                    }
+                }
+                if (jv < jq && mbar_test_wait(p_full, jv & 1)) {
+                    tc_fence_after_thread_sync();
+                    for (int m = 0; m < blocks; m++) {
+                        const int slot = (jv * tile_units + m) % units;
+                        const uint32_t d = tmem_base + m * N;
+                        const uint32_t a_lo = umma_desc_sw128_lo(sbase + slot * L_UNIT, L_PANEL);
+#pragma unroll
+                        for (int part = 0; part < 2; part++) {
+                            const uint32_t b_lo = umma_desc_sw128_lo(w_base + part * (N * 128), 16);
+#pragma unroll
+                            for (int kk = 0; kk < 4; kk++)
+                                umma_ss_f16(d, umma_desc_pack(a_lo + ((kk * 2048) >> 4), DESC_HI), umma_desc_pack(b_lo + ((kk * 32) >> 4), DESC_HI),
+                                            IDESC_PV, (jv > 0 || part > 0 || kk > 0) ? 1u : 0u);
+                        }
+                        umma_commit(empty + 8 * slot);
+                    }
+                    umma_commit(o_done);
+                    jv++;
+                    since = clock64();
+                    continue;
+                }
+                if (clock64() - since > p.wait_limit) {
+                    report(p.status, STATUS_FULL_WAIT_TIMEOUT);
+                    live = false;
+                }
+            }
+        }
+    } else {
+        // ---- queries: latent part as it comes, shared part turned by the row's position, zeros up to the pool's row
+        {
+            const bool whole = p.kv_rank % 8 == 0 && reinterpret_cast<uintptr_t>(p.q_lat) % 16 == 0;
+            const __nv_bfloat16* q_lat = static_cast<const __nv_bfloat16*>(p.q_lat);
+            const __nv_bfloat16* q_rot = static_cast<const __nv_bfloat16*>(p.q_rot);
+            const int half = p.rot / 2, rot_g = p.kv_rank / 8;  // granules below rot_g hold latent elements only
+            auto line = [&](int r, int g) { return q_base + (g >> 3) * (N * 128) + r * 128 + (((g & 7) ^ (r & 7)) << 4); };
+            const int lat_g = whole ? rot_g : 0;
+            for (int r = warp; r < N; r += 4) {
+                const int rr = row_lo + r, token = token0 + rr / H, head = rr % H;
+                const uint4* src = reinterpret_cast<const uint4*>(q_lat + ((size_t)token * H + head) * p.kv_rank);
+                for (int g = lane; g < lat_g; g += 32) {
+                    const uint4 v = r < n_rows ? __ldg(src + g) : make_uint4(0u, 0u, 0u, 0u);
+                    sts128(line(r, g), (int)v.x, (int)v.y, (int)v.z, (int)v.w);
+                }
+            }
+            for (int i = tid; i < N * (gpr - lat_g); i += 128) {
+                const int r = i / (gpr - lat_g), g = lat_g + i % (gpr - lat_g), rr = row_lo + r, token = token0 + rr / H, head = rr % H;
+                uint4 v = make_uint4(0u, 0u, 0u, 0u);
+                if (r < n_rows && 8 * g < p.kv_rank + p.rot) {
+                    const __nv_bfloat16* src = q_lat + ((size_t)token * H + head) * p.kv_rank;
                     const __nv_bfloat16* qr = q_rot + (size_t)token * p.q_rot_row + (size_t)head * p.q_rot_head;
+                    const float pos = (float)p.positions[token];
                     float x[8];
 #pragma unroll
                     for (int k = 0; k < 8; k++) {
@@ -144,277 +286,217 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                         } else if (d < p.rot) {
                             const int pair = d < half ? d : d - half;
                             float sn, cs;
-                            fast_sincos((float)p.positions[token] * p.freq[pair], &sn, &cs);
+                            fast_sincos(pos * __ldg(p.freq + pair), &sn, &cs);
                             const float a = __bfloat162float(qr[pair]), b = __bfloat162float(qr[pair + half]);
                             x[k] = d < half ? a * cs - b * sn : b * cs + a * sn;
                         }
                     }
                     v = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
                 }
+                sts128(line(r, g), (int)v.x, (int)v.y, (int)v.z, (int)v.w);
             }
-            sts128(q_base + staged<ROWS>(r, g), (int)v.x, (int)v.y, (int)v.z, (int)v.w);
+            fence_proxy_async();
+            mbar_arrive(q_ready);
         }
-    }
 
-    // ---- roles: rows and tokens of the first product, columns of the second
-    const int my_m = warp % MT, my_run = warp / MT;
-    const bool busy = my_m < m_tiles;
-    int lo[2], hi[2];  // positions a row sees, relative to `first`
-#pragma unroll
-    for (int h = 0; h < 2; h++) {
-        const int r = my_m * 16 + (lane >> 2) + 8 * h;
-        lo[h] = hi[h] = 0;
-        if (r < n_rows) {
-            const int pos = p.positions[token0 + (row_lo + r) / H] - first;
-            hi[h] = min(pos + 1, end);
-            lo[h] = p.window > 0 ? pos - p.window + 1 : 0;
+        // ---- softmax: thread tid has PER tokens of row tid / TPR: fours of tokens, TPR threads side by side
+        const int row = tid / TPR, part = tid % TPR;
+        int lo = 0, hi = 0;  // what the row sees, relative to `first`
+        if (row < n_rows) {
+            const int pos = p.positions[token0 + (row_lo + row) / H] - first;
+            hi = min(pos + 1, end);
+            lo = p.window > 0 ? pos - p.window + 1 : 0;
         }
-    }
-    float o[MT][NV][4], m[2] = {L_NEG_BIG, L_NEG_BIG}, l[2] = {0.f, 0.f};
-#pragma unroll
-    for (int a = 0; a < MT; a++)
-#pragma unroll
-        for (int i = 0; i < NV; i++)
-#pragma unroll
-            for (int k = 0; k < 4; k++) o[a][i][k] = 0.f;
-    const int mat = lane >> 3, r8 = lane & 7;
-    __syncthreads();  // the queries are staged
-
-    for (int j = 0; j < n_tiles; j++) {
-        const uint32_t tile = ring + (j % stages) * stage_bytes;
-        bool ok = mbar_wait_bounded(bars + 8 * (j % stages), (j / stages) & 1, p.wait_limit);
-        ok = __all_sync(0xffffffffu, ok);
-        const int at = start + j * NT, lines = min(NT, end - at);
-        if (lines < NT) {
-            // the lines behind the stored ones meet weights of zero and only have to be finite
-            for (int i = tid; i < panels * (NT - lines) * 8; i += L_THREADS) {
-                const int pn = i / ((NT - lines) * 8), q = i % ((NT - lines) * 8);
-                sts128_zero(tile + pn * (NT * 128) + lines * 128 + q * 16);
+        const float scale = fabsf(p.scale_log2), sign = p.scale_log2 < 0.f ? -1.f : 1.f;
+        const uint32_t lane_addr = tmem_base + ((uint32_t)(warp * 32) << 16);
+        float m_used = L_NEG_BIG, l = 0.f;
+        bool live = true;
+        for (int j = 0; j < n_tiles; j++) {
+            const int b = j & 1, at = start + j * L_TOK;
+            // a wait that has run out lets everything run through without waiting: the warps keep meeting at their barriers
+            if (live) {
+                live = mbar_wait_bounded(s_full + 8 * b, (j >> 1) & 1, p.wait_limit);
+                live = __all_sync(0xffffffffu, live);
+                if (!live && lane == 0) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
             }
-        }
-        // ---- scores of 16 rows x RUN tokens
-        float s[NB][4];
+            tc_fence_after_thread_sync();
+            // M = 64: token 16 w + i is lane i of warp w
 #pragma unroll
-        for (int i = 0; i < NB; i++)
+            for (int c = 0; c < N; c += CH) {
+                uint32_t s[CH];
+                tmem_ld<CH>(lane_addr + COL_S + b * S_COLS + c, s);
+                tmem_wait_ld();
+                if (lane < 16) {
 #pragma unroll
-            for (int k = 0; k < 4; k++) s[i][k] = 0.f;
-        const int tb = my_run * RUN;
-        if (busy && ok) {
-            const int a_row = my_m * 16 + (lane & 15), a_g = lane >> 4;
-            if (NB == 2) {
-#pragma unroll 4
-                for (int ks = 0; ks < gpr / 2; ks++) {
-                    uint32_t a[4], b0, b1, b2, b3;
-                    ldsm_x4(a[0], a[1], a[2], a[3], q_base + staged<ROWS>(a_row, 2 * ks + a_g));
-                    ldsm_x4(b0, b1, b2, b3, tile + staged<NT>(tb + (mat >> 1) * 8 + r8, 2 * ks + (mat & 1)));
-                    mma_bf16(s[0], a, b0, b1);
-                    mma_bf16(s[NB - 1], a, b2, b3);
+                    for (int i = 0; i < CH; i++) sc[(c + i) * (L_TOK + 4) + warp * 16 + lane] = __uint_as_float(s[i]);
                 }
-            } else {
-                float s2[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-                for (int ks = 0; ks < gpr / 2; ks += 2) {
-                    uint32_t a[4], c[4], b0, b1, b2, b3;
-                    ldsm_x4(a[0], a[1], a[2], a[3], q_base + staged<ROWS>(a_row, 2 * ks + a_g));
-                    ldsm_x4(c[0], c[1], c[2], c[3], q_base + staged<ROWS>(a_row, 2 * ks + 2 + a_g));
-                    ldsm_x4(b0, b1, b2, b3, tile + staged<NT>(tb + r8, 2 * ks + mat));
-                    mma_bf16(s[0], a, b0, b1);
-                    mma_bf16(s2, c, b2, b3);
+            }
+            tc_fence_before_thread_sync();
+            softmax_warps_sync();
+            if (tid == 0) flag_s[b ^ 1] = 0;  // everyone has read it in the tile before
+            float x[PER];
+            float mx = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < PER / 4; i++) {
+                const int t = (i * TPR + part) * 4;
+                const float4 v = *reinterpret_cast<const float4*>(sc + row * (L_TOK + 4) + t);
+                const float in[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+                for (int k = 0; k < 4; k++) {
+                    const int c = at + t + k;
+                    x[4 * i + k] = c >= lo && c < hi ? in[k] * sign : -INFINITY;
+                    mx = fmaxf(mx, x[4 * i + k]);
                 }
-#pragma unroll
-                for (int k = 0; k < 4; k++) s[0][k] += s2[k];
-            }
-        }
-        const int col = at + tb + (lane & 3) * 2;  // of s[i][0], relative to `first`: + 8 i
-        float mx[2] = {L_NEG_BIG, L_NEG_BIG};
-#pragma unroll
-        for (int i = 0; i < NB; i++)
-#pragma unroll
-            for (int k = 0; k < 4; k++) {
-                const int c = col + 8 * i + (k & 1);
-                s[i][k] = c >= lo[k >> 1] && c < hi[k >> 1] ? s[i][k] * p.scale_log2 : -INFINITY;
-                mx[k >> 1] = fmaxf(mx[k >> 1], s[i][k]);
             }
 #pragma unroll
-        for (int h = 0; h < 2; h++) {
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-            if ((lane & 3) == 0) red[my_run][my_m * 16 + (lane >> 2) + 8 * h] = mx[h];
-        }
-        if (!__syncthreads_and(ok)) {
-            if (tid == 0) {
-                atomicCAS(p.status, STATUS_OK, STATUS_FULL_WAIT_TIMEOUT);
-                for (int f = j; f < min(n_tiles, j + stages - 1); f++)
-                    mbar_wait_bounded(bars + 8 * (f % stages), (f / stages) & 1, p.wait_limit);
+            for (int o = 1; o < TPR; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            mx = scale == 0.f ? 0.f : fmaxf(mx * scale, L_NEG_BIG);
+            float alpha = 1.f;
+            if (j == 0) {
+                m_used = mx;
+            } else if (mx > m_used + L_RESCALE_STEP) {
+                alpha = fast_exp2(m_used - mx);
+                m_used = mx;
+                l *= alpha;
+                flag_s[b] = 1;
             }
-            return;
-        }
-        // every warp is past tile j - 1: its slot takes tile j + stages - 1
-        if (tid == 0 && j + stages - 1 < n_tiles) copy_tile(j + stages - 1);
-        if (busy) {
-            float alpha[2];
-#pragma unroll
-            for (int h = 0; h < 2; h++) {
-                const int r = my_m * 16 + (lane >> 2) + 8 * h;
-                float mn = m[h];
-#pragma unroll
-                for (int t = 0; t < TS; t++) mn = fmaxf(mn, red[t][r]);
-                alpha[h] = fast_exp2(m[h] - mn);
-                m[h] = mn;
-                if (my_run == 0 && (lane & 3) == 0) alpha_s[r] = alpha[h];
-                float sum = 0.f;
-#pragma unroll
-                for (int i = 0; i < NB; i++) {
-                    const float a = fast_exp2(s[i][2 * h] - mn), b = fast_exp2(s[i][2 * h + 1] - mn);
-                    sum += a + b;
-                    const uint32_t hw = pack_bf16(a, b);
-                    const uint32_t lw = pack_bf16(a - __uint_as_float(hw << 16), b - __uint_as_float(hw & 0xffff0000u));
-                    const int t = tb + 8 * i + (lane & 3) * 2;
-                    sts32(w_base + weight_at<MT>(0, r, t >> 3) + (t & 7) * 2, hw);
-                    sts32(w_base + weight_at<MT>(1, r, t >> 3) + (t & 7) * 2, lw);
+            if (part == 0) alpha_s[row] = alpha;
+            softmax_warps_sync();
+            if (j > 0) {
+                // the second product of tile j - 1 is complete: O may be rescaled and the weights replaced
+                if (live) {
+                    live = mbar_wait_bounded(o_done, (j - 1) & 1, p.wait_limit);
+                    live = __all_sync(0xffffffffu, live);
+                    if (!live && lane == 0) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
                 }
-                l[h] = l[h] * alpha[h] + sum;  // this lane's tokens only
-            }
-        }
-        __syncthreads();
-        // ---- O += P V over this warp's columns
-        const int c0 = warp * (8 * NV);
-        if (c0 < p.geo.d_value) {
+                if (*reinterpret_cast<volatile int*>(flag_s + b)) {
+                    tc_fence_after_thread_sync();
+                    for (int m = 0; m < blocks; m++)
 #pragma unroll
-            for (int a = 0; a < MT; a++)
-                if (a < m_tiles) {
-                    const float x = alpha_s[a * 16 + (lane >> 2)], y = alpha_s[a * 16 + (lane >> 2) + 8];
-                    if (__any_sync(0xffffffffu, x != 1.f || y != 1.f)) {
+                        for (int c = 0; c < N; c += CH) {
+                            uint32_t o[CH];
+                            tmem_ld<CH>(lane_addr + m * N + c, o);
+                            tmem_wait_ld();
 #pragma unroll
-                        for (int i = 0; i < NV; i++) {
-                            o[a][i][0] *= x;
-                            o[a][i][1] *= x;
-                            o[a][i][2] *= y;
-                            o[a][i][3] *= y;
+                            for (int i = 0; i < CH; i++) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha_s[c + i]);
+                            if constexpr (CH == 32) tmem_st32(lane_addr + m * N + c, o);
+                            else tmem_st16(lane_addr + m * N + c, o);
                         }
-                    }
+                    tmem_wait_st();
                 }
-#pragma unroll
-            for (int kk = 0; kk < NT / 16; kk++) {
-                uint32_t b[NV][2];
-#pragma unroll
-                for (int i = 0; i < NV; i += 2) {
-                    // columns past d_value (NV rounded up) are neither read nor stored
-                    const int c = c0 + 8 * i < p.geo.d_value ? c0 + 8 * i : c0;
-                    ldsm_x4_trans(b[i][0], b[i][1], b[i + 1][0], b[i + 1][1],
-                                  tile + staged<NT>(16 * kk + (mat & 1) * 8 + r8, c / 8 + (mat >> 1)));
-                }
-#pragma unroll
-                for (int a = 0; a < MT; a++)
-                    if (a < m_tiles) {
-                        uint32_t hw[4], lw[4];
-                        const int r = a * 16 + (lane & 15), g = 2 * kk + (lane >> 4);
-                        ldsm_x4(hw[0], hw[1], hw[2], hw[3], w_base + weight_at<MT>(0, r, g));
-                        ldsm_x4(lw[0], lw[1], lw[2], lw[3], w_base + weight_at<MT>(1, r, g));
-#pragma unroll
-                        for (int i = 0; i < NV; i++) {
-                            mma_bf16(o[a][i], hw, b[i][0], b[i][1]);
-                            mma_bf16(o[a][i], lw, b[i][0], b[i][1]);
-                        }
-                    }
             }
+#pragma unroll
+            for (int i = 0; i < PER / 4; i++) {
+                const int t = (i * TPR + part) * 4;
+                float e[4];
+#pragma unroll
+                for (int k = 0; k < 4; k++) {
+                    e[k] = x[4 * i + k] == -INFINITY ? 0.f : fast_exp2(fmaf(x[4 * i + k], scale, -m_used));
+                    l += e[k];
+                }
+                const uint32_t h0 = pack_bf16(e[0], e[1]), h1 = pack_bf16(e[2], e[3]);
+                const uint32_t l0 = pack_bf16(e[0] - __uint_as_float(h0 << 16), e[1] - __uint_as_float(h0 & 0xffff0000u));
+                const uint32_t l1 = pack_bf16(e[2] - __uint_as_float(h1 << 16), e[3] - __uint_as_float(h1 & 0xffff0000u));
+                const uint32_t dst = w_base + row * 128 + (((t >> 3) ^ (row & 7)) << 4) + (t & 4) * 2;
+                sts64(dst, h0, h1);
+                sts64(dst + N * 128, l0, l1);
+            }
+            fence_proxy_async();
+            tc_fence_before_thread_sync();
+            mbar_arrive(p_full);
         }
-    }
-
-    // ---- sums of the runs, then every warp stores its columns
-    __syncthreads();
-#pragma unroll
-    for (int h = 0; h < 2; h++) {
-        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
-        l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
-        const int r = my_m * 16 + (lane >> 2) + 8 * h;
-        if ((lane & 3) == 0) {
-            red[my_run][r] = l[h];
-            if (my_run == 0) m_s[r] = m[h];
+        if (n_tiles > 0 && live) {
+            live = mbar_wait_bounded(o_done, (n_tiles - 1) & 1, p.wait_limit);
+            live = __all_sync(0xffffffffu, live);
+            if (!live && lane == 0) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
         }
-    }
-    __syncthreads();
-    const int c0 = warp * (8 * NV);
+        tc_fence_after_thread_sync();
+        // ---- epilogue: the factor of every row through shared memory, then lane = value element, column = row
 #pragma unroll
-    for (int a = 0; a < MT; a++)
-#pragma unroll
-        for (int h = 0; h < 2; h++) {
-            const int r = a * 16 + (lane >> 2) + 8 * h;
-            if (r >= n_rows) continue;
-            float M = m_s[r], L = 0.f;
-#pragma unroll
-            for (int t = 0; t < TS; t++) L += red[t][r];
-            const int rr = row_lo + r, token = token0 + rr / H, head = rr % H;
+        for (int o = 1; o < TPR; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+        if (part == 0) {
+            const int rr = row_lo + row, head = rr % H;
+            float f = 1.f;
             if (SPAN) {
-                float f = 1.f;
-                if (p.sink) {
-                    const float sk = p.sink[head] * L_LOG2E, top = fmaxf(M, sk);
-                    f = fast_exp2(M - top);
-                    L = L * f + fast_exp2(sk - top);
+                float total = l, M = m_used;
+                if (p.sink && row < n_rows) {
+                    const float sk = p.sink[head] * L_LOG2E;
+                    M = fmaxf(m_used, sk);
+                    total = l * fast_exp2(m_used - M) + fast_exp2(sk - M);
                 }
-                f = L > 0.f ? f / L : 0.f;
-                __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + ((size_t)token * H + head) * p.kv_rank;
+                f = total > 0.f ? fast_exp2(m_used - M) / total : 0.f;
+            } else if (row < n_rows && live) {
+                p.part_ml[((size_t)slot_base + rr / H) * H + head] = make_float2(m_used, l);
+            }
+            alpha_s[row] = f;
+        }
+        softmax_warps_sync();
+        if (live) {
+            for (int m = 0; m < blocks; m++) {
+                const int e = m * 128 + warp * 32 + lane;
 #pragma unroll
-                for (int i = 0; i < NV; i++) {
-                    const int c = c0 + 8 * i + (lane & 3) * 2;
-                    const float x = o[a][i][2 * h] * f, y = o[a][i][2 * h + 1] * f;
-                    if (p.kv_rank % 2 == 0) {
-                        if (c < p.kv_rank) *reinterpret_cast<uint32_t*>(out + c) = pack_bf16(x, y);
+                for (int c = 0; c < N; c += CH) {
+                    uint32_t o[CH];
+                    if (n_tiles > 0) {
+                        tmem_ld<CH>(lane_addr + m * N + c, o);
+                        tmem_wait_ld();
                     } else {
-                        if (c < p.kv_rank) out[c] = __float2bfloat16_rn(x);
-                        if (c + 1 < p.kv_rank) out[c + 1] = __float2bfloat16_rn(y);
-                    }
-                }
-            } else {
-                const size_t slot = (size_t)slot_base * H + (size_t)(rr / H) * H + head;
-                if (warp == 0 && (lane & 3) == 0) p.part_ml[slot] = make_float2(M, L);
-                float* dst = p.part_o + slot * p.part_width;
 #pragma unroll
-                for (int i = 0; i < NV; i++) {
-                    const int c = c0 + 8 * i + (lane & 3) * 2;
-                    if (c < p.part_width) *reinterpret_cast<float2*>(dst + c) = make_float2(o[a][i][2 * h], o[a][i][2 * h + 1]);
+                        for (int i = 0; i < CH; i++) o[i] = 0u;
+                    }
+#pragma unroll
+                    for (int i = 0; i < CH; i++) {
+                        const int r = c + i, rr = row_lo + r;
+                        if (r >= n_rows) break;
+                        if (SPAN) {  // rows are consecutive (token, head) pairs
+                            if (e < p.kv_rank)
+                                static_cast<__nv_bfloat16*>(p.out)[((size_t)token0 * H + rr) * p.kv_rank + e] = __float2bfloat16_rn(__uint_as_float(o[i]) * alpha_s[r]);
+                        } else if (e < p.part_width) {
+                            p.part_o[((size_t)slot_base * H + rr) * p.part_width + e] = __uint_as_float(o[i]);
+                        }
+                    }
                 }
             }
         }
-}
-
-constexpr int L_SMEM_LIMIT = 227 * 1024 - 2048;  // static shared memory and alignment taken off
-
-template <int MT, int NV> cudaError_t launch(const LatentParams& p, cudaStream_t stream) {
-    const int q_bytes = 16 * MT * p.geo.gpr * 16, stage = tile_tokens<MT>() * p.geo.gpr * 16, weights = weight_bytes<MT>();
-    const int room = (L_SMEM_LIMIT - q_bytes - weights) / stage;
-    if (room < 2) return cudaErrorInvalidValue;
-    const int stages = std::min(room, L_MAX_STAGES), smem = q_bytes + stages * stage + weights;
-    const unsigned subs = (unsigned)((p.path_off ? p.block_rows * p.n_heads : std::max(p.n_heads, p.item_rows)) + 16 * MT - 1) / (16 * MT);
-    if (p.path_off) {
-        auto* k = latent_rows_kernel<MT, NV, true>;
-        cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-        if (e != cudaSuccess) return e;
-        k<<<dim3(p.n_blocks, subs), L_THREADS, smem, stream>>>(p, stages);
-    } else {
-        auto* k = latent_rows_kernel<MT, NV, false>;
-        cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-        if (e != cudaSuccess) return e;
-        k<<<dim3(p.n_items, subs), L_THREADS, smem, stream>>>(p, stages);
     }
-    return cudaGetLastError();
+    // ---- common exit: nobody touches TMEM after this barrier, then the allocating warp frees it
+    tc_fence_before_thread_sync();
+    __syncthreads();
+    if (warp == 5) {
+        tc_fence_after_thread_sync();
+        tmem_dealloc(tmem_base, COLS);
+    }
 }
 
-template <int MT> cudaError_t by_width(const LatentParams& p, cudaStream_t stream) {
-    if (p.geo.d_value <= 128) return launch<MT, 2>(p, stream);
-    if (p.geo.d_value <= 256) return launch<MT, 4>(p, stream);
-    return launch<MT, 8>(p, stream);
+constexpr int L_SMEM_LIMIT = 227 * 1024;
+constexpr int L_CONTROL = (2 * L_MAX_UNITS + 5) * 8 + L_MAX_ROWS * 4 + 16;  // barriers, row factors, flags, TMEM address
+
+template <int N> cudaError_t launch(const LatentParams& p, cudaStream_t stream) {
+    const int tile_units = ((p.geo.gpr >> 3) + 1) / 2, fixed = layout_of<N>(p.geo.gpr, 0).end + L_CONTROL;
+    // three tiles keep the copies ahead of the products; more would only keep other CTAs off the SM
+    const int units = std::min({L_MAX_UNITS, 3 * tile_units, (L_SMEM_LIMIT - fixed) / L_UNIT});
+    if (units < tile_units + 1) return cudaErrorInvalidValue;
+    const int smem = units * L_UNIT + fixed;
+    const int rows = p.path_off ? p.block_rows * p.n_heads : std::max(p.n_heads, p.item_rows);
+    auto* span = latent_rows_kernel<N, true>;
+    auto* items = latent_rows_kernel<N, false>;
+    auto* k = p.path_off ? span : items;
+    cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(k, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    if (e != cudaSuccess) return e;
+    k<<<dim3(p.path_off ? p.n_blocks : p.n_items, (rows + N - 1) / N), L_THREADS, smem, stream>>>(p, units);
+    return cudaGetLastError();
 }
 
 }  // namespace
 
 bool latent_rows_serves(const Geometry& g) {
-    return g.esize == 2 && g.chunk_size == L_CHUNK && g.swz && g.d_head <= 640 && g.d_value <= 512;
+    return g.esize == 2 && g.chunk_size == L_TOK && g.swz && g.d_head <= 640 && g.d_value <= 512;
 }
 
 cudaError_t launch_latent_rows(const LatentParams& p, cudaStream_t stream) {
-    const int rows = p.path_off ? std::min(64, p.block_rows * p.n_heads) : std::max(p.n_heads, p.item_rows);
-    cudaError_t e = rows <= 16 ? by_width<1>(p, stream) : (rows <= 32 ? by_width<2>(p, stream) : by_width<4>(p, stream));
+    const int rows = p.path_off ? p.block_rows * p.n_heads : std::max(p.n_heads, p.item_rows);
+    cudaError_t e = rows <= 16 ? launch<16>(p, stream) : (rows <= 32 ? launch<32>(p, stream) : launch<64>(p, stream));
     if (e != cudaSuccess || p.path_off) return e;
     RowsParams r{};
     r.geo = p.geo;

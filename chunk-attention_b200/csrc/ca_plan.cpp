@@ -28,7 +28,7 @@ std::string fmt(const char* f, long a = 0, long b = 0, long c = 0) {
 // remaining_tiles / n_ctas tiles, clamped to [1, MAX_TILES_PER_ITEM], so the list starts with
 // full-size items and ends with single tiles.
 void cut_units(Plan& plan, const std::vector<Unit>& units, size_t ubegin, size_t uend, int n_ctas, int n_heads,
-               int32_t& n_slots, int64_t tiles_elsewhere = 0) {
+               int32_t& n_slots, int64_t tiles_elsewhere = 0, int even_len = 0) {
     // tiles_elsewhere: work of the same step that other kernels do (the short tails); counting it keeps
     // the pieces of shared runs long - every piece of a run costs a partial row per sharer, so they
     // are not tapered down to single tiles for the sake of the last microsecond
@@ -38,12 +38,17 @@ void cut_units(Plan& plan, const std::vector<Unit>& units, size_t ubegin, size_t
     for (size_t u = ubegin; u < uend; u++) {
         const Unit& un = units[u];
         const int n_tiles = un.n_chunks;
-        int j = 0;
+        const int pieces = even_len > 0 ? (n_tiles + even_len - 1) / even_len : 0;
+        int j = 0, piece = 0;
         while (j < n_tiles) {
             int want = (int)std::min<int64_t>(MAX_TILES_PER_ITEM - 1, std::max<int64_t>(1, remaining / n_ctas));
+            if (pieces > 0) {
+                piece++;
+                want = (int)((int64_t)n_tiles * piece / pieces) - j;
+            }
             // a sequence's tail chunk (partially filled or still empty) rides along with the piece
             // before it instead of becoming an item of its own
-            if (n_tiles - (j + want) == 1 && un.tail) want++;
+            if (n_tiles - (j + want) == 1 && un.tail && pieces == 0) want++;
             const int len = std::min(want, n_tiles - j);
             plan.items.emplace_back();
             PlanItem& it = plan.items.back();
@@ -61,6 +66,29 @@ void cut_units(Plan& plan, const std::vector<Unit>& units, size_t ubegin, size_t
             remaining -= (int64_t)len * n_heads;
         }
     }
+}
+
+// Largest item for which n_ctas CTAs at a time, one item each, are done soonest: every wave takes as long as its largest
+// item, plus what setting up and storing an item costs.
+int even_length(const std::vector<Unit>& units, int n_ctas, int n_heads) {
+    constexpr double ITEM_OVERHEAD = 2.0;  // in tiles
+    int best = 1;
+    double best_cost = 0;
+    for (int len = 1; len <= MAX_TILES_PER_ITEM; len++) {
+        int64_t items = 0;
+        int longest = 0;
+        for (const Unit& u : units) {
+            const int pieces = (u.n_chunks + len - 1) / len;
+            items += (int64_t)pieces * n_heads;
+            if (pieces > 0) longest = std::max(longest, (u.n_chunks + pieces - 1) / pieces);
+        }
+        const double cost = (double)((items + n_ctas - 1) / n_ctas) * (longest + ITEM_OVERHEAD);
+        if (len == 1 || cost <= best_cost) {
+            best = len;
+            best_cost = cost;
+        }
+    }
+    return best;
 }
 
 // Position of the first token of every entry of a depth-first chunk list.
@@ -102,7 +130,7 @@ void build_paths(Plan& plan) {
 std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int n_seqs, int n_heads,
                        int chunk_size, int tpp_threshold, int n_ctas, int64_t max_chunks,
                        bool split_phases, int d_head, int esize, bool fast_path, bool seq_first_tensor, int wide_mode,
-                       bool want_paths, int rows_per_item, bool one_partial_per_row, int window) {
+                       bool want_paths, int rows_per_item, bool one_partial_per_row, int window, bool even_items) {
     if (rows_per_item < 1) rows_per_item = 1;
     plan.window = window;
     // the vectors keep their capacity from one rebuild to the next
@@ -305,7 +333,7 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
     }
     const int64_t short_tiles = (int64_t)short_units.size() * n_heads;
     if (!split_phases) {
-        cut_units(plan, units, 0, units.size(), n_ctas, n_heads, n_slots, short_tiles);
+        cut_units(plan, units, 0, units.size(), n_ctas, n_heads, n_slots, short_tiles, even_items ? even_length(units, n_ctas, n_heads) : 0);
         plan.n_items_cf = 0;
         for (const PlanItem& it : plan.items) plan.n_items_cf += it.n_rows > 1 ? 1 : 0;
     } else {

@@ -91,7 +91,8 @@ std::string build_plan(Plan& plan, const ca_chunk_info* infos, int n_infos, int 
                        bool want_paths = true,   // also build the per-row path lists of the any-geometry kernel
                        int rows_per_item = MAX_ROWS_PER_ITEM,
                        bool one_partial_per_row = false,   // items of shared runs do not emit a partial per token split
-                       int window = 0);  // > 0: chunks that lie before the window of every row they serve are left out
+                       int window = 0,  // > 0: chunks that lie before the window of every row they serve are left out
+                       bool even_items = false);  // items of about equal size, as many as fill whole waves of n_ctas CTAs
 // The per-row path lists (path_off / path_chunks / path_tokens) from plan.infos, for a plan built without them.
 void build_paths(Plan& plan);
 
