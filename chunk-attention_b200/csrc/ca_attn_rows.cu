@@ -378,12 +378,10 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
     if (pair >= p.n_rows * H) return;
     const int row = pair / H, head = pair % H;
     const int b = p.merge_off[row], n = p.merge_off[row + 1] - b;
-    const bool has_sink = p.sink || p.sink_scores;
-    const float sink = p.sink_scores ? p.sink_scores[head] * 1.4426950408889634f : 0.f;  // in log2 units
-    float M = has_sink ? sink : R_NEG_BIG;
+    float M = p.sink ? 0.f : R_NEG_BIG;
     for (int i = lane; i < n; i += 32) M = fmaxf(M, p.part_ml[(size_t)p.merge_slots[b + i] * H + head].x);
     M = warp_max(M);
-    float acc[K][2], L = has_sink && lane == 0 ? fast_exp2(sink - M) : 0.f;  // pairs lane + 32 k
+    float acc[K][2], L = p.sink && lane == 0 ? fast_exp2(-M) : 0.f;  // pairs lane + 32 k
 #pragma unroll
     for (int k = 0; k < K; k++) acc[k][0] = acc[k][1] = 0.f;
     const int pairs = p.part_width / 2;
@@ -397,7 +395,7 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
             L = fmaf(w, ml.y, L);
         }
         const int m = min(32, n - i0);
-        constexpr int AHEAD = K == 8 ? 4 : 8;  // partial rows requested together
+        constexpr int AHEAD = 8;  // partial rows requested together
         for (int ib = 0; ib < m; ib += AHEAD) {
             float2 x[AHEAD][K];
 #pragma unroll
@@ -441,21 +439,6 @@ __global__ void __launch_bounds__(256) rows_merge_kernel(const RowsParams p) {
     }
 }
 
-}  // namespace
-
-cudaError_t launch_rows_merge(const RowsParams& p, cudaStream_t stream) {
-    const int64_t pairs = (int64_t)p.n_rows * p.geo.n_heads * p.group;
-    const unsigned grid = (unsigned)((pairs + 7) / 8);
-    if (p.part_width <= 64) rows_merge_kernel<1><<<grid, 256, 0, stream>>>(p);
-    else if (p.part_width <= 128) rows_merge_kernel<2><<<grid, 256, 0, stream>>>(p);
-    else if (p.part_width <= 256) rows_merge_kernel<4><<<grid, 256, 0, stream>>>(p);
-    else if (p.part_width <= 512) rows_merge_kernel<8><<<grid, 256, 0, stream>>>(p);
-    else return cudaErrorInvalidValue;
-    return cudaGetLastError();
-}
-
-namespace {
-
 template <int DK, int DV, int STAGES, bool BULK>
 cudaError_t launch(const RowsParams& p, cudaStream_t stream) {
     constexpr int ring = STAGES * R_TILE * (DK + DV) * 2 + (BULK ? STAGES * 8 : 0), out = 4 * 16 * (DV + 4) * 4 + 64 * 8;
@@ -472,7 +455,11 @@ cudaError_t launch(const RowsParams& p, cudaStream_t stream) {
         k<<<dim3(p.n_items * p.geo.n_heads, p.subs), R_THREADS, smem, stream>>>(p);
         e = cudaGetLastError();
         if (e != cudaSuccess) return e;
-        return launch_rows_merge(p, stream);
+        const int64_t pairs = (int64_t)p.n_rows * p.geo.n_heads * p.group;
+        const unsigned grid = (unsigned)((pairs + 7) / 8);
+        if (p.part_width <= 64) rows_merge_kernel<1><<<grid, 256, 0, stream>>>(p);
+        else if (p.part_width <= 128) rows_merge_kernel<2><<<grid, 256, 0, stream>>>(p);
+        else rows_merge_kernel<4><<<grid, 256, 0, stream>>>(p);
     }
     return cudaGetLastError();
 }

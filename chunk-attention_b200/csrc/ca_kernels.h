@@ -162,7 +162,6 @@ struct RowsParams {
     int n_rows;
     float scale_log2;            // scale * log2(e)
     int sink;
-    const float* sink_scores = nullptr;  // [query heads]: a score per head instead of the sink's 0 (merge kernel only)
     const int32_t* positions;    // [n_rows]
     const float* value_freq;     // null: values are not rotated
     int subs;                    // 64-row sub-blocks of a block
@@ -185,8 +184,6 @@ struct RowsParams {
     long long wait_limit;
 };
 cudaError_t launch_attn_rows(const RowsParams& p, cudaStream_t stream);
-// one warp per (row, query head): combines the row's partials
-cudaError_t launch_rows_merge(const RowsParams& p, cudaStream_t stream);
 
 // ---- latent caches (ca_latent.cu, ca_latent_rows.cu) -----------------------------------------------------------
 struct LatentStoreParams {

@@ -4,15 +4,17 @@
 // A token's pool row is key and value of every head at once, so the query heads of a token, and the tokens of a block, are
 // rows of ONE product against the rows staged in shared memory: row r is head r % H of token r / H.  There are few of them
 // (up to 64) and the values are long, so the products are formed transposed, cache rows and value elements on the M side:
-//   S^T = K Q^T   M = 64 tokens, N = query rows; D in TMEM, two buffers, so that the scores of tile j + 1 are computed under
-//                 the softmax of tile j
-//   softmax       the scores go through shared memory once, so that 128 / N threads share a query row; fp32, log2 units;
+//   S^T = K Q^T   two 64-element panels at a time: M = 64 tokens of one panel and the same 64 of the next, N = query rows of one
+//                 panel and of the next; the blocks on the diagonal of D are the two panels' shares of the scores (the others
+//                 are not used).  D in TMEM, two buffers, so that tile j + 1 is scored under the softmax of tile j
+//   softmax       the shares go through shared memory once, so that 128 / N threads share a query row; fp32, log2 units;
 //                 every row has a window.  O is rescaled only when a row's maximum has grown by more than 8.  The
 //                 weights go back to shared memory as bf16 hi + lo parts, whose sum has 16 bits of the fp32 weight
-//   O^T += V^T P^T  M = 128 value elements (one TMEM block each), N = query rows; A = the same staged rows read the other way
+//   O^T += V^T P^T  M = 128 value elements (one TMEM block each), N = hi and lo parts of the query rows (up to 32 rows: side by
+//                 side in one product; 64: one after the other); A = the same staged rows read the other way
 // Cache rows arrive by 1-D TMA bulk copies, verbatim (the pool's lines are the swizzled operand layout), in a ring of
 // 16 KiB units: two 64-element panels of a 64-token chunk, released one by one as the second product has used them.  Decode
-// emits one partial per row and item, combined by the merge kernel of ca_attn_rows.cu; portions emit finished rows.
+// emits one partial per row and item, combined by a merge kernel; portions emit finished rows.
 // Warp roles: 0-3 softmax and epilogue, 4 TMA producer, 5 TMEM and the MMA issue.
 //
 // Every wait is bounded: on expiry a status code is recorded, every role runs out without waiting further, nothing is
@@ -53,8 +55,8 @@ template <int N> __host__ __device__ inline Layout layout_of(int gpr, int units)
     l.units = units;
     l.q = units * L_UNIT;                        // queries: [gpr / 8 panels][N lines of 128 bytes]
     l.weights = l.q + N * gpr * 16;              // weights: hi and lo, [N lines of 64 tokens] each
-    l.scores = l.weights + 2 * N * 128;          // fp32 [N][L_TOK + 4]
-    l.end = l.scores + N * (L_TOK + 4) * 4;
+    l.scores = l.weights + 2 * N * 128;          // fp32 [2 shares][N][L_TOK + 4]
+    l.end = l.scores + 2 * N * (L_TOK + 4) * 4;
     return l;
 }
 
@@ -63,7 +65,8 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int TPR = 128 / N, PER = L_TOK / TPR;  // threads of a row, tokens of a thread
     constexpr int CH = N < 32 ? N : 32;              // TMEM columns read at a time
-    constexpr int S_COLS = N;
+    constexpr bool WIDE = N <= 32;                   // hi and lo weights in one product
+    constexpr int S_COLS = 2 * N, O_COLS = WIDE ? 2 * N : N;
     const int gpr = p.geo.gpr, panels = gpr >> 3, tile_units = (panels + 1) >> 1, blocks = (p.geo.d_value + 127) >> 7;
     const Layout lay = layout_of<N>(gpr, units);
     const uint32_t sbase = smem_u32(smem);
@@ -133,8 +136,9 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
         }
         fence_proxy_async();
     }
-    constexpr uint32_t COLS = 2 * S_COLS + 4 * N <= 128 ? 128 : (2 * S_COLS + 4 * N <= 256 ? 256 : 512);
-    constexpr uint32_t COL_S = 4 * N;  // O blocks at columns 0, N, 2 N, 3 N
+    constexpr uint32_t COL_S = 4 * O_COLS;  // O blocks at columns 0, O_COLS, ...
+    constexpr uint32_t COLS = 2 * S_COLS + COL_S <= 256 ? 256 : 512;
+    static_assert(2 * S_COLS + COL_S <= 512, "tensor memory");
     if (warp == 5) {  // the warp that allocates is the warp that frees
         tmem_alloc(smem_u32(tmem_slot), COLS);
         tmem_relinquish_alloc_permit();
@@ -147,7 +151,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     if (warp == 4) {
         // ---- producer
         if (lane == 0) {
-            int issued = 0;
+            int issued = 0, slot = 0, parity = 1;
             bool live = true;
             for (int j = 0; j < n_tiles && live; j++) {
                 const int at = start + j * L_TOK;
@@ -159,8 +163,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                 }
                 const uint8_t* src = static_cast<const uint8_t*>(p.pool) + (size_t)chunk * (L_TOK * 16) * gpr;
                 for (int u = 0; u < tile_units; u++, issued++) {
-                    const int slot = issued % units;
-                    if (!mbar_wait_bounded(empty + 8 * slot, ((issued / units) & 1) ^ 1, p.wait_limit)) {
+                    if (!mbar_wait_bounded(empty + 8 * slot, parity, p.wait_limit)) {
                         report(p.status, STATUS_EMPTY_WAIT_TIMEOUT);
                         live = false;
                         break;
@@ -174,6 +177,10 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                         bulk_copy_g2s(dst, src + 2 * u * L_PANEL, bytes, bar);
                         if (two) bulk_copy_g2s(dst + L_PANEL, src + (2 * u + 1) * L_PANEL, bytes, bar);
                     }
+                    if (++slot == units) {
+                        slot = 0;
+                        parity ^= 1;
+                    }
                 }
             }
             for (int f = issued > units ? issued - units : 0; f < issued; f++) {
@@ -184,65 +191,76 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             }
         }
     } else if (warp == 5) {
-        // ---- MMA issuer: one thread.  Whatever is ready goes first: the scores of the next tile when its rows have
-        // arrived (at most one tile ahead of the second product: there are two score buffers), or the second product
+        // ---- MMA issuer: one thread.  Whatever is ready goes first: the second product, which frees units, or the
+        // scores of the next tile when its rows have arrived (at most one tile ahead: there are two score buffers)
         if (elect_one() && n_tiles > 0) {
             constexpr uint32_t DESC_HI = umma_desc_sw128_hi(1024);
-            constexpr uint32_t IDESC_QK = idesc_bf16(L_TOK, N, false), IDESC_PV = idesc_bf16(128, N, true);
+            constexpr uint32_t IDESC_QK2 = idesc_bf16(128, 2 * N, false), IDESC_QK1 = idesc_bf16(128, N, false);
+            constexpr uint32_t IDESC_PV = idesc_bf16(128, O_COLS, true);
             bool live = mbar_wait_bounded(q_ready, 0, p.wait_limit);
             if (!live) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
             const uint32_t q_lo = umma_desc_sw128_lo(q_base, 16);
+            // units in the ring, each product's next one: slot, and parity of its current use
+            struct Place {
+                int slot = 0, parity = 0;
+                __device__ __forceinline__ void next(int units) {
+                    if (++slot == units) {
+                        slot = 0;
+                        parity ^= 1;
+                    }
+                }
+            } k_at, v_at, last;
+            for (int u = 1; u < tile_units; u++) last.next(units);  // the last unit of the next tile
             int jq = 0, jv = 0;
             long long since = clock64();
             while (live && jv < n_tiles) {
-                if (jq < n_tiles && jq <= jv + 1) {
-                    const int last = jq * tile_units + tile_units - 1;
-                    if (mbar_test_wait(full + 8 * (last % units), (last / units) & 1)) {
-                        const uint32_t d = tmem_base + COL_S + (jq & 1) * S_COLS;
-                        for (int u = 0; u < tile_units && live; u++) {
-                            const int g = jq * tile_units + u, slot = g % units;
-                            live = mbar_wait_bounded(full + 8 * slot, (g / units) & 1, p.wait_limit);
-                            if (!live) break;
-                            tc_fence_after_thread_sync();
-                            const uint32_t a_lo = umma_desc_sw128_lo(sbase + slot * L_UNIT, 16);
-                            const int n_pan = 2 * u + 1 < panels ? 2 : 1;
-                            for (int pn = 0; pn < n_pan; pn++)
-#pragma unroll
-                                for (int ks = 0; ks < 4; ks++) {
-                                    const uint64_t a = umma_desc_pack(a_lo + ((pn * L_PANEL + ks * 32) >> 4), DESC_HI);
-                                    const uint64_t b = umma_desc_pack(q_lo + (((2 * u + pn) * (N * 128) + ks * 32) >> 4), DESC_HI);
-                                    umma_ss_f16(d, a, b, IDESC_QK, (u > 0 || pn > 0 || ks > 0) ? 1u : 0u);
-                                }
-                            if (u >= blocks) umma_commit(empty + 8 * slot);  // holds no values
-                        }
-                        if (!live) {
-                            report(p.status, STATUS_FULL_WAIT_TIMEOUT);
-                            break;
-                        }
-                        umma_commit(s_full + 8 * (jq & 1));
-                        jq++;
-                        since = clock64();
-                        continue;
-                    }
-                }
                 if (jv < jq && mbar_test_wait(p_full, jv & 1)) {
                     tc_fence_after_thread_sync();
-                    for (int m = 0; m < blocks; m++) {
-                        const int slot = (jv * tile_units + m) % units;
-                        const uint32_t d = tmem_base + m * N;
-                        const uint32_t a_lo = umma_desc_sw128_lo(sbase + slot * L_UNIT, L_PANEL);
+                    const uint32_t b_lo = umma_desc_sw128_lo(w_base, 16);
+                    for (int m = 0; m < tile_units; m++) {
+                        if (m < blocks) {
+                            const uint32_t d = tmem_base + m * O_COLS;
+                            const uint32_t a_lo = umma_desc_sw128_lo(sbase + v_at.slot * L_UNIT, L_PANEL);
 #pragma unroll
-                        for (int part = 0; part < 2; part++) {
-                            const uint32_t b_lo = umma_desc_sw128_lo(w_base + part * (N * 128), 16);
+                            for (int part = 0; part < (WIDE ? 1 : 2); part++)
 #pragma unroll
-                            for (int kk = 0; kk < 4; kk++)
-                                umma_ss_f16(d, umma_desc_pack(a_lo + ((kk * 2048) >> 4), DESC_HI), umma_desc_pack(b_lo + ((kk * 32) >> 4), DESC_HI),
-                                            IDESC_PV, (jv > 0 || part > 0 || kk > 0) ? 1u : 0u);
+                                for (int kk = 0; kk < 4; kk++)
+                                    umma_ss_f16(d, umma_desc_pack(a_lo + 128 * kk, DESC_HI), umma_desc_pack(b_lo + part * (N * 8) + 2 * kk, DESC_HI), IDESC_PV,
+                                                part + kk > 0 ? 1u : (jv > 0 ? 1u : 0u));
+                            umma_commit(empty + 8 * v_at.slot);
                         }
-                        umma_commit(empty + 8 * slot);
+                        v_at.next(units);
                     }
                     umma_commit(o_done);
                     jv++;
+                    since = clock64();
+                    continue;
+                }
+                if (jq < n_tiles && jq <= jv + 1 && mbar_test_wait(full + 8 * last.slot, last.parity)) {
+                    const uint32_t d = tmem_base + COL_S + (jq & 1) * S_COLS;
+                    uint32_t b_lo = q_lo;
+                    for (int u = 0; u < tile_units; u++) {
+                        live = live && mbar_wait_bounded(full + 8 * k_at.slot, k_at.parity, p.wait_limit);
+                        if (!live) break;
+                        tc_fence_after_thread_sync();
+                        const uint32_t a_lo = umma_desc_sw128_lo(sbase + k_at.slot * L_UNIT, 16);
+                        // a last panel without a partner: its share only (the lower half of D is not used)
+                        const uint32_t idesc = 2 * u + 1 < panels ? IDESC_QK2 : IDESC_QK1;
+                        umma_ss_f16(d, umma_desc_pack(a_lo, DESC_HI), umma_desc_pack(b_lo, DESC_HI), idesc, u > 0 ? 1u : 0u);
+#pragma unroll
+                        for (int ks = 1; ks < 4; ks++)
+                            umma_ss_f16(d, umma_desc_pack(a_lo + 2 * ks, DESC_HI), umma_desc_pack(b_lo + 2 * ks, DESC_HI), idesc, 1u);
+                        if (u >= blocks) umma_commit(empty + 8 * k_at.slot);  // holds no values
+                        b_lo += 2 * N * 8;
+                        k_at.next(units);
+                        last.next(units);
+                    }
+                    if (!live) {
+                        report(p.status, STATUS_FULL_WAIT_TIMEOUT);
+                        break;
+                    }
+                    umma_commit(s_full + 8 * (jq & 1));
+                    jq++;
                     since = clock64();
                     continue;
                 }
@@ -253,54 +271,99 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             }
         }
     } else {
-        // ---- queries: latent part as it comes, shared part turned by the row's position, zeros up to the pool's row
+        // ---- queries: latent part as it comes, shared part turned by the row's position, zeros up to the pool's row.  Loads
+        // are requested in batches before any of them is used
         {
-            const bool whole = p.kv_rank % 8 == 0 && reinterpret_cast<uintptr_t>(p.q_lat) % 16 == 0;
-            const __nv_bfloat16* q_lat = static_cast<const __nv_bfloat16*>(p.q_lat);
+            const __nv_bfloat16* q_lat = static_cast<const __nv_bfloat16*>(p.q_lat) + ((size_t)token0 * H + row_lo) * p.kv_rank;  // rows follow one another
             const __nv_bfloat16* q_rot = static_cast<const __nv_bfloat16*>(p.q_rot);
-            const int half = p.rot / 2, rot_g = p.kv_rank / 8;  // granules below rot_g hold latent elements only
+            const int half = p.rot / 2;
             auto line = [&](int r, int g) { return q_base + (g >> 3) * (N * 128) + r * 128 + (((g & 7) ^ (r & 7)) << 4); };
-            const int lat_g = whole ? rot_g : 0;
-            for (int r = warp; r < N; r += 4) {
-                const int rr = row_lo + r, token = token0 + rr / H, head = rr % H;
-                const uint4* src = reinterpret_cast<const uint4*>(q_lat + ((size_t)token * H + head) * p.kv_rank);
-                for (int g = lane; g < lat_g; g += 32) {
-                    const uint4 v = r < n_rows ? __ldg(src + g) : make_uint4(0u, 0u, 0u, 0u);
-                    sts128(line(r, g), (int)v.x, (int)v.y, (int)v.z, (int)v.w);
+            auto aligned = [](const void* x) { return reinterpret_cast<uintptr_t>(x) % 16 == 0; };
+            const bool whole = p.kv_rank % 8 == 0 && aligned(p.q_lat);
+            const bool pairs = whole && half % 8 == 0 && half > 0 && p.q_rot_row % 8 == 0 && p.q_rot_head % 8 == 0 && aligned(p.q_rot) && aligned(p.freq);
+            const int done_g = whole ? p.kv_rank / 8 : 0;  // granules below it hold latent elements only
+            constexpr int AHEAD = N >= 32 ? 16 : 8;
+            uint4 v[AHEAD];
+#pragma unroll
+            for (int k = 0; k < AHEAD; k++) {
+                const int i = tid + 128 * k;
+                v[k] = make_uint4(0u, 0u, 0u, 0u);
+                if (i < n_rows * done_g) v[k] = __ldg(reinterpret_cast<const uint4*>(q_lat) + i);
+            }
+            if (pairs) {  // a granule of the rotated part's first half and its partner in the second
+                const int units_r = half / 8;
+                for (int i = tid; i < N * units_r; i += 128) {
+                    const int r = i / units_r, u = i % units_r, rr = row_lo + r, token = token0 + rr / H;
+                    uint4 a = make_uint4(0u, 0u, 0u, 0u), b = a;
+                    if (r < n_rows) {
+                        const uint4* src = reinterpret_cast<const uint4*>(q_rot + (size_t)token * p.q_rot_row + (size_t)(rr % H) * p.q_rot_head);
+                        a = __ldg(src + u);
+                        b = __ldg(src + units_r + u);
+                        const float pos = (float)p.positions[token];
+                        const float4 f0 = *reinterpret_cast<const float4*>(p.freq + 8 * u), f1 = *reinterpret_cast<const float4*>(p.freq + 8 * u + 4);
+                        const float f[8] = {f0.x, f0.y, f0.z, f0.w, f1.x, f1.y, f1.z, f1.w};
+                        uint32_t* aw = reinterpret_cast<uint32_t*>(&a);
+                        uint32_t* bw = reinterpret_cast<uint32_t*>(&b);
+#pragma unroll
+                        for (int k = 0; k < 4; k++) {
+                            const float x0 = __uint_as_float(aw[k] << 16), x1 = __uint_as_float(aw[k] & 0xffff0000u);
+                            const float y0 = __uint_as_float(bw[k] << 16), y1 = __uint_as_float(bw[k] & 0xffff0000u);
+                            float s0, c0, s1, c1;
+                            fast_sincos(pos * f[2 * k], &s0, &c0);
+                            fast_sincos(pos * f[2 * k + 1], &s1, &c1);
+                            aw[k] = pack_bf16(x0 * c0 - y0 * s0, x1 * c1 - y1 * s1);
+                            bw[k] = pack_bf16(y0 * c0 + x0 * s0, y1 * c1 + x1 * s1);
+                        }
+                    }
+                    sts128(line(r, done_g + u), (int)a.x, (int)a.y, (int)a.z, (int)a.w);
+                    sts128(line(r, done_g + units_r + u), (int)b.x, (int)b.y, (int)b.z, (int)b.w);
+                }
+                const int behind = gpr - done_g - 2 * units_r;
+                for (int i = tid; i < N * behind; i += 128) sts128_zero(line(i / behind, done_g + 2 * units_r + i % behind));
+            }
+            for (int i0 = tid; i0 < N * done_g; i0 += 128 * AHEAD) {
+#pragma unroll
+                for (int k = 0; k < AHEAD; k++) {
+                    const int i = i0 + 128 * k;
+                    if (i < N * done_g) sts128(line(i / done_g, i % done_g), (int)v[k].x, (int)v[k].y, (int)v[k].z, (int)v[k].w);
+                }
+#pragma unroll
+                for (int k = 0; k < AHEAD; k++) {
+                    const int i = i0 + 128 * (AHEAD + k);
+                    v[k] = make_uint4(0u, 0u, 0u, 0u);
+                    if (i < n_rows * done_g) v[k] = __ldg(reinterpret_cast<const uint4*>(q_lat) + i);
                 }
             }
-            for (int i = tid; i < N * (gpr - lat_g); i += 128) {
-                const int r = i / (gpr - lat_g), g = lat_g + i % (gpr - lat_g), rr = row_lo + r, token = token0 + rr / H, head = rr % H;
-                uint4 v = make_uint4(0u, 0u, 0u, 0u);
-                if (r < n_rows && 8 * g < p.kv_rank + p.rot) {
-                    const __nv_bfloat16* src = q_lat + ((size_t)token * H + head) * p.kv_rank;
-                    const __nv_bfloat16* qr = q_rot + (size_t)token * p.q_rot_row + (size_t)head * p.q_rot_head;
-                    const float pos = (float)p.positions[token];
+            if (!pairs) {  // any sizes, element by element
+                const int rest = gpr - done_g;
+                for (int i = tid; i < N * rest; i += 128) {
+                    const int r = i / rest, g = done_g + i % rest, rr = row_lo + r, token = token0 + rr / H;
                     float x[8];
 #pragma unroll
                     for (int k = 0; k < 8; k++) {
                         const int e = 8 * g + k, d = e - p.kv_rank;
                         x[k] = 0.f;
+                        if (r >= n_rows) continue;
                         if (d < 0) {
-                            x[k] = __bfloat162float(src[e]);
+                            x[k] = __bfloat162float(q_lat[(size_t)r * p.kv_rank + e]);
                         } else if (d < p.rot) {
+                            const __nv_bfloat16* qr = q_rot + (size_t)token * p.q_rot_row + (size_t)(rr % H) * p.q_rot_head;
                             const int pair = d < half ? d : d - half;
                             float sn, cs;
-                            fast_sincos(pos * __ldg(p.freq + pair), &sn, &cs);
+                            fast_sincos((float)p.positions[token] * __ldg(p.freq + pair), &sn, &cs);
                             const float a = __bfloat162float(qr[pair]), b = __bfloat162float(qr[pair + half]);
                             x[k] = d < half ? a * cs - b * sn : b * cs + a * sn;
                         }
                     }
-                    v = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+                    sts128(line(r, g), (int)pack_bf16(x[0], x[1]), (int)pack_bf16(x[2], x[3]), (int)pack_bf16(x[4], x[5]), (int)pack_bf16(x[6], x[7]));
                 }
-                sts128(line(r, g), (int)v.x, (int)v.y, (int)v.z, (int)v.w);
             }
             fence_proxy_async();
             mbar_arrive(q_ready);
         }
 
         // ---- softmax: thread tid has PER tokens of row tid / TPR: fours of tokens, TPR threads side by side
-        const int row = tid / TPR, part = tid % TPR;
+        const int row = tid / TPR, part = tid % TPR, shares = panels > 1 ? 2 : 1;
         int lo = 0, hi = 0;  // what the row sees, relative to `first`
         if (row < n_rows) {
             const int pos = p.positions[token0 + (row_lo + row) / H] - first;
@@ -320,15 +383,16 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                 if (!live && lane == 0) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
             }
             tc_fence_after_thread_sync();
-            // M = 64: token 16 w + i is lane i of warp w
+            // lane = token of a share: warps 0 and 1 the first panels', columns 0 .., warps 2 and 3 the second ones', columns N ..
+            if (shares == 2 || warp < 2) {
+                float* const mine = sc + (warp >> 1) * N * (L_TOK + 4) + (warp & 1) * 32 + lane;
 #pragma unroll
-            for (int c = 0; c < N; c += CH) {
-                uint32_t s[CH];
-                tmem_ld<CH>(lane_addr + COL_S + b * S_COLS + c, s);
-                tmem_wait_ld();
-                if (lane < 16) {
+                for (int c = 0; c < N; c += CH) {
+                    uint32_t s[CH];
+                    tmem_ld<CH>(lane_addr + COL_S + b * S_COLS + (warp >> 1) * N + c, s);
+                    tmem_wait_ld();
 #pragma unroll
-                    for (int i = 0; i < CH; i++) sc[(c + i) * (L_TOK + 4) + warp * 16 + lane] = __uint_as_float(s[i]);
+                    for (int i = 0; i < CH; i++) mine[(c + i) * (L_TOK + 4)] = __uint_as_float(s[i]);
                 }
             }
             tc_fence_before_thread_sync();
@@ -340,7 +404,14 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             for (int i = 0; i < PER / 4; i++) {
                 const int t = (i * TPR + part) * 4;
                 const float4 v = *reinterpret_cast<const float4*>(sc + row * (L_TOK + 4) + t);
-                const float in[4] = {v.x, v.y, v.z, v.w};
+                float in[4] = {v.x, v.y, v.z, v.w};
+                if (shares == 2) {
+                    const float4 w = *reinterpret_cast<const float4*>(sc + (N + row) * (L_TOK + 4) + t);
+                    in[0] += w.x;
+                    in[1] += w.y;
+                    in[2] += w.z;
+                    in[3] += w.w;
+                }
 #pragma unroll
                 for (int k = 0; k < 4; k++) {
                     const int c = at + t + k;
@@ -373,14 +444,14 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                     tc_fence_after_thread_sync();
                     for (int m = 0; m < blocks; m++)
 #pragma unroll
-                        for (int c = 0; c < N; c += CH) {
+                        for (int c = 0; c < O_COLS; c += CH) {
                             uint32_t o[CH];
-                            tmem_ld<CH>(lane_addr + m * N + c, o);
+                            tmem_ld<CH>(lane_addr + m * O_COLS + c, o);
                             tmem_wait_ld();
 #pragma unroll
-                            for (int i = 0; i < CH; i++) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha_s[c + i]);
-                            if constexpr (CH == 32) tmem_st32(lane_addr + m * N + c, o);
-                            else tmem_st16(lane_addr + m * N + c, o);
+                            for (int i = 0; i < CH; i++) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha_s[(c + i) % N]);
+                            if constexpr (CH == 32) tmem_st32(lane_addr + m * O_COLS + c, o);
+                            else tmem_st16(lane_addr + m * O_COLS + c, o);
                         }
                     tmem_wait_st();
                 }
@@ -434,26 +505,35 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
         if (live) {
             for (int m = 0; m < blocks; m++) {
                 const int e = m * 128 + warp * 32 + lane;
+                // rows are consecutive (token, head) pairs
+                __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + ((size_t)token0 * H + row_lo) * p.kv_rank + e;
+                float* part_o = p.part_o + ((size_t)slot_base * H + row_lo) * p.part_width + e;
 #pragma unroll
                 for (int c = 0; c < N; c += CH) {
                     uint32_t o[CH];
                     if (n_tiles > 0) {
-                        tmem_ld<CH>(lane_addr + m * N + c, o);
+                        tmem_ld<CH>(lane_addr + m * O_COLS + c, o);
                         tmem_wait_ld();
+                        if (WIDE) {
+                            uint32_t o2[CH];
+                            tmem_ld<CH>(lane_addr + m * O_COLS + N + c, o2);
+                            tmem_wait_ld();
+#pragma unroll
+                            for (int i = 0; i < CH; i++) o[i] = __float_as_uint(__uint_as_float(o[i]) + __uint_as_float(o2[i]));
+                        }
                     } else {
 #pragma unroll
                         for (int i = 0; i < CH; i++) o[i] = 0u;
                     }
+                    if (SPAN) {
+                        if (e < p.kv_rank)
 #pragma unroll
-                    for (int i = 0; i < CH; i++) {
-                        const int r = c + i, rr = row_lo + r;
-                        if (r >= n_rows) break;
-                        if (SPAN) {  // rows are consecutive (token, head) pairs
-                            if (e < p.kv_rank)
-                                static_cast<__nv_bfloat16*>(p.out)[((size_t)token0 * H + rr) * p.kv_rank + e] = __float2bfloat16_rn(__uint_as_float(o[i]) * alpha_s[r]);
-                        } else if (e < p.part_width) {
-                            p.part_o[((size_t)slot_base * H + rr) * p.part_width + e] = __uint_as_float(o[i]);
-                        }
+                            for (int i = 0; i < CH; i++, out += p.kv_rank)
+                                if (c + i < n_rows) *out = __float2bfloat16_rn(__uint_as_float(o[i]) * alpha_s[c + i]);
+                    } else if (e < p.part_width) {
+#pragma unroll
+                        for (int i = 0; i < CH; i++, part_o += p.part_width)
+                            if (c + i < n_rows) *part_o = __uint_as_float(o[i]);
                     }
                 }
             }
@@ -465,6 +545,59 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     if (warp == 5) {
         tc_fence_after_thread_sync();
         tmem_dealloc(tmem_base, COLS);
+    }
+}
+
+// One CTA per (row, query head), four value elements per thread: combines the row's partials and the sink, stores bf16.
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p) {
+    const int H = p.n_heads, row = blockIdx.x / H, head = blockIdx.x % H, e = threadIdx.x * 4;
+    const int b = p.merge_off[row], n = p.merge_off[row + 1] - b;
+    constexpr int AHEAD = 4;
+    const bool on = e < p.part_width;
+    float M = L_NEG_BIG, L = 0.f, acc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (p.sink) {
+        M = p.sink[head] * L_LOG2E;
+        L = 1.f;
+    }
+    for (int i0 = 0; i0 < n; i0 += AHEAD) {
+        float2 ml[AHEAD];
+        float4 o[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; i++) {
+            ml[i] = make_float2(L_NEG_BIG, 0.f);
+            o[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i0 + i < n) {
+                const size_t slot = (size_t)p.merge_slots[b + i0 + i] * H + head;
+                ml[i] = p.part_ml[slot];
+                if (on) o[i] = *reinterpret_cast<const float4*>(p.part_o + slot * p.part_width + e);
+            }
+        }
+        float top = M;
+#pragma unroll
+        for (int i = 0; i < AHEAD; i++) top = fmaxf(top, ml[i].x);
+        const float keep = fast_exp2(M - top);
+        M = top;
+        L *= keep;
+#pragma unroll
+        for (int k = 0; k < 4; k++) acc[k] *= keep;
+#pragma unroll
+        for (int i = 0; i < AHEAD; i++) {
+            const float w = fast_exp2(ml[i].x - top);
+            L = fmaf(w, ml[i].y, L);
+            acc[0] = fmaf(w, o[i].x, acc[0]);
+            acc[1] = fmaf(w, o[i].y, acc[1]);
+            acc[2] = fmaf(w, o[i].z, acc[2]);
+            acc[3] = fmaf(w, o[i].w, acc[3]);
+        }
+    }
+    const float inv = L > 0.f ? 1.f / L : 0.f;
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t)blockIdx.x * p.kv_rank;
+    if (p.kv_rank % 4 == 0) {
+        if (e < p.kv_rank) *reinterpret_cast<uint2*>(out + e) = make_uint2(pack_bf16(acc[0] * inv, acc[1] * inv), pack_bf16(acc[2] * inv, acc[3] * inv));
+    } else {
+#pragma unroll
+        for (int k = 0; k < 4; k++)
+            if (e + k < p.kv_rank) out[e + k] = __float2bfloat16_rn(acc[k] * inv);
     }
 }
 
@@ -498,19 +631,10 @@ cudaError_t launch_latent_rows(const LatentParams& p, cudaStream_t stream) {
     const int rows = p.path_off ? p.block_rows * p.n_heads : std::max(p.n_heads, p.item_rows);
     cudaError_t e = rows <= 16 ? launch<16>(p, stream) : (rows <= 32 ? launch<32>(p, stream) : launch<64>(p, stream));
     if (e != cudaSuccess || p.path_off) return e;
-    RowsParams r{};
-    r.geo = p.geo;
-    r.group = p.n_heads;
-    r.out = p.out;
-    r.out_width = p.kv_rank;
-    r.n_rows = p.n_rows;
-    r.sink_scores = p.sink;
-    r.part_o = p.part_o;
-    r.part_ml = p.part_ml;
-    r.part_width = p.part_width;
-    r.merge_off = p.merge_off;
-    r.merge_slots = p.merge_slots;
-    return launch_rows_merge(r, stream);
+    const int64_t pairs = (int64_t)p.n_rows * p.n_heads;
+    if (pairs > 0x7fffffff) return cudaErrorInvalidValue;
+    latent_merge_kernel<<<(unsigned)pairs, 128, 0, stream>>>(p);
+    return cudaGetLastError();
 }
 
 }  // namespace ca

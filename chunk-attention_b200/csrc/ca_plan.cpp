@@ -71,7 +71,7 @@ void cut_units(Plan& plan, const std::vector<Unit>& units, size_t ubegin, size_t
 // Largest item for which n_ctas CTAs at a time, one item each, are done soonest: every wave takes as long as its largest
 // item, plus what setting up and storing an item costs.
 int even_length(const std::vector<Unit>& units, int n_ctas, int n_heads) {
-    constexpr double ITEM_OVERHEAD = 2.0;  // in tiles
+    constexpr double ITEM_OVERHEAD = 2.5;  // in tiles
     int best = 1;
     double best_cost = 0;
     for (int len = 1; len <= MAX_TILES_PER_ITEM; len++) {
