@@ -27,7 +27,7 @@ from .configuration_bikelix import BikelixConfig
 
 GATE_SLOPE = 1.702
 EXPAND_MIN_TOKENS = 32   # of a step
-ABSORBED_COST = 3        # of a product in the latent space, in units of one between expanded heads
+ABSORBED_COST = 2        # of a product in the latent space, in units of one between expanded heads
 
 
 class LatentAttentionMixer:

@@ -1216,7 +1216,7 @@ int ca_latent_gather(ca_context* c, const ca_latent_gather_args* a, ca_stream st
     if (!c->shape.latent) return fail(CA_ERR_INVALID, "latent_gather needs a latent context");
     if (a->n_rows < 0) return fail(CA_ERR_INVALID, "negative row count");
     if (a->n_rows == 0) return CA_OK;
-    if (!a->lat || !a->rot || !a->row_span || !a->base || !a->first || !a->path_off || !a->path_chunks)
+    if (!a->lat || !a->rot || !a->src_row)
         return fail(CA_ERR_INVALID, "an operand is null");
     if (a->rot_stride < c->shape.d_key - c->shape.d_value || a->rot_stride % 8 || reinterpret_cast<uintptr_t>(a->lat) % 16 ||
         reinterpret_cast<uintptr_t>(a->rot) % 16)
@@ -1232,11 +1232,7 @@ int ca_latent_gather(ca_context* c, const ca_latent_gather_args* a, ca_stream st
     p.rot = a->rot;
     p.rot_stride = a->rot_stride;
     p.n_rows = a->n_rows;
-    p.row_span = a->row_span;
-    p.base = a->base;
-    p.first = a->first;
-    p.path_off = a->path_off;
-    p.path_chunks = a->path_chunks;
+    p.src_row = a->src_row;
     p.max_chunks = (int)c->max_chunks;
     p.status = c->status;
     CA_CUDA(ca::launch_latent_gather(p, c->dtype, static_cast<cudaStream_t>(stream_)));

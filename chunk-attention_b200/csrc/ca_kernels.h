@@ -278,11 +278,7 @@ struct LatentGatherParams {
     void* rot;                   // [n_rows, rot_stride]
     int rot_stride;
     int n_rows;
-    const int32_t* row_span;
-    const int32_t* base;
-    const int32_t* first;
-    const int32_t* path_off;
-    const int32_t* path_chunks;
+    const int32_t* src_row;      // [n_rows]: chunk * chunk_size + row in the chunk
     int max_chunks;
     int* status;
 };

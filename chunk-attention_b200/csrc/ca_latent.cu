@@ -11,8 +11,9 @@ namespace ca {
 namespace {
 
 // ---- projections -> query latent and pool row --------------------------------------------------------------------
-// One CTA per token.  V elements per access (whole granules), or 1.
-constexpr int LS_THREADS = 256;
+// One CTA per token.  V elements per access (whole granules), or 1.  Everything the token needs is requested before the
+// reduction; what a thread does not keep in registers (longer rows) is read again.
+constexpr int LS_THREADS = 128, LS_KEEP_Q = 2;
 
 __device__ __forceinline__ float2 block_sum2(float a, float b) {
     __shared__ float2 sums[LS_THREADS / 32];
@@ -31,13 +32,12 @@ __device__ __forceinline__ float2 block_sum2(float a, float b) {
 
 template <typename T, int V>
 __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentStoreParams p) {
-    const int t = blockIdx.x, tid = threadIdx.x;
+    using P = Pack<T, V>;
+    using W = Pack<float, V>;
+    const int t = blockIdx.x, tid = threadIdx.x, c0 = tid * V, step = LS_THREADS * V;
     const T* row = static_cast<const T*>(p.in) + (size_t)t * p.row_stride;
     const T* kv = row + p.q_rank;
-    using P = Pack<T, V>;
-    // the first vectors of both latents stay in registers; anything longer is read again
-    P q_keep{}, kv_keep{};
-    float sq = 0.f, skv = 0.f;
+    const T* r = kv + p.kv_rank;
     auto squares = [](const P& a) {
         float s = 0.f;
 #pragma unroll
@@ -47,26 +47,13 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentSt
         }
         return s;
     };
-    const int c0 = tid * V, step = LS_THREADS * V;
-    if (c0 < p.q_rank) q_keep = *reinterpret_cast<const P*>(row + c0);
-    if (c0 < p.kv_rank) kv_keep = *reinterpret_cast<const P*>(kv + c0);
-    sq = squares(q_keep);
-    skv = squares(kv_keep);
-    for (int c = c0 + step; c < p.q_rank; c += step) sq += squares(*reinterpret_cast<const P*>(row + c));
-    for (int c = c0 + step; c < p.kv_rank; c += step) skv += squares(*reinterpret_cast<const P*>(kv + c));
-    const float2 ss = block_sum2(sq, skv);
-
-    if (p.q_rank > 0) {
-        const float inv = 1.f / sqrtf(ss.x / p.q_rank + p.eps);
-        T* out = static_cast<T*>(p.q_out) + (size_t)t * p.q_rank;
-        for (int c = c0; c < p.q_rank; c += step) {
-            const P a = c == c0 ? q_keep : *reinterpret_cast<const P*>(row + c);
-            P o;
+    P q_keep[LS_KEEP_Q], kv_keep{};
 #pragma unroll
-            for (int i = 0; i < V; i++) o.v[i] = from_f32<T>(to_f32(a.v[i]) * inv * p.q_norm[c + i]);
-            *reinterpret_cast<P*>(out + c) = o;
-        }
+    for (int k = 0; k < LS_KEEP_Q; k++) {
+        q_keep[k] = P{};
+        if (c0 + k * step < p.q_rank) q_keep[k] = *reinterpret_cast<const P*>(row + c0 + k * step);
     }
+    if (c0 < p.kv_rank) kv_keep = *reinterpret_cast<const P*>(kv + c0);
     int chunk, slot;
     if (p.tok_slot) {
         const int s = p.tok_slot[t];
@@ -77,25 +64,51 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentSt
         slot = p.tail_tokens[t] + p.delta_tokens;
         if (slot >= p.geo.chunk_size) chunk = -1;  // rejected on the host; never write past the tile
     }
+    const int half = p.rot / 2;
+    float rot_u = 0.f, rot_v = 0.f, sn = 0.f, cs = 0.f;
+    if (tid < half) {
+        sincos_for<T>((float)p.positions[t] * p.freq[tid], &sn, &cs);
+        rot_u = to_f32(r[tid]);
+        rot_v = to_f32(r[tid + half]);
+    }
+    float sq = 0.f, skv = squares(kv_keep);
+#pragma unroll
+    for (int k = 0; k < LS_KEEP_Q; k++) sq += squares(q_keep[k]);
+    for (int c = c0 + LS_KEEP_Q * step; c < p.q_rank; c += step) sq += squares(*reinterpret_cast<const P*>(row + c));
+    for (int c = c0 + step; c < p.kv_rank; c += step) skv += squares(*reinterpret_cast<const P*>(kv + c));
+    const float2 ss = block_sum2(sq, skv);
+
+    auto scaled = [](const P& a, float inv, const float* w) {
+        const W ww = *reinterpret_cast<const W*>(w);
+        P o;
+#pragma unroll
+        for (int i = 0; i < V; i++) o.v[i] = from_f32<T>(to_f32(a.v[i]) * inv * ww.v[i]);
+        return o;
+    };
+    if (p.q_rank > 0) {
+        const float inv = 1.f / sqrtf(ss.x / p.q_rank + p.eps);
+        T* out = static_cast<T*>(p.q_out) + (size_t)t * p.q_rank;
+#pragma unroll
+        for (int k = 0; k < LS_KEEP_Q; k++) {
+            const int c = c0 + k * step;
+            if (c < p.q_rank) *reinterpret_cast<P*>(out + c) = scaled(q_keep[k], inv, p.q_norm + c);
+        }
+        for (int c = c0 + LS_KEEP_Q * step; c < p.q_rank; c += step)
+            *reinterpret_cast<P*>(out + c) = scaled(*reinterpret_cast<const P*>(row + c), inv, p.q_norm + c);
+    }
     if (chunk < 0) return;
     T* tile = static_cast<T*>(p.pool) + tile_base_elems(p.geo, chunk, 0, 0);
     const float inv = 1.f / sqrtf(ss.y / p.kv_rank + p.eps);
-    for (int c = c0; c < p.kv_rank; c += step) {
-        const P a = c == c0 ? kv_keep : *reinterpret_cast<const P*>(kv + c);
-        P o;
-#pragma unroll
-        for (int i = 0; i < V; i++) o.v[i] = from_f32<T>(to_f32(a.v[i]) * inv * p.kv_norm[c + i]);
-        *reinterpret_cast<P*>(tile + tile_elem_offset(p.geo, slot, c)) = o;
-    }
-    const int half = p.rot / 2;
-    const float pos = (float)p.positions[t];
-    const T* r = kv + p.kv_rank;
+    for (int c = c0; c < p.kv_rank; c += step)
+        *reinterpret_cast<P*>(tile + tile_elem_offset(p.geo, slot, c)) = scaled(c == c0 ? kv_keep : *reinterpret_cast<const P*>(kv + c), inv, p.kv_norm + c);
     for (int i = tid; i < half; i += LS_THREADS) {
-        float sn, cs;
-        sincos_for<T>(pos * p.freq[i], &sn, &cs);
-        const float u = to_f32(r[i]), v = to_f32(r[i + half]);
-        tile[tile_elem_offset(p.geo, slot, p.kv_rank + i)] = from_f32<T>(u * cs - v * sn);
-        tile[tile_elem_offset(p.geo, slot, p.kv_rank + half + i)] = from_f32<T>(v * cs + u * sn);
+        if (i != tid) {
+            sincos_for<T>((float)p.positions[t] * p.freq[i], &sn, &cs);
+            rot_u = to_f32(r[i]);
+            rot_v = to_f32(r[i + half]);
+        }
+        tile[tile_elem_offset(p.geo, slot, p.kv_rank + i)] = from_f32<T>(rot_u * cs - rot_v * sn);
+        tile[tile_elem_offset(p.geo, slot, p.kv_rank + half + i)] = from_f32<T>(rot_v * cs + rot_u * sn);
     }
     for (int c = p.kv_rank + p.rot + tid; c < p.geo.d_head; c += LS_THREADS) tile[tile_elem_offset(p.geo, slot, c)] = from_f32<T>(0.f);
 }
@@ -103,7 +116,9 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentSt
 template <typename T> void run_latent_store(const LatentStoreParams& p, cudaStream_t stream) {
     constexpr int V = 16 / sizeof(T);
     auto aligned = [](const void* q) { return reinterpret_cast<uintptr_t>(q) % 16 == 0; };
-    if (p.q_rank % V == 0 && p.kv_rank % V == 0 && p.row_stride % V == 0 && aligned(p.in) && aligned(p.q_out))
+    auto aligned32 = [](const void* q) { return reinterpret_cast<uintptr_t>(q) % 32 == 0; };
+    if (p.q_rank % V == 0 && p.kv_rank % V == 0 && p.row_stride % V == 0 && aligned(p.in) && aligned(p.q_out) && aligned32(p.q_norm) &&
+        aligned32(p.kv_norm))
         latent_store_kernel<T, V><<<p.n_tokens, LS_THREADS, 0, stream>>>(p);
     else
         latent_store_kernel<T, 1><<<p.n_tokens, LS_THREADS, 0, stream>>>(p);
@@ -229,10 +244,10 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentGatherPa
     constexpr int EPG = 16 / sizeof(T);
     const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= p.n_rows) return;
-    const int e = p.row_span[row], pos = p.first[e] + row - p.base[e], C = p.geo.chunk_size;
-    int chunk = p.path_chunks[p.path_off[e] + pos / C];
-    if (chunk < 0 || chunk >= p.max_chunks) {
-        atomicCAS(p.status, STATUS_OK, STATUS_BAD_WORK_LIST);
+    const int C = p.geo.chunk_size, src = p.src_row[row], at = src % C;
+    int chunk = src / C;
+    if (src < 0 || chunk >= p.max_chunks) {
+        if (lane == 0) atomicCAS(p.status, STATUS_OK, STATUS_BAD_WORK_LIST);
         chunk = 0;
     }
     const T* tile = static_cast<const T*>(p.pool) + tile_base_elems(p.geo, chunk, 0, 0);
@@ -242,16 +257,16 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const LatentGatherPa
         const int n = p.kv_rank / EPG;
         using P = Pack<T, EPG>;
         for (int g = lane; g < n; g += 32)
-            reinterpret_cast<P*>(lat)[g] = *reinterpret_cast<const P*>(tile + tile_granule_index(p.geo, pos % C, g) * EPG);
+            reinterpret_cast<P*>(lat)[g] = *reinterpret_cast<const P*>(tile + tile_granule_index(p.geo, at, g) * EPG);
         for (int g = lane; g < p.rot_stride / EPG; g += 32) {  // what lies behind the rotated elements is zero in the pool, too
             P a{};
-            if (n + g < p.geo.gpr) a = *reinterpret_cast<const P*>(tile + tile_granule_index(p.geo, pos % C, n + g) * EPG);
+            if (n + g < p.geo.gpr) a = *reinterpret_cast<const P*>(tile + tile_granule_index(p.geo, at, n + g) * EPG);
             reinterpret_cast<P*>(rot)[g] = a;
         }
     } else {
-        for (int c = lane; c < p.kv_rank; c += 32) lat[c] = tile[tile_elem_offset(p.geo, pos % C, c)];
+        for (int c = lane; c < p.kv_rank; c += 32) lat[c] = tile[tile_elem_offset(p.geo, at, c)];
         for (int c = lane; c < p.rot_stride; c += 32)
-            rot[c] = c < p.rot_dims ? tile[tile_elem_offset(p.geo, pos % C, p.kv_rank + c)] : from_f32<T>(0.f);
+            rot[c] = c < p.rot_dims ? tile[tile_elem_offset(p.geo, at, p.kv_rank + c)] : from_f32<T>(0.f);
     }
 }
 

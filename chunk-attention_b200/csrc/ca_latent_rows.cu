@@ -50,13 +50,15 @@ template <> __device__ __forceinline__ void tmem_ld<32>(uint32_t taddr, uint32_t
 struct Layout {
     int units, q, weights, scores, end;
 };
+// floats between the score rows: the rows that eight threads read together fall into different banks
+template <int N> __host__ __device__ constexpr int score_pitch() { return N == 32 ? L_TOK + 16 : L_TOK + 8; }
 template <int N> __host__ __device__ inline Layout layout_of(int gpr, int units) {
     Layout l;
     l.units = units;
     l.q = units * L_UNIT;                        // queries: [gpr / 8 panels][N lines of 128 bytes]
     l.weights = l.q + N * gpr * 16;              // weights: hi and lo, [N lines of 64 tokens] each
-    l.scores = l.weights + 2 * N * 128;          // fp32 [2 shares][N][L_TOK + 4]
-    l.end = l.scores + 2 * N * (L_TOK + 4) * 4;
+    l.scores = l.weights + 2 * N * 128;          // fp32 [2 shares][N][score_pitch]
+    l.end = l.scores + 2 * N * score_pitch<N>() * 4;
     return l;
 }
 
@@ -64,6 +66,7 @@ template <int N, bool SPAN>
 __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentParams p, int units) {
     extern __shared__ __align__(1024) uint8_t smem[];
     constexpr int TPR = 128 / N, PER = L_TOK / TPR;  // threads of a row, tokens of a thread
+    constexpr int PITCH = score_pitch<N>();
     constexpr int CH = N < 32 ? N : 32;              // TMEM columns read at a time
     constexpr bool WIDE = N <= 32;                   // hi and lo weights in one product
     constexpr int S_COLS = 2 * N, O_COLS = WIDE ? 2 * N : N;
@@ -80,6 +83,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     uint32_t* const tmem_slot = reinterpret_cast<uint32_t*>(flag_s + 2);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int H = p.n_heads;
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");  // the merge kernel may be set up; it waits for this one's end
 
     // ---- the block of rows and its tokens: [start, end) relative to position `first` of list[0]
     int token0, n_rows, first, end, low, row_lo = (int)blockIdx.y * N, slot_base = 0;
@@ -321,17 +325,26 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                 const int behind = gpr - done_g - 2 * units_r;
                 for (int i = tid; i < N * behind; i += 128) sts128_zero(line(i / behind, done_g + 2 * units_r + i % behind));
             }
-            for (int i0 = tid; i0 < N * done_g; i0 += 128 * AHEAD) {
+            if (done_g > 0) {
+                const int step_r = 128 / done_g, step_g = 128 % done_g;
+                int r = tid / done_g, g = tid % done_g;
+                for (int i0 = tid; i0 < N * done_g; i0 += 128 * AHEAD) {
 #pragma unroll
-                for (int k = 0; k < AHEAD; k++) {
-                    const int i = i0 + 128 * k;
-                    if (i < N * done_g) sts128(line(i / done_g, i % done_g), (int)v[k].x, (int)v[k].y, (int)v[k].z, (int)v[k].w);
-                }
+                    for (int k = 0; k < AHEAD; k++) {
+                        if (r < N) sts128(line(r, g), (int)v[k].x, (int)v[k].y, (int)v[k].z, (int)v[k].w);
+                        r += step_r;
+                        g += step_g;
+                        if (g >= done_g) {
+                            g -= done_g;
+                            r++;
+                        }
+                    }
 #pragma unroll
-                for (int k = 0; k < AHEAD; k++) {
-                    const int i = i0 + 128 * (AHEAD + k);
-                    v[k] = make_uint4(0u, 0u, 0u, 0u);
-                    if (i < n_rows * done_g) v[k] = __ldg(reinterpret_cast<const uint4*>(q_lat) + i);
+                    for (int k = 0; k < AHEAD; k++) {
+                        const int i = i0 + 128 * (AHEAD + k);
+                        v[k] = make_uint4(0u, 0u, 0u, 0u);
+                        if (i < n_rows * done_g) v[k] = __ldg(reinterpret_cast<const uint4*>(q_lat) + i);
+                    }
                 }
             }
             if (!pairs) {  // any sizes, element by element
@@ -385,14 +398,14 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             tc_fence_after_thread_sync();
             // lane = token of a share: warps 0 and 1 the first panels', columns 0 .., warps 2 and 3 the second ones', columns N ..
             if (shares == 2 || warp < 2) {
-                float* const mine = sc + (warp >> 1) * N * (L_TOK + 4) + (warp & 1) * 32 + lane;
+                float* const mine = sc + (warp >> 1) * N * PITCH + (warp & 1) * 32 + lane;
 #pragma unroll
                 for (int c = 0; c < N; c += CH) {
                     uint32_t s[CH];
                     tmem_ld<CH>(lane_addr + COL_S + b * S_COLS + (warp >> 1) * N + c, s);
                     tmem_wait_ld();
 #pragma unroll
-                    for (int i = 0; i < CH; i++) mine[(c + i) * (L_TOK + 4)] = __uint_as_float(s[i]);
+                    for (int i = 0; i < CH; i++) mine[(c + i) * PITCH] = __uint_as_float(s[i]);
                 }
             }
             tc_fence_before_thread_sync();
@@ -403,22 +416,27 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
 #pragma unroll
             for (int i = 0; i < PER / 4; i++) {
                 const int t = (i * TPR + part) * 4;
-                const float4 v = *reinterpret_cast<const float4*>(sc + row * (L_TOK + 4) + t);
+                const float4 v = *reinterpret_cast<const float4*>(sc + row * PITCH + t);
                 float in[4] = {v.x, v.y, v.z, v.w};
                 if (shares == 2) {
-                    const float4 w = *reinterpret_cast<const float4*>(sc + (N + row) * (L_TOK + 4) + t);
+                    const float4 w = *reinterpret_cast<const float4*>(sc + (N + row) * PITCH + t);
                     in[0] += w.x;
                     in[1] += w.y;
                     in[2] += w.z;
                     in[3] += w.w;
                 }
 #pragma unroll
-                for (int k = 0; k < 4; k++) {
-                    const int c = at + t + k;
-                    x[4 * i + k] = c >= lo && c < hi ? in[k] * sign : -INFINITY;
-                    mx = fmaxf(mx, x[4 * i + k]);
+                for (int k = 0; k < 4; k++) x[4 * i + k] = in[k] * sign;
+            }
+            if (at < lo || at + L_TOK > hi) {
+#pragma unroll
+                for (int i = 0; i < PER; i++) {
+                    const int c = at + ((i >> 2) * TPR + part) * 4 + (i & 3);
+                    if (c < lo || c >= hi) x[i] = -INFINITY;
                 }
             }
+#pragma unroll
+            for (int i = 0; i < PER; i++) mx = fmaxf(mx, x[i]);
 #pragma unroll
             for (int o = 1; o < TPR; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
             mx = scale == 0.f ? 0.f : fmaxf(mx * scale, L_NEG_BIG);
@@ -552,6 +570,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
 __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p) {
     const int H = p.n_heads, row = blockIdx.x / H, head = blockIdx.x % H, e = threadIdx.x * 4;
     const int b = p.merge_off[row], n = p.merge_off[row + 1] - b;
+    asm volatile("griddepcontrol.wait;" ::: "memory");  // what comes before is not written by the kernel before this one
     constexpr int AHEAD = 4;
     const bool on = e < p.part_width;
     float M = L_NEG_BIG, L = 0.f, acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -633,8 +652,16 @@ cudaError_t launch_latent_rows(const LatentParams& p, cudaStream_t stream) {
     if (e != cudaSuccess || p.path_off) return e;
     const int64_t pairs = (int64_t)p.n_rows * p.n_heads;
     if (pairs > 0x7fffffff) return cudaErrorInvalidValue;
-    latent_merge_kernel<<<(unsigned)pairs, 128, 0, stream>>>(p);
-    return cudaGetLastError();
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3((unsigned)pairs);
+    cfg.blockDim = dim3(128);
+    cfg.stream = stream;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    return cudaLaunchKernelEx(&cfg, latent_merge_kernel, p);
 }
 
 }  // namespace ca

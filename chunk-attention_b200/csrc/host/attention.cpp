@@ -605,7 +605,7 @@ const Attention::WindowTables& Attention::window_tables() {
     if (f != all.end()) return f->second;
     const size_t E = tables_->lens.size();
     WindowTables w;
-    std::vector<int32_t> span, base{0}, first;
+    std::vector<int32_t> src, base{0}, first;
     for (size_t i = 0; i < E; i++) {
         const int64_t start = tables_->starts[i], len = tables_->lens[i], win = shape_.window > 0 ? shape_.window : start + len;
         first.push_back((int32_t)std::max<int64_t>(0, start - win + 1));
@@ -613,12 +613,13 @@ const Attention::WindowTables& Attention::window_tables() {
         // positions start .. start + len - 1 see min(position + 1, win) tokens each
         const int64_t growing = std::min(len, std::max<int64_t>(0, win - start));
         w.pairs += growing * (2 * start + growing + 1) / 2 + (len - growing) * win;
-        span.insert(span.end(), base[i + 1] - base[i], (int32_t)i);
+        const int32_t* path = shared_tables_->data.data() + tables_->path_chunks + shared_tables_->data[tables_->path_off + (int64_t)i];
+        for (int64_t pos = first.back(); pos < start + len; pos++) src.push_back(path[pos / chunk_size_] * chunk_size_ + (int32_t)(pos % chunk_size_));
     }
     w.rows = base.back();
-    span.insert(span.end(), base.begin(), base.end());
-    span.insert(span.end(), first.begin(), first.end());
-    w.device = upload(span, options_.device());
+    src.insert(src.end(), base.begin(), base.end());
+    src.insert(src.end(), first.begin(), first.end());
+    w.device = upload(src, options_.device());
     return all.emplace(shape_.window, w).first->second;
 }
 
@@ -714,7 +715,7 @@ std::pair<torch::Tensor, torch::Tensor> Attention::gather_latents() {
     if (tables_->n_tokens < 0) throw std::runtime_error("gather_latents: extend must have described the tokens");
     c10::cuda::CUDAGuard guard(options_.device());
     const WindowTables& w = window_tables();
-    const int64_t E = (int64_t)tables_->lens.size(), pad = (shape_.d_key - shape_.d_value + 63) / 64 * 64;
+    const int64_t pad = (shape_.d_key - shape_.d_value + 63) / 64 * 64;
     torch::Tensor lat = torch::empty({w.rows, shape_.d_value}, options_), rot = torch::empty({w.rows, std::max<int64_t>(pad, 64)}, options_);
     const int32_t* t = w.device.data_ptr<int32_t>();
     ca_latent_gather_args a{};
@@ -722,11 +723,7 @@ std::pair<torch::Tensor, torch::Tensor> Attention::gather_latents() {
     a.rot = rot.data_ptr();
     a.rot_stride = (int32_t)rot.size(1);
     a.n_rows = (int32_t)w.rows;
-    a.row_span = t;
-    a.base = t + w.rows;
-    a.first = t + w.rows + E + 1;
-    a.path_off = tables_->device.data_ptr<int32_t>() + tables_->path_off;
-    a.path_chunks = tables_->device.data_ptr<int32_t>() + tables_->path_chunks;
+    a.src_row = t;
     check_rc(ca_latent_gather(ctx_, &a, stream()), "gather_latents");
     return {lat, rot};
 }

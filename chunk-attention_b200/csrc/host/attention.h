@@ -165,7 +165,7 @@ class Attention {
 
     // The device tables of the current portions (extend), shared the same way: equal tables are uploaded once.
     struct WindowTables {
-        torch::Tensor device;  // row_span [rows] | base [entries + 1] | first [entries]
+        torch::Tensor device;  // src_row [rows] | base [entries + 1] | first [entries]
         int64_t rows = 0, pairs = 0;
     };
     struct SharedTables {

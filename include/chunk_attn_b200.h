@@ -431,27 +431,23 @@ CA_API int ca_latent_attention(ca_context* ctx, const ca_latent_args* args, ca_s
  * as portions */
 CA_API int ca_latent_decodes(const ca_context* ctx);
 
-/* The cached rows a step of portions reads, laid out densely: workspace row base[e] + i is position first[e] + i of span
- * e, for i < base[e + 1] - base[e].  lat: [base[n], d_value], rot: [base[n], rot_stride] (zeros behind the rotated
- * elements; rot_stride a multiple of 8). */
+/* The cached rows a step of portions reads, laid out densely: workspace row i is pool row src_row[i] (chunk * chunk_size +
+ * row in the chunk).  lat: [n_rows, d_value], rot: [n_rows, rot_stride] (zeros behind the rotated elements; rot_stride a
+ * multiple of 8). */
 typedef struct ca_latent_gather_args {
     void* lat;
     void* rot;
     int32_t rot_stride;
-    int32_t n_rows;             /* base[n_entries]                  */
-    const int32_t* row_span;    /* [n_rows]: span of each row       */
-    const int32_t* base;        /* [n_entries + 1]                  */
-    const int32_t* first;       /* [n_entries]                      */
-    const int32_t* path_off;
-    const int32_t* path_chunks;
+    int32_t n_rows;
+    const int32_t* src_row;     /* [n_rows]                         */
 } ca_latent_gather_args;
 CA_API int ca_latent_gather(ca_context* ctx, const ca_latent_gather_args* args, ca_stream stream);
 
 /* Attention of portions over keys and values expanded from gathered rows (bf16, head sizes of whole granules up to 128, a
  * positive scale: ca_latent_expands).  kv: [kv_rows, kv_stride], per workspace row the unrotated keys of all heads (dim
  * each), then their values (vdim each); rot: the gathered shared key parts, [kv_rows, rot_stride], at least 64 (128 for more
- * than 64 rotated elements) wide; q: [n_rows, n_heads, dim + rotated], not yet rotated; out: [n_rows, n_heads, vdim].  base and
- * first as in ca_latent_gather, blocks of at most ca_latent_expanded_block() rows. */
+ * than 64 rotated elements) wide; q: [n_rows, n_heads, dim + rotated], not yet rotated; out: [n_rows, n_heads, vdim].
+ * Workspace row base[e] + i is position first[e] + i of span e; blocks of at most ca_latent_expanded_block() rows. */
 typedef struct ca_latent_expanded_args {
     const void* q;
     const void* kv;
