@@ -7,7 +7,7 @@
 //   S^T = K Q^T   two 64-element panels at a time: M = 64 tokens of one panel and the same 64 of the next, N = query rows of one
 //                 panel and of the next; the blocks on the diagonal of D are the two panels' shares of the scores (the others
 //                 are not used).  D in TMEM, two buffers, so that tile j + 1 is scored under the softmax of tile j
-//   softmax       the shares go through shared memory once, so that 128 / N threads share a query row; fp32, log2 units;
+//   softmax       the shares go through shared memory once, so that 256 / N threads share a query row; fp32, log2 units;
 //                 every row has a window.  O is rescaled only when a row's maximum has grown by more than 8.  The
 //                 weights go back to shared memory as bf16 hi + lo parts, whose sum has 16 bits of the fp32 weight
 //   O^T += V^T P^T  M = 128 value elements (one TMEM block each), N = hi and lo parts of the query rows (up to 32 rows: side by
@@ -15,7 +15,7 @@
 // Cache rows arrive by 1-D TMA bulk copies, verbatim (the pool's lines are the swizzled operand layout), in a ring of
 // 16 KiB units: two 64-element panels of a 64-token chunk, released one by one as the second product has used them.  Decode
 // emits one partial per row and item, combined by a merge kernel; portions emit finished rows.
-// Warp roles: 0-3 softmax and epilogue, 4 TMA producer, 5 TMEM and the MMA issue.
+// Warp roles: 0-7 softmax and epilogue, 8 TMA producer, 9 TMEM and the first product's issue, 10 the second one's.
 //
 // Every wait is bounded: on expiry a status code is recorded, every role runs out without waiting further, nothing is
 // stored, and the TMEM columns are freed at the common exit.
@@ -30,7 +30,9 @@ namespace ca {
 namespace {
 using namespace ptx;
 
-constexpr int L_THREADS = 192, L_TOK = 64, L_PANEL = L_TOK * 128, L_UNIT = 2 * L_PANEL, L_MAX_UNITS = 16, L_MAX_ROWS = 64;
+constexpr int L_PITCH = 68;                           // floats between score rows
+constexpr int L_SOFT = 256, L_THREADS = L_SOFT + 96,  // softmax threads, and all
+              L_TOK = 64, L_PANEL = L_TOK * 128, L_UNIT = 2 * L_PANEL, L_MAX_UNITS = 16, L_MAX_ROWS = 64;
 constexpr float L_NEG_BIG = -1.0e30f, L_LOG2E = 1.4426950408889634f, L_RESCALE_STEP = 8.f;
 
 __host__ __device__ constexpr uint32_t idesc_bf16(int m, int n, bool a_mn_major) { return umma_idesc_f16(m, n, a_mn_major, false) | (1u << 7) | (1u << 10); }
@@ -39,7 +41,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&h);
 }
-__device__ __forceinline__ void softmax_warps_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void softmax_warps_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 __device__ __forceinline__ void sts64(uint32_t addr, uint32_t x, uint32_t y) { asm volatile("st.shared.v2.u32 [%0], {%1,%2};" ::"r"(addr), "r"(x), "r"(y) : "memory"); }
 
 template <int N> __device__ __forceinline__ void tmem_ld(uint32_t taddr, uint32_t (&r)[N]);
@@ -50,25 +52,23 @@ template <> __device__ __forceinline__ void tmem_ld<32>(uint32_t taddr, uint32_t
 struct Layout {
     int units, q, weights, scores, end;
 };
-// floats between the score rows: the rows that eight threads read together fall into different banks
-template <int N> __host__ __device__ constexpr int score_pitch() { return N == 32 ? L_TOK + 16 : L_TOK + 8; }
 template <int N> __host__ __device__ inline Layout layout_of(int gpr, int units) {
     Layout l;
     l.units = units;
     l.q = units * L_UNIT;                        // queries: [gpr / 8 panels][N lines of 128 bytes]
     l.weights = l.q + N * gpr * 16;              // weights: hi and lo, [N lines of 64 tokens] each
-    l.scores = l.weights + 2 * N * 128;          // fp32 [2 shares][N][score_pitch]
-    l.end = l.scores + 2 * N * score_pitch<N>() * 4;
+    l.scores = l.weights + 2 * N * 128;          // fp32 [2 shares][N][L_PITCH]
+    l.end = l.scores + 2 * N * L_PITCH * 4;
     return l;
 }
 
 template <int N, bool SPAN>
 __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentParams p, int units) {
     extern __shared__ __align__(1024) uint8_t smem[];
-    constexpr int TPR = 128 / N, PER = L_TOK / TPR;  // threads of a row, tokens of a thread
-    constexpr int PITCH = score_pitch<N>();
+    constexpr int TPR = L_SOFT / N, PER = L_TOK / TPR;  // threads of a row, tokens of a thread
     constexpr int CH = N < 32 ? N : 32;              // TMEM columns read at a time
     constexpr bool WIDE = N <= 32;                   // hi and lo weights in one product
+    constexpr uint32_t DESC_HI = umma_desc_sw128_hi(1024);
     constexpr int S_COLS = 2 * N, O_COLS = WIDE ? 2 * N : N;
     const int gpr = p.geo.gpr, panels = gpr >> 3, tile_units = (panels + 1) >> 1, blocks = (p.geo.d_value + 127) >> 7;
     const Layout lay = layout_of<N>(gpr, units);
@@ -77,8 +77,8 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     float* const sc = reinterpret_cast<float*>(smem + lay.scores);
     uint64_t* const bar_mem = reinterpret_cast<uint64_t*>(smem + lay.end);
     const uint32_t full = smem_u32(bar_mem), empty = full + 8 * L_MAX_UNITS, s_full = empty + 8 * L_MAX_UNITS, p_full = s_full + 16,
-                   o_done = p_full + 8, q_ready = o_done + 8;
-    float* const alpha_s = reinterpret_cast<float*>(bar_mem + 2 * L_MAX_UNITS + 5);  // [N]
+                   o_done = p_full + 8, q_ready = o_done + 8, s_empty = q_ready + 8;
+    float* const alpha_s = reinterpret_cast<float*>(bar_mem + 2 * L_MAX_UNITS + 7);  // [N]
     int* const flag_s = reinterpret_cast<int*>(alpha_s + L_MAX_ROWS);                 // [2]
     uint32_t* const tmem_slot = reinterpret_cast<uint32_t*>(flag_s + 2);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -123,9 +123,11 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
         }
         mbar_init(s_full, 1);
         mbar_init(s_full + 8, 1);
-        mbar_init(p_full, 128);
+        mbar_init(p_full, L_SOFT);
         mbar_init(o_done, 1);
-        mbar_init(q_ready, 128);
+        mbar_init(q_ready, L_SOFT);
+        mbar_init(s_empty, L_SOFT / 32);
+        mbar_init(s_empty + 8, L_SOFT / 32);
         flag_s[0] = flag_s[1] = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -143,7 +145,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     constexpr uint32_t COL_S = 4 * O_COLS;  // O blocks at columns 0, O_COLS, ...
     constexpr uint32_t COLS = 2 * S_COLS + COL_S <= 256 ? 256 : 512;
     static_assert(2 * S_COLS + COL_S <= 512, "tensor memory");
-    if (warp == 5) {  // the warp that allocates is the warp that frees
+    if (warp == 9) {  // the warp that allocates is the warp that frees
         tmem_alloc(smem_u32(tmem_slot), COLS);
         tmem_relinquish_alloc_permit();
     }
@@ -152,7 +154,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     tc_fence_after_thread_sync();
     const uint32_t tmem_base = *tmem_slot;
 
-    if (warp == 4) {
+    if (warp == 8) {
         // ---- producer
         if (lane == 0) {
             int issued = 0, slot = 0, parity = 1;
@@ -194,84 +196,72 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                 }
             }
         }
-    } else if (warp == 5) {
-        // ---- MMA issuer: one thread.  Whatever is ready goes first: the second product, which frees units, or the
-        // scores of the next tile when its rows have arrived (at most one tile ahead: there are two score buffers)
-        if (elect_one() && n_tiles > 0) {
-            constexpr uint32_t DESC_HI = umma_desc_sw128_hi(1024);
+    } else if (warp == 9) {
+        // ---- scores: one thread issues, unit by unit as a tile's rows arrive, up to two tiles ahead of the softmax
+        if (elect_one()) {
             constexpr uint32_t IDESC_QK2 = idesc_bf16(128, 2 * N, false), IDESC_QK1 = idesc_bf16(128, N, false);
-            constexpr uint32_t IDESC_PV = idesc_bf16(128, O_COLS, true);
-            bool live = mbar_wait_bounded(q_ready, 0, p.wait_limit);
-            if (!live) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
+            bool live = true;
+            auto wait = [&](uint32_t bar, int parity) {
+                if (live && !mbar_wait_bounded(bar, parity, p.wait_limit)) {
+                    report(p.status, STATUS_FULL_WAIT_TIMEOUT);
+                    live = false;
+                }
+            };
             const uint32_t q_lo = umma_desc_sw128_lo(q_base, 16);
-            // units in the ring, each product's next one: slot, and parity of its current use
-            struct Place {
-                int slot = 0, parity = 0;
-                __device__ __forceinline__ void next(int units) {
+            int slot = 0, parity = 0;
+            wait(q_ready, 0);
+            for (int j = 0; j < n_tiles && live; j++) {
+                if (j >= 2) wait(s_empty + 8 * (j & 1), ((j >> 1) - 1) & 1);
+                const uint32_t d = tmem_base + COL_S + (j & 1) * S_COLS;
+                uint32_t b_lo = q_lo;
+                for (int u = 0; u < tile_units; u++) {
+                    wait(full + 8 * slot, parity);
+                    if (!live) break;
+                    tc_fence_after_thread_sync();
+                    const uint32_t a_lo = umma_desc_sw128_lo(sbase + slot * L_UNIT, 16);
+                    // a last panel without a partner: its share only (the lower half of D is not used)
+                    const uint32_t idesc = 2 * u + 1 < panels ? IDESC_QK2 : IDESC_QK1;
+                    umma_ss_f16(d, umma_desc_pack(a_lo, DESC_HI), umma_desc_pack(b_lo, DESC_HI), idesc, u > 0 ? 1u : 0u);
+#pragma unroll
+                    for (int ks = 1; ks < 4; ks++)
+                        umma_ss_f16(d, umma_desc_pack(a_lo + 2 * ks, DESC_HI), umma_desc_pack(b_lo + 2 * ks, DESC_HI), idesc, 1u);
+                    if (u >= blocks) umma_commit(empty + 8 * slot);  // holds no values
+                    b_lo += 2 * N * 8;
                     if (++slot == units) {
                         slot = 0;
                         parity ^= 1;
                     }
                 }
-            } k_at, v_at, last;
-            for (int u = 1; u < tile_units; u++) last.next(units);  // the last unit of the next tile
-            int jq = 0, jv = 0;
-            long long since = clock64();
-            while (live && jv < n_tiles) {
-                if (jv < jq && mbar_test_wait(p_full, jv & 1)) {
-                    tc_fence_after_thread_sync();
-                    const uint32_t b_lo = umma_desc_sw128_lo(w_base, 16);
-                    for (int m = 0; m < tile_units; m++) {
-                        if (m < blocks) {
-                            const uint32_t d = tmem_base + m * O_COLS;
-                            const uint32_t a_lo = umma_desc_sw128_lo(sbase + v_at.slot * L_UNIT, L_PANEL);
-#pragma unroll
-                            for (int part = 0; part < (WIDE ? 1 : 2); part++)
-#pragma unroll
-                                for (int kk = 0; kk < 4; kk++)
-                                    umma_ss_f16(d, umma_desc_pack(a_lo + 128 * kk, DESC_HI), umma_desc_pack(b_lo + part * (N * 8) + 2 * kk, DESC_HI), IDESC_PV,
-                                                part + kk > 0 ? 1u : (jv > 0 ? 1u : 0u));
-                            umma_commit(empty + 8 * v_at.slot);
-                        }
-                        v_at.next(units);
-                    }
-                    umma_commit(o_done);
-                    jv++;
-                    since = clock64();
-                    continue;
-                }
-                if (jq < n_tiles && jq <= jv + 1 && mbar_test_wait(full + 8 * last.slot, last.parity)) {
-                    const uint32_t d = tmem_base + COL_S + (jq & 1) * S_COLS;
-                    uint32_t b_lo = q_lo;
-                    for (int u = 0; u < tile_units; u++) {
-                        live = live && mbar_wait_bounded(full + 8 * k_at.slot, k_at.parity, p.wait_limit);
-                        if (!live) break;
-                        tc_fence_after_thread_sync();
-                        const uint32_t a_lo = umma_desc_sw128_lo(sbase + k_at.slot * L_UNIT, 16);
-                        // a last panel without a partner: its share only (the lower half of D is not used)
-                        const uint32_t idesc = 2 * u + 1 < panels ? IDESC_QK2 : IDESC_QK1;
-                        umma_ss_f16(d, umma_desc_pack(a_lo, DESC_HI), umma_desc_pack(b_lo, DESC_HI), idesc, u > 0 ? 1u : 0u);
-#pragma unroll
-                        for (int ks = 1; ks < 4; ks++)
-                            umma_ss_f16(d, umma_desc_pack(a_lo + 2 * ks, DESC_HI), umma_desc_pack(b_lo + 2 * ks, DESC_HI), idesc, 1u);
-                        if (u >= blocks) umma_commit(empty + 8 * k_at.slot);  // holds no values
-                        b_lo += 2 * N * 8;
-                        k_at.next(units);
-                        last.next(units);
-                    }
-                    if (!live) {
-                        report(p.status, STATUS_FULL_WAIT_TIMEOUT);
-                        break;
-                    }
-                    umma_commit(s_full + 8 * (jq & 1));
-                    jq++;
-                    since = clock64();
-                    continue;
-                }
-                if (clock64() - since > p.wait_limit) {
+                if (live) umma_commit(s_full + 8 * (j & 1));
+            }
+        }
+    } else if (warp == 10) {
+        // ---- the second product: one thread issues, and frees the units block by block
+        if (elect_one()) {
+            constexpr uint32_t IDESC_PV = idesc_bf16(128, O_COLS, true);
+            const uint32_t p_lo = umma_desc_sw128_lo(w_base, 16);
+            int slot = 0;
+            for (int j = 0; j < n_tiles; j++) {
+                if (!mbar_wait_bounded(p_full, j & 1, p.wait_limit)) {
                     report(p.status, STATUS_FULL_WAIT_TIMEOUT);
-                    live = false;
+                    break;
                 }
+                tc_fence_after_thread_sync();
+                for (int m = 0; m < tile_units; m++) {
+                    if (m < blocks) {
+                        const uint32_t d = tmem_base + m * O_COLS;
+                        const uint32_t a_lo = umma_desc_sw128_lo(sbase + slot * L_UNIT, L_PANEL);
+#pragma unroll
+                        for (int part = 0; part < (WIDE ? 1 : 2); part++)
+#pragma unroll
+                            for (int kk = 0; kk < 4; kk++)
+                                umma_ss_f16(d, umma_desc_pack(a_lo + 128 * kk, DESC_HI), umma_desc_pack(p_lo + part * (N * 8) + 2 * kk, DESC_HI), IDESC_PV,
+                                            part + kk > 0 ? 1u : (j > 0 ? 1u : 0u));
+                        umma_commit(empty + 8 * slot);
+                    }
+                    if (++slot == units) slot = 0;
+                }
+                umma_commit(o_done);
             }
         }
     } else {
@@ -286,17 +276,17 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             const bool whole = p.kv_rank % 8 == 0 && aligned(p.q_lat);
             const bool pairs = whole && half % 8 == 0 && half > 0 && p.q_rot_row % 8 == 0 && p.q_rot_head % 8 == 0 && aligned(p.q_rot) && aligned(p.freq);
             const int done_g = whole ? p.kv_rank / 8 : 0;  // granules below it hold latent elements only
-            constexpr int AHEAD = N >= 32 ? 16 : 8;
+            constexpr int AHEAD = 8;
             uint4 v[AHEAD];
 #pragma unroll
             for (int k = 0; k < AHEAD; k++) {
-                const int i = tid + 128 * k;
+                const int i = tid + L_SOFT * k;
                 v[k] = make_uint4(0u, 0u, 0u, 0u);
                 if (i < n_rows * done_g) v[k] = __ldg(reinterpret_cast<const uint4*>(q_lat) + i);
             }
             if (pairs) {  // a granule of the rotated part's first half and its partner in the second
                 const int units_r = half / 8;
-                for (int i = tid; i < N * units_r; i += 128) {
+                for (int i = tid; i < N * units_r; i += L_SOFT) {
                     const int r = i / units_r, u = i % units_r, rr = row_lo + r, token = token0 + rr / H;
                     uint4 a = make_uint4(0u, 0u, 0u, 0u), b = a;
                     if (r < n_rows) {
@@ -323,12 +313,12 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                     sts128(line(r, done_g + units_r + u), (int)b.x, (int)b.y, (int)b.z, (int)b.w);
                 }
                 const int behind = gpr - done_g - 2 * units_r;
-                for (int i = tid; i < N * behind; i += 128) sts128_zero(line(i / behind, done_g + 2 * units_r + i % behind));
+                for (int i = tid; i < N * behind; i += L_SOFT) sts128_zero(line(i / behind, done_g + 2 * units_r + i % behind));
             }
             if (done_g > 0) {
-                const int step_r = 128 / done_g, step_g = 128 % done_g;
+                const int step_r = L_SOFT / done_g, step_g = L_SOFT % done_g;
                 int r = tid / done_g, g = tid % done_g;
-                for (int i0 = tid; i0 < N * done_g; i0 += 128 * AHEAD) {
+                for (int i0 = tid; i0 < N * done_g; i0 += L_SOFT * AHEAD) {
 #pragma unroll
                     for (int k = 0; k < AHEAD; k++) {
                         if (r < N) sts128(line(r, g), (int)v[k].x, (int)v[k].y, (int)v[k].z, (int)v[k].w);
@@ -341,7 +331,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                     }
 #pragma unroll
                     for (int k = 0; k < AHEAD; k++) {
-                        const int i = i0 + 128 * (AHEAD + k);
+                        const int i = i0 + L_SOFT * (AHEAD + k);
                         v[k] = make_uint4(0u, 0u, 0u, 0u);
                         if (i < n_rows * done_g) v[k] = __ldg(reinterpret_cast<const uint4*>(q_lat) + i);
                     }
@@ -349,7 +339,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             }
             if (!pairs) {  // any sizes, element by element
                 const int rest = gpr - done_g;
-                for (int i = tid; i < N * rest; i += 128) {
+                for (int i = tid; i < N * rest; i += L_SOFT) {
                     const int r = i / rest, g = done_g + i % rest, rr = row_lo + r, token = token0 + rr / H;
                     float x[8];
 #pragma unroll
@@ -376,7 +366,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
         }
 
         // ---- softmax: thread tid has PER tokens of row tid / TPR: fours of tokens, TPR threads side by side
-        const int row = tid / TPR, part = tid % TPR, shares = panels > 1 ? 2 : 1;
+        const int row = tid / TPR, part = tid % TPR, shares = panels > 1 ? 2 : 1, quarter = warp & 3, side = warp >> 2;
         int lo = 0, hi = 0;  // what the row sees, relative to `first`
         if (row < n_rows) {
             const int pos = p.positions[token0 + (row_lo + row) / H] - first;
@@ -384,7 +374,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
             lo = p.window > 0 ? pos - p.window + 1 : 0;
         }
         const float scale = fabsf(p.scale_log2), sign = p.scale_log2 < 0.f ? -1.f : 1.f;
-        const uint32_t lane_addr = tmem_base + ((uint32_t)(warp * 32) << 16);
+        const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
         float m_used = L_NEG_BIG, l = 0.f;
         bool live = true;
         for (int j = 0; j < n_tiles; j++) {
@@ -396,19 +386,20 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                 if (!live && lane == 0) report(p.status, STATUS_FULL_WAIT_TIMEOUT);
             }
             tc_fence_after_thread_sync();
-            // lane = token of a share: warps 0 and 1 the first panels', columns 0 .., warps 2 and 3 the second ones', columns N ..
-            if (shares == 2 || warp < 2) {
-                float* const mine = sc + (warp >> 1) * N * PITCH + (warp & 1) * 32 + lane;
+            // lane = token of a share: quarters 0 and 1 of the lanes the first panels', columns 0 .., quarters 2 and 3 the second
+            // ones', columns N ..; the two warps of a quarter take half of the columns each
+            if ((shares == 2 || quarter < 2) && (N >= 32 || side == 0)) {
+                constexpr int SC = N >= 32 ? N / 2 : N;
+                float* const mine = sc + ((quarter >> 1) * N + side * SC) * L_PITCH + (quarter & 1) * 32 + lane;
+                uint32_t s[SC];
+                tmem_ld<SC>(lane_addr + COL_S + b * S_COLS + (quarter >> 1) * N + side * SC, s);
+                tmem_wait_ld();
 #pragma unroll
-                for (int c = 0; c < N; c += CH) {
-                    uint32_t s[CH];
-                    tmem_ld<CH>(lane_addr + COL_S + b * S_COLS + (warp >> 1) * N + c, s);
-                    tmem_wait_ld();
-#pragma unroll
-                    for (int i = 0; i < CH; i++) mine[(c + i) * PITCH] = __uint_as_float(s[i]);
-                }
+                for (int i = 0; i < SC; i++) mine[i * L_PITCH] = __uint_as_float(s[i]);
             }
             tc_fence_before_thread_sync();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(s_empty + 8 * b);
             softmax_warps_sync();
             if (tid == 0) flag_s[b ^ 1] = 0;  // everyone has read it in the tile before
             float x[PER];
@@ -416,10 +407,10 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
 #pragma unroll
             for (int i = 0; i < PER / 4; i++) {
                 const int t = (i * TPR + part) * 4;
-                const float4 v = *reinterpret_cast<const float4*>(sc + row * PITCH + t);
+                const float4 v = *reinterpret_cast<const float4*>(sc + row * L_PITCH + t);
                 float in[4] = {v.x, v.y, v.z, v.w};
                 if (shares == 2) {
-                    const float4 w = *reinterpret_cast<const float4*>(sc + (N + row) * PITCH + t);
+                    const float4 w = *reinterpret_cast<const float4*>(sc + (N + row) * L_PITCH + t);
                     in[0] += w.x;
                     in[1] += w.y;
                     in[2] += w.z;
@@ -460,7 +451,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
                 }
                 if (*reinterpret_cast<volatile int*>(flag_s + b)) {
                     tc_fence_after_thread_sync();
-                    for (int m = 0; m < blocks; m++)
+                    for (int m = side; m < blocks; m += 2)
 #pragma unroll
                         for (int c = 0; c < O_COLS; c += CH) {
                             uint32_t o[CH];
@@ -521,8 +512,8 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
         }
         softmax_warps_sync();
         if (live) {
-            for (int m = 0; m < blocks; m++) {
-                const int e = m * 128 + warp * 32 + lane;
+            for (int m = side; m < blocks; m += 2) {
+                const int e = m * 128 + quarter * 32 + lane;
                 // rows are consecutive (token, head) pairs
                 __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + ((size_t)token0 * H + row_lo) * p.kv_rank + e;
                 float* part_o = p.part_o + ((size_t)slot_base * H + row_lo) * p.part_width + e;
@@ -560,7 +551,7 @@ __global__ void __launch_bounds__(L_THREADS) latent_rows_kernel(const LatentPara
     // ---- common exit: nobody touches TMEM after this barrier, then the allocating warp frees it
     tc_fence_before_thread_sync();
     __syncthreads();
-    if (warp == 5) {
+    if (warp == 9) {
         tc_fence_after_thread_sync();
         tmem_dealloc(tmem_base, COLS);
     }
@@ -621,7 +612,7 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentParams p)
 }
 
 constexpr int L_SMEM_LIMIT = 227 * 1024;
-constexpr int L_CONTROL = (2 * L_MAX_UNITS + 5) * 8 + L_MAX_ROWS * 4 + 16;  // barriers, row factors, flags, TMEM address
+constexpr int L_CONTROL = (2 * L_MAX_UNITS + 7) * 8 + L_MAX_ROWS * 4 + 16;  // barriers, row factors, flags, TMEM address
 
 template <int N> cudaError_t launch(const LatentParams& p, cudaStream_t stream) {
     const int tile_units = ((p.geo.gpr >> 3) + 1) / 2, fixed = layout_of<N>(p.geo.gpr, 0).end + L_CONTROL;
