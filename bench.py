@@ -1550,11 +1550,6 @@ def run_bikelix(args):
                 pairs = pairs_of([0] * E, lens, window)
                 kernel("forward_expanded window %d %s" % (window, tag), lambda: cache.forward_expanded(q, kv, rot, sp.positions, freq, sink, dv),
                        2.0 * T * H * (d + r + dv + d + dv) + 2.0 * T * r, flops=2.0 * pairs * H * (d + r + dv), like="attention_rows kv32")
-                if window == 1024:
-                    ql = rnd(T, H, R)
-                    kernel("forward_latent portions window %d %s" % (window, tag), lambda: cache.forward_latent(ql, q, sp.positions, freq, sink, sp.entry_of),
-                           2.0 * T * H * (2 * R + r) + 2.0 * T * (R + r), flops=2.0 * pairs * H * (2 * R + r), like="attention_rows kv32")
-                    del ql
                 del cache, lat, rot, kv, q
             del x, r_, gate, u, gu, proj
         for batch, ctx in bench.DECODES:
@@ -1581,6 +1576,33 @@ def run_bikelix(args):
                 kernel("forward_latent decode window %d %s" % (window, tag), lambda: cache.forward_latent(ql, q, sp.positions, freq, sink),
                        2.0 * batch * seen * (R + r) + 4.0 * batch * H * R, flops=2.0 * batch * seen * H * (2 * R + r), like="attention_rows decode kv8 / kv32")
                 del cache
+        # short portions behind a context: 32 sequences bring 8 tokens each
+        E, n, ctx, window = 32, 8, 2048, 1024
+        ids, more = [prompt(i, ctx) for i in range(E)], [prompt(100 + i, n) for i in range(E)]
+        tag = "portions %dx%d behind %d" % (E, n, ctx)
+        sp = SpanBatch(more, [ctx] * E, list(range(E)), dev)
+        for kvh in (32, 8):
+            cache = chunk_attn.Attention.shaped(n_heads=H, n_kv_heads=kvh, d_key=d, d_value=d, scale=d ** -0.5, sink=True, memory_mb=4096, dtype=bf, device=dev)
+            k3 = rnd(ctx, kvh, d)
+            for p in ids:
+                cache.add_seq(tokens=p, k=k3, v=k3)
+            rows = list(range(E))
+            cache.extend(rows, more)
+            q = cache.store_qkv(rnd(E * n, (H + 2 * kvh) * d), sp.positions)
+            kernel("attention_rows kv%d %s" % (kvh, tag), lambda: cache.forward_rows(q, sp.positions, None, sp.entry_of), 4.0 * E * ctx * kvh * d,
+                   flops=4.0 * pairs_of([ctx] * E, [n] * E, 1 << 30) * H * d)
+            del cache
+        cache = latent_cache(window)
+        for i, p in enumerate(ids):
+            cache.extend([-1], [p])
+            cache.store_latent(rnd(ctx, QR + R + r), SpanBatch([p], [0], [i], dev).positions, qn, kn, 1e-5, freq)
+        cache.extend(list(range(E)), more)
+        cache.store_latent(rnd(E * n, QR + R + r), sp.positions, qn, kn, 1e-5, freq)
+        ql, q = rnd(E * n, H, R), rnd(E * n, H, d + r)
+        kernel("forward_latent %s, window %d" % (tag, window), lambda: cache.forward_latent(ql, q, sp.positions, freq, sink, sp.entry_of),
+               2.0 * E * (window + n - 1) * (R + r) + 4.0 * E * n * H * R, flops=2.0 * pairs_of([ctx] * E, [n] * E, window) * H * (2 * R + r),
+               like="attention_rows kv8 / kv32 portions")
+        del cache
     value = bench.layers["window 1024"]["decode_64_at_1024"]
     line = {"metric": "bikelix_decode_tokens_per_s", "value": value["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": bench.steps,
             "warmup": bench.warm, "ms_per_step": value["us"] * 1e-3, "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
