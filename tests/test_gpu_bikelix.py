@@ -188,7 +188,7 @@ def sharp_weights(cfg, w, layer, owner):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("reader", [False, True])
-@pytest.mark.parametrize("window", [40, 64, 150])
+@pytest.mark.parametrize("window", [41, 64, 150])
 def test_keys_on_the_edge_of_a_window(dtype, reader, window):
     """One key that dwarfs all others, just inside the window (it decides the logits) and just outside (it must not be seen): in
     a prompt, in a portion of two tokens, and decoded; in a layer with rows of its own and in one that reads another's."""
