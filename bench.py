@@ -1485,6 +1485,7 @@ def run_bikelix(args):
     from chunk_attn.models.bikelix.modeling_bikelix import random_weights
     from chunk_attn.models.gagorax import GagoraxConfig, GagoraxForCausalLM
     from chunk_attn.models.gagorax.modeling_gagorax import random_weights as gagorax_weights
+    from chunk_attn.models.span_decoder import split_frequencies
     bench = LayerBench(args, measured_bf16_peak())
     dev, prompt, kernel = bench.dev, bench.prompt, bench.kernel
     bf, f32, f16 = torch.bfloat16, torch.float32, torch.float16
@@ -1508,7 +1509,7 @@ def run_bikelix(args):
 
         W, F, H, d, r, dv, QR, R = 4096, 11008, 32, 128, 64, 128, 1536, 512
         scale = (d + r) ** -0.5
-        freq = (10000.0 ** (-torch.arange(r // 2, device=dev) * 2.0 / r)).float()
+        freq = split_frequencies(r, 10000.0, dev)
         qn, kn, sink = 1 + 0.1 * rnd(QR, dtype=f32), 1 + 0.1 * rnd(R, dtype=f32), rnd(H, dtype=f32)
         w_ukv = rnd(H * (d + dv), R) * R ** -0.5
 

@@ -22,7 +22,7 @@ import chunk_attn
 from chunk_attn import ops
 
 from ..recurrent_state import RecurrentState
-from ..span_decoder import SpanDecoder, Weights, linear_f32, pair_frequencies
+from ..span_decoder import SpanDecoder, Weights, linear_f32, split_frequencies
 from .configuration_bikelix import BikelixConfig
 
 GATE_SLOPE = 1.702
@@ -45,7 +45,7 @@ class LatentAttentionMixer:
         self.w_uk = self.w_ukv[:uk.shape[0]].view(self.heads, self.dim, m["kv_rank"])
         self.w_uv = self.w_ukv[uk.shape[0]:].view(self.heads, self.vdim, m["kv_rank"])
         self.sink = w.vector(p + "sink")
-        self.freq = pair_frequencies(self.rot, m["rot"]["base"], config.torch_device)
+        self.freq = split_frequencies(self.rot, m["rot"]["base"], config.torch_device)
         self.cache = None
 
     def geometry(self):

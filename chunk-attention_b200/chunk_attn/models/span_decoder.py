@@ -28,6 +28,13 @@ def pair_frequencies(dims, base, device):
     return f.to(torch.float32).to(device)
 
 
+def split_frequencies(dims, base, device):
+    """[2, dims / 2]: the frequencies rounded to fp32, and what rounding left out."""
+    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    hi = f.to(torch.float32)
+    return torch.stack([hi, (f - hi.double()).to(torch.float32)]).to(device)
+
+
 class Weights:
     """The named tensors of a model, placed on the device: matrices in the model's dtype, vectors in fp32."""
 

@@ -196,7 +196,7 @@ struct LatentStoreParams {
     const float* q_norm;
     const float* kv_norm;
     float eps;
-    const float* freq;           // [rot / 2]
+    const float* freq;           // [2][rot / 2]: rounded, and what rounding left out
     const int32_t* positions;
     const int32_t* tok_slot;     // as in QkvParams
     const int32_t* tail_chunk;
@@ -219,7 +219,7 @@ struct LatentParams {
     float scale, scale_log2;     // scale and scale * log2(e)
     const float* sink;           // [n_heads] or null
     const int32_t* positions;    // [n_rows]
-    const float* freq;           // [rot / 2]
+    const float* freq;           // [2][rot / 2]: rounded, and what rounding left out
     // portions
     const int32_t* row_entry;
     const int32_t* path_off;     // null: decode
@@ -257,7 +257,7 @@ struct LatentSpanParams {
     float scale_log2;            // > 0
     const float* sink;           // [n_heads] or null
     const int32_t* positions;
-    const float* freq;           // [rot / 2]
+    const float* freq;           // [2][rot / 2]: rounded, and what rounding left out
     const int32_t* base;         // workspace row of position first[e] of span e
     const int32_t* first;
     const int32_t* blocks;       // [n_blocks][4]: span, first token, end token, 0; at most 256 tokens each

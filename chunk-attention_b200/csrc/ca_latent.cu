@@ -67,7 +67,7 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentSt
     const int half = p.rot / 2;
     float rot_u = 0.f, rot_v = 0.f, sn = 0.f, cs = 0.f;
     if (tid < half) {
-        sincos_for<T>((float)p.positions[t] * p.freq[tid], &sn, &cs);
+        turn_for<T>((float)p.positions[t], p.freq[tid], p.freq[half + tid], &sn, &cs);
         rot_u = to_f32(r[tid]);
         rot_v = to_f32(r[tid + half]);
     }
@@ -103,7 +103,7 @@ __global__ void __launch_bounds__(LS_THREADS) latent_store_kernel(const LatentSt
         *reinterpret_cast<P*>(tile + tile_elem_offset(p.geo, slot, c)) = scaled(c == c0 ? kv_keep : *reinterpret_cast<const P*>(kv + c), inv, p.kv_norm + c);
     for (int i = tid; i < half; i += LS_THREADS) {
         if (i != tid) {
-            sincos_for<T>((float)p.positions[t] * p.freq[i], &sn, &cs);
+            turn_for<T>((float)p.positions[t], p.freq[i], p.freq[half + i], &sn, &cs);
             rot_u = to_f32(r[i]);
             rot_v = to_f32(r[i + half]);
         }
@@ -148,7 +148,7 @@ __global__ void __launch_bounds__(LG_WARPS * 32) latent_generic_kernel(const Lat
         const int half = rot / 2;
         for (int i = threadIdx.x; i < half; i += blockDim.x) {
             float sn, cs;
-            sincos_for<T>((float)pos * p.freq[i], &sn, &cs);
+            turn_for<T>((float)pos, p.freq[i], p.freq[half + i], &sn, &cs);
             const float u = to_f32(qr[i]), v = to_f32(qr[i + half]);
             // rounded as the tensor-core kernels' operands are
             q_s[kv_rank + i] = to_f32(from_f32<T>(u * cs - v * sn)) * p.scale;

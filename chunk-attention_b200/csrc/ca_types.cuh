@@ -50,6 +50,17 @@ __device__ __forceinline__ void fast_sincos(float a, float* sn, float* cs) {
 template <typename T> __device__ __forceinline__ void sincos_for(float a, float* sn, float* cs) { fast_sincos(a, sn, cs); }
 template <> __device__ __forceinline__ void sincos_for<float>(float a, float* sn, float* cs) { sincosf(a, sn, cs); }
 
+// sine and cosine of pos * f, f = hi + lo.  fp32 kernels keep what the product's rounding and hi leave out; in 16-bit kernels
+// it is far below the results' own rounding.
+template <typename T> __device__ __forceinline__ void turn_for(float pos, float hi, float lo, float* sn, float* cs) { fast_sincos(pos * hi, sn, cs); }
+template <> __device__ __forceinline__ void turn_for<float>(float pos, float hi, float lo, float* sn, float* cs) {
+    const float a = pos * hi, rest = fmaf(pos, lo, fmaf(pos, hi, -a));
+    float s, c;
+    sincosf(a, &s, &c);
+    *sn = fmaf(rest, c, s);
+    *cs = fmaf(-rest, s, c);
+}
+
 // one MUFU operation; results below 2^-126 are 0
 __device__ __forceinline__ float exp2_approx(float x) {
     float y;

@@ -646,7 +646,7 @@ torch::Tensor Attention::store_latent(torch::Tensor in, torch::Tensor positions,
     a.q_norm = f32_ptr(q_norm, q_rank, "store_latent: q_norm must be fp32 [q_rank]");
     a.kv_norm = f32_ptr(kv_norm, shape_.d_value, "store_latent: kv_norm must be fp32 [latent size]");
     a.eps = (float)eps;
-    a.freq = f32_ptr(freq, rot / 2, "store_latent: freq must be fp32 [rotated / 2]");
+    a.freq = f32_ptr(freq, rot, "store_latent: freq must be fp32 [2, rotated / 2]");
     a.positions = i32_ptr(positions, n, "store_latent: positions must be int32 [n_tokens]");
     a.n_tokens = (int32_t)n;
     c10::cuda::CUDAGuard guard(options_.device());
@@ -689,7 +689,7 @@ torch::Tensor Attention::forward_latent(torch::Tensor q_lat, torch::Tensor q, to
     a.out = out.data_ptr();
     a.n_rows = (int32_t)n;
     a.positions = i32_ptr(positions, n, "forward_latent: positions must be int32 [n_rows]");
-    a.freq = f32_ptr(freq, rot / 2, "forward_latent: freq must be fp32 [rotated / 2]");
+    a.freq = f32_ptr(freq, rot, "forward_latent: freq must be fp32 [2, rotated / 2]");
     a.sink = f32_ptr(sink, n_heads_, "forward_latent: sink must be fp32 [n_heads]");
     a.delta_tokens = -1;
     if (row_entry.has_value()) {
@@ -757,7 +757,7 @@ torch::Tensor Attention::forward_expanded(torch::Tensor q, torch::Tensor kv, tor
     a.dim = dim;
     a.vdim = vdim;
     a.positions = i32_ptr(positions, n, "forward_expanded: positions must be int32 [n_rows]");
-    a.freq = f32_ptr(freq, rotated / 2, "forward_expanded: freq must be fp32 [rotated / 2]");
+    a.freq = f32_ptr(freq, rotated, "forward_expanded: freq must be fp32 [2, rotated / 2]");
     a.sink = f32_ptr(sink, n_heads_, "forward_expanded: sink must be fp32 [n_heads]");
     a.base = t + w.rows;
     a.first = t + w.rows + (int64_t)tables_->lens.size() + 1;

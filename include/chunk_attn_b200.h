@@ -385,7 +385,8 @@ CA_API int ca_attention_rows(ca_context* ctx, const ca_rows_args* args, ca_strea
 /* Latent caches.  in: [n_tokens, row_stride] of the context's type, q_rank elements of the query latent | d_value of the
  * key/value latent | d_key - d_value of the shared key part.  The query latent is RMS-normed (q_norm, fp32 [q_rank]) into
  * q_out [n_tokens, q_rank] (q_rank 0: there is none); the key/value latent is RMS-normed (kv_norm, fp32 [d_value]), the
- * shared key part rotated (element i with element i + half, by position * freq[i], fp32 [half]), both go to the pool.
+ * shared key part rotated (element i with element i + half, by position * (freq[i] + freq[half + i]):
+ * fp32 [2][half], the frequencies rounded and what rounding left out), both go to the pool.
  * tok_slot as in ca_store_qkv. */
 typedef struct ca_latent_store_args {
     const void* in;

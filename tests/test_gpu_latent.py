@@ -81,7 +81,10 @@ class Feeder:
 
     def __init__(self, dtype, q_rank, latent, rot, heads, window, scale=1.0, chunk=64, base=100.0, tokens=4096):
         self.dtype, self.q_rank, self.R, self.r, self.base = dtype, q_rank, latent, rot, base
-        self.freq = torch.from_numpy(oracle.half_frequencies(rot, base)).float().to(DEV) if rot else None
+        self.freq = None
+        if rot:  # rounded, and what rounding left out
+            f = torch.from_numpy(oracle.half_frequencies(rot, base))
+            self.freq = torch.stack([f.float(), (f - f.float().double()).float()]).to(DEV)
         line = 128 // (2 if dtype == torch.bfloat16 else 4)
         mb = -(-(latent + rot) // line) * 128 * (tokens + 64 * chunk) / 2 ** 20
         self.cache = chunk_attn.Attention.latent(n_heads=heads, latent=latent, rotated=rot, scale=scale, window=window, chunk_size=chunk,
@@ -379,3 +382,15 @@ def test_readers(dtype):
     with pytest.raises(RuntimeError, match="separate keys"):
         f.cache.add_seq(tokens=[1], k=torch.zeros(1, 1, R + r, device=DEV), v=torch.zeros(1, 1, R, device=DEV))
     assert all(v[0].device_status() == 0 for v in views.values())
+
+
+def test_angles_far_from_the_start():
+    """In fp32 the rotation at position 100 000 is as exact as at the start: angles are not rounded to one fp32 number."""
+    f = Feeder(torch.float32, 8, 32, 16, heads=1, window=0, base=3.0, tokens=128)
+    x = rnd(3, 1, 8 + 32 + 16).to(DEV)
+    pos = 100_000
+    sp = SpanBatch([[1]], [pos], [0], DEV)
+    f.cache.extend([-1], [[1]])
+    f.cache.store_latent(x, sp.positions, f.q_norm, f.kv_norm, 0.1, f.freq)
+    _, kr = f.cache.gather_latents()
+    close(kr[:, :16], oracle.rotate_halves(f64(x)[:, 40:], [pos], 16, 3.0), torch.float32)
